@@ -503,6 +503,7 @@ class NativeInferConfig:
     pausable_kv_cache: bool = False
     kv_cache_dtype: str = "bfloat16"
     use_cuda_graph: bool = True
+    compute_dtype: str = "bfloat16"  # float32: matrices, activations and cache in 32 bits (mixer stacks only)
     weight_dtype: str = "bfloat16"  # or float8_e4m3fn (block-scaled)
     random_seed: int = 1
     share_trainer_weights: bool = True  # colocated mode: read the trainer's parameters in place

@@ -17,6 +17,7 @@ from __future__ import annotations
 
 import asyncio
 import collections
+import contextlib
 import math
 import threading
 import time
@@ -36,10 +37,10 @@ from ..models.decoder import CausalLM, PackedBatch, build_model
 from ..ops import functional as OF
 from ..ops import lib as oplib
 from ..utils import logging as alog
+from .ragged_step import DECODE_BUCKETS, Entry, RaggedRunner
+from .state_cache import Carried, PagePool, StateCache
 
 logger = alog.getLogger("infer_engine")
-
-DECODE_BUCKETS = (1, 2, 4, 8, 16, 32, 64, 128, 256, 512)
 
 
 @dataclass
@@ -71,14 +72,15 @@ class _Seq:
     stop_window: int = 16                  # tokens decoded per check
     mm: Any = None                         # vision-language request: {"pixel_values", "image_grid_thw"}
     rope_delta: int = 0                    # M-RoPE: rotary position of token i (after the prompt) = i + rope_delta
+    carry: Optional[Carried] = None        # mixer stacks: pages and state slot while running
     hstate: Any = None                     # recurrent-state models: models.hybrid.SequenceState once the prompt is absorbed
 
 
-class PagedKVCache:
+class PagedKVCache(PagePool):
     """K and V pages for all layers: ``[layers, 2, num_pages * page_size, Hkv, D]``."""
 
     def __init__(self, cfg: ModelConfig, num_pages: int, page_size: int, device, dtype, pausable: bool = False):
-        self.page_size, self.num_pages = page_size, num_pages
+        super().__init__(num_pages, page_size)
         shape = (cfg.num_layers, 2, num_pages * page_size, cfg.num_kv_heads, cfg.head_dim)
         self.pausable = None
         if pausable:
@@ -93,32 +95,6 @@ class PagedKVCache:
                 self.data.zero_()
         if self.pausable is None:
             self.data = torch.zeros(*shape, device=device, dtype=dtype)
-        self.free = list(range(num_pages - 1, -1, -1))
-        self.ref = [0] * num_pages          # users of a page: its sequence, plus the prefix cache and other sequences when shared
-
-    def alloc(self, n: int) -> Optional[list[int]]:
-        if len(self.free) < n:
-            return None
-        out = self.free[-n:] if n else []
-        if n:
-            del self.free[-n:]
-        for p in out:
-            self.ref[p] = 1
-        return out
-
-    def share(self, pages: list[int]) -> None:
-        for p in pages:
-            self.ref[p] += 1
-
-    def release(self, pages: list[int]) -> None:
-        for p in pages:
-            self.ref[p] -= 1
-            if self.ref[p] <= 0:
-                self.ref[p] = 0
-                self.free.append(p)
-
-    def pages_needed(self, tokens: int) -> int:
-        return (tokens + self.page_size - 1) // self.page_size
 
 
 class NativeInferenceEngine(InferenceEngine):
@@ -157,7 +133,9 @@ class NativeInferenceEngine(InferenceEngine):
         self.stats = collections.Counter()
         self._prefix: collections.OrderedDict = collections.OrderedDict()     # prompt bytes -> shared pages + last-token logits
         self.device = torch.device("cpu")
-        self.cache: Optional[PagedKVCache] = None
+        self.cache: Optional[PagePool] = None
+        self.runner: Optional[RaggedRunner] = None
+        self._ragged = False
 
     # ------------------------------------------------------------------ lifecycle
     def initialize(self, device=None, seed: int = 1, train_data_parallel_size: int = 1, model_path: Optional[str] = None,
@@ -173,6 +151,10 @@ class NativeInferenceEngine(InferenceEngine):
                     raise ValueError("inference engine needs a model, a model_config or a model_path")
                 self.model_config = ModelConfig.from_pretrained(model_path)
             dtype = torch.bfloat16 if self.device.type == "cuda" else torch.float32
+            if self.icfg.compute_dtype == "float32":
+                if not self.model_config.is_mixer_stack:
+                    raise NotImplementedError("32-bit compute is built for mixer stacks only")
+                dtype = torch.float32
             self.model = build_model(self.model_config, dtype=dtype, device=self.device, seed=seed)
             if model_path:
                 from ..models import hf_io
@@ -192,11 +174,16 @@ class NativeInferenceEngine(InferenceEngine):
         # convolution tail, keys / values of the full-attention layers) and then advance one token per
         # step on that state (``_step_recurrent``).
         self._recompute_decode = bool(getattr(self.model_config, "is_hybrid", False))
-        if self.device.type == "cuda" and not self._recompute_decode:
+        self._ragged = bool(getattr(self.model_config, "is_mixer_stack", False))
+        if self._ragged:
+            self._init_ragged()
+        elif self.device.type == "cuda" and not self._recompute_decode:
             self._init_cuda_state()
         elif self.device.type == "cuda":
             self.stream = torch.cuda.Stream(device=self.device)
         self._t_start = time.perf_counter()
+        if not kwargs.get("start_loop", True):
+            return self                     # the caller steps the engine itself (trace runner)
         self._thread = threading.Thread(target=self._engine_main, name="infer-engine", daemon=True)
         self._thread.start()
         if start_executor:
@@ -209,8 +196,8 @@ class NativeInferenceEngine(InferenceEngine):
         """Replaces the freshly built (or loaded) full model by this rank's tensor-parallel slice."""
         from ..parallel import tp as TP
 
-        if self.model_config.is_vlm:
-            raise NotImplementedError("tensor-parallel rollout of vision-language models")
+        if self.model_config.is_vlm or self.model_config.is_mixer_stack:
+            raise NotImplementedError("tensor-parallel rollout of vision-language models and mixer stacks")
         full, full_cfg = self.model, self.model_config
         self.full_model_config = full_cfg
         self.model_config = TP.local_config(full_cfg, self.tp_size)
@@ -301,6 +288,46 @@ class NativeInferenceEngine(InferenceEngine):
         oplib.get_lib().ab2_runtime_init()
         logger.info("KV cache: %d pages x %d tokens (%.1f GB)", n_pages, ic.page_size, n_pages * per_page / 2 ** 30)
 
+    def _init_ragged(self):
+        """Cache, runner and sampling buffers of a mixer stack (any device)."""
+        ic, dev = self.icfg, self.device
+        if self.tp_size > 1:
+            raise NotImplementedError("tensor-parallel rollout of mixer stacks")
+        mixers = [l.mix for l in self.model.layers]
+        dtype = self.model.dtype
+        self.max_batch = B = max(b for b in DECODE_BUCKETS if b <= max(1, ic.max_running_requests))
+        want = ic.max_running_requests * (ic.context_length // ic.page_size + 1)
+        n_pages = ic.num_pages
+        if n_pages is None:
+            n_pages = want
+            per_page = StateCache.bytes_per_page(mixers, ic.page_size, torch.empty(0, dtype=dtype).element_size())
+            if dev.type == "cuda" and per_page:
+                torch.cuda.empty_cache()
+                free, _ = torch.cuda.mem_get_info(dev)
+                budget = free - int(ic.reserve_free_gb * (1 << 30)) if ic.reserve_free_gb > 0 else int(free * ic.mem_fraction_static) - (2 << 30)
+                n_pages = max(16, min(want, (budget - B * StateCache.bytes_per_slot(mixers)) // per_page))
+        self._ragged_shape = (n_pages, ic.page_size, B)
+        if dev.type == "cuda":
+            if dtype == torch.float32:
+                torch.backends.cuda.matmul.allow_tf32 = False       # 32-bit compute means 32-bit products
+            self.s_inv_temp = torch.ones(B, dtype=torch.float32, device=dev)
+            self.s_greedy, self.s_seeds, self.s_out_tok = (torch.zeros(B, dtype=torch.int32, device=dev) for _ in range(3))
+            self.s_out_lp = torch.zeros(B, dtype=torch.float32, device=dev)
+            self.h_out = torch.zeros(2, B, dtype=torch.int32).pin_memory()
+            self.hn_out_tok, self.hn_out_lp = self.h_out.numpy()[0], self.h_out.numpy()[1].view(np.float32)
+            self.stream = torch.cuda.Stream(device=dev, priority=-1)
+            self._err_poll = oplib.ErrorPoller()
+            oplib.get_lib().ab2_runtime_init()
+        self._make_ragged_runner()
+
+    def _make_ragged_runner(self):
+        ic = self.icfg
+        n_pages, ps, slots = self._ragged_shape
+        self.cache = StateCache([l.mix for l in self.model.layers], n_pages, ps, slots, self.device, self.model.dtype)
+        self.runner = RaggedRunner(self.model, self.cache, self.device, slots, ic.context_length, ic.use_cuda_graph)
+        if self.device.type == "cuda":
+            self.runner.stream = self.stream
+
     def destroy(self):
         self._stop.set()
         if self._executor is not None:
@@ -310,7 +337,7 @@ class NativeInferenceEngine(InferenceEngine):
             self._thread.join(timeout=10)
             self._thread = None
         self._graphs.clear()
-        self.cache = None
+        self.cache = self.runner = None
 
     # ------------------------------------------------------------------ versions / weights
     def set_version(self, version: int) -> None:
@@ -400,7 +427,7 @@ class NativeInferenceEngine(InferenceEngine):
         """Gives the KV pool's memory back to the device. With a pausable pool the addresses (and the
         CUDA graphs that point into them) survive; otherwise the pool and the graphs are dropped."""
         self.pause_generation()
-        if self.cache is not None and self.cache.pausable is not None:
+        if not self._ragged and self.cache is not None and self.cache.pausable is not None:
             self._abort_all_now()
             self._prefix.clear()
             self.cache.free = list(range(self.cache.num_pages - 1, -1, -1))
@@ -409,6 +436,12 @@ class NativeInferenceEngine(InferenceEngine):
             self.cache.pausable.pause()
             return
         self._graphs.clear()
+        if self._ragged:
+            self._abort_all_now()
+            self.cache = self.runner = None
+            if self.device.type == "cuda":
+                torch.cuda.empty_cache()
+            return
         if self.cache is not None:
             self._saved_cache_shape = (self.cache.num_pages, self.cache.page_size)
             self.cache = None
@@ -419,6 +452,11 @@ class NativeInferenceEngine(InferenceEngine):
         self._abort_all()
 
     def onload(self, tags=None):
+        if self._ragged:
+            if self.cache is None:
+                self._make_ragged_runner()
+            self.continue_generation()
+            return
         if self.cache is not None and self.cache.pausable is not None:
             if self.cache.pausable.paused:
                 self.cache.pausable.resume()
@@ -553,7 +591,10 @@ class NativeInferenceEngine(InferenceEngine):
                     continue
                 self._idle.clear()
                 t_busy = time.perf_counter()
-                if self.device.type == "cuda" and self._recompute_decode:
+                if self._ragged:
+                    with torch.no_grad(), (torch.cuda.stream(self.stream) if self.device.type == "cuda" else contextlib.nullcontext()):
+                        self._step_ragged()
+                elif self.device.type == "cuda" and self._recompute_decode:
                     with torch.cuda.stream(self.stream), torch.no_grad():
                         self._step_recurrent()
                 elif self.device.type == "cuda":
@@ -606,6 +647,10 @@ class NativeInferenceEngine(InferenceEngine):
         if self.cache is not None and seq.pages:
             self.cache.release(seq.pages)
             seq.pages = []
+        if seq.carry is not None:
+            if self.cache is not None:
+                self.cache.close(seq.carry)
+            seq.carry = None
         if seq.row >= 0:
             self._free_row(seq)
         if seq.future is None:          # follower of a tensor-parallel replica: the leader answers the client
@@ -717,6 +762,77 @@ class NativeInferenceEngine(InferenceEngine):
         for s, _ in done:
             s.hstate = None
         self._retire(done)
+
+    def _step_ragged(self):
+        """Mixer stacks: one ragged batch per iteration. Running requests bring the token they sampled last, requests
+        whose prompt is not absorbed yet bring the next portion of it (``max_prefill_tokens`` per step over all of
+        them); those whose last known token was absorbed sample their next one."""
+        cache, ic = self.cache, self.icfg
+        with self._lock:
+            while self._waiting and len(self._running) < self.max_batch:
+                s = self._waiting[0]
+                # pages of the prompt's first portion now, the rest as the sequence grows; a page per running request
+                # stays free so that growth rarely has to pre-empt
+                first = min(len(s.tokens), ic.max_prefill_tokens)
+                if self._running and cache.has_kv and len(cache.free) < cache.pages_needed(first) + len(self._running):
+                    break
+                s.carry = cache.open()
+                if s.carry is None:
+                    break
+                cache.grow(s.carry, first)          # (alone in the pool it may be short: growing below settles that)
+                self._running.append(self._waiting.popleft())
+            batch = list(self._running)
+        if not batch:
+            return
+        budget = ic.max_prefill_tokens
+        plan = []
+        for s in batch:
+            n = len(s.tokens) - s.carry.length
+            if n > 1:
+                n = min(n, budget)
+                budget -= n
+            if n > 0:
+                plan.append((s, n))
+        plan = self._grow_ragged(plan, batch)
+        entries = []
+        for s, n in plan:
+            a = s.carry.length
+            entries.append(Entry(s.carry, s.tokens[a:a + n], [n - 1] if a + n == len(s.tokens) else []))
+        if not entries:
+            return
+        logits = self.runner.step(entries)
+        self.stats["prefill_tokens"] += sum(n for _, n in plan if n > 1)
+        self.stats["decode_steps"] += 1
+        ready = [s for (s, _), e in zip(plan, entries) if e.want]
+        done: list = []
+        if ready:
+            if self.device.type == "cuda":
+                toks, lps = self._sample_cuda(logits, ready)
+            else:
+                self._step += 1
+                toks, lps = zip(*[self._sample_cpu(logits[i], s) for i, s in enumerate(ready)])
+            for s, tok, lp in zip(ready, toks, lps):
+                self._accept_token(s, tok, lp, done)
+        self._retire(done)
+
+    def _grow_ragged(self, plan: list, running: list) -> list:
+        """Pages for every planned portion. When the pool is dry the most recently admitted other request is pre-empted
+        (it leaves with what it has generated and its client resubmits it)."""
+        gone: set = set()
+        for s, n in plan:
+            if id(s) in gone:
+                continue
+            while not self.cache.grow(s.carry, s.carry.length + n):
+                victims = [v for v in running if id(v) not in gone and v is not s]
+                if not victims:
+                    raise RuntimeError("KV page pool too small for a single sequence")
+                v = max(victims, key=lambda q: (q.t_submit, q.rid))
+                gone.add(id(v))
+                self.stats["preempted"] += 1
+                with self._lock:
+                    self._running = [q for q in self._running if q is not v]
+                self._resolve(v, "abort")
+        return [(s, n) for s, n in plan if id(s) not in gone]
 
     def _sample_cpu(self, logits: torch.Tensor, s: _Seq):
         if s.greedy:

@@ -1,5 +1,5 @@
 """Architecture description of the supported decoder families (Qwen2 / Qwen2.5, Qwen3,
-Qwen3-MoE) and conversion from / to Hugging Face ``config.json``.
+Qwen3-MoE, Qwen3.5, mixer stacks) and conversion from / to Hugging Face ``config.json``.
 
 Reference model zoo: ``areal/experimental/models/archon/{qwen2,qwen3}/model/args.py`` and
 the HF path of ``areal/engine/fsdp_engine.py:375-560``.
@@ -14,7 +14,7 @@ from typing import Optional
 
 @dataclass
 class ModelConfig:
-    arch: str = "qwen2"                 # qwen2 | qwen3 | qwen3_moe | qwen2_moe
+    arch: str = "qwen2"                 # qwen2 | qwen3 | qwen3_moe | qwen2_moe | qwen3_5 | qwen3_5_moe | kagolix
     vocab_size: int = 151936
     hidden_size: int = 1536
     num_layers: int = 28
@@ -63,6 +63,16 @@ class ModelConfig:
     partial_rotary_factor: float = 1.0
     attn_output_gate: bool = False
     rms_norm_offset: bool = False
+    # mixer stacks (Kagolix): one entry per layer, {"type": mixer kind, "mixer": its sizes, "mlp": feed-forward or
+    # None} as in config.json (see models/mixers.py); grouped RMS norms and a capped output
+    mixer_layers: list[dict] = field(default_factory=list)
+    norm_groups: int = 1
+    logit_softcap: float = 0.0
+
+    @property
+    def is_mixer_stack(self) -> bool:
+        """Layers built from per-layer mixer specs; served by the ragged step (engine/ragged_step.py)."""
+        return bool(self.mixer_layers)
 
     @property
     def is_hybrid(self) -> bool:
@@ -100,6 +110,10 @@ class ModelConfig:
         return self.is_moe and i not in self.mlp_only_layers and (i + 1) % max(1, self.decoder_sparse_step) == 0
 
     def num_params(self) -> int:
+        if self.is_mixer_stack:
+            from .decoder import build_model
+
+            return sum(p.numel() for p in build_model(self, device="meta").parameters())
         H, V, L = self.hidden_size, self.vocab_size, self.num_layers
         attn = H * (self.q_size + 2 * self.kv_size) + self.q_size * H
         if self.attention_bias:
@@ -137,6 +151,8 @@ class ModelConfig:
     # ------------------------------------------------------------------ HF interop
     @classmethod
     def from_hf_dict(cls, d: dict) -> "ModelConfig":
+        if "architecture" in d:
+            return cls._from_mixer_stack_dict(d)
         mt = d.get("model_type", "qwen2")
         vl = None
         if mt == "qwen3_vl":
@@ -219,12 +235,40 @@ class ModelConfig:
         )
 
     @classmethod
+    def _from_mixer_stack_dict(cls, d: dict) -> "ModelConfig":
+        """config.json of a mixer stack: ``architecture`` names the design, ``layers`` lists every layer's mixer
+        and feed-forward with their sizes."""
+        if d["architecture"] != "Kagolix":
+            raise ValueError(f"unsupported architecture '{d['architecture']}'")
+        from .mixers import check_layer_specs
+
+        layers = [dict(type=e["type"], mixer=dict(e["mixer"]), mlp=dict(e["mlp"]) if e.get("mlp") else None) for e in d["layers"]]
+        check_layer_specs(layers, d["width"], d["norm"].get("groups", 1))
+        att = [e["mixer"] for e in layers if e["type"] == "attention"]
+        moe = [e["mlp"] for e in layers if e["mlp"] and e["mlp"]["kind"] == "moe"]
+        return cls(arch="kagolix", vocab_size=d["vocab"], hidden_size=d["width"], num_layers=len(layers),
+                   # engine-wide summaries; every layer reads its own sizes from its spec
+                   num_heads=max((m["heads"] for m in att), default=1), num_kv_heads=max((m["kv_heads"] for m in att), default=1),
+                   head_dim=max((m["dim"] for m in att), default=1),
+                   intermediate_size=max((e["mlp"]["ff"] for e in layers if e["mlp"] and e["mlp"]["kind"] == "dense"), default=0),
+                   num_experts=max((m["router"]["experts"] for m in moe), default=0),
+                   num_experts_per_tok=max((m["router"]["top"] for m in moe), default=0),
+                   moe_intermediate_size=max((m["expert"]["ff"] for m in moe), default=0), norm_topk_prob=False,
+                   rms_norm_eps=float(d["norm"]["eps"]), norm_groups=int(d["norm"].get("groups", 1)),
+                   logit_softcap=float(d.get("logit_softcap") or 0.0), tie_word_embeddings=False, attention_bias=False,
+                   mixer_layers=layers, max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)))
+
+    @classmethod
     def from_pretrained(cls, path: str) -> "ModelConfig":
         with open(os.path.join(path, "config.json")) as f:
             return cls.from_hf_dict(json.load(f))
 
     def to_hf_dict(self) -> dict:
         mt = self.arch
+        if self.is_mixer_stack:
+            return dict(architecture="Kagolix", vocab=self.vocab_size, width=self.hidden_size,
+                        norm=dict(eps=self.rms_norm_eps, groups=self.norm_groups), logit_softcap=self.logit_softcap,
+                        layers=[dict(e) for e in self.mixer_layers])
         d = dict(
             model_type=mt, architectures=[{"qwen2": "Qwen2ForCausalLM", "qwen3": "Qwen3ForCausalLM", "qwen3_5": "Qwen3_5ForCausalLM", "qwen3_5_moe": "Qwen3_5MoeForCausalLM",
                                            "qwen3_moe": "Qwen3MoeForCausalLM", "qwen2_moe": "Qwen2MoeForCausalLM"}[mt]],
@@ -342,9 +386,37 @@ PRESETS = {
 }
 
 
+def _mixer_stack_preset(vocab, width, pattern, att, ssm, lru, dense_ff, moe, groups, eps=1e-6, softcap=20.0):
+    """A mixer stack from a pattern of letters: a / m / r pick the mixer (attention, mamba2, rglru), upper case
+    gives the layer experts instead of a dense feed-forward."""
+    kinds = {"a": ("attention", att), "m": ("mamba2", ssm), "r": ("rglru", lru)}
+    layers = []
+    for c in pattern:
+        t, m = kinds[c.lower()]
+        mlp = dict(kind="moe", expert=dict(ff=moe[2]), router=dict(experts=moe[0], top=moe[1])) if c.isupper() else dict(kind="dense", ff=dense_ff)
+        layers.append(dict(type=t, mixer=dict(m), mlp=mlp))
+    return dict(architecture="Kagolix", vocab=vocab, width=width, norm=dict(eps=eps, groups=groups), logit_softcap=softcap, layers=layers)
+
+
+MIXER_STACK_PRESETS = {
+    "tiny-kagolix": _mixer_stack_preset(
+        320, 128, "aMrM", dict(heads=4, kv_heads=2, dim=32, vdim=48, scale=0.2, softcap=25.0, mask=dict(size=40)),
+        dict(heads=4, vdim=32, state=16, groups=2, norm_groups=2, conv=4), dict(width=96, blocks=3, conv=4), 160, (6, 2, 64), 2),
+    # layer sizes of an 8B-class model; one of every kind of layer
+    "kagolix-8b-layers": _mixer_stack_preset(
+        32768, 4096, "amRM", dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, mask=dict(size=4096)),
+        dict(heads=64, vdim=64, state=128, groups=8, norm_groups=8, conv=4), dict(width=4096, blocks=16, conv=4), 12288, (64, 8, 768), 8),
+}
+
+
 def preset(name: str, **overrides) -> ModelConfig:
+    if name in MIXER_STACK_PRESETS:
+        cfg = ModelConfig.from_hf_dict(MIXER_STACK_PRESETS[name])
+        for k, v in overrides.items():
+            setattr(cfg, k, v)
+        return cfg
     if name not in PRESETS:
-        raise KeyError(f"unknown model preset '{name}' (have {sorted(PRESETS)})")
+        raise KeyError(f"unknown model preset '{name}' (have {sorted([*PRESETS, *MIXER_STACK_PRESETS])})")
     d = dict(PRESETS[name])
     d.update(overrides)
     return ModelConfig(**d)

@@ -359,7 +359,9 @@ class CausalLM(nn.Module):
         self.dtype = dtype
         H = cfg.hidden_size
         self.embed_tokens = nn.Parameter(torch.empty(cfg.vocab_size, H, dtype=dtype, device=device))
-        if cfg.layer_types:
+        if cfg.is_mixer_stack:
+            from .mixers import MixerLayer as layer_cls
+        elif cfg.layer_types:
             from .hybrid import HybridDecoderLayer as layer_cls   # linear / gated full attention per layer (Qwen3.5)
         else:
             layer_cls = DecoderLayer
@@ -511,4 +513,8 @@ def build_model(cfg: ModelConfig, dtype=torch.bfloat16, device="cpu", seed: Opti
         from .vlm import VisionLanguageModel
 
         return VisionLanguageModel(cfg, dtype=dtype, device=device, seed=seed)
+    if cfg.is_mixer_stack:
+        from .mixers import MixerStackLM
+
+        return MixerStackLM(cfg, dtype=dtype, device=device, seed=seed)
     return CausalLM(cfg, dtype=dtype, device=device, seed=seed)

@@ -21,6 +21,10 @@ from .config import ModelConfig
 # --------------------------------------------------------------------------- name mapping
 def hf_to_native_plan(cfg: ModelConfig) -> dict[str, list[tuple[str, Optional[tuple[int, int]], Optional[int]]]]:
     """native name -> list of (hf name, row range in the native tensor or None, expert idx or None)."""
+    if cfg.is_mixer_stack:
+        from .mixers import checkpoint_plan
+
+        return checkpoint_plan(cfg)
     D, nq, nkv = cfg.head_dim, cfg.num_heads, cfg.num_kv_heads
     plan: dict = {"embed_tokens": [("model.embed_tokens.weight", None, None)], "norm": [("model.norm.weight", None, None)]}
     if cfg.is_critic:

@@ -22,6 +22,9 @@ HERE = Path(__file__).resolve().parent
 CSRC = HERE / "csrc"
 BUILD = HERE / "build"
 LIB = HERE / "libab2_kernels.so"
+# the kernels that serve a mixer stack, linked alone: what a fresh checkout compiles before its first trace
+STEP_LIB = HERE / "libab2_step.so"
+STEP_SOURCES = ("runtime", "gemm", "gemm2sm", "gemm_grouped", "router", "infer", "mixer_attention", "mixer_ops", "mixer_scan")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -46,24 +49,34 @@ def _digest(paths) -> str:
     return h.hexdigest()
 
 
-def sources():
-    return sorted(CSRC.glob("*.cu"))
+def sources(names=None):
+    return sorted(p for p in CSRC.glob("*.cu") if names is None or p.stem in names)
 
 
-def is_current() -> bool:
-    stamp = BUILD / "stamp"
-    if not LIB.exists() or not stamp.exists():
+def _headers() -> list:
+    return list(CSRC.glob("*.cuh")) + list(CSRC.glob("*.h"))
+
+
+def is_current(lib: Path = LIB, names=None) -> bool:
+    stamp = BUILD / ("stamp" if lib == LIB else "stamp-" + lib.stem)
+    if not lib.exists() or not stamp.exists():
         return False
-    return stamp.read_text().strip() == _digest(list(sources()) + list(CSRC.glob("*.cuh")) + list(CSRC.glob("*.h")))
+    return stamp.read_text().strip() == _digest(sources(names) + _headers())
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
-    """Compiles and links the library if sources changed. Returns the library path."""
-    if not force and is_current():
-        return LIB
+def build_step_library() -> Path:
+    """The library a mixer stack is served from: the whole one when it is up to date, else its own subset."""
+    return LIB if is_current() else build(lib=STEP_LIB, names=STEP_SOURCES)
+
+
+def build(force: bool = False, verbose: bool = False, lib: Path = LIB, names=None) -> Path:
+    """Compiles and links the library if sources changed. Returns the library path. ``names``: the sources of a
+    library that holds a subset of the kernels."""
+    if not force and is_current(lib, names):
+        return lib
     BUILD.mkdir(exist_ok=True)
     nvcc = _nvcc()
-    srcs = sources()
+    srcs = sources(names)
     logs = {}
 
     def compile_one(src: Path):
@@ -84,13 +97,15 @@ def build(force: bool = False, verbose: bool = False) -> Path:
             sys.stderr.write(f"== {src.name}\n{r.stderr}\n")
         objs.append(str(obj))
     (BUILD / "ptxas.log").write_text("\n".join(f"== {k}\n{v}" for k, v in logs.items()))
-    link = [nvcc, "-shared", "-o", str(LIB), *objs, "-lcudart"]
+    part = lib.with_suffix(".part.so")
+    link = [nvcc, "-shared", "-o", str(part), *objs, "-lcudart"]
     r = subprocess.run(link, capture_output=True, text=True)
     if r.returncode != 0:
         sys.stderr.write(r.stdout + r.stderr)
         raise RuntimeError("link failed")
-    (BUILD / "stamp").write_text(_digest(list(srcs) + list(CSRC.glob("*.cuh")) + list(CSRC.glob("*.h"))))
-    return LIB
+    os.replace(part, lib)
+    (BUILD / ("stamp" if lib == LIB else "stamp-" + lib.stem)).write_text(_digest(srcs + _headers()))
+    return lib
 
 
 if __name__ == "__main__":

@@ -142,14 +142,14 @@ class Routing:
     a list; the copy was started when the routing was made, so a caller that asks late (the weight
     gradients in backward) does not stall the stream."""
 
-    def __init__(self, tope, topw, probs, counts, offs, order, token_of, inv, row_tiles, num_row_tiles, k):
+    def __init__(self, tope, topw, probs, counts, offs, order, token_of, inv, row_tiles, num_row_tiles, k, want_host: bool = True):
         self.tope, self.topw, self.probs = tope, topw, probs
         self.counts, self.offs, self.order, self.token_of, self.inv = counts, offs, order, token_of, inv
         self.row_tiles, self.num_row_tiles, self.k = row_tiles, num_row_tiles, k
         self.rows = order.shape[0]
         self._host = None
         self._event = None
-        if counts.is_cuda:
+        if counts.is_cuda and want_host:
             self._host = torch.empty(counts.shape, dtype=counts.dtype, pin_memory=True)
             self._host.copy_(counts, non_blocking=True)
             self._event = torch.cuda.Event()
@@ -187,10 +187,12 @@ def moe_route_ref(logits, k: int, bias=None, sigmoid: bool = False, norm: bool =
 
 
 def moe_route(logits: torch.Tensor, k: int, bias: Optional[torch.Tensor] = None, sigmoid: bool = False, norm: bool = True,
-              scale: float = 1.0, tope: Optional[torch.Tensor] = None, want_probs: bool = True) -> Routing:
+              scale: float = 1.0, tope: Optional[torch.Tensor] = None, want_probs: bool = True,
+              want_host: bool = True) -> Routing:
     """Scores, top-k choice, stable sort by expert, group sizes and the grouped-GEMM tile list from fp32
     router logits [T, E], in four small launches and without a host read. With ``tope`` given (the choice
-    was made elsewhere, e.g. group-limited routing) only the sort / counts / tiles are produced."""
+    was made elsewhere, e.g. group-limited routing) only the sort / counts / tiles are produced. ``want_host=False``
+    leaves out the copy of the group sizes to the host (inference has no use for it)."""
     T, E = logits.shape
     if not logits.is_cuda or E > 256 or k > 16:
         return moe_route_ref(logits, k, bias, sigmoid, norm, scale, tope)
@@ -215,7 +217,7 @@ def moe_route(logits: torch.Tensor, k: int, bias: Optional[torch.Tensor] = None,
                          tope_.data_ptr(), counts.data_ptr(), offs.data_ptr(), order.data_ptr(), token_of.data_ptr(),
                          inv.data_ptr(), row_tiles.data_ptr(), num_rt.data_ptr(), max_rt, ws.data_ptr(), _s())
     _lib.check(rc, "ab2_moe_route")
-    return Routing(tope_, topw, probs, counts, offs, order, token_of, inv, row_tiles, num_rt, k)
+    return Routing(tope_, topw, probs, counts, offs, order, token_of, inv, row_tiles, num_rt, k, want_host)
 
 
 def grouped_gemm_rt(x: torch.Tensor, w: torch.Tensor, routing: Routing, b_mn: bool = False) -> torch.Tensor:

@@ -74,6 +74,14 @@ def lib_path() -> Path:
     return _LIB_PATH
 
 
+def use_library(path) -> None:
+    """Loads the kernels from another build of the library (before the first op)."""
+    global _LIB_PATH
+    if _LIB is not None and Path(path) != _LIB_PATH:
+        raise KernelLibraryError("the kernel library is already loaded")
+    _LIB_PATH = Path(path)
+
+
 def available() -> bool:
     """True when CUDA is usable and the kernel library can be loaded."""
     if not torch.cuda.is_available():
