@@ -1,0 +1,552 @@
+// Elementwise, norm, convolution and small-product kernels of mixer stacks (bf16 or fp32 activations, fp32 residual
+// stream, norm weights and states): grouped sandwich norms, whole-projection q / k norms fused with the cache append,
+// causal convolutions with carried tails, xIELU, SiLU gate, expert combine, capped logits, and a plain grouped product
+// for 32-bit experts and odd sizes.
+#include "mixer_common.cuh"
+
+namespace ab2 {
+
+// ------------------------------------------------------------------ grouped norms
+// How a CTA shares `groups` equal parts of a row: with no more groups than warps every group gets wpg warps (its
+// elements interleaved over their lanes), otherwise a warp walks several groups. Sums have a fixed order.
+struct GroupMap {
+  int groups, part, wpg, warp, lane, nw;
+  __device__ GroupMap(int groups_, int H) : groups(groups_), part(H / groups_) {
+    warp = threadIdx.x >> 5;
+    lane = threadIdx.x & 31;
+    nw = blockDim.x >> 5;
+    wpg = groups <= nw ? nw / groups : 1;
+  }
+  __device__ int first() const { return groups <= nw ? warp / wpg : warp; }
+  __device__ int step() const { return groups <= nw ? groups : nw; }       // one group per warp, or every nw-th
+  __device__ int offset() const { return groups <= nw ? (warp % wpg) * 32 + lane : lane; }
+  __device__ int stride() const { return wpg * 32; }
+  __device__ int sub() const { return groups <= nw ? warp % wpg : 0; }
+  __device__ float total(const float* sums, int g) const {
+    float s = 0.f;
+    for (int i = 0; i < wpg; ++i) s += sums[g * wpg + i];
+    return s;
+  }
+};
+
+// Row by row: v = h (or the fp32 residual taken from an embedding row); with w_post: resid += norm(h) * w_post;
+// then x = norm(resid) * w_next. The row stays in shared memory between the passes.
+template <typename T, int V>
+__global__ void sandwich_norm_kernel(const int* __restrict__ ids, const T* __restrict__ table, int vocab, const T* __restrict__ h,
+                                     long long ldh, const float* __restrict__ w_post, float* __restrict__ resid,
+                                     const float* __restrict__ w_next, T* __restrict__ x, int H, int groups, float eps) {
+  extern __shared__ __align__(16) float srow[];       // [H] values, then the partial sums
+  pdl_wait();
+  pdl_trigger();
+  const GroupMap gm(groups, H);
+  float* sums = srow + ((H + 3) & ~3);
+  float* sums2 = sums + groups * gm.wpg;
+  const int row = blockIdx.x;
+  float* rr = resid + (size_t)row * H;
+  const int pv = gm.part / V;
+  if (h != nullptr) {
+    const T* hr = h + (size_t)row * ldh;
+    for (int g = gm.first(); g < groups; g += gm.step()) {
+      float ss = 0.f;
+      for (int i = gm.offset(); i < pv; i += gm.stride()) {
+        float v[V];
+        ldv<V>(hr + g * gm.part + i * V, v);
+        for (int e = 0; e < V; ++e) ss += v[e] * v[e];
+        stv<V>(srow + g * gm.part + i * V, v);
+      }
+      ss = warp_sum(ss);
+      if (gm.lane == 0) sums[g * gm.wpg + gm.sub()] = ss;
+    }
+    __syncthreads();
+  }
+  int id = 0;
+  if (h == nullptr) {
+    id = ids[row];
+    id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+  }
+  for (int g = gm.first(); g < groups; g += gm.step()) {
+    const float rstd = h != nullptr ? 1.f / sqrtf(gm.total(sums, g) / gm.part + eps) : 0.f;
+    float ss = 0.f;
+    for (int i = gm.offset(); i < pv; i += gm.stride()) {
+      const int c = g * gm.part + i * V;
+      float v[V];
+      if (h != nullptr) {
+        float r[V], w[V];
+        ldv<V>(srow + c, v);
+        ldv<V>(rr + c, r);
+        ldv<V>(w_post + c, w);
+        for (int e = 0; e < V; ++e) v[e] = r[e] + v[e] * rstd * w[e];
+      } else {
+        ldv<V>(table + (size_t)id * H + c, v);
+      }
+      stv<V>(rr + c, v);
+      stv<V>(srow + c, v);
+      for (int e = 0; e < V; ++e) ss += v[e] * v[e];
+    }
+    ss = warp_sum(ss);
+    if (gm.lane == 0) sums2[g * gm.wpg + gm.sub()] = ss;
+  }
+  __syncthreads();
+  for (int g = gm.first(); g < groups; g += gm.step()) {
+    const float rstd = 1.f / sqrtf(gm.total(sums2, g) / gm.part + eps);
+    for (int i = gm.offset(); i < pv; i += gm.stride()) {
+      const int c = g * gm.part + i * V;
+      float v[V], w[V];
+      ldv<V>(srow + c, v);
+      ldv<V>(w_next + c, w);
+      for (int e = 0; e < V; ++e) v[e] = v[e] * rstd * w[e];
+      stv<V>(x + (size_t)row * H + c, v);
+    }
+  }
+}
+
+// out = norm(y * silu(z)) * w in groups; y fp32.
+template <typename T, int V>
+__global__ void gated_norm_kernel(const float* __restrict__ y, const T* __restrict__ z, long long ldz, const float* __restrict__ w,
+                                  T* __restrict__ out, int C, int groups, float eps) {
+  extern __shared__ __align__(16) float srow[];
+  pdl_wait();
+  pdl_trigger();
+  const GroupMap gm(groups, C);
+  float* sums = srow + ((C + 3) & ~3);
+  const int row = blockIdx.x;
+  const int pv = gm.part / V;
+  for (int g = gm.first(); g < groups; g += gm.step()) {
+    float ss = 0.f;
+    for (int i = gm.offset(); i < pv; i += gm.stride()) {
+      const int c = g * gm.part + i * V;
+      float a[V], b[V];
+      ldv<V>(y + (size_t)row * C + c, a);
+      ldv<V>(z + (size_t)row * ldz + c, b);
+      for (int e = 0; e < V; ++e) {
+        a[e] *= siluf(b[e]);
+        ss += a[e] * a[e];
+      }
+      stv<V>(srow + c, a);
+    }
+    ss = warp_sum(ss);
+    if (gm.lane == 0) sums[g * gm.wpg + gm.sub()] = ss;
+  }
+  __syncthreads();
+  for (int g = gm.first(); g < groups; g += gm.step()) {
+    const float rstd = 1.f / sqrtf(gm.total(sums, g) / gm.part + eps);
+    for (int i = gm.offset(); i < pv; i += gm.stride()) {
+      const int c = g * gm.part + i * V;
+      float a[V], b[V];
+      ldv<V>(srow + c, a);
+      ldv<V>(w + c, b);
+      for (int e = 0; e < V; ++e) a[e] = a[e] * rstd * b[e];
+      stv<V>(out + (size_t)row * C + c, a);
+    }
+  }
+}
+
+static inline int norm_threads(int H) { return H <= 1024 ? 128 : (H <= 4096 ? 256 : 512); }
+static inline size_t norm_smem(int H, int groups, int threads) {
+  const int nw = threads / 32;
+  const int per = groups <= nw ? groups * (nw / groups) : groups;
+  return (size_t)(((H + 3) & ~3) + 2 * per) * 4;
+}
+
+// ------------------------------------------------------------------ q / k norm + cache append
+template <typename T, int V>
+__global__ void qk_norm_append_kernel(const T* __restrict__ qkv, long long ld, const float* __restrict__ wq, const float* __restrict__ wk,
+                                      const int* __restrict__ slots, T* __restrict__ q, T* __restrict__ kc, T* __restrict__ vc, int nq, int nk,
+                                      int nv, float eps) {
+  __shared__ float red[2][32];
+  pdl_wait();
+  pdl_trigger();
+  const int row = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nw = blockDim.x >> 5;
+  const T* src = qkv + (size_t)row * ld;
+  float sq = 0.f, sk = 0.f;
+  for (int i = tid * V; i < nq + nk; i += blockDim.x * V) {
+    float v[V];
+    ldv<V>(src + i, v);
+    float s = 0.f;
+    for (int e = 0; e < V; ++e) s += v[e] * v[e];
+    if (i < nq) sq += s; else sk += s;
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+  __syncthreads();
+  sq = sk = 0.f;
+  for (int w = 0; w < nw; ++w) { sq += red[0][w]; sk += red[1][w]; }
+  const float rq = 1.f / sqrtf(sq / nq + eps), rk = 1.f / sqrtf(sk / nk + eps);
+  const int slot = slots[row];
+  for (int i = tid * V; i < nq + nk + nv; i += blockDim.x * V) {
+    float v[V], w[V];
+    ldv<V>(src + i, v);
+    if (i < nq) {
+      ldv<V>(wq + i, w);
+      for (int e = 0; e < V; ++e) v[e] = v[e] * rq * w[e];
+      stv<V>(q + (size_t)row * nq + i, v);
+    } else if (slot >= 0) {
+      if (i < nq + nk) {
+        ldv<V>(wk + i - nq, w);
+        for (int e = 0; e < V; ++e) v[e] = v[e] * rk * w[e];
+        stv<V>(kc + (size_t)slot * nk + i - nq, v);
+      } else {
+        stv<V>(vc + (size_t)slot * nv + i - nq - nk, v);
+      }
+    }
+  }
+}
+
+// ------------------------------------------------------------------ causal convolution
+// Single-token rows: the window is the slot's tail plus the row; the tail moves on by one.
+template <typename T>
+__global__ void conv_decode_kernel(const T* __restrict__ x, long long ld, const float* __restrict__ bin, const float* __restrict__ w,
+                                   const float* __restrict__ bias, int silu, const int* __restrict__ start, const int* __restrict__ state,
+                                   float* __restrict__ tail, T* __restrict__ out, int C, int K) {
+  pdl_wait();
+  pdl_trigger();
+  const int row = blockIdx.y, c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (c >= C) return;
+  const int slot = state[row];
+  if (slot < 0) { stf(out + (size_t)row * C + c, 0.f); return; }
+  const bool fresh = start[row] <= 0;
+  float* tl = tail + ((size_t)slot * C + c) * (K - 1);
+  const float cur = ldf(x + (size_t)row * ld + c) + (bin ? bin[c] : 0.f);
+  float acc = bias[c] + w[(size_t)c * K + K - 1] * cur;
+  for (int m = 0; m < K - 1; ++m) acc += w[(size_t)c * K + m] * (fresh ? 0.f : tl[m]);
+  for (int m = 0; m + 1 < K - 1; ++m) tl[m] = fresh ? 0.f : tl[m + 1];
+  if (K > 1) tl[K - 2] = cur;
+  stf(out + (size_t)row * C + c, silu ? siluf(acc) : acc);
+}
+
+// Portions: a CTA walks the rows of one block (64 rows of one entry) for 128 channels, the last inputs in registers.
+// KT = taps (1..8), 0: any number, inputs re-read.
+template <typename T, int KT>
+__global__ void conv_prefill_kernel(const T* __restrict__ x, long long ld, const float* __restrict__ bin, const float* __restrict__ w,
+                                    const float* __restrict__ bias, int silu, const int* __restrict__ cu, const int* __restrict__ start,
+                                    const int* __restrict__ state, const int4* __restrict__ blocks, const float* __restrict__ tail,
+                                    T* __restrict__ out, int C, int Kdyn) {
+  const int K = KT > 0 ? KT : Kdyn;
+  const int4 blk = blocks[blockIdx.y];
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (c >= C) return;
+  const int e = blk.x, r0 = blk.y, n = blk.z, first = cu[e];
+  const int slot = state[e];
+  const bool fresh = start[e] <= 0;
+  const float bi = bin ? bin[c] : 0.f, b0 = bias[c];
+  const float* tl = tail + ((size_t)slot * C + c) * (K - 1);
+  auto at = [&](int r) -> float {                       // input at row r of this entry (before its first row: the tail)
+    if (r >= first) return ldf(x + (size_t)r * ld + c) + bi;
+    const int m = K - 1 + (r - first);
+    return (fresh || m < 0) ? 0.f : tl[m];
+  };
+  if constexpr (KT > 0) {
+    float wv[KT], win[KT];
+#pragma unroll
+    for (int j = 0; j < KT; ++j) wv[j] = w[(size_t)c * KT + j];
+#pragma unroll
+    for (int j = 0; j < KT - 1; ++j) win[j + 1] = at(r0 - (KT - 1) + j);
+    for (int i = 0; i < n; ++i) {
+#pragma unroll
+      for (int j = 0; j < KT - 1; ++j) win[j] = win[j + 1];
+      win[KT - 1] = ldf(x + (size_t)(r0 + i) * ld + c) + bi;
+      float acc = b0;
+#pragma unroll
+      for (int j = 0; j < KT; ++j) acc += wv[j] * win[j];
+      stf(out + (size_t)(r0 + i) * C + c, silu ? siluf(acc) : acc);
+    }
+  } else {
+    for (int i = 0; i < n; ++i) {
+      float acc = b0;
+      for (int j = 0; j < K; ++j) acc += w[(size_t)c * K + j] * at(r0 + i - (K - 1) + j);
+      stf(out + (size_t)(r0 + i) * C + c, silu ? siluf(acc) : acc);
+    }
+  }
+}
+
+// After the convolution: the last K - 1 inputs of every portion become its slot's tail.
+template <typename T>
+__global__ void conv_tail_kernel(const T* __restrict__ x, long long ld, const float* __restrict__ bin, const int* __restrict__ cu,
+                                 const int* __restrict__ start, const int* __restrict__ state, int n_dec, float* __restrict__ tail, int C, int K) {
+  const int e = n_dec + blockIdx.y, c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (c >= C) return;
+  const int slot = state[e];
+  if (slot < 0) return;
+  const int r0 = cu[e], L = cu[e + 1] - r0;
+  const bool fresh = start[e] <= 0;
+  float* tl = tail + ((size_t)slot * C + c) * (K - 1);
+  for (int m = 0; m < K - 1; ++m) {                     // ascending: a slot entry is read before it is overwritten
+    const int r = L - (K - 1) + m;
+    tl[m] = r >= 0 ? ldf(x + (size_t)(r0 + r) * ld + c) + (bin ? bin[c] : 0.f) : (fresh ? 0.f : tl[m + L]);
+  }
+}
+
+// ------------------------------------------------------------------ activations, combine, cap
+template <typename T, int V>
+__global__ void xielu_kernel(const T* __restrict__ x, long long ld, const float* __restrict__ pq, T* __restrict__ out, long long total, int C) {
+  pdl_wait();
+  pdl_trigger();
+  const float sp = softplusf(pq[0]), sq = 0.5f + softplusf(pq[1]);
+  const int cv = C / V;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / cv;
+    const int c = (int)(i - r * cv) * V;
+    float v[V];
+    ldv<V>(x + r * ld + c, v);
+    for (int e = 0; e < V; ++e) v[e] = 0.5f * v[e] + (v[e] > 0.f ? sp * v[e] * v[e] : sq * (expm1f(v[e]) - v[e]));
+    stv<V>(out + r * C + c, v);
+  }
+}
+
+template <typename T, int V>
+__global__ void glu_silu_kernel(const T* __restrict__ gu, long long ld, T* __restrict__ out, long long total, int I) {
+  pdl_wait();
+  pdl_trigger();
+  const int cv = I / V;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / cv;
+    const int c = (int)(i - r * cv) * V;
+    float g[V], u[V];
+    ldv<V>(gu + r * ld + c, g);
+    ldv<V>(gu + r * ld + I + c, u);
+    for (int e = 0; e < V; ++e) g[e] = siluf(g[e]) * u[e];
+    stv<V>(out + r * I + c, g);
+  }
+}
+
+template <typename T, int V>
+__global__ void expert_combine_kernel(const T* __restrict__ y, const int* __restrict__ inv, const float* __restrict__ topw, T* __restrict__ out,
+                                      long long total, int k, int H, int n_rows) {
+  pdl_wait();
+  pdl_trigger();
+  const int hv = H / V;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long t = i / hv;
+    const int c = (int)(i - t * hv) * V;
+    float acc[V];
+    for (int e = 0; e < V; ++e) acc[e] = 0.f;
+    for (int s = 0; s < k; ++s) {
+      const int r = inv[t * k + s];
+      if (r < 0 || r >= n_rows) continue;
+      const float w = topw[t * k + s];
+      float v[V];
+      ldv<V>(y + (size_t)r * H + c, v);
+      for (int e = 0; e < V; ++e) acc[e] += w * v[e];
+    }
+    stv<V>(out + t * H + c, acc);
+  }
+}
+
+__global__ void softcap_kernel(float* __restrict__ z, long long ld, int R, int C, float cap, float inv_cap) {
+  pdl_wait();
+  pdl_trigger();
+  const int r = blockIdx.y;
+  for (int c = blockIdx.x * blockDim.x + threadIdx.x; c < C; c += gridDim.x * blockDim.x) {
+    float* p = z + (size_t)r * ld + c;
+    *p = cap * tanhf(*p * inv_cap);
+  }
+}
+
+// ------------------------------------------------------------------ plain grouped product
+// 128 x 64 output tile per CTA, fp32 FMA; rows of `tiles` are (expert, first row, valid rows, -).
+template <typename T>
+__global__ void __launch_bounds__(256)
+grouped_plain_kernel(const T* __restrict__ x, const T* __restrict__ w, T* __restrict__ out, const int4* __restrict__ tiles,
+                     const int* __restrict__ n_tiles, int N, int K) {
+  if ((int)blockIdx.x >= *n_tiles) return;
+  __shared__ float sa[16][132], sb[16][68];
+  const int4 t = tiles[blockIdx.x];
+  const int n0 = blockIdx.y * 64, tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  const T* we = w + (size_t)t.x * N * K;
+  float acc[8][4] = {};
+  for (int k0 = 0; k0 < K; k0 += 16) {
+    for (int i = threadIdx.x; i < 128 * 16; i += 256) {
+      const int r = i >> 4, k = i & 15;
+      sa[k][r] = (r < t.z && k0 + k < K) ? ldf(x + (size_t)(t.y + r) * K + k0 + k) : 0.f;
+    }
+    for (int i = threadIdx.x; i < 64 * 16; i += 256) {
+      const int n = i >> 4, k = i & 15;
+      sb[k][n] = (n0 + n < N && k0 + k < K) ? ldf(we + (size_t)(n0 + n) * K + k0 + k) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 16; ++k) {
+      float a[8], b[4];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) a[i] = sa[k][ty * 8 + i];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) b[j] = sb[k][tx * 4 + j];
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] += a[i] * b[j];
+    }
+    __syncthreads();
+  }
+  for (int i = 0; i < 8; ++i)
+    for (int j = 0; j < 4; ++j)
+      if (ty * 8 + i < t.z && n0 + tx * 4 + j < N) stf(out + (size_t)(t.y + ty * 8 + i) * N + n0 + tx * 4 + j, acc[i][j]);
+}
+
+static inline int flat_grid(long long n) {
+  const long long g = (n + 255) / 256;
+  return (int)(g < 148 * 16 ? g : 148 * 16);
+}
+
+}  // namespace ab2
+
+// T = __nv_bfloat16 (dt 0) or float (dt 1); V = 4 when every row start and length allows it.
+#define AB2_TYPED(dt, vec, ...)                                                                              \
+  do {                                                                                                       \
+    if ((dt) == 0) {                                                                                         \
+      using T = __nv_bfloat16;                                                                               \
+      if (vec) { constexpr int V = 4; __VA_ARGS__; } else { constexpr int V = 1; __VA_ARGS__; }                 \
+    } else {                                                                                                 \
+      using T = float;                                                                                       \
+      if (vec) { constexpr int V = 4; __VA_ARGS__; } else { constexpr int V = 1; __VA_ARGS__; }                 \
+    }                                                                                                        \
+  } while (0)
+#define AB2_DONE return cudaGetLastError() == cudaSuccess ? 0 : 1
+
+extern "C" {
+using namespace ab2;
+
+// resid [R, H] fp32, x [R, H]. With h: resid += norm(h) * w_post first; without: resid = table[ids].
+int ab2_sandwich_norm(const int* ids, const void* table, int vocab, const void* h, long long ldh, const float* w_post, float* resid,
+                      const float* w_next, void* x, int R, int H, int groups, float eps, int dt, void* stream) {
+  if (R <= 0) return 0;
+  if (groups < 1 || H % groups) return 10;
+  const int th = norm_threads(H);
+  const size_t smem = norm_smem(H, groups, th);
+  if (smem > 200 * 1024) return 11;
+  const int eb = dt == 0 ? 2 : 4;
+  const bool vec = (H / groups) % 4 == 0 && ldh % 4 == 0 && aligned_to(h ? h : table, 4 * eb) && aligned_to(x, 4 * eb);
+  AB2_TYPED(dt, vec, {
+    auto kern = sandwich_norm_kernel<T, V>;
+    static ab2host::DevState st;
+    if (ab2host::prepare_launch(kern, 200 * 1024, st, nullptr)) return 12;
+    launch_pdl(kern, dim3(R), dim3(th), smem, (cudaStream_t)stream, ids, (const T*)table, vocab, (const T*)h, ldh, w_post, resid, w_next, (T*)x, H,
+               groups, eps);
+  });
+  AB2_DONE;
+}
+
+int ab2_gated_group_norm(const float* y, const void* z, long long ldz, const float* w, void* out, int R, int C, int groups, float eps, int dt,
+                         void* stream) {
+  if (R <= 0) return 0;
+  if (groups < 1 || C % groups) return 10;
+  const int th = norm_threads(C);
+  const size_t smem = norm_smem(C, groups, th);
+  if (smem > 200 * 1024) return 11;
+  const int eb = dt == 0 ? 2 : 4;
+  const bool vec = (C / groups) % 4 == 0 && ldz % 4 == 0 && aligned_to(z, 4 * eb);
+  AB2_TYPED(dt, vec, {
+    auto kern = gated_norm_kernel<T, V>;
+    static ab2host::DevState st;
+    if (ab2host::prepare_launch(kern, 200 * 1024, st, nullptr)) return 12;
+    launch_pdl(kern, dim3(R), dim3(th), smem, (cudaStream_t)stream, y, (const T*)z, ldz, w, (T*)out, C, groups, eps);
+  });
+  AB2_DONE;
+}
+
+int ab2_qk_norm_append(const void* qkv, long long ld, const float* wq, const float* wk, const int* slots, void* q, void* kc, void* vc, int R,
+                       int nq, int nk, int nv, float eps, int dt, void* stream) {
+  if (R <= 0) return 0;
+  const int eb = dt == 0 ? 2 : 4;
+  const bool vec = nq % 4 == 0 && nk % 4 == 0 && nv % 4 == 0 && ld % 4 == 0 && aligned_to(qkv, 4 * eb);
+  AB2_TYPED(dt, vec, {
+    launch_pdl(qk_norm_append_kernel<T, V>, dim3(R), dim3(256), 0, (cudaStream_t)stream, (const T*)qkv, ld, wq, wk, slots, (T*)q, (T*)kc, (T*)vc, nq,
+               nk, nv, eps);
+  });
+  AB2_DONE;
+}
+
+// Rows of the first n_dec entries are single tokens; `blocks` lists the 64-row blocks of the other entries.
+int ab2_causal_conv(const void* x, long long ld, const float* bin, const float* w, const float* bias, int silu, const int* cu, const int* start,
+                    const int* state, const void* blocks, int nb, int n_dec, int n_entries, float* tail, void* out, int C, int K, int dt,
+                    void* stream) {
+  if (C <= 0 || K < 1) return 10;
+  cudaStream_t s = (cudaStream_t)stream;
+  const int gx = (C + 127) / 128;
+  if (n_dec > 0) {
+    if (n_dec > 65535) return 11;
+    if (dt == 0)
+      launch_pdl(conv_decode_kernel<__nv_bfloat16>, dim3(gx, n_dec), dim3(128), 0, s, (const __nv_bfloat16*)x, ld, bin, w, bias, silu, start, state,
+                 tail, (__nv_bfloat16*)out, C, K);
+    else
+      launch_pdl(conv_decode_kernel<float>, dim3(gx, n_dec), dim3(128), 0, s, (const float*)x, ld, bin, w, bias, silu, start, state, tail,
+                 (float*)out, C, K);
+  }
+  if (nb > 0) {
+    if (nb > 65535 || n_entries - n_dec > 65535) return 11;
+#define AB2_CONV(TT, KK) conv_prefill_kernel<TT, KK><<<dim3(gx, nb), 128, 0, s>>>((const TT*)x, ld, bin, w, bias, silu, cu, start, state, \
+                                                                              (const int4*)blocks, tail, (TT*)out, C, K)
+#define AB2_CONV_K(TT)                                                                         \
+  switch (K) {                                                                                 \
+    case 1: AB2_CONV(TT, 1); break;                                                            \
+    case 2: AB2_CONV(TT, 2); break;                                                            \
+    case 3: AB2_CONV(TT, 3); break;                                                            \
+    case 4: AB2_CONV(TT, 4); break;                                                            \
+    default: AB2_CONV(TT, 0);                                                                  \
+  }
+    if (dt == 0) { AB2_CONV_K(__nv_bfloat16) } else { AB2_CONV_K(float) }
+#undef AB2_CONV_K
+#undef AB2_CONV
+    if (K > 1) {
+      if (dt == 0)
+        conv_tail_kernel<__nv_bfloat16><<<dim3(gx, n_entries - n_dec), 128, 0, s>>>((const __nv_bfloat16*)x, ld, bin, cu, start, state, n_dec, tail, C, K);
+      else
+        conv_tail_kernel<float><<<dim3(gx, n_entries - n_dec), 128, 0, s>>>((const float*)x, ld, bin, cu, start, state, n_dec, tail, C, K);
+    }
+  }
+  AB2_DONE;
+}
+
+int ab2_xielu(const void* x, long long ld, const float* pq, void* out, int R, int C, int dt, void* stream) {
+  if (R <= 0) return 0;
+  const int eb = dt == 0 ? 2 : 4;
+  const bool vec = C % 4 == 0 && ld % 4 == 0 && aligned_to(x, 4 * eb);
+  AB2_TYPED(dt, vec, {
+    const long long n = (long long)R * (C / V);
+    launch_pdl(xielu_kernel<T, V>, dim3(flat_grid(n)), dim3(256), 0, (cudaStream_t)stream, (const T*)x, ld, pq, (T*)out, n, C);
+  });
+  AB2_DONE;
+}
+
+int ab2_glu_silu(const void* gu, long long ld, void* out, int R, int I, int dt, void* stream) {
+  if (R <= 0) return 0;
+  const int eb = dt == 0 ? 2 : 4;
+  const bool vec = I % 4 == 0 && ld % 4 == 0 && aligned_to(gu, 4 * eb);
+  AB2_TYPED(dt, vec, {
+    const long long n = (long long)R * (I / V);
+    launch_pdl(glu_silu_kernel<T, V>, dim3(flat_grid(n)), dim3(256), 0, (cudaStream_t)stream, (const T*)gu, ld, (T*)out, n, I);
+  });
+  AB2_DONE;
+}
+
+int ab2_expert_combine(const void* y, const int* inv, const float* topw, void* out, int T_, int k, int H, int dt, void* stream) {
+  if (T_ <= 0) return 0;
+  AB2_TYPED(dt, H % 4 == 0, {
+    const long long n = (long long)T_ * (H / V);
+    launch_pdl(expert_combine_kernel<T, V>, dim3(flat_grid(n)), dim3(256), 0, (cudaStream_t)stream, (const T*)y, inv, topw, (T*)out, n, k, H, T_ * k);
+  });
+  AB2_DONE;
+}
+
+int ab2_softcap(float* z, long long ld, int R, int C, float cap, void* stream) {
+  if (R <= 0) return 0;
+  if (R > 65535 || cap <= 0.f) return 10;
+  const int gx = (C + 1023) / 1024;
+  launch_pdl(softcap_kernel, dim3(gx < 64 ? gx : 64, R), dim3(256), 0, (cudaStream_t)stream, z, ld, R, C, cap, 1.f / cap);
+  AB2_DONE;
+}
+
+int ab2_grouped_plain(const void* x, const void* w, void* out, const void* tiles, const int* n_tiles, int max_tiles, int N, int K, int dt,
+                      void* stream) {
+  if (max_tiles <= 0) return 0;
+  if ((N + 63) / 64 > 65535) return 10;
+  const dim3 grid(max_tiles, (N + 63) / 64);
+  if (dt == 0)
+    grouped_plain_kernel<__nv_bfloat16><<<grid, 256, 0, (cudaStream_t)stream>>>((const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (__nv_bfloat16*)out,
+                                                                                (const int4*)tiles, n_tiles, N, K);
+  else
+    grouped_plain_kernel<float><<<grid, 256, 0, (cudaStream_t)stream>>>((const float*)x, (const float*)w, (float*)out, (const int4*)tiles, n_tiles, N, K);
+  AB2_DONE;
+}
+}

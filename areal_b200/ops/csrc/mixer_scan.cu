@@ -1,0 +1,336 @@
+// Recurrences of mixer stacks on per-request state slots: the RG-LRU (block-diagonal gates on tensor cores, then a
+// blocked linear scan) and the Mamba-2 state update. Gates, decays and states are fp32 throughout.
+#include "mixer_common.cuh"
+
+namespace ab2 {
+
+// ------------------------------------------------------------------ RG-LRU gates
+// One CTA: 64 rows x 32 channels of one block of the block-diagonal gate matrices, both gates at once (64 product
+// columns: 32 of r, 32 of i), so the thread that holds r of a channel also holds its i. The epilogue turns the two
+// logits into the decay a = exp(-8 r softplus(lam)) and the input sqrt(1 - a^2) i u, and either stores both for the
+// scan or (single-token rows) advances the state at once.
+constexpr int GT_R = 64, GT_C = 32, GT_K = 64;
+
+struct GateEpi {
+  const float *gb, *lam, *yb;
+  const int *start, *state;
+  float *S, *a, *x;
+  int W, bs, nblk;
+};
+
+template <typename T, bool DECODE>
+__device__ __forceinline__ void gate_epilogue(const GateEpi& p, const T* u, const T* y, long long ldy, T* out, int row, int ch, float zr, float zi) {
+  const float r = sigmoidf(zr + p.gb[ch]), i = sigmoidf(zi + p.gb[p.W + ch]);
+  const float la = -8.f * r * softplusf(p.lam[ch]);
+  const float a = expf(la);
+  const float xin = sqrtf(-expm1f(2.f * la)) * i * ldf(u + (size_t)row * p.W + ch);
+  const size_t o = (size_t)row * p.W + ch;
+  if constexpr (DECODE) {
+    const int slot = p.state[row];
+    if (slot < 0) { stf(out + o, 0.f); return; }
+    float* s = p.S + (size_t)slot * p.W + ch;
+    const float h = (p.start[row] > 0 ? a * *s : 0.f) + xin;
+    *s = h;
+    stf(out + o, h * gelu_tanhf(ldf(y + (size_t)row * ldy + ch) + p.yb[ch]));
+  } else {
+    p.a[o] = a;
+    p.x[o] = xin;
+  }
+}
+
+template <typename T, bool DECODE>
+__global__ void __launch_bounds__(128)
+rglru_gate_kernel(const T* __restrict__ u, const T* __restrict__ y, long long ldy, const T* __restrict__ gw, GateEpi p, T* __restrict__ out, int R) {
+  constexpr bool MMA = sizeof(T) == 2;
+  constexpr int LD = MMA ? GT_K + 8 : GT_K + 1;          // padded rows: no bank conflicts on fragment reads
+  __shared__ __align__(16) T sA[GT_R * LD];
+  __shared__ __align__(16) T sB[2 * GT_C * LD];
+  pdl_wait();
+  pdl_trigger();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int cpb = (p.bs + GT_C - 1) / GT_C;              // channel tiles per block
+  const int blk = blockIdx.x / cpb, c0 = (blockIdx.x % cpb) * GT_C, r0 = blockIdx.y * GT_R;
+  const T zero = T(0.f);
+  float acc[8][4];
+#pragma unroll
+  for (int i = 0; i < 8; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+  const bool vec = MMA && p.bs % 8 == 0 && p.W % 8 == 0;
+  for (int k0 = 0; k0 < p.bs; k0 += GT_K) {
+    if (vec) {
+      for (int i = tid; i < GT_R * (GT_K / 8); i += 128) {
+        const int r = i / (GT_K / 8), k = (i % (GT_K / 8)) * 8;
+        uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        if (r0 + r < R && k0 + k < p.bs) v = *reinterpret_cast<const uint4*>(u + (size_t)(r0 + r) * p.W + blk * p.bs + k0 + k);
+        *reinterpret_cast<uint4*>(sA + r * LD + k) = v;
+        const int g = r >> 5, c = c0 + (r & 31);          // 2 x 32 weight rows: as many as there are token rows
+        uint4 w = make_uint4(0u, 0u, 0u, 0u);
+        if (c < p.bs && k0 + k < p.bs) w = *reinterpret_cast<const uint4*>(gw + (((size_t)g * p.nblk + blk) * p.bs + c) * p.bs + k0 + k);
+        *reinterpret_cast<uint4*>(sB + r * LD + k) = w;
+      }
+    } else {
+      for (int i = tid; i < GT_R * GT_K; i += 128) {
+        const int r = i / GT_K, k = i % GT_K;
+        sA[r * LD + k] = (r0 + r < R && k0 + k < p.bs) ? u[(size_t)(r0 + r) * p.W + blk * p.bs + k0 + k] : zero;
+        const int g = r >> 5, c = c0 + (r & 31);
+        sB[r * LD + k] = (c < p.bs && k0 + k < p.bs) ? gw[(((size_t)g * p.nblk + blk) * p.bs + c) * p.bs + k0 + k] : zero;
+      }
+    }
+    __syncthreads();
+    if constexpr (MMA) {
+      const int gq = lane >> 2, tq = lane & 3;
+      const uint32_t* A = reinterpret_cast<const uint32_t*>(sA);
+      const uint32_t* B = reinterpret_cast<const uint32_t*>(sB);
+      constexpr int LW = LD / 2;
+#pragma unroll
+      for (int kk = 0; kk < GT_K / 16; ++kk) {
+        const int ar = (warp * 16 + gq) * LW + kk * 8 + tq;
+        const uint32_t a0 = A[ar], a1 = A[ar + 8 * LW], a2 = A[ar + 4], a3 = A[ar + 8 * LW + 4];
+#pragma unroll
+        for (int t = 0; t < 8; ++t) {
+          const int br = (t * 8 + gq) * LW + kk * 8 + tq;
+          asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                       : "+f"(acc[t][0]), "+f"(acc[t][1]), "+f"(acc[t][2]), "+f"(acc[t][3])
+                       : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(B[br]), "r"(B[br + 4]));
+        }
+      }
+    } else {
+      // thread = 4 rows x (4 channels of r and the same 4 of i): channels tx + 8 j
+      const int tx = tid & 7, ty = tid >> 3;
+      for (int k = 0; k < GT_K; ++k) {
+        float av[4], bv[8];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) av[i] = ldf(sA + (ty * 4 + i) * LD + k);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) bv[j] = ldf(sB + (tx + 8 * j) * LD + k);
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+#pragma unroll
+          for (int i = 0; i < 4; ++i) acc[j][i] += av[i] * bv[j];
+      }
+    }
+    __syncthreads();
+  }
+  if constexpr (MMA) {
+    const int gq = lane >> 2, tq = lane & 3;
+#pragma unroll
+    for (int t = 0; t < 4; ++t)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int row = r0 + warp * 16 + gq + (j >> 1) * 8, c = c0 + t * 8 + tq * 2 + (j & 1);
+        if (row < R && c < p.bs) gate_epilogue<T, DECODE>(p, u, y, ldy, out, row, blk * p.bs + c, acc[t][j], acc[t + 4][j]);
+      }
+  } else {
+    const int tx = tid & 7, ty = tid >> 3;
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int row = r0 + ty * 4 + i, c = c0 + tx + 8 * j;
+        if (row < R && c < p.bs) gate_epilogue<T, DECODE>(p, u, y, ldy, out, row, blk * p.bs + c, acc[j][i], acc[j + 4][i]);
+      }
+  }
+}
+
+// Blocked scan h = a h + x over the 64-row blocks of every portion: per block the product of a and the state from
+// zero; the states between blocks; then every block from its true start, gated on the way out. Row indices of
+// `blocks` count from the first row of the step, a / x / y / out from row0.
+__global__ void __launch_bounds__(128)
+lru_block_kernel(const float* __restrict__ a, const float* __restrict__ x, const int4* __restrict__ blocks, int row0, float* __restrict__ carry, int nb,
+                 int W) {
+  const int4 b = blocks[blockIdx.y];
+  const int c = blockIdx.x * 128 + threadIdx.x;
+  if (c >= W) return;
+  float A = 1.f, h = 0.f;
+  const size_t o = (size_t)(b.y - row0) * W + c;
+#pragma unroll 8
+  for (int t = 0; t < b.z; ++t) {
+    const float at = a[o + (size_t)t * W];
+    h = at * h + x[o + (size_t)t * W];
+    A *= at;
+  }
+  carry[(size_t)blockIdx.y * W + c] = A;
+  carry[((size_t)nb + blockIdx.y) * W + c] = h;
+}
+
+__global__ void __launch_bounds__(128)
+lru_carry_kernel(const int4* __restrict__ blocks, const int* __restrict__ start, const int* __restrict__ state, float* __restrict__ S,
+                 float* __restrict__ carry, int nb, int W) {
+  const int c = blockIdx.x * 128 + threadIdx.x;
+  if (c >= W) return;
+  float h = 0.f;
+#pragma unroll 4
+  for (int k = 0; k < nb; ++k) {
+    const int4 b = blocks[k];
+    if (b.w) h = start[b.x] > 0 ? S[(size_t)state[b.x] * W + c] : 0.f;
+    const float A = carry[(size_t)k * W + c], x = carry[((size_t)nb + k) * W + c];
+    carry[(size_t)k * W + c] = h;                        // state before this block
+    h = A * h + x;
+    if (k + 1 == nb || blocks[k + 1].w) S[(size_t)state[b.x] * W + c] = h;
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+lru_apply_kernel(const float* __restrict__ a, const float* __restrict__ x, const int4* __restrict__ blocks, int row0, const float* __restrict__ carry,
+                 const T* __restrict__ y, long long ldy, const float* __restrict__ yb, T* __restrict__ out, int W) {
+  const int4 b = blocks[blockIdx.y];
+  const int c = blockIdx.x * 128 + threadIdx.x;
+  if (c >= W) return;
+  float h = carry[(size_t)blockIdx.y * W + c];
+  const float bias = yb[c];
+  const int r0 = b.y - row0;
+#pragma unroll 4
+  for (int t = 0; t < b.z; ++t) {
+    const size_t o = (size_t)(r0 + t) * W + c;
+    h = a[o] * h + x[o];
+    stf(out + o, h * gelu_tanhf(ldf(y + (size_t)(r0 + t) * ldy + c) + bias));
+  }
+}
+
+// ------------------------------------------------------------------ Mamba-2, token by token
+// A warp owns 8 channels p of one head: lane l holds the states n = l, l + 32, ... of each. Serves single-token rows
+// (one pass over the state) and any sizes; portions with aligned sizes take the blocked form below.
+constexpr int M2_P = 8;
+
+template <typename T, int NL>
+__global__ void __launch_bounds__(128)
+mamba2_scan_kernel(const T* __restrict__ xbc, long long ldx, const T* __restrict__ dtr, long long ldd, const float* __restrict__ dt_bias,
+                   const float* __restrict__ A_log, const float* __restrict__ Dp, const int* __restrict__ cu, const int* __restrict__ start,
+                   const int* __restrict__ state, float* __restrict__ S, float* __restrict__ y, int H, int P, int N, int G) {
+  pdl_wait();
+  pdl_trigger();
+  const int e = blockIdx.x, hd = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int p0 = (blockIdx.z * 4 + warp) * M2_P;
+  if (p0 >= P) return;
+  const int np = min(M2_P, P - p0);
+  const int inner = H * P, g = hd / (H / G);
+  const int r0 = cu[e], r1 = cu[e + 1], slot = state[e];
+  if (slot < 0) {
+    for (int r = r0; r < r1; ++r)
+      if (lane < np) y[(size_t)r * inner + hd * P + p0 + lane] = 0.f;
+    return;
+  }
+  float* Sp = S + (((size_t)slot * H + hd) * P + p0) * N;
+  float s[M2_P][NL];
+  const bool fresh = start[e] <= 0;
+#pragma unroll
+  for (int i = 0; i < M2_P; ++i)
+#pragma unroll
+    for (int j = 0; j < NL; ++j) {
+      const int n = lane + 32 * j;
+      s[i][j] = (!fresh && i < np && n < N) ? Sp[(size_t)i * N + n] : 0.f;
+    }
+  const float A = -expf(A_log[hd]), bias = dt_bias[hd], Dh = Dp[hd];
+  const T* Bb = xbc + inner + g * N;
+  const T* Cb = Bb + G * N;
+  const T* xb = xbc + hd * P + p0;
+  float bn[NL], cn[NL], xn, dn;
+  auto fetch = [&](int r) {
+#pragma unroll
+    for (int j = 0; j < NL; ++j) {
+      const int n = lane + 32 * j;
+      bn[j] = n < N ? ldf(Bb + (size_t)r * ldx + n) : 0.f;
+      cn[j] = n < N ? ldf(Cb + (size_t)r * ldx + n) : 0.f;
+    }
+    xn = lane < np ? ldf(xb + (size_t)r * ldx + lane) : 0.f;
+    dn = ldf(dtr + (size_t)r * ldd + hd);
+  };
+  if (r0 < r1) fetch(r0);
+  for (int r = r0; r < r1; ++r) {
+    float b[NL], c[NL];
+#pragma unroll
+    for (int j = 0; j < NL; ++j) { b[j] = bn[j]; c[j] = cn[j]; }
+    const float x = xn, dt = softplusf(dn + bias);
+    if (r + 1 < r1) fetch(r + 1);
+    const float dec = expf(A * dt);
+    float mine = 0.f;
+#pragma unroll
+    for (int i = 0; i < M2_P; ++i) {
+      const float dx = dt * __shfl_sync(0xffffffffu, x, i);
+      float acc = 0.f;
+#pragma unroll
+      for (int j = 0; j < NL; ++j) {
+        s[i][j] = dec * s[i][j] + dx * b[j];
+        acc += s[i][j] * c[j];
+      }
+      acc = warp_sum(acc);
+      if (lane == i) mine = acc;
+    }
+    if (lane < np) y[(size_t)r * inner + hd * P + p0 + lane] = mine + Dh * x;
+  }
+#pragma unroll
+  for (int i = 0; i < M2_P; ++i)
+#pragma unroll
+    for (int j = 0; j < NL; ++j) {
+      const int n = lane + 32 * j;
+      if (i < np && n < N) Sp[(size_t)i * N + n] = s[i][j];
+    }
+}
+
+template <typename T>
+static int launch_rglru(bool decode, const void* u, const void* y, long long ldy, const float* yb, const void* gw, const float* gb, const float* lam,
+                        const int* start, const int* state, float* S, float* a, float* x, void* out, int R, int n, int bs, cudaStream_t s) {
+  const dim3 grid(n * ((bs + GT_C - 1) / GT_C), (R + GT_R - 1) / GT_R);
+  if (grid.y > 65535) return 11;
+  GateEpi p{gb, lam, yb, start, state, S, a, x, n * bs, bs, n};
+  if (decode)
+    launch_pdl(rglru_gate_kernel<T, true>, grid, dim3(128), 0, s, (const T*)u, (const T*)y, ldy, (const T*)gw, p, (T*)out, R);
+  else
+    launch_pdl(rglru_gate_kernel<T, false>, grid, dim3(128), 0, s, (const T*)u, (const T*)y, ldy, (const T*)gw, p, (T*)out, R);
+  return cudaGetLastError() == cudaSuccess ? 0 : 1;
+}
+
+}  // namespace ab2
+
+extern "C" {
+using namespace ab2;
+
+// Single-token rows. u [R, W], y [R, W] (row stride ldy), gw [2, n, bs, bs], gb [2, W], S [slots, W].
+int ab2_rglru_decode(const void* u, const void* y, long long ldy, const float* yb, const void* gw, const float* gb, const float* lam,
+                     const int* start, const int* state, float* S, void* out, int R, int n, int bs, int dt, void* stream) {
+  if (R <= 0) return 0;
+  return dt == 0 ? launch_rglru<__nv_bfloat16>(true, u, y, ldy, yb, gw, gb, lam, start, state, S, nullptr, nullptr, out, R, n, bs, (cudaStream_t)stream)
+                 : launch_rglru<float>(true, u, y, ldy, yb, gw, gb, lam, start, state, S, nullptr, nullptr, out, R, n, bs, (cudaStream_t)stream);
+}
+
+// Portions: R rows from row row0 of the step on, in nb blocks. a, x [R, W] and carry [2, nb, W] are scratch.
+int ab2_rglru_prefill(const void* u, const void* y, long long ldy, const float* yb, const void* gw, const float* gb, const float* lam,
+                      const void* blocks, int nb, int row0, int R, const int* start, const int* state, float* S, float* a, float* x, float* carry,
+                      void* out, int n, int bs, int dt, void* stream) {
+  if (R <= 0 || nb <= 0) return 0;
+  if (nb > 65535) return 11;
+  cudaStream_t s = (cudaStream_t)stream;
+  const int W = n * bs, gx = (W + 127) / 128;
+  const int rc = dt == 0 ? launch_rglru<__nv_bfloat16>(false, u, y, ldy, yb, gw, gb, lam, start, state, S, a, x, out, R, n, bs, s)
+                         : launch_rglru<float>(false, u, y, ldy, yb, gw, gb, lam, start, state, S, a, x, out, R, n, bs, s);
+  if (rc) return rc;
+  lru_block_kernel<<<dim3(gx, nb), 128, 0, s>>>(a, x, (const int4*)blocks, row0, carry, nb, W);
+  lru_carry_kernel<<<gx, 128, 0, s>>>((const int4*)blocks, start, state, S, carry, nb, W);
+  if (dt == 0)
+    lru_apply_kernel<__nv_bfloat16><<<dim3(gx, nb), 128, 0, s>>>(a, x, (const int4*)blocks, row0, carry, (const __nv_bfloat16*)y, ldy, yb,
+                                                                 (__nv_bfloat16*)out, W);
+  else
+    lru_apply_kernel<float><<<dim3(gx, nb), 128, 0, s>>>(a, x, (const int4*)blocks, row0, carry, (const float*)y, ldy, yb, (float*)out, W);
+  return cudaGetLastError() == cudaSuccess ? 0 : 1;
+}
+
+// Entries 0 .. E - 1, each over its rows. xbc rows: x [H * P] | B [G * N] | C [G * N]; S [slots, H, P, N]; y [rows, H * P] fp32.
+int ab2_mamba2_scan(const void* xbc, long long ldx, const void* dtr, long long ldd, const float* dt_bias, const float* A_log, const float* D,
+                    const int* cu, const int* start, const int* state, int E, float* S, float* y, int H, int P, int N, int G, int dt, void* stream) {
+  if (E <= 0) return 0;
+  if (G < 1 || H % G || H > 65535) return 10;
+  const dim3 grid(E, H, (P + 4 * M2_P - 1) / (4 * M2_P));
+  const int nl = (N + 31) / 32;
+#define AB2_M2(TT, NLV)                                                                                                                       \
+  launch_pdl(mamba2_scan_kernel<TT, NLV>, grid, dim3(128), 0, (cudaStream_t)stream, (const TT*)xbc, ldx, (const TT*)dtr, ldd, dt_bias, A_log, D, \
+             cu, start, state, S, y, H, P, N, G)
+#define AB2_M2_N(TT)                                                                                                                   \
+  if (nl <= 1) AB2_M2(TT, 1); else if (nl <= 2) AB2_M2(TT, 2); else if (nl <= 4) AB2_M2(TT, 4); else if (nl <= 8) AB2_M2(TT, 8); else if (nl <= 16) AB2_M2(TT, 16); else return 12
+  if (dt == 0) { AB2_M2_N(__nv_bfloat16); } else { AB2_M2_N(float); }
+#undef AB2_M2_N
+#undef AB2_M2
+  return cudaGetLastError() == cudaSuccess ? 0 : 1;
+}
+}

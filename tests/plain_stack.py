@@ -42,18 +42,21 @@ def attend(q, k, v, scale, softcap, r1, r2, chunk):
     the earlier positions of the query's own chunk."""
     L, H, _ = q.shape
     per = H // k.shape[1]
-    out = q.new_zeros(L, H, v.shape[-1])
-    for i in range(L):
-        js = [j for j in range(i + 1) if not chunk or i // chunk == j // chunk]
-        dist = torch.tensor([i - j for j in js], dtype=q.dtype)
-        for h in range(H):
-            s = (k[js, h // per] @ q[i, h]) * scale
-            if softcap:
-                s = softcap * torch.tanh(s / softcap)
-            s = s - r1[h] * torch.log(1 + r2[h] * dist)
-            w = torch.exp(s - s.max())
-            out[i, h] = (w / w.sum()) @ v[js, h // per]
-    return out
+    at = torch.arange(L)
+    dist = (at[:, None] - at[None, :]).to(q.dtype)
+    seen = dist >= 0
+    if chunk:
+        seen &= (at // chunk)[:, None] == (at // chunk)[None, :]
+    out = []
+    for h in range(H):
+        s = q[:, h] @ k[:, h // per].T * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
+        s = s - r1[h] * torch.log(1 + r2[h] * dist.clamp(min=0))
+        s = torch.where(seen, s, torch.full_like(s, -math.inf))
+        w = torch.exp(s - s.max(-1, keepdim=True).values)
+        out.append(w / w.sum(-1, keepdim=True) @ v[:, h // per])
+    return torch.stack(out, 1)
 
 
 def attention(W, pre, h, cfg, eps):
@@ -69,12 +72,9 @@ def attention(W, pre, h, cfg, eps):
 
 def causal_conv(x, w, b):
     """out[t, c] = b[c] + sum_j w[c, K - 1 - j] x[t - j, c], zeros before the start."""
-    L, K = x.shape[0], w.shape[1]
     out = b.expand_as(x).clone()
-    for t in range(L):
-        for j in range(K):
-            if t - j >= 0:
-                out[t] += w[:, K - 1 - j] * x[t - j]
+    for j in range(w.shape[1]):
+        out[j:] += w[:, w.shape[1] - 1 - j] * x[:x.shape[0] - j]
     return out
 
 
@@ -104,13 +104,13 @@ def mamba2(W, pre, h, cfg, eps):
     x, B, C = torch.split(xbc, [inner, G * N, G * N], dim=-1)
     x, B, C = x.view(L, H, P), B.view(L, G, N), C.view(L, G, N)
     dt = softplus(dt + W[pre + "dt_bias"])
-    y = torch.zeros(L, H, P, dtype=h.dtype)
-    for hd in range(H):
-        g = hd // (H // G)
-        S = torch.zeros(N, P, dtype=h.dtype)
-        for t in range(L):
-            S = torch.exp(-torch.exp(W[pre + "A_log"][hd]) * dt[t, hd]) * S + dt[t, hd] * torch.outer(B[t, g], x[t, hd])
-            y[t, hd] = S.T @ C[t, g] + W[pre + "D"][hd] * x[t, hd]
+    B, C = (t[:, [hd // (H // G) for hd in range(H)]] for t in (B, C))          # each head's group
+    decay = torch.exp(-torch.exp(W[pre + "A_log"]) * dt)
+    S, y = torch.zeros(H, N, P, dtype=h.dtype), []
+    for t in range(L):
+        S = decay[t][:, None, None] * S + dt[t][:, None, None] * B[t][:, :, None] * x[t][:, None, :]
+        y.append(torch.einsum("hnp,hn->hp", S, C[t]) + W[pre + "D"][:, None] * x[t])
+    y = torch.stack(y)
     y = y.reshape(L, inner) * silu(z)
     return root_mean_square_norm(y, W[pre + "norm"], eps, m["norm_groups"]) @ W[pre + "o"].T
 
@@ -132,10 +132,11 @@ def feed_forward(W, pre, h, mlp):
         return xielu(h @ W[pre + "up"].T, p, q) @ W[pre + "down"].T
     chosen, weight = route(h, W[pre + "router"], W[pre + "correction"], mlp["router"]["top"])
     out = torch.zeros_like(h)
-    for t in range(h.shape[0]):
-        for e, w in zip(chosen[t].tolist(), weight[t]):
-            p = f"{pre}e{e}."
-            out[t] += w * (W[p + "down"] @ (silu(W[p + "gate"] @ h[t]) * (W[p + "up"] @ h[t])))
+    for e in range(mlp["router"]["experts"]):
+        t, slot = torch.where(chosen == e)
+        p = f"{pre}e{e}."
+        y = (silu(h[t] @ W[p + "gate"].T) * (h[t] @ W[p + "up"].T)) @ W[p + "down"].T
+        out[t] += weight[t, slot, None] * y
     return out
 
 
