@@ -1,0 +1,331 @@
+"""Serving throughput of a mixer stack beside the framework's closest existing models at equal layer sizes, and the time of
+every kernel against its roofline (``bench.py --workload mixer-serve``). Random weights, synthetic tokens, one GPU.
+
+Kernel times are CUDA events around one launch with the L2 flushed in between (a 256 MB buffer is written); step times
+are CUDA events around whole steps of the serving path, whose weights alone exceed L2."""
+from __future__ import annotations
+
+import json
+import math
+import os
+import time
+
+import torch
+import torch.nn.functional as F
+
+from ..ops import functional as OF
+from ..ops import lib as oplib
+from ..ops import mixer_ops as M
+
+ROOT = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
+
+
+def peaks() -> tuple[float, float, str]:
+    try:
+        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+            p = json.load(f)
+        return p["hbm_gbs"] * 1e9, p["bf16_tflops"] * 1e12, "measured"
+    except (OSError, KeyError, ValueError):
+        return 6.65e12, 1.59e15, "fallback"
+
+
+def timed(fn, iters: int = 10, warmup: int = 3, flush=None) -> float:
+    """Median seconds of one call."""
+    for _ in range(warmup):
+        fn()
+    torch.cuda.synchronize()
+    ts = []
+    for _ in range(iters):
+        if flush is not None:
+            flush.zero_()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        fn()
+        b.record()
+        b.synchronize()
+        ts.append(a.elapsed_time(b) * 1e-3)
+    return sorted(ts)[len(ts) // 2]
+
+
+def _batch(lens, starts, dev, page_size=64):
+    """A ragged batch over consecutive pages; single-token entries first. Returns (batch, cache rows)."""
+    from ..engine.ragged_step import Entry, RaggedRunner
+    from ..engine.state_cache import Carried
+
+    ents, at = [], 0
+    for i, (n, s) in enumerate(zip(lens, starts)):
+        k = -(-(n + s) // page_size)
+        ents.append(Entry(Carried(slot=i, pages=list(range(at, at + k)), length=s), [1] * n, []))
+        at += k
+    r = RaggedRunner.__new__(RaggedRunner)
+    r.device = torch.device(dev)
+    r.cache = type("C", (), dict(page_size=page_size, has_kv=True))
+    return RaggedRunner._layout(r, ents)[0], at * page_size
+
+
+def kernel_table(cfg, prefill=(4, 2048), decode=(64, 1024), dev="cuda") -> list[dict]:
+    """Time, roofline time and fraction of the new design's kernels, each beside the like kernel of the existing models.
+    ``prefill`` = (sequences, tokens each), ``decode`` = (sequences, cached tokens each)."""
+    bw, fl, _ = peaks()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    bf = dict(device=dev, dtype=torch.bfloat16)
+    f32 = dict(device=dev, dtype=torch.float32)
+    rows = []
+
+    def add(name, fn, nbytes=0.0, flops=0.0, like=None):
+        t = timed(fn, flush=flush)
+        roof = max(nbytes / bw, flops / fl)
+        rows.append(dict(kernel=name, us=round(t * 1e6, 1), roofline_us=round(roof * 1e6, 1), fraction=round(roof / t, 3), like=like))
+
+    H = cfg.hidden_size
+    spec = {e["type"]: e["mixer"] for e in cfg.mixer_layers}
+    at, m2, lr = spec["attention"], spec["mamba2"], spec["rglru"]
+    B, L = prefill
+    T = B * L
+    pb, prow = _batch([L] * B, [0] * B, dev)
+    nB, ctx = decode
+    db, drow = _batch([1] * nB, [ctx] * nB, dev)
+    w = torch.ones(H, **f32)
+    for tag, R in (("prefill", T), ("decode", nB)):
+        h, res = torch.randn(R, H, **bf), torch.randn(R, H, **f32)
+        add(f"sandwich_norm {tag}", lambda: M.sandwich_norm(h, w, res, w, cfg.norm_groups, 1e-6), R * H * 12, like=f"rmsnorm {tag}")
+        r16, w16 = res.bfloat16(), w.bfloat16()
+        with torch.no_grad():
+            add(f"rmsnorm {tag}", lambda: OF.rmsnorm(h, w16, 1e-6, r16), R * H * 8)
+    # attention
+    nq, nk, D, Dv = at["heads"], at["kv_heads"], at["dim"], at["vdim"]
+    chunk = at["mask"]["size"]
+    r1, r2 = torch.rand(nq, **f32), torch.rand(nq, **f32)
+    for tag, b, R, rows_ in (("prefill", pb, T, prow), ("decode", db, nB, drow)):
+        kc, vc, q = torch.randn(rows_, nk, D, **bf), torch.randn(rows_, nk, Dv, **bf), torch.randn(R, nq, D, **bf)
+        qkv = torch.randn(R, nq * D + nk * (D + Dv), **bf)
+        wq, wk = torch.ones(nq * D, **f32), torch.ones(nk * D, **f32)
+        add(f"qk_norm_append {tag}", lambda: M.qk_norm_append(qkv, wq, wk, 1e-6, b, kc, vc, nq), qkv.numel() * 4)
+        if tag == "prefill":
+            pairs = B * sum(p % chunk + 1 for p in range(L))
+            fn = lambda: M.chunk_attention(q, kc, vc, b, D ** -0.5, at["softcap"], r1, r2, chunk)      # noqa: E731
+            add("chunk_attention prefill", fn, (q.numel() * 2 + (nk * (D + Dv)) * T) * 2, 2.0 * nq * (D + Dv) * pairs, like="attn_fwd prefill")
+            if D == Dv and D in (64, 128):
+                k, v = torch.randn(T, nk, D, **bf), torch.randn(T, nk, D, **bf)
+                cu = torch.arange(0, T + 1, L, device=dev, dtype=torch.int32)
+                ti = OF.attn_tile_table(cu, T)
+                add("attn_fwd prefill", lambda: OF.attention_fwd(q, k, v, cu, True, D ** -0.5, ti), 0, 4.0 * nq * D * B * L * (L + 1) / 2)
+        else:
+            see = ctx % chunk + 1
+            add("chunk_attention decode", lambda: M.chunk_attention(q, kc, vc, b, D ** -0.5, at["softcap"], r1, r2, chunk), nB * see * nk * (D + Dv) * 2,
+                like="paged_decode decode")
+            if D == Dv and D in (64, 128):
+                lens = torch.full((nB,), ctx + 1, device=dev, dtype=torch.int32)
+                po, ml = torch.empty(nB * nq * 4 * D, **f32), torch.empty(nB * nq * 8, **f32)
+                o = torch.empty_like(q)
+
+                def paged():
+                    oplib.check(oplib.get_lib().ab2_paged_decode_strided(
+                        q.data_ptr(), kc.data_ptr(), vc.data_ptr(), b.pages.data_ptr(), lens.data_ptr(), po.data_ptr(), ml.data_ptr(), o.data_ptr(), nB, nq,
+                        nk, D, 64, b.pages.shape[1], 4, D ** -0.5, q.stride(0), oplib.stream_ptr()), "paged_decode")
+                add("paged_decode decode", paged, nB * (ctx + 1) * nk * 2 * D * 2)
+    # recurrences
+    Hm, P, N, G = m2["heads"], m2["vdim"], m2["state"], m2["groups"]
+    I, C = Hm * P, Hm * P + 2 * G * N
+    dtb, Al, Dd = torch.randn(Hm, **f32) - 4, torch.rand(Hm, **f32), torch.ones(Hm, **f32)
+    W, nb_ = lr["width"], lr["blocks"]
+    gw, gb, lam = torch.randn(2, nb_, W // nb_, W // nb_, **bf) * 0.05, torch.zeros(2, nb_, W // nb_, **f32), torch.full((W,), -3.0, **f32)
+    for tag, b, R, ne in (("prefill", pb, T, B), ("decode", db, nB, nB)):
+        x, taps = torch.randn(R, I + C + Hm, **bf), m2["conv"]
+        cw, cb, tail = torch.randn(C, taps, **f32), torch.randn(C, **f32), torch.zeros(ne, C, taps - 1, **f32)
+        add(f"causal_conv {tag}", lambda: M.causal_conv(x[:, I:I + C], None, cw, cb, True, b, tail), R * C * 4 + (ne * C * (taps - 1) * 8))
+        xbc, S = torch.randn(R, C, **bf), torch.zeros(ne, Hm, P, N, **f32)
+        add(f"mamba2_scan {tag}", lambda: M.mamba2_scan(xbc, x[:, I + C:], dtb, Al, Dd, Hm, P, N, G, b, S), R * (C * 2 + I * 4) + 2 * S.numel() * 4, 0,
+            like=f"gated_delta_rule {tag}")
+        y, nw = torch.randn(R, I, **f32), torch.ones(I, **f32)
+        add(f"gated_group_norm {tag}", lambda: M.gated_group_norm(y, x[:, :I], nw, m2["norm_groups"], 1e-6), R * I * 8)
+        yx, SL, yb = torch.randn(R, 2 * W, **bf), torch.zeros(ne, W, **f32), torch.zeros(W, **f32)
+        u = torch.randn(R, W, **bf)
+        add(f"rglru {tag}", lambda: M.rglru(u, yx[:, :W], yb, gw, gb, lam, b, SL), R * W * 6 + gw.numel() * 2 + 2 * SL.numel() * 4,
+            4.0 * R * W * (W // nb_), like=f"gated_delta_rule {tag}")
+        # the existing linear-attention rule at the same state size (heads x 128 x 64 / 128)
+        from ..models.hybrid import gated_delta_rule_chunked, gated_delta_rule_recurrent
+
+        shp = (ne, R // ne, Hm)
+        q_, k_ = torch.randn(*shp, N, **f32), F.normalize(torch.randn(*shp, N, **f32), dim=-1)
+        v_, g_, be = torch.randn(*shp, P, **f32), -torch.rand(*shp, **f32), torch.rand(*shp, **f32)
+        rule = gated_delta_rule_chunked if tag == "prefill" else gated_delta_rule_recurrent
+        S0 = torch.zeros(ne, Hm, N, P, **f32)
+        add(f"gated_delta_rule {tag}", lambda: rule(q_, k_, v_, g_, be, state=S0), R * Hm * (2 * N + 2 * P) * 2 + 2 * S0.numel() * 4)
+    # feed-forward pieces
+    ff = max([e["mlp"]["ff"] for e in cfg.mixer_layers if e["mlp"] and e["mlp"]["kind"] == "dense"], default=4 * H)
+    pq = torch.ones(2, **f32)
+    for tag, R in (("prefill", T), ("decode", nB)):
+        x = torch.randn(R, ff, **bf)
+        add(f"xielu {tag}", lambda: M.xielu(x, pq), R * ff * 4, like=f"swiglu {tag}")
+        gu = torch.randn(R, 2 * ff, **bf)
+        add(f"glu_silu {tag}", lambda: M.glu_silu(gu), R * ff * 6, like=f"swiglu {tag}")
+        with torch.no_grad():
+            add(f"swiglu {tag}", lambda: OF.swiglu(gu), R * ff * 6)
+        lg = torch.randn(min(R, 256), cfg.vocab_size, **f32)
+        add(f"softcap {tag}", lambda: M.softcap_(lg, 30.0), lg.numel() * 8)
+        moe = next((e["mlp"] for e in cfg.mixer_layers if e["mlp"] and e["mlp"]["kind"] == "moe"), None)
+        if moe:
+            E, k, If = moe["router"]["experts"], moe["router"]["top"], moe["expert"]["ff"]
+            rt = OF.moe_route(torch.randn(R, E, **f32), k, norm=False, want_probs=False, want_host=False)
+            ys, wgu, wd = torch.randn(R * k, H, **bf), torch.randn(E, 2 * If, H, **bf), torch.randn(E, H, If, **bf)
+            hh = torch.randn(R * k, If, **bf)
+            live = min(E, R * k)
+            add(f"expert_linear up {tag}", lambda: M.expert_linear(ys, wgu, rt), (live * 2 * If * H + R * k * (H + 2 * If)) * 2, 4.0 * R * k * H * If)
+            add(f"expert_linear down {tag}", lambda: M.expert_linear(hh, wd, rt), (live * If * H + R * k * (H + If)) * 2, 2.0 * R * k * H * If)
+            add(f"expert_combine {tag}", lambda: M.expert_combine(ys, rt, rt.topw), R * (k + 1) * H * 2, like=f"gather and sum {tag}")
+            add(f"gather and sum {tag}", lambda: (ys.index_select(0, rt.inv).view(R, k, H) * rt.topw.to(ys.dtype).unsqueeze(-1)).sum(1), R * (k + 1) * H * 2)
+    return rows
+
+
+# ----------------------------------------------------------------------------- whole steps
+def _engine(cfg, seqs, total, prefill_tokens):
+    from ..api.cli_args import InferenceEngineConfig, NativeInferConfig
+    from ..engine.infer_engine import NativeInferenceEngine
+    from ..models.decoder import build_model
+
+    ic = NativeInferConfig(page_size=64, num_pages=seqs * (total // 64 + 2), max_running_requests=seqs, context_length=total + 64,
+                           max_prefill_tokens=prefill_tokens)
+    model = build_model(cfg, dtype=torch.bfloat16, device="cuda", seed=1)
+    return NativeInferenceEngine(InferenceEngineConfig(), ic, model=model).initialize(device="cuda", start_executor=False, start_loop=False)
+
+
+def mixer_steps(cfg, prefill, decode) -> dict:
+    from ..engine.ragged_step import Entry
+
+    (B, L), (nB, ctx) = prefill, decode
+    eng = _engine(cfg, max(B, nB), max(L, ctx + 64), B * L)
+    toks = torch.randint(0, cfg.vocab_size, (L,)).tolist()
+
+    def fill(n, length):
+        cs = []
+        for _ in range(n):
+            c = eng.cache.open()
+            assert eng.cache.grow(c, length)
+            cs.append(c)
+        return cs
+
+    def prompt():
+        cs = fill(B, L)
+        eng.runner.step([Entry(c, toks, [L - 1]) for c in cs])
+        for c in cs:
+            eng.cache.close(c)
+    with torch.cuda.stream(eng.stream):
+        tp = timed(prompt, iters=5, warmup=2)
+        cs = fill(nB, ctx)
+        for c in cs:
+            eng.runner.step([Entry(c, (toks * (ctx // L + 1))[:ctx], [])])
+
+        def one():
+            for c in cs:
+                eng.cache.grow(c, c.length + 1)
+            eng.runner.step([Entry(c, [7], [0]) for c in cs])
+        td = timed(one, iters=20, warmup=4)
+        t0 = time.perf_counter()
+        for _ in range(10):
+            one()
+        torch.cuda.synchronize()
+        wall = (time.perf_counter() - t0) / 10
+    n = oplib.launch_count()
+    out = dict(prefill_tokens_per_s=round(B * L / tp), prefill_ms=round(tp * 1e3, 3), decode_tokens_per_s=round(nB / td), decode_ms=round(td * 1e3, 3),
+               decode_wall_ms=round(wall * 1e3, 3), launches=n, params_m=round(sum(p.numel() for p in eng.model.parameters()) / 1e6, 1))
+    eng.destroy()
+    return out
+
+
+def decoder_steps(cfg, prefill, decode) -> dict:
+    """A dense / routed decoder of the framework: packed prefill and graph-captured paged decode of the rollout engine."""
+    from ..engine.infer_engine import _Seq
+
+    (B, L), (nB, ctx) = prefill, decode
+    eng = _engine(cfg, max(B, nB), max(L, ctx + 64), max(B * L, ctx * 8))
+
+    def seq(i, n):
+        return _Seq(rid=str(i), tokens=torch.randint(0, cfg.vocab_size, (n,)).tolist(), prompt_len=n, max_new=1 << 20, min_new=0, temperature=1.0, greedy=True,
+                    stop_ids=set(), ignore_eos=True, seed=1)
+
+    def prompt():
+        ss = [seq(i, L) for i in range(B)]
+        for s in ss:
+            s.pages = eng.cache.alloc(eng.cache.pages_needed(L + 1))
+        eng._prefill(ss, [])
+        for s in ss:
+            eng.cache.release(s.pages)
+    with torch.cuda.stream(eng.stream), torch.no_grad():
+        tp = timed(prompt, iters=5, warmup=2)
+        run = [seq(i, ctx) for i in range(nB)]
+        for i in range(0, nB, 8):
+            for s in run[i:i + 8]:
+                s.pages = eng.cache.alloc(eng.cache.pages_needed(ctx + 64))
+            eng._prefill(run[i:i + 8], [])
+        for s in run:
+            eng._assign_row(s)
+        td = timed(lambda: eng._decode(run, []), iters=20, warmup=4)
+    out = dict(prefill_tokens_per_s=round(B * L / tp), prefill_ms=round(tp * 1e3, 3), decode_tokens_per_s=round(nB / td), decode_ms=round(td * 1e3, 3),
+               params_m=round(sum(p.numel() for p in eng.model.parameters()) / 1e6, 1))
+    eng.destroy()
+    return out
+
+
+def hybrid_steps(cfg, prefill, decode) -> dict:
+    """The framework's linear / full attention stack (carried state outside pages and graphs)."""
+    from ..models.decoder import build_model
+    from ..models.hybrid import decode_states, prefill_states
+
+    (B, L), (nB, ctx) = prefill, decode
+    model = build_model(cfg, dtype=torch.bfloat16, device="cuda", seed=1).eval()
+    with torch.no_grad():
+        ids = torch.randint(0, cfg.vocab_size, (B * L,), device="cuda")
+        cu = torch.arange(0, B * L + 1, L, device="cuda", dtype=torch.int32)
+        tp = timed(lambda: model.logits(prefill_states(model, ids, cu, L)[0][(cu[1:] - 1).long()]), iters=3, warmup=1)
+        states = []
+        for _ in range(0, nB, 8):
+            n = min(8, nB)
+            c2 = torch.arange(0, n * ctx + 1, ctx, device="cuda", dtype=torch.int32)
+            states += prefill_states(model, torch.randint(0, cfg.vocab_size, (n * ctx,), device="cuda"), c2, ctx)[1]
+        t1 = torch.randint(0, cfg.vocab_size, (nB,), device="cuda")
+        td = timed(lambda: model.logits(decode_states(model, t1, states[:nB])), iters=5, warmup=2)
+    return dict(prefill_tokens_per_s=round(B * L / tp), prefill_ms=round(tp * 1e3, 3), decode_tokens_per_s=round(nB / td), decode_ms=round(td * 1e3, 3),
+                params_m=round(sum(p.numel() for p in model.parameters()) / 1e6, 1))
+
+
+def like_sized(cfg):
+    """The closest existing models with the same width, heads, feed-forward and vocabulary: (hybrid stack, dense decoder,
+    routed decoder), as many layers as ``cfg`` has."""
+    from ..models.config import ModelConfig
+
+    at = next(e["mixer"] for e in cfg.mixer_layers if e["type"] == "attention")
+    moe = next(e["mlp"] for e in cfg.mixer_layers if e["mlp"] and e["mlp"]["kind"] == "moe")
+    n = cfg.num_layers
+    base = dict(vocab_size=cfg.vocab_size, hidden_size=cfg.hidden_size, num_layers=n, num_heads=at["heads"], num_kv_heads=at["kv_heads"], head_dim=at["dim"],
+                intermediate_size=cfg.intermediate_size, tie_word_embeddings=False, attention_bias=False, qk_norm=True)
+    hyb = ModelConfig(arch="qwen3_5", **base, layer_types=["full_attention" if i == 0 else "linear_attention" for i in range(n)], linear_key_head_dim=128,
+                      linear_value_head_dim=128, linear_num_key_heads=cfg.hidden_size // 256, linear_num_value_heads=cfg.hidden_size // 128,
+                      partial_rotary_factor=0.25, attn_output_gate=True, rms_norm_offset=True)
+    routed = ModelConfig(arch="qwen3_moe", **base, num_experts=moe["router"]["experts"], num_experts_per_tok=moe["router"]["top"],
+                         moe_intermediate_size=moe["expert"]["ff"])
+    return hyb, ModelConfig(arch="qwen3", **base), routed
+
+
+def run(steps=True, kernels=True, sizes=("kagolix-8b-layers", "kagolix-2b-layers")) -> dict:
+    from ..models.config import preset
+
+    torch.manual_seed(0)
+    bw, fl, src = peaks()
+    out = dict(workload="mixer-serve", dtype="bf16", data="synthetic tokens, random weights", roofline=f"{src}: {bw / 1e9:.0f} GB/s, {fl / 1e12:.0f} TFLOP/s",
+               sizes={})
+    for name in sizes:
+        cfg = preset(name)
+        prefill, decode = (4, 2048), (64, 1024)
+        r = dict(prefill=f"{prefill[0]} x {prefill[1]} tokens", decode=f"{decode[0]} sequences at {decode[1]} tokens")
+        if steps:
+            hyb, dense, routed = like_sized(cfg)
+            r["mixer_stack"] = mixer_steps(cfg, prefill, decode)
+            torch.cuda.empty_cache()
+            for key, fn, c in (("decoder_dense", decoder_steps, dense), ("decoder_routed", decoder_steps, routed), ("hybrid", hybrid_steps, hyb)):
+                r[key] = fn(c, prefill, decode)
+                torch.cuda.empty_cache()
+        if kernels:
+            r["kernels"] = kernel_table(cfg, prefill, decode)
+        out["sizes"][name] = r
+    return out

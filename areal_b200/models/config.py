@@ -406,6 +406,9 @@ MIXER_STACK_PRESETS = {
     "kagolix-8b-layers": _mixer_stack_preset(
         32768, 4096, "amRM", dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, mask=dict(size=4096)),
         dict(heads=64, vdim=64, state=128, groups=8, norm_groups=8, conv=4), dict(width=4096, blocks=16, conv=4), 12288, (64, 8, 768), 8),
+    "kagolix-2b-layers": _mixer_stack_preset(
+        32768, 2048, "amRM", dict(heads=16, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, mask=dict(size=1024)),
+        dict(heads=64, vdim=64, state=128, groups=4, norm_groups=4, conv=4), dict(width=2560, blocks=10, conv=4), 8192, (64, 8, 768), 8),
 }
 
 

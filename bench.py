@@ -52,6 +52,9 @@ def parse_args():
     ap.add_argument("--steps", type=int, default=3)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", type=str, default="native", choices=["native", "reference"])
+    ap.add_argument("--workload", type=str, default="train", choices=["train", "mixer-serve"],
+                    help="train: the headline job; mixer-serve: prefill and decode throughput of the mixer stack beside the closest existing "
+                         "models, and its kernels against their rooflines (one GPU, prints its own JSON line)")
     ap.add_argument("--model", type=str, default="qwen3-8b")
     ap.add_argument("--preset", type=str, default="driver", choices=sorted(PRESETS))
     ap.add_argument("--length-scale", type=float, default=None, help="scales prompt / median / cap lengths of the preset")
@@ -179,10 +182,24 @@ def run_reference(args):
     return 0
 
 
+def run_mixer_serve():
+    os.environ.setdefault("AB2_PDL", "1")
+    from areal_b200.infra.bench_mixers import run
+
+    clocks = ClockSampler()
+    clocks.start()
+    result = run()
+    result["clocks"] = clocks.stop()
+    print(json.dumps(result))
+    return 0
+
+
 def main():
     args = parse_args()
     if args.impl == "reference":
         return run_reference(args)
+    if args.workload == "mixer-serve":
+        return run_mixer_serve()
     import faulthandler
 
     # decode-path switches of the kernel library, read once per process at first use: programmatic

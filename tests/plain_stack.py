@@ -126,11 +126,15 @@ def route(h, router, correction, top):
     return chosen, s.gather(1, chosen)
 
 
-def feed_forward(W, pre, h, mlp):
+def feed_forward(W, pre, h, mlp, margins=None):
     if mlp["kind"] == "dense":
         p, q = W[pre + "act"]
         return xielu(h @ W[pre + "up"].T, p, q) @ W[pre + "down"].T
     chosen, weight = route(h, W[pre + "router"], W[pre + "correction"], mlp["router"]["top"])
+    if margins is not None:
+        c = torch.softmax(h @ W[pre + "router"].T, -1) + W[pre + "correction"]
+        c = c.sort(-1, descending=True).values
+        margins.append(c[:, mlp["router"]["top"] - 1] - c[:, mlp["router"]["top"]])
     out = torch.zeros_like(h)
     for e in range(mlp["router"]["experts"]):
         t, slot = torch.where(chosen == e)
@@ -140,8 +144,9 @@ def feed_forward(W, pre, h, mlp):
     return out
 
 
-def forward(W, config, tokens):
-    """Logits [L, vocab] of one sequence, and the residual stream after every layer."""
+def forward(W, config, tokens, margins=None):
+    """Logits [L, vocab] of one sequence, and the residual stream after every layer. ``margins`` (a list) collects, per
+    routed layer, how far each token's last chosen expert is ahead of the first one left out."""
     eps, groups = config["norm"]["eps"], config["norm"]["groups"]
 
     def norm(x, name):
@@ -153,7 +158,7 @@ def forward(W, config, tokens):
         pre = f"l{i}."
         x = x + norm(MIXERS[layer["type"]](W, pre + "mix.", norm(x, pre + "norm1"), layer, eps), pre + "norm1b")
         if layer["mlp"] is not None:
-            x = x + norm(feed_forward(W, pre + "mlp.", norm(x, pre + "norm2"), layer["mlp"]), pre + "norm2b")
+            x = x + norm(feed_forward(W, pre + "mlp.", norm(x, pre + "norm2"), layer["mlp"], margins), pre + "norm2b")
         states.append(x)
     logits = norm(x, "final.norm") @ W["head"].T
     cap = config["logit_softcap"]

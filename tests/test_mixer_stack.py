@@ -68,7 +68,7 @@ CONFIGS = {
     "odd": config((rglru(width=42, blocks=3, conv=2), moe(experts=5, top=3, ff=20)), (attention(heads=3, kv=1, dim=20, vdim=12, size=33), dense(36)),
                   (mamba2(heads=3, vdim=10, state=7, groups=1, norm_groups=3, conv=3), dense(33)), vocab=101, width=60, groups=3),
     # chunks longer than a page and than a query tile, several heads per group, wide values, states of two lane rows
-    "wide": config((attention(heads=8, kv=2, dim=64, vdim=96, size=320), moe(8, 3, 64)), (mamba2(heads=2, vdim=64, state=64, groups=1, norm_groups=1), None),
+    "wide": config((attention(heads=8, kv=2, dim=64, vdim=96, size=320), dense(96)), (mamba2(heads=2, vdim=64, state=64, groups=1, norm_groups=1), None),
                    (rglru(width=128, blocks=1, conv=1), dense(128)), width=128, groups=1, vocab=96),
     "dim128": config((attention(heads=2, kv=2, dim=128, vdim=128, size=200), dense(64)), (mamba2(heads=2, vdim=16, state=128, groups=2, norm_groups=4), None),
                      width=64, groups=4),
@@ -173,9 +173,13 @@ def tokens(n, vocab, seed):
     return [r.randrange(vocab) for _ in range(n)]
 
 
-def assert_close(got, want, dtype, what=""):
+def assert_close(got, want, dtype, what="", sure=None):
+    """``sure``: rows whose choice of experts is clear (bf16 rounding may turn a close one, which is another result)."""
     scale = want.pow(2).mean().sqrt()
     err = (got - want).pow(2).mean(-1).sqrt() / scale
+    if sure is not None and dtype == torch.bfloat16:
+        assert len(sure) < 20 or sure.double().mean() > 0.6
+        err = err * sure
     assert torch.isfinite(got).all() and err.max() < TOL[dtype], f"{what}: row {int(err.argmax())} off by {float(err.max()):.2e}"
 
 
@@ -183,11 +187,14 @@ _ORACLE: dict = {}
 
 
 def oracle(name, n, seed):
-    """Logits of a random prompt under a named configuration (cached: shared by the targets and the schedules)."""
+    """Tokens, logits and rows with a clear choice of experts of a random prompt under a named configuration (cached:
+    shared by the targets and the schedules)."""
     if (name, n, seed) not in _ORACLE:
         cfg = CONFIGS[name]
         t = tokens(n, cfg["vocab"], seed)
-        _ORACLE[name, n, seed] = (t, plain.forward(make_weights(cfg), cfg, t)[0])
+        margins = [torch.ones(n)]
+        logits = plain.forward(make_weights(cfg), cfg, t, margins)[0]
+        _ORACLE[name, n, seed] = (t, logits, torch.stack([m.double() for m in margins]).amin(0) > 0.02)
     return _ORACLE[name, n, seed]
 
 
@@ -198,7 +205,7 @@ def test_whole_prompt_portions_and_single_tokens_agree(name, target):
     cfg = CONFIGS[name]
     eng = make_engine(cfg, make_weights(cfg), target)
     n = 150
-    t, want = oracle(name, n, 1)
+    t, want, sure = oracle(name, n, 1)
     cuts = {"whole": [n], "decoded": [100] + [1] * 50, "pairs": [2] * 35 + [80], "ragged": [1, 2, 61, 3, 64, 2, 1, 16]}
     for what, sizes in cuts.items():
         d, at = Driver(eng), 0
@@ -206,7 +213,7 @@ def test_whole_prompt_portions_and_single_tokens_agree(name, target):
         for s in sizes:
             d.step([("a", t[at:at + s])], end=["a"] if at + s == n else [])
             at += s
-        assert_close(d.logits("a"), want, target[1], f"{name} {what}")
+        assert_close(d.logits("a"), want, target[1], f"{name} {what}", sure)
     assert len(eng.cache.free) == eng.cache.num_pages and len(eng.cache.free_slots) == eng.cache.num_slots
 
 
@@ -215,11 +222,11 @@ def test_long_prompt_and_long_decoding_cross_many_chunks(target):
     name = "wide"
     cfg = CONFIGS[name]
     n = 700
-    t, want = oracle(name, n, 2)
+    t, want, sure = oracle(name, n, 2)
     eng = make_engine(cfg, make_weights(cfg), target)
     d = Driver(eng)
     d.step([("a", t)], end=["a"])
-    assert_close(d.logits("a"), want, target[1], "whole")
+    assert_close(d.logits("a"), want, target[1], "whole", sure)
     d = Driver(eng)
     d.step([("a", t[:300])])
     for i in range(300, 345):                      # decoding walks over the chunk border at 320
@@ -228,7 +235,7 @@ def test_long_prompt_and_long_decoding_cross_many_chunks(target):
     d.step([("a", t[345:637])])
     for i in range(637, n):                        # and the next one at 640
         d.step([("a", t[i:i + 1])], end=["a"] if i == n - 1 else [])
-    assert_close(d.logits("a"), want, target[1], "decoded")
+    assert_close(d.logits("a"), want, target[1], "decoded", sure)
 
 
 @pytest.mark.parametrize("target", TARGETS)
@@ -259,7 +266,7 @@ def test_mixed_batches_on_reused_pages_and_slots(target, page_size):
         d.step(portions, end=done)
         live = [r for r in live if r not in done]
     for rid in lens:
-        assert_close(d.logits(rid), ref[rid][1], target[1], rid)
+        assert_close(d.logits(rid), ref[rid][1], target[1], rid, ref[rid][2])
     assert len(eng.cache.free) == eng.cache.num_pages
 
 
@@ -604,8 +611,8 @@ def test_trace_runner_replays_steps(tmp_path, target):
     save_file({n: t.bfloat16().contiguous() for n, t in make_weights(cfg).items()}, str(model / "model.safetensors"))
     eng = trace_engine(str(model), "float32" if target[1] == torch.float32 else "bfloat16", 256, target[0])
     assert eng.cache.num_pages == 4 and eng.cache.num_slots == 4
-    ta, wa = oracle(name, 97, 12)
-    tb, wb = oracle(name, 7, 11)
+    ta, wa, sure = oracle(name, 97, 12)
+    tb, wb, _ = oracle(name, 7, 11)
     steps = [dict(step=0, entries=[dict(id="a", tokens=ta[:90], want=[3, 89])], end=[]),
              dict(step=1, entries=[dict(id="a", tokens=ta[90:92], want=[]), dict(id="b", tokens=tb[:1], want=[])], end=[]),
              dict(step=2, entries=[dict(id="a", tokens=ta[92:], want=[4, 0]), dict(id="b", tokens=tb[1:2], want=[0])], end=["a"]),
@@ -615,7 +622,7 @@ def test_trace_runner_replays_steps(tmp_path, target):
     assert said == [f"done {i}" for i in range(4)]
     got = {i: torch.from_numpy(np.fromfile(out / f"{i}.f32", dtype="<f4")).view(-1, cfg["vocab"]).double() for i in (0, 2, 3)}
     assert not (out / "1.f32").exists()
-    assert_close(got[0], wa[[3, 89]], target[1])
+    assert_close(got[0], wa[[3, 89]], target[1], sure=sure[[3, 89]])
     assert_close(got[2], torch.stack([wa[96], wa[92], wb[1]]), target[1])
     assert_close(got[3], wb[[6]], target[1])
     assert len(eng.cache.free) == 4 and len(eng.cache.free_slots) == 4
