@@ -119,7 +119,7 @@ __global__ void gated_norm_kernel(const float* __restrict__ y, const T* __restri
       ldv<V>(y + (size_t)row * C + c, a);
       ldv<V>(z + (size_t)row * ldz + c, b);
       for (int e = 0; e < V; ++e) {
-        a[e] *= siluf(b[e]);
+        a[e] *= silu_t<sizeof(T) == 2>(b[e]);
         ss += a[e] * a[e];
       }
       stv<V>(srow + c, a);
@@ -212,50 +212,77 @@ __global__ void conv_decode_kernel(const T* __restrict__ x, long long ld, const 
   for (int m = 0; m < K - 1; ++m) acc += w[(size_t)c * K + m] * (fresh ? 0.f : tl[m]);
   for (int m = 0; m + 1 < K - 1; ++m) tl[m] = fresh ? 0.f : tl[m + 1];
   if (K > 1) tl[K - 2] = cur;
-  stf(out + (size_t)row * C + c, silu ? siluf(acc) : acc);
+  stf(out + (size_t)row * C + c, silu ? silu_t<sizeof(T) == 2>(acc) : acc);
 }
 
-// Portions: a CTA walks the rows of one block (64 rows of one entry) for 128 channels, the last inputs in registers.
-// KT = taps (1..8), 0: any number, inputs re-read.
-template <typename T, int KT>
-__global__ void conv_prefill_kernel(const T* __restrict__ x, long long ld, const float* __restrict__ bin, const float* __restrict__ w,
-                                    const float* __restrict__ bias, int silu, const int* __restrict__ cu, const int* __restrict__ start,
-                                    const int* __restrict__ state, const int4* __restrict__ blocks, const float* __restrict__ tail,
-                                    T* __restrict__ out, int C, int Kdyn) {
+// Portions: a CTA walks the rows of one block (64 rows of one entry), every thread V neighbouring channels with their
+// last inputs in registers. KT = taps (1..4), 0: any number, inputs re-read.
+template <typename T, int KT, int V>
+__global__ void __launch_bounds__(128)
+conv_prefill_kernel(const T* __restrict__ x, long long ld, const float* __restrict__ bin, const float* __restrict__ w, const float* __restrict__ bias,
+                    int silu, const int* __restrict__ cu, const int* __restrict__ start, const int* __restrict__ state,
+                    const int4* __restrict__ blocks, const float* __restrict__ tail, T* __restrict__ out, int C, int Kdyn) {
   const int K = KT > 0 ? KT : Kdyn;
   const int4 blk = blocks[blockIdx.y];
-  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
   if (c >= C) return;
   const int e = blk.x, r0 = blk.y, n = blk.z, first = cu[e];
   const int slot = state[e];
   const bool fresh = start[e] <= 0;
-  const float bi = bin ? bin[c] : 0.f, b0 = bias[c];
+  float bi[V], b0[V];
+  for (int v = 0; v < V; ++v) {
+    bi[v] = bin ? bin[c + v] : 0.f;
+    b0[v] = bias[c + v];
+  }
   const float* tl = tail + ((size_t)slot * C + c) * (K - 1);
-  auto at = [&](int r) -> float {                       // input at row r of this entry (before its first row: the tail)
-    if (r >= first) return ldf(x + (size_t)r * ld + c) + bi;
-    const int m = K - 1 + (r - first);
-    return (fresh || m < 0) ? 0.f : tl[m];
+  auto at = [&](int r, float (&o)[V]) {                 // inputs at row r of this entry (before its first row: the tail)
+    if (r >= first) {
+      ldv<V>(x + (size_t)r * ld + c, o);
+      for (int v = 0; v < V; ++v) o[v] += bi[v];
+    } else {
+      const int m = K - 1 + (r - first);
+      for (int v = 0; v < V; ++v) o[v] = (fresh || m < 0) ? 0.f : tl[v * (K - 1) + m];
+    }
   };
   if constexpr (KT > 0) {
-    float wv[KT], win[KT];
+    float wv[KT][V], win[KT][V];
 #pragma unroll
-    for (int j = 0; j < KT; ++j) wv[j] = w[(size_t)c * KT + j];
+    for (int j = 0; j < KT; ++j)
 #pragma unroll
-    for (int j = 0; j < KT - 1; ++j) win[j + 1] = at(r0 - (KT - 1) + j);
+      for (int v = 0; v < V; ++v) wv[j][v] = w[(size_t)(c + v) * KT + j];
+#pragma unroll
+    for (int j = 0; j < KT - 1; ++j) at(r0 - (KT - 1) + j, win[j + 1]);
+    float nxt[V];
+    ldv<V>(x + (size_t)r0 * ld + c, nxt);
     for (int i = 0; i < n; ++i) {
 #pragma unroll
-      for (int j = 0; j < KT - 1; ++j) win[j] = win[j + 1];
-      win[KT - 1] = ldf(x + (size_t)(r0 + i) * ld + c) + bi;
-      float acc = b0;
+      for (int j = 0; j < KT - 1; ++j)
 #pragma unroll
-      for (int j = 0; j < KT; ++j) acc += wv[j] * win[j];
-      stf(out + (size_t)(r0 + i) * C + c, silu ? siluf(acc) : acc);
+        for (int v = 0; v < V; ++v) win[j][v] = win[j + 1][v];
+#pragma unroll
+      for (int v = 0; v < V; ++v) win[KT - 1][v] = nxt[v] + bi[v];
+      if (i + 1 < n) ldv<V>(x + (size_t)(r0 + i + 1) * ld + c, nxt);
+      float acc[V];
+#pragma unroll
+      for (int v = 0; v < V; ++v) {
+        acc[v] = b0[v];
+#pragma unroll
+        for (int j = 0; j < KT; ++j) acc[v] += wv[j][v] * win[j][v];
+        if (silu) acc[v] = silu_t<sizeof(T) == 2>(acc[v]);
+      }
+      stv<V>(out + (size_t)(r0 + i) * C + c, acc);
     }
   } else {
     for (int i = 0; i < n; ++i) {
-      float acc = b0;
-      for (int j = 0; j < K; ++j) acc += w[(size_t)c * K + j] * at(r0 + i - (K - 1) + j);
-      stf(out + (size_t)(r0 + i) * C + c, silu ? siluf(acc) : acc);
+      float acc[V], o[V];
+      for (int v = 0; v < V; ++v) acc[v] = b0[v];
+      for (int j = 0; j < K; ++j) {
+        at(r0 + i - (K - 1) + j, o);
+        for (int v = 0; v < V; ++v) acc[v] += w[(size_t)(c + v) * K + j] * o[v];
+      }
+      for (int v = 0; v < V; ++v)
+        if (silu) acc[v] = silu_t<sizeof(T) == 2>(acc[v]);
+      stv<V>(out + (size_t)(r0 + i) * C + c, acc);
     }
   }
 }
@@ -289,7 +316,11 @@ __global__ void xielu_kernel(const T* __restrict__ x, long long ld, const float*
     const int c = (int)(i - r * cv) * V;
     float v[V];
     ldv<V>(x + r * ld + c, v);
-    for (int e = 0; e < V; ++e) v[e] = 0.5f * v[e] + (v[e] > 0.f ? sp * v[e] * v[e] : sq * (expm1f(v[e]) - v[e]));
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      const float n = fminf(v[e], 0.f), q = v[e] > 0.f ? sp * v[e] * v[e] : sq * (expm1_neg<sizeof(T) == 2>(n) - n);
+      v[e] = 0.5f * v[e] + q;
+    }
     stv<V>(out + r * C + c, v);
   }
 }
@@ -305,7 +336,7 @@ __global__ void glu_silu_kernel(const T* __restrict__ gu, long long ld, T* __res
     float g[V], u[V];
     ldv<V>(gu + r * ld + c, g);
     ldv<V>(gu + r * ld + I + c, u);
-    for (int e = 0; e < V; ++e) g[e] = siluf(g[e]) * u[e];
+    for (int e = 0; e < V; ++e) g[e] = silu_t<sizeof(T) == 2>(g[e]) * u[e];
     stv<V>(out + r * I + c, g);
   }
 }
@@ -402,6 +433,12 @@ static inline int flat_grid(long long n) {
       if (vec) { constexpr int V = 4; __VA_ARGS__; } else { constexpr int V = 1; __VA_ARGS__; }                 \
     }                                                                                                        \
   } while (0)
+// as AB2_TYPED with a third width: V = 8 when `vec8`
+#define AB2_TYPED8(dt, vec8, vec, ...)                                                                       \
+  do {                                                                                                       \
+    if ((dt) == 0 && (vec8)) { using T = __nv_bfloat16; constexpr int V = 8; __VA_ARGS__; }                  \
+    else AB2_TYPED(dt, vec, __VA_ARGS__);                                                                    \
+  } while (0)
 #define AB2_DONE return cudaGetLastError() == cudaSuccess ? 0 : 1
 
 extern "C" {
@@ -450,7 +487,7 @@ int ab2_qk_norm_append(const void* qkv, long long ld, const float* wq, const flo
   if (R <= 0) return 0;
   const int eb = dt == 0 ? 2 : 4;
   const bool vec = nq % 4 == 0 && nk % 4 == 0 && nv % 4 == 0 && ld % 4 == 0 && aligned_to(qkv, 4 * eb);
-  AB2_TYPED(dt, vec, {
+  AB2_TYPED8(dt, nq % 8 == 0 && nk % 8 == 0 && nv % 8 == 0 && ld % 8 == 0 && aligned_to(qkv, 16), vec, {
     launch_pdl(qk_norm_append_kernel<T, V>, dim3(R), dim3(256), 0, (cudaStream_t)stream, (const T*)qkv, ld, wq, wk, slots, (T*)q, (T*)kc, (T*)vc, nq,
                nk, nv, eps);
   });
@@ -475,18 +512,17 @@ int ab2_causal_conv(const void* x, long long ld, const float* bin, const float* 
   }
   if (nb > 0) {
     if (nb > 65535 || n_entries - n_dec > 65535) return 11;
-#define AB2_CONV(TT, KK) conv_prefill_kernel<TT, KK><<<dim3(gx, nb), 128, 0, s>>>((const TT*)x, ld, bin, w, bias, silu, cu, start, state, \
-                                                                              (const int4*)blocks, tail, (TT*)out, C, K)
-#define AB2_CONV_K(TT)                                                                         \
-  switch (K) {                                                                                 \
-    case 1: AB2_CONV(TT, 1); break;                                                            \
-    case 2: AB2_CONV(TT, 2); break;                                                            \
-    case 3: AB2_CONV(TT, 3); break;                                                            \
-    case 4: AB2_CONV(TT, 4); break;                                                            \
-    default: AB2_CONV(TT, 0);                                                                  \
-  }
-    if (dt == 0) { AB2_CONV_K(__nv_bfloat16) } else { AB2_CONV_K(float) }
-#undef AB2_CONV_K
+    const bool vec = C % 4 == 0 && ld % 4 == 0 && aligned_to(x, dt == 0 ? 8 : 16);
+#define AB2_CONV(KK)                                                                                                                       \
+  AB2_TYPED(dt, vec, conv_prefill_kernel<T, KK, V><<<dim3((C / V + 127) / 128, nb), 128, 0, s>>>((const T*)x, ld, bin, w, bias, silu, cu, start, \
+                                                                                                 state, (const int4*)blocks, tail, (T*)out, C, K))
+    switch (K) {
+      case 1: AB2_CONV(1); break;
+      case 2: AB2_CONV(2); break;
+      case 3: AB2_CONV(3); break;
+      case 4: AB2_CONV(4); break;
+      default: AB2_CONV(0);
+    }
 #undef AB2_CONV
     if (K > 1) {
       if (dt == 0)
@@ -502,7 +538,7 @@ int ab2_xielu(const void* x, long long ld, const float* pq, void* out, int R, in
   if (R <= 0) return 0;
   const int eb = dt == 0 ? 2 : 4;
   const bool vec = C % 4 == 0 && ld % 4 == 0 && aligned_to(x, 4 * eb);
-  AB2_TYPED(dt, vec, {
+  AB2_TYPED8(dt, C % 8 == 0 && ld % 8 == 0 && aligned_to(x, 16), vec, {
     const long long n = (long long)R * (C / V);
     launch_pdl(xielu_kernel<T, V>, dim3(flat_grid(n)), dim3(256), 0, (cudaStream_t)stream, (const T*)x, ld, pq, (T*)out, n, C);
   });
@@ -513,7 +549,7 @@ int ab2_glu_silu(const void* gu, long long ld, void* out, int R, int I, int dt, 
   if (R <= 0) return 0;
   const int eb = dt == 0 ? 2 : 4;
   const bool vec = I % 4 == 0 && ld % 4 == 0 && aligned_to(gu, 4 * eb);
-  AB2_TYPED(dt, vec, {
+  AB2_TYPED8(dt, I % 8 == 0 && ld % 8 == 0 && aligned_to(gu, 16), vec, {
     const long long n = (long long)R * (I / V);
     launch_pdl(glu_silu_kernel<T, V>, dim3(flat_grid(n)), dim3(256), 0, (cudaStream_t)stream, (const T*)gu, ld, (T*)out, n, I);
   });
@@ -522,7 +558,7 @@ int ab2_glu_silu(const void* gu, long long ld, void* out, int R, int I, int dt, 
 
 int ab2_expert_combine(const void* y, const int* inv, const float* topw, void* out, int T_, int k, int H, int dt, void* stream) {
   if (T_ <= 0) return 0;
-  AB2_TYPED(dt, H % 4 == 0, {
+  AB2_TYPED8(dt, H % 8 == 0, H % 4 == 0, {
     const long long n = (long long)T_ * (H / V);
     launch_pdl(expert_combine_kernel<T, V>, dim3(flat_grid(n)), dim3(256), 0, (cudaStream_t)stream, (const T*)y, inv, topw, (T*)out, n, k, H, T_ * k);
   });

@@ -7,35 +7,25 @@ namespace ab2 {
 // ------------------------------------------------------------------ RG-LRU gates
 // One CTA: 64 rows x 32 channels of one block of the block-diagonal gate matrices, both gates at once (64 product
 // columns: 32 of r, 32 of i), so the thread that holds r of a channel also holds its i. The epilogue turns the two
-// logits into the decay a = exp(-8 r softplus(lam)) and the input sqrt(1 - a^2) i u, and either stores both for the
-// scan or (single-token rows) advances the state at once.
+// logits into the decay a = exp(-8 r softplus(lam)) and the input sqrt(1 - a^2) i u. Single-token rows advance their
+// state at once; for portions the 64 rows are one block of the scan, and the CTA scans them from zero before it stores
+// (running product of a, state from zero).
 constexpr int GT_R = 64, GT_C = 32, GT_K = 64;
 
 struct GateEpi {
   const float *gb, *lam, *yb;
   const int *start, *state;
-  float *S, *a, *x;
-  int W, bs, nblk;
+  const int4* blocks;
+  float *S, *a, *x, *carry;
+  int W, bs, nblk, row0, nb;
 };
 
-template <typename T, bool DECODE>
-__device__ __forceinline__ void gate_epilogue(const GateEpi& p, const T* u, const T* y, long long ldy, T* out, int row, int ch, float zr, float zi) {
-  const float r = sigmoidf(zr + p.gb[ch]), i = sigmoidf(zi + p.gb[p.W + ch]);
-  const float la = -8.f * r * softplusf(p.lam[ch]);
-  const float a = expf(la);
-  const float xin = sqrtf(-expm1f(2.f * la)) * i * ldf(u + (size_t)row * p.W + ch);
-  const size_t o = (size_t)row * p.W + ch;
-  if constexpr (DECODE) {
-    const int slot = p.state[row];
-    if (slot < 0) { stf(out + o, 0.f); return; }
-    float* s = p.S + (size_t)slot * p.W + ch;
-    const float h = (p.start[row] > 0 ? a * *s : 0.f) + xin;
-    *s = h;
-    stf(out + o, h * gelu_tanhf(ldf(y + (size_t)row * ldy + ch) + p.yb[ch]));
-  } else {
-    p.a[o] = a;
-    p.x[o] = xin;
-  }
+// decay and scaled input of one channel; nsp = -8 softplus(lam)
+template <bool FAST>
+__device__ __forceinline__ void gate_values(float zr, float zi, float nsp, float u, float& a, float& xin) {
+  const float la = nsp * sigmoid_t<FAST>(zr);
+  a = exp_t<FAST>(la);
+  xin = sqrtf(-expm1_neg<FAST>(2.f * la)) * sigmoid_t<FAST>(zi) * u;
 }
 
 template <typename T, bool DECODE>
@@ -43,13 +33,29 @@ __global__ void __launch_bounds__(128)
 rglru_gate_kernel(const T* __restrict__ u, const T* __restrict__ y, long long ldy, const T* __restrict__ gw, GateEpi p, T* __restrict__ out, int R) {
   constexpr bool MMA = sizeof(T) == 2;
   constexpr int LD = MMA ? GT_K + 8 : GT_K + 1;          // padded rows: no bank conflicts on fragment reads
-  __shared__ __align__(16) T sA[GT_R * LD];
-  __shared__ __align__(16) T sB[2 * GT_C * LD];
+  constexpr int SCAN_BYTES = DECODE ? 0 : 2 * GT_R * (GT_C + 1) * 4;       // a and x of the block, over the operands
+  constexpr int OP_BYTES = (GT_R + 2 * GT_C) * LD * (int)sizeof(T);
+  __shared__ __align__(16) unsigned char s_raw[OP_BYTES > SCAN_BYTES ? OP_BYTES : SCAN_BYTES];
+  __shared__ float s_par[3][GT_C];                       // r bias, i bias, -8 softplus(lam)
+  T* sA = reinterpret_cast<T*>(s_raw);
+  T* sB = sA + GT_R * LD;
   pdl_wait();
   pdl_trigger();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int cpb = (p.bs + GT_C - 1) / GT_C;              // channel tiles per block
-  const int blk = blockIdx.x / cpb, c0 = (blockIdx.x % cpb) * GT_C, r0 = blockIdx.y * GT_R;
+  const int blk = blockIdx.x / cpb, c0 = (blockIdx.x % cpb) * GT_C;
+  int r0 = blockIdx.y * GT_R;
+  if constexpr (!DECODE) {
+    const int4 b = p.blocks[blockIdx.y];
+    r0 = b.y - p.row0;
+    R = r0 + b.z;
+  }
+  if (tid < GT_C && c0 + tid < p.bs) {
+    const int ch = blk * p.bs + c0 + tid;
+    s_par[0][tid] = p.gb[ch];
+    s_par[1][tid] = p.gb[p.W + ch];
+    s_par[2][tid] = -8.f * softplusf(p.lam[ch]);
+  }
   const T zero = T(0.f);
   float acc[8][4];
 #pragma unroll
@@ -112,48 +118,83 @@ rglru_gate_kernel(const T* __restrict__ u, const T* __restrict__ y, long long ld
     }
     __syncthreads();
   }
+  float* s_a = reinterpret_cast<float*>(s_raw);
+  float* s_x = s_a + GT_R * (GT_C + 1);
+  auto finish = [&](int rr, int c, float zr, float zi) {   // row rr and channel c of the tile
+    const int row = r0 + rr, ch = blk * p.bs + c0 + c;
+    float a = 1.f, xin = 0.f;
+    if (row < R && c0 + c < p.bs)
+      gate_values<MMA>(zr + s_par[0][c], zi + s_par[1][c], s_par[2][c], ldf(u + (size_t)row * p.W + ch), a, xin);
+    if constexpr (DECODE) {
+      if (row >= R || c0 + c >= p.bs) return;
+      const int slot = p.state[row];
+      T* o = out + (size_t)row * p.W + ch;
+      if (slot < 0) { stf(o, 0.f); return; }
+      float* s = p.S + (size_t)slot * p.W + ch;
+      const float h = (p.start[row] > 0 ? a * *s : 0.f) + xin;
+      *s = h;
+      stf(o, h * gelu_tanh_t<MMA>(ldf(y + (size_t)row * ldy + ch) + p.yb[ch]));
+    } else {
+      s_a[rr * (GT_C + 1) + c] = a;
+      s_x[rr * (GT_C + 1) + c] = xin;
+    }
+  };
   if constexpr (MMA) {
     const int gq = lane >> 2, tq = lane & 3;
 #pragma unroll
     for (int t = 0; t < 4; ++t)
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int row = r0 + warp * 16 + gq + (j >> 1) * 8, c = c0 + t * 8 + tq * 2 + (j & 1);
-        if (row < R && c < p.bs) gate_epilogue<T, DECODE>(p, u, y, ldy, out, row, blk * p.bs + c, acc[t][j], acc[t + 4][j]);
-      }
+      for (int j = 0; j < 4; ++j) finish(warp * 16 + gq + (j >> 1) * 8, t * 8 + tq * 2 + (j & 1), acc[t][j], acc[t + 4][j]);
   } else {
     const int tx = tid & 7, ty = tid >> 3;
 #pragma unroll
     for (int j = 0; j < 4; ++j)
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int row = r0 + ty * 4 + i, c = c0 + tx + 8 * j;
-        if (row < R && c < p.bs) gate_epilogue<T, DECODE>(p, u, y, ldy, out, row, blk * p.bs + c, acc[j][i], acc[j + 4][i]);
+      for (int i = 0; i < 4; ++i) finish(ty * 4 + i, tx + 8 * j, acc[j][i], acc[j + 4][i]);
+  }
+  if constexpr (!DECODE) {
+    // a warp scans 16 of the 64 rows, a lane one channel; the warps' ends are chained through shared memory
+    __shared__ float s_end[2][4][GT_C];
+    __syncthreads();
+    float pa[16], hx[16], P = 1.f, h = 0.f;
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      const int o = (warp * 16 + i) * (GT_C + 1) + lane;
+      const float at = s_a[o];
+      h = at * h + s_x[o];
+      P *= at;
+      pa[i] = P;
+      hx[i] = h;
+    }
+    s_end[0][warp][lane] = P;
+    s_end[1][warp][lane] = h;
+    __syncthreads();
+    float Pp = 1.f, hp = 0.f;
+    for (int w = 0; w < warp; ++w) {
+      hp = s_end[0][w][lane] * hp + s_end[1][w][lane];
+      Pp *= s_end[0][w][lane];
+    }
+    if (c0 + lane < p.bs) {
+      const int ch = blk * p.bs + c0 + lane;
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        const int row = r0 + warp * 16 + i;
+        if (row < R) {
+          p.a[(size_t)row * p.W + ch] = pa[i] * Pp;
+          p.x[(size_t)row * p.W + ch] = hx[i] + pa[i] * hp;
+        }
       }
+      if (warp == 3) {                                     // rows past the block's end have a = 1, x = 0
+        p.carry[(size_t)blockIdx.y * p.W + ch] = pa[15] * Pp;
+        p.carry[((size_t)p.nb + blockIdx.y) * p.W + ch] = hx[15] + pa[15] * hp;
+      }
+    }
   }
 }
 
-// Blocked scan h = a h + x over the 64-row blocks of every portion: per block the product of a and the state from
-// zero; the states between blocks; then every block from its true start, gated on the way out. Row indices of
-// `blocks` count from the first row of the step, a / x / y / out from row0.
-__global__ void __launch_bounds__(128)
-lru_block_kernel(const float* __restrict__ a, const float* __restrict__ x, const int4* __restrict__ blocks, int row0, float* __restrict__ carry, int nb,
-                 int W) {
-  const int4 b = blocks[blockIdx.y];
-  const int c = blockIdx.x * 128 + threadIdx.x;
-  if (c >= W) return;
-  float A = 1.f, h = 0.f;
-  const size_t o = (size_t)(b.y - row0) * W + c;
-#pragma unroll 8
-  for (int t = 0; t < b.z; ++t) {
-    const float at = a[o + (size_t)t * W];
-    h = at * h + x[o + (size_t)t * W];
-    A *= at;
-  }
-  carry[(size_t)blockIdx.y * W + c] = A;
-  carry[((size_t)nb + blockIdx.y) * W + c] = h;
-}
-
+// The states between the blocks of every portion (carry: product and state of each block, then the state before it),
+// and the rows from their block's true start, gated on the way out. Row indices of `blocks` count from the first row of
+// the step, a / x / y / out from row0.
 __global__ void __launch_bounds__(128)
 lru_carry_kernel(const int4* __restrict__ blocks, const int* __restrict__ start, const int* __restrict__ state, float* __restrict__ S,
                  float* __restrict__ carry, int nb, int W) {
@@ -171,21 +212,27 @@ lru_carry_kernel(const int4* __restrict__ blocks, const int* __restrict__ start,
   }
 }
 
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(128)
 lru_apply_kernel(const float* __restrict__ a, const float* __restrict__ x, const int4* __restrict__ blocks, int row0, const float* __restrict__ carry,
                  const T* __restrict__ y, long long ldy, const float* __restrict__ yb, T* __restrict__ out, int W) {
   const int4 b = blocks[blockIdx.y];
-  const int c = blockIdx.x * 128 + threadIdx.x;
+  const int c = (blockIdx.x * 128 + threadIdx.x) * V;
   if (c >= W) return;
-  float h = carry[(size_t)blockIdx.y * W + c];
-  const float bias = yb[c];
+  float h0[V], bias[V];
+  ldv<V>(carry + (size_t)blockIdx.y * W + c, h0);
+  ldv<V>(yb + c, bias);
   const int r0 = b.y - row0;
-#pragma unroll 4
-  for (int t = 0; t < b.z; ++t) {
+#pragma unroll 2
+  for (int t = blockIdx.z; t < b.z; t += gridDim.z) {
     const size_t o = (size_t)(r0 + t) * W + c;
-    h = a[o] * h + x[o];
-    stf(out + o, h * gelu_tanhf(ldf(y + (size_t)(r0 + t) * ldy + c) + bias));
+    float av[V], xv[V], yv[V];
+    ldv<V>(a + o, av);
+    ldv<V>(x + o, xv);
+    ldv<V>(y + (size_t)(r0 + t) * ldy + c, yv);
+#pragma unroll
+    for (int v = 0; v < V; ++v) yv[v] = (av[v] * h0[v] + xv[v]) * gelu_tanh_t<sizeof(T) == 2>(yv[v] + bias[v]);
+    stv<V>(out + o, yv);
   }
 }
 
@@ -269,16 +316,23 @@ mamba2_scan_kernel(const T* __restrict__ xbc, long long ldx, const T* __restrict
     }
 }
 
-template <typename T>
-static int launch_rglru(bool decode, const void* u, const void* y, long long ldy, const float* yb, const void* gw, const float* gb, const float* lam,
-                        const int* start, const int* state, float* S, float* a, float* x, void* out, int R, int n, int bs, cudaStream_t s) {
-  const dim3 grid(n * ((bs + GT_C - 1) / GT_C), (R + GT_R - 1) / GT_R);
+template <typename T, bool DECODE>
+static int launch_gates(const void* u, const void* y, long long ldy, const void* gw, const GateEpi& p, void* out, int R, cudaStream_t s) {
+  const dim3 grid(p.nblk * ((p.bs + GT_C - 1) / GT_C), DECODE ? (R + GT_R - 1) / GT_R : p.nb);
   if (grid.y > 65535) return 11;
-  GateEpi p{gb, lam, yb, start, state, S, a, x, n * bs, bs, n};
-  if (decode)
-    launch_pdl(rglru_gate_kernel<T, true>, grid, dim3(128), 0, s, (const T*)u, (const T*)y, ldy, (const T*)gw, p, (T*)out, R);
+  launch_pdl(rglru_gate_kernel<T, DECODE>, grid, dim3(128), 0, s, (const T*)u, (const T*)y, ldy, (const T*)gw, p, (T*)out, R);
+  return cudaGetLastError() == cudaSuccess ? 0 : 1;
+}
+
+template <typename T>
+static int launch_lru_prefill(const void* u, const void* y, long long ldy, const void* gw, const GateEpi& p, void* out, cudaStream_t s) {
+  if (const int rc = launch_gates<T, false>(u, y, ldy, gw, p, out, 0, s)) return rc;
+  lru_carry_kernel<<<(p.W + 127) / 128, 128, 0, s>>>(p.blocks, p.start, p.state, p.S, p.carry, p.nb, p.W);
+  const bool vec = p.W % 4 == 0 && ldy % 4 == 0 && aligned_to(y, 16) && aligned_to(out, 16) && aligned_to(p.yb, 16);
+  if (vec)
+    lru_apply_kernel<T, 4><<<dim3((p.W / 4 + 127) / 128, p.nb, 4), 128, 0, s>>>(p.a, p.x, p.blocks, p.row0, p.carry, (const T*)y, ldy, p.yb, (T*)out, p.W);
   else
-    launch_pdl(rglru_gate_kernel<T, false>, grid, dim3(128), 0, s, (const T*)u, (const T*)y, ldy, (const T*)gw, p, (T*)out, R);
+    lru_apply_kernel<T, 1><<<dim3((p.W + 127) / 128, p.nb, 1), 128, 0, s>>>(p.a, p.x, p.blocks, p.row0, p.carry, (const T*)y, ldy, p.yb, (T*)out, p.W);
   return cudaGetLastError() == cudaSuccess ? 0 : 1;
 }
 
@@ -291,8 +345,10 @@ using namespace ab2;
 int ab2_rglru_decode(const void* u, const void* y, long long ldy, const float* yb, const void* gw, const float* gb, const float* lam,
                      const int* start, const int* state, float* S, void* out, int R, int n, int bs, int dt, void* stream) {
   if (R <= 0) return 0;
-  return dt == 0 ? launch_rglru<__nv_bfloat16>(true, u, y, ldy, yb, gw, gb, lam, start, state, S, nullptr, nullptr, out, R, n, bs, (cudaStream_t)stream)
-                 : launch_rglru<float>(true, u, y, ldy, yb, gw, gb, lam, start, state, S, nullptr, nullptr, out, R, n, bs, (cudaStream_t)stream);
+  GateEpi p{};
+  p.gb = gb; p.lam = lam; p.yb = yb; p.start = start; p.state = state; p.S = S; p.W = n * bs; p.bs = bs; p.nblk = n;
+  return dt == 0 ? launch_gates<__nv_bfloat16, true>(u, y, ldy, gw, p, out, R, (cudaStream_t)stream)
+                 : launch_gates<float, true>(u, y, ldy, gw, p, out, R, (cudaStream_t)stream);
 }
 
 // Portions: R rows from row row0 of the step on, in nb blocks. a, x [R, W] and carry [2, nb, W] are scratch.
@@ -302,18 +358,10 @@ int ab2_rglru_prefill(const void* u, const void* y, long long ldy, const float* 
   if (R <= 0 || nb <= 0) return 0;
   if (nb > 65535) return 11;
   cudaStream_t s = (cudaStream_t)stream;
-  const int W = n * bs, gx = (W + 127) / 128;
-  const int rc = dt == 0 ? launch_rglru<__nv_bfloat16>(false, u, y, ldy, yb, gw, gb, lam, start, state, S, a, x, out, R, n, bs, s)
-                         : launch_rglru<float>(false, u, y, ldy, yb, gw, gb, lam, start, state, S, a, x, out, R, n, bs, s);
-  if (rc) return rc;
-  lru_block_kernel<<<dim3(gx, nb), 128, 0, s>>>(a, x, (const int4*)blocks, row0, carry, nb, W);
-  lru_carry_kernel<<<gx, 128, 0, s>>>((const int4*)blocks, start, state, S, carry, nb, W);
-  if (dt == 0)
-    lru_apply_kernel<__nv_bfloat16><<<dim3(gx, nb), 128, 0, s>>>(a, x, (const int4*)blocks, row0, carry, (const __nv_bfloat16*)y, ldy, yb,
-                                                                 (__nv_bfloat16*)out, W);
-  else
-    lru_apply_kernel<float><<<dim3(gx, nb), 128, 0, s>>>(a, x, (const int4*)blocks, row0, carry, (const float*)y, ldy, yb, (float*)out, W);
-  return cudaGetLastError() == cudaSuccess ? 0 : 1;
+  GateEpi p{};
+  p.gb = gb; p.lam = lam; p.yb = yb; p.start = start; p.state = state; p.S = S; p.W = n * bs; p.bs = bs; p.nblk = n;
+  p.blocks = (const int4*)blocks; p.nb = nb; p.row0 = row0; p.a = a; p.x = x; p.carry = carry;
+  return dt == 0 ? launch_lru_prefill<__nv_bfloat16>(u, y, ldy, gw, p, out, s) : launch_lru_prefill<float>(u, y, ldy, gw, p, out, s);
 }
 
 // Entries 0 .. E - 1, each over its rows. xbc rows: x [H * P] | B [G * N] | C [G * N]; S [slots, H, P, N]; y [rows, H * P] fp32.

@@ -282,23 +282,15 @@ def mamba2_scan(xbc, dt_raw, dt_bias, A_log, D, heads: int, vdim: int, state: in
             S[sl] = h
         return y.reshape(R, inner)
     y = torch.empty(R, inner, device=xbc.device, dtype=torch.float32)
-    nb = 0 if b.blocks is None else b.blocks.shape[0]
-    common = (heads, vdim, state, groups, _dt(xbc))
-    nd = b.n_dec
-    if nb and xbc.dtype == torch.bfloat16 and MAMBA2_BLOCKED and vdim % 16 == 0 and vdim <= 128 and state % 16 == 0 and state <= 128:
-        if nd:
-            _call("ab2_mamba2_scan", _p(xbc), xbc.stride(0), _p(dt_raw), dt_raw.stride(0), _p(dt_bias), _p(A_log), _p(D), _p(b.cu), _p(b.start),
-                  _p(b.state), nd, _p(S), _p(y), *common)
-        ws = torch.empty(nb * heads * (state * vdim + 1), device=xbc.device, dtype=torch.float32)
-        _call("ab2_mamba2_blocked", _p(xbc), xbc.stride(0), _p(dt_raw), dt_raw.stride(0), _p(dt_bias), _p(A_log), _p(D), _p(b.blocks), nb, nd,
-              b.n_entries, _p(b.start), _p(b.state), _p(S), _p(ws), _p(y), *common)
-        return y
-    _call("ab2_mamba2_scan", _p(xbc), xbc.stride(0), _p(dt_raw), dt_raw.stride(0), _p(dt_bias), _p(A_log), _p(D), _p(b.cu), _p(b.start),
-          _p(b.state), b.n_entries, _p(S), _p(y), *common)
+    args = (_p(xbc), xbc.stride(0), _p(dt_raw), dt_raw.stride(0), _p(dt_bias), _p(A_log), _p(D), _p(b.cu), _p(b.start), _p(b.state))
+    E, nd = b.n_entries, b.n_dec
+    if E > nd and xbc.dtype == torch.bfloat16 and vdim % 8 == 0 and state % 8 == 0 and state <= 128 and xbc.stride(0) % 8 == 0:
+        # portions in blocks on the tensor cores, single tokens with one pass over their state
+        _call("ab2_mamba2_ssd", *args, nd, E, _p(S), _p(y), heads, vdim, state, groups)
+        E = nd
+    if E:
+        _call("ab2_mamba2_scan", *args, E, _p(S), _p(y), heads, vdim, state, groups, _dt(xbc))
     return y
-
-
-MAMBA2_BLOCKED = False
 
 
 def gated_group_norm(y, z, w, groups: int, eps: float):
@@ -376,7 +368,7 @@ for _n, _a in {
     "ab2_rglru_decode": [_V, _V, _lib.c_ll] + [_V] * 8 + [_I] * 4,
     "ab2_rglru_prefill": [_V, _V, _lib.c_ll] + [_V] * 5 + [_I] * 3 + [_V] * 7 + [_I] * 3,
     "ab2_mamba2_scan": [_V, _lib.c_ll, _V, _lib.c_ll] + [_V] * 6 + [_I] + [_V] * 2 + [_I] * 5,
-    "ab2_mamba2_blocked": [_V, _lib.c_ll, _V, _lib.c_ll] + [_V] * 4 + [_I] * 3 + [_V] * 5 + [_I] * 5,
+    "ab2_mamba2_ssd": [_V, _lib.c_ll, _V, _lib.c_ll] + [_V] * 6 + [_I, _I] + [_V] * 2 + [_I] * 4,
     "ab2_gated_group_norm": [_V, _V, _lib.c_ll, _V, _V, _I, _I, _I, _F, _I],
     "ab2_xielu": [_V, _lib.c_ll, _V, _V, _I, _I, _I],
     "ab2_glu_silu": [_V, _lib.c_ll, _V, _I, _I, _I],
