@@ -43,7 +43,7 @@ from .state_cache import Carried, PagePool, StateCache
 logger = alog.getLogger("infer_engine")
 
 
-@dataclass
+@dataclass(eq=False)
 class _Seq:
     rid: str
     tokens: list[int]                      # prompt + generated so far
@@ -136,6 +136,7 @@ class NativeInferenceEngine(InferenceEngine):
         self.cache: Optional[PagePool] = None
         self.runner: Optional[RaggedRunner] = None
         self._ragged = False
+        self._sampled: list = []            # mixer stacks: requests whose sampling parameters the device buffers hold
 
     # ------------------------------------------------------------------ lifecycle
     def initialize(self, device=None, seed: int = 1, train_data_parallel_size: int = 1, model_path: Optional[str] = None,
@@ -807,7 +808,13 @@ class NativeInferenceEngine(InferenceEngine):
         done: list = []
         if ready:
             if self.device.type == "cuda":
-                toks, lps = self._sample_cuda(logits, ready)
+                if ready == self._sampled and all(s.top_p >= 1.0 and s.top_k <= 0 for s in ready):
+                    # the rows of the step before: their sampling parameters are on the device
+                    self._sample_rows(logits, len(ready), self.s_inv_temp, self.s_greedy, self.s_seeds)
+                    toks, lps = self._fetch_samples(len(ready))
+                else:
+                    toks, lps = self._sample_cuda(logits, ready)
+                    self._sampled = ready
             else:
                 self._step += 1
                 toks, lps = zip(*[self._sample_cpu(logits[i], s) for i, s in enumerate(ready)])

@@ -191,6 +191,8 @@ def main(argv=None):
     ap.add_argument("--port", type=int, default=0)
     ap.add_argument("--max-running-requests", type=int, default=256)
     ap.add_argument("--context-length", type=int, default=32768)
+    ap.add_argument("--compute-dtype", choices=["bfloat16", "float32"], default="bfloat16", help="float32: 32-bit compute (mixer stacks only)")
+    ap.add_argument("--max-prefill-tokens", type=int, default=16384, help="prompt tokens absorbed per engine step")
     ap.add_argument("--mem-fraction-static", type=float, default=0.85)
     ap.add_argument("--experiment-name", default="")
     ap.add_argument("--trial-name", default="")
@@ -203,6 +205,8 @@ def main(argv=None):
     mc = preset(a.preset) if a.preset else None
     eng = NativeInferenceEngine(InferenceEngineConfig(), NativeInferConfig(max_running_requests=a.max_running_requests,
                                                                            context_length=a.context_length,
+                                                                           compute_dtype=a.compute_dtype,
+                                                                           max_prefill_tokens=a.max_prefill_tokens,
                                                                            mem_fraction_static=a.mem_fraction_static),
                                 model_config=mc)
     eng.initialize(model_path=a.model_path or None, seed=a.seed, start_executor=False)

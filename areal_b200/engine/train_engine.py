@@ -363,6 +363,8 @@ class B200TrainEngine(TrainEngine):
                 model_config = ModelConfig.from_pretrained(cfg.path)
             else:
                 raise ValueError("no model architecture: give model_config, config.model_config or a checkpoint path")
+        if model_config.is_mixer_stack:
+            raise NotImplementedError(f"{model_config.arch}: mixer stacks are served, not trained (their ops have no backward pass)")
         if cfg.is_critic:
             model_config.is_critic = True
             model_config.tie_word_embeddings = False

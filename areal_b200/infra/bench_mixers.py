@@ -63,7 +63,7 @@ def _batch(lens, starts, dev, page_size=64):
     return RaggedRunner._layout(r, ents)[0], at * page_size
 
 
-def kernel_table(cfg, prefill=(4, 2048), decode=(64, 1024), dev="cuda") -> list[dict]:
+def kernel_table(cfg, prefill=(4, 2048), decode=(64, 960), dev="cuda") -> list[dict]:
     """Time, roofline time and fraction of the new design's kernels, each beside the like kernel of the existing models.
     ``prefill`` = (sequences, tokens each), ``decode`` = (sequences, cached tokens each)."""
     bw, fl, _ = peaks()
@@ -221,14 +221,13 @@ def mixer_steps(cfg, prefill, decode) -> dict:
                 eng.cache.grow(c, c.length + 1)
             eng.runner.step([Entry(c, [7], [0]) for c in cs])
         td = timed(one, iters=20, warmup=4)
-        t0 = time.perf_counter()
+        n0, t0 = oplib.launch_count(), time.perf_counter()
         for _ in range(10):
             one()
         torch.cuda.synchronize()
-        wall = (time.perf_counter() - t0) / 10
-    n = oplib.launch_count()
+        wall, n = (time.perf_counter() - t0) / 10, (oplib.launch_count() - n0) // 10
     out = dict(prefill_tokens_per_s=round(B * L / tp), prefill_ms=round(tp * 1e3, 3), decode_tokens_per_s=round(nB / td), decode_ms=round(td * 1e3, 3),
-               decode_wall_ms=round(wall * 1e3, 3), launches=n, params_m=round(sum(p.numel() for p in eng.model.parameters()) / 1e6, 1))
+               decode_wall_ms=round(wall * 1e3, 3), decode_launches=n, params_m=round(sum(p.numel() for p in eng.model.parameters()) / 1e6, 1))
     eng.destroy()
     return out
 
@@ -316,7 +315,7 @@ def run(steps=True, kernels=True, sizes=("kagolix-8b-layers", "kagolix-2b-layers
                sizes={})
     for name in sizes:
         cfg = preset(name)
-        prefill, decode = (4, 2048), (64, 1024)
+        prefill, decode = (4, 2048), (64, 960)
         r = dict(prefill=f"{prefill[0]} x {prefill[1]} tokens", decode=f"{decode[0]} sequences at {decode[1]} tokens")
         if steps:
             hyb, dense, routed = like_sized(cfg)

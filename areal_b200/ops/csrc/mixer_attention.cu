@@ -241,6 +241,11 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
     float alpha[2];
 #pragma unroll
     for (int hh = 0; hh < 2; ++hh) {
+      if (hh * 8 >= G) {                                // a group of up to 8 heads leaves the lower half of the tile empty
+        pa[hh] = pa[2 + hh] = 0u;
+        alpha[hh] = 1.f;
+        continue;
+      }
       float v[4];
       float mx = -INFINITY;
 #pragma unroll
@@ -630,7 +635,7 @@ template <int DK, int DV, bool CAP>
 static int launch_decode(const void* q, const int* pos, const int* slots, void* out, int R, const ChunkArgs& a, cudaStream_t s) {
   constexpr int SMEM = ChunkDecodeCfg<DK, DV>::SMEM;
   static_assert(2 * ChunkDecodeCfg<DK, DV>::STAGE >= (4 * 16 * DV + 8 * 16) * 4, "the merge buffers alias the stage memory");
-  const int spl = R * a.Hkv >= 444 ? 1 : (R * a.Hkv >= 111 ? 4 : 8);       // at least one wave of three CTAs per SM
+  const int spl = R * a.Hkv >= 1776 ? 1 : (R * a.Hkv >= 111 ? 4 : 8);      // several waves of three CTAs per SM, or all there is
   auto go = [&](auto kern, ab2host::DevState& st) -> int {
     if (ab2host::prepare_launch(kern, SMEM, st, nullptr)) return 300;
     launch_pdl(kern, dim3(R, a.Hkv, spl), dim3(128), (size_t)SMEM, s, (const __nv_bfloat16*)q, pos, slots, (__nv_bfloat16*)out, a);

@@ -198,18 +198,30 @@ rglru_gate_kernel(const T* __restrict__ u, const T* __restrict__ y, long long ld
 __global__ void __launch_bounds__(128)
 lru_carry_kernel(const int4* __restrict__ blocks, const int* __restrict__ start, const int* __restrict__ state, float* __restrict__ S,
                  float* __restrict__ carry, int nb, int W) {
-  const int c = blockIdx.x * 128 + threadIdx.x;
-  if (c >= W) return;
-  float h = 0.f;
-#pragma unroll 4
-  for (int k = 0; k < nb; ++k) {
-    const int4 b = blocks[k];
-    if (b.w) h = start[b.x] > 0 ? S[(size_t)state[b.x] * W + c] : 0.f;
-    const float A = carry[(size_t)k * W + c], x = carry[((size_t)nb + k) * W + c];
-    carry[(size_t)k * W + c] = h;                        // state before this block
-    h = A * h + x;
-    if (k + 1 == nb || blocks[k + 1].w) S[(size_t)state[b.x] * W + c] = h;
+  const int c = blockIdx.x * 128 + threadIdx.x, k0 = blockIdx.y;
+  const int4 b0 = blocks[k0];
+  if (c >= W || !b0.w) return;                            // one CTA row per entry: that of its first block
+  float* st = S + (size_t)state[b0.x] * W + c;
+  float h = start[b0.x] > 0 ? *st : 0.f;
+  bool more = true;
+  for (int k = k0; more; k += 8) {
+    float A[8], x[8];
+    int n = 0;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {                         // up to eight blocks' values before the chain of products
+      const bool in = more && k + i < nb && blocks[k + i].x == b0.x;
+      more = in;
+      n += in;
+      A[i] = in ? carry[(size_t)(k + i) * W + c] : 1.f;
+      x[i] = in ? carry[((size_t)nb + k + i) * W + c] : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      if (i < n) carry[(size_t)(k + i) * W + c] = h;      // state before the block
+      h = A[i] * h + x[i];
+    }
   }
+  *st = h;
 }
 
 template <typename T, int V>
@@ -327,7 +339,7 @@ static int launch_gates(const void* u, const void* y, long long ldy, const void*
 template <typename T>
 static int launch_lru_prefill(const void* u, const void* y, long long ldy, const void* gw, const GateEpi& p, void* out, cudaStream_t s) {
   if (const int rc = launch_gates<T, false>(u, y, ldy, gw, p, out, 0, s)) return rc;
-  lru_carry_kernel<<<(p.W + 127) / 128, 128, 0, s>>>(p.blocks, p.start, p.state, p.S, p.carry, p.nb, p.W);
+  lru_carry_kernel<<<dim3((p.W + 127) / 128, p.nb), 128, 0, s>>>(p.blocks, p.start, p.state, p.S, p.carry, p.nb, p.W);
   const bool vec = p.W % 4 == 0 && ldy % 4 == 0 && aligned_to(y, 16) && aligned_to(out, 16) && aligned_to(p.yb, 16);
   if (vec)
     lru_apply_kernel<T, 4><<<dim3((p.W / 4 + 127) / 128, p.nb, 4), 128, 0, s>>>(p.a, p.x, p.blocks, p.row0, p.carry, (const T*)y, ldy, p.yb, (T*)out, p.W);
