@@ -70,10 +70,13 @@ class RaggedRunner:
         slots = pt[row_entry, pos // ps - base[row_entry]].astype(np.int64) * ps + pos % ps if self.cache.has_kv else pos * 0
         n_dec = int((n == 1).sum())
         blocks, tiles = [], []
+        span = getattr(self.cache, "span", 0)
         for i in range(n_dec, len(entries)):
             for r in range(0, int(n[i]), SCAN_BLOCK):
                 blocks.append((i, cu[i] + r, min(SCAN_BLOCK, n[i] - r), int(r == 0)))
             tiles += [(i, cu[i] + r) for r in range(0, int(n[i]), ATTN_TILE)]
+        # tiles that see the most keys start first: the last ones to run are short
+        tiles.sort(key=lambda t: -(pos[t[1]] % span if span else pos[t[1]]))
         toks = np.concatenate([np.asarray(e.tokens, np.int64) for e in entries])
         state = np.array([e.carry.slot for e in entries])
         arrs = [toks, pos, slots, row_entry, cu, start, state, pt, base]

@@ -131,7 +131,7 @@ def feed_forward(W, pre, h, mlp, margins=None):
         p, q = W[pre + "act"]
         return xielu(h @ W[pre + "up"].T, p, q) @ W[pre + "down"].T
     chosen, weight = route(h, W[pre + "router"], W[pre + "correction"], mlp["router"]["top"])
-    if margins is not None:
+    if margins is not None and mlp["router"]["top"] < mlp["router"]["experts"]:
         c = torch.softmax(h @ W[pre + "router"].T, -1) + W[pre + "correction"]
         c = c.sort(-1, descending=True).values
         margins.append(c[:, mlp["router"]["top"] - 1] - c[:, mlp["router"]["top"]])
