@@ -241,7 +241,7 @@ static int launch_ssd(const void* xbc, long long ldx, const void* dtr, long long
 
 }  // namespace ab2
 
-// Entries e0 .. E - 1 (contract of ab2_mamba2_scan, bf16). P and N multiples of 8, N <= 128, rows of xbc 16-byte aligned.
+// Entries e0 .. E - 1 (arguments as of ab2_mamba2_scan, bf16). P and N multiples of 8, N <= 128, rows of xbc 16-byte aligned.
 extern "C" int ab2_mamba2_ssd(const void* xbc, long long ldx, const void* dtr, long long ldd, const float* dt_bias, const float* A_log, const float* D,
                               const int* cu, const int* start, const int* state, int e0, int E, float* S, float* y, int H, int P, int N, int G,
                               void* stream) {
