@@ -184,6 +184,7 @@ def run_reference(args):
 
 def run_mixer_serve():
     os.environ.setdefault("AB2_PDL", "1")
+    os.environ.setdefault("AB2_DECODE_SPLITK", "1")
     from areal_b200.infra.bench_mixers import run
 
     clocks = ClockSampler()
