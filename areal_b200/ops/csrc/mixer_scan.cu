@@ -12,6 +12,15 @@ namespace ab2 {
 // (running product of a, state from zero).
 constexpr int GT_R = 64, GT_C = 32, GT_K = 64;
 
+// Operand stages: bf16 operands are brought in by asynchronous copies, several 64-wide pieces ahead (single-token rows:
+// few CTAs, all pieces of a 256-wide block at once); the 32-bit form uses one stage.
+template <typename T, bool DECODE>
+struct GateCfg {
+  static constexpr int LD = sizeof(T) == 2 ? GT_K + 8 : GT_K + 1;          // padded rows: no bank conflicts on fragment reads
+  static constexpr int NS = sizeof(T) == 2 ? (DECODE ? 4 : 2) : 1;
+  static constexpr int OP_BYTES = (GT_R + 2 * GT_C) * LD * (int)sizeof(T);
+};
+
 struct GateEpi {
   const float *gb, *lam, *yb;
   const int *start, *state;
@@ -32,13 +41,11 @@ template <typename T, bool DECODE>
 __global__ void __launch_bounds__(128)
 rglru_gate_kernel(const T* __restrict__ u, const T* __restrict__ y, long long ldy, const T* __restrict__ gw, GateEpi p, T* __restrict__ out, int R) {
   constexpr bool MMA = sizeof(T) == 2;
-  constexpr int LD = MMA ? GT_K + 8 : GT_K + 1;          // padded rows: no bank conflicts on fragment reads
+  constexpr int LD = GateCfg<T, DECODE>::LD, NS = GateCfg<T, DECODE>::NS, OP_BYTES = GateCfg<T, DECODE>::OP_BYTES;
   constexpr int SCAN_BYTES = DECODE ? 0 : 2 * GT_R * (GT_C + 1) * 4;       // a and x of the block, over the operands
-  constexpr int OP_BYTES = (GT_R + 2 * GT_C) * LD * (int)sizeof(T);
-  __shared__ __align__(16) unsigned char s_raw[OP_BYTES > SCAN_BYTES ? OP_BYTES : SCAN_BYTES];
+  static_assert(NS * OP_BYTES >= SCAN_BYTES, "the scan's values fit over the operand stages");
+  extern __shared__ __align__(16) unsigned char s_raw[];     // NS operand stages
   __shared__ float s_par[3][GT_C];                       // r bias, i bias, -8 softplus(lam)
-  T* sA = reinterpret_cast<T*>(s_raw);
-  T* sB = sA + GT_R * LD;
   pdl_wait();
   pdl_trigger();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -62,19 +69,49 @@ rglru_gate_kernel(const T* __restrict__ u, const T* __restrict__ y, long long ld
   for (int i = 0; i < 8; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+  // element q of this thread's 16 results: row and channel of the tile (r in acc[q / 4][q % 4], i four columns on)
+  auto rr_of = [&](int q) { return MMA ? warp * 16 + (lane >> 2) + ((q & 3) >> 1) * 8 : (tid >> 3) * 4 + (q & 3); };
+  auto c_of = [&](int q) { return MMA ? (q >> 2) * 8 + (lane & 3) * 2 + (q & 1) : (tid & 7) + 8 * (q >> 2); };
   const bool vec = MMA && p.bs % 8 == 0 && p.W % 8 == 0;
-  for (int k0 = 0; k0 < p.bs; k0 += GT_K) {
-    if (vec) {
+  const int nk = (p.bs + GT_K - 1) / GT_K;
+  auto copy = [&](int kt) {                                // piece kt of both operands into its stage (vec only)
+    if (kt < nk) {
+      const uint32_t dA = smem_u32(s_raw) + (kt % NS) * OP_BYTES, dB = dA + GT_R * LD * (int)sizeof(T);
       for (int i = tid; i < GT_R * (GT_K / 8); i += 128) {
-        const int r = i / (GT_K / 8), k = (i % (GT_K / 8)) * 8;
-        uint4 v = make_uint4(0u, 0u, 0u, 0u);
-        if (r0 + r < R && k0 + k < p.bs) v = *reinterpret_cast<const uint4*>(u + (size_t)(r0 + r) * p.W + blk * p.bs + k0 + k);
-        *reinterpret_cast<uint4*>(sA + r * LD + k) = v;
-        const int g = r >> 5, c = c0 + (r & 31);          // 2 x 32 weight rows: as many as there are token rows
-        uint4 w = make_uint4(0u, 0u, 0u, 0u);
-        if (c < p.bs && k0 + k < p.bs) w = *reinterpret_cast<const uint4*>(gw + (((size_t)g * p.nblk + blk) * p.bs + c) * p.bs + k0 + k);
-        *reinterpret_cast<uint4*>(sB + r * LD + k) = w;
+        const int r = i / (GT_K / 8), kc = (i % (GT_K / 8)) * 8, k = kt * GT_K + kc;
+        const int g = r >> 5, c = c0 + (r & 31);           // 2 x 32 weight rows: as many as there are token rows
+        const bool oa = r0 + r < R && k < p.bs, ob = c < p.bs && k < p.bs;
+        const T* pa = oa ? u + (size_t)(r0 + r) * p.W + blk * p.bs + k : u;
+        const T* pb = ob ? gw + (((size_t)g * p.nblk + blk) * p.bs + c) * p.bs + k : gw;
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dA + (r * LD + kc) * (int)sizeof(T)), "l"(pa), "r"(oa ? 16 : 0) : "memory");
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dB + (r * LD + kc) * (int)sizeof(T)), "l"(pb), "r"(ob ? 16 : 0) : "memory");
       }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  if (vec)
+    for (int kt = 0; kt < NS - 1; ++kt) copy(kt);
+  // single-token rows: what the epilogue needs is asked for before the products, all of it at once
+  float ev_u[16], ev_y[16], ev_s[16];
+  int ev_slot[16];
+#pragma unroll
+  for (int q = 0; q < 16; ++q) {
+    const int row = r0 + rr_of(q), c = c0 + c_of(q), ch = blk * p.bs + c;
+    const bool in = row < R && c < p.bs;
+    ev_u[q] = in ? ldf(u + (size_t)row * p.W + ch) : 0.f;
+    if constexpr (DECODE) {
+      ev_slot[q] = in ? p.state[row] : -1;
+      ev_y[q] = in ? ldf(y + (size_t)row * ldy + ch) + p.yb[ch] : 0.f;
+      ev_s[q] = ev_slot[q] >= 0 && p.start[row] > 0 ? p.S[(size_t)ev_slot[q] * p.W + ch] : 0.f;
+    }
+  }
+  for (int kt = 0; kt < nk; ++kt) {
+    const int k0 = kt * GT_K;
+    T* sA = reinterpret_cast<T*>(s_raw + (vec ? (kt % NS) * OP_BYTES : 0));
+    T* sB = sA + GT_R * LD;
+    if (vec) {
+      copy(kt + NS - 1);                                   // its stage was read in the previous turn
+      asm volatile("cp.async.wait_group %0;" ::"n"(NS - 1) : "memory");
     } else {
       for (int i = tid; i < GT_R * GT_K; i += 128) {
         const int r = i / GT_K, k = i % GT_K;
@@ -120,37 +157,23 @@ rglru_gate_kernel(const T* __restrict__ u, const T* __restrict__ y, long long ld
   }
   float* s_a = reinterpret_cast<float*>(s_raw);
   float* s_x = s_a + GT_R * (GT_C + 1);
-  auto finish = [&](int rr, int c, float zr, float zi) {   // row rr and channel c of the tile
-    const int row = r0 + rr, ch = blk * p.bs + c0 + c;
+#pragma unroll
+  for (int q = 0; q < 16; ++q) {
+    const int rr = rr_of(q), c = c_of(q), row = r0 + rr;
+    const bool in = row < R && c0 + c < p.bs;
     float a = 1.f, xin = 0.f;
-    if (row < R && c0 + c < p.bs)
-      gate_values<MMA>(zr + s_par[0][c], zi + s_par[1][c], s_par[2][c], ldf(u + (size_t)row * p.W + ch), a, xin);
+    if (in) gate_values<MMA>(acc[q >> 2][q & 3] + s_par[0][c], acc[(q >> 2) + 4][q & 3] + s_par[1][c], s_par[2][c], ev_u[q], a, xin);
     if constexpr (DECODE) {
-      if (row >= R || c0 + c >= p.bs) return;
-      const int slot = p.state[row];
-      T* o = out + (size_t)row * p.W + ch;
-      if (slot < 0) { stf(o, 0.f); return; }
-      float* s = p.S + (size_t)slot * p.W + ch;
-      const float h = (p.start[row] > 0 ? a * *s : 0.f) + xin;
-      *s = h;
-      stf(o, h * gelu_tanh_t<MMA>(ldf(y + (size_t)row * ldy + ch) + p.yb[ch]));
+      if (in) {
+        const int ch = blk * p.bs + c0 + c;
+        const float h = a * ev_s[q] + xin;
+        if (ev_slot[q] >= 0) p.S[(size_t)ev_slot[q] * p.W + ch] = h;
+        stf(out + (size_t)row * p.W + ch, ev_slot[q] >= 0 ? h * gelu_tanh_t<MMA>(ev_y[q]) : 0.f);
+      }
     } else {
       s_a[rr * (GT_C + 1) + c] = a;
       s_x[rr * (GT_C + 1) + c] = xin;
     }
-  };
-  if constexpr (MMA) {
-    const int gq = lane >> 2, tq = lane & 3;
-#pragma unroll
-    for (int t = 0; t < 4; ++t)
-#pragma unroll
-      for (int j = 0; j < 4; ++j) finish(warp * 16 + gq + (j >> 1) * 8, t * 8 + tq * 2 + (j & 1), acc[t][j], acc[t + 4][j]);
-  } else {
-    const int tx = tid & 7, ty = tid >> 3;
-#pragma unroll
-    for (int j = 0; j < 4; ++j)
-#pragma unroll
-      for (int i = 0; i < 4; ++i) finish(ty * 4 + i, tx + 8 * j, acc[j][i], acc[j + 4][i]);
   }
   if constexpr (!DECODE) {
     // a warp scans 16 of the 64 rows, a lane one channel; the warps' ends are chained through shared memory
@@ -332,7 +355,11 @@ template <typename T, bool DECODE>
 static int launch_gates(const void* u, const void* y, long long ldy, const void* gw, const GateEpi& p, void* out, int R, cudaStream_t s) {
   const dim3 grid(p.nblk * ((p.bs + GT_C - 1) / GT_C), DECODE ? (R + GT_R - 1) / GT_R : p.nb);
   if (grid.y > 65535) return 11;
-  launch_pdl(rglru_gate_kernel<T, DECODE>, grid, dim3(128), 0, s, (const T*)u, (const T*)y, ldy, (const T*)gw, p, (T*)out, R);
+  auto kern = rglru_gate_kernel<T, DECODE>;
+  constexpr int SMEM = GateCfg<T, DECODE>::NS * GateCfg<T, DECODE>::OP_BYTES;
+  static ab2host::DevState st;
+  if (ab2host::prepare_launch(kern, SMEM, st, nullptr)) return 300;
+  launch_pdl(kern, grid, dim3(128), (size_t)SMEM, s, (const T*)u, (const T*)y, ldy, (const T*)gw, p, (T*)out, R);
   return cudaGetLastError() == cudaSuccess ? 0 : 1;
 }
 
