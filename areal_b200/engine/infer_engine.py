@@ -136,6 +136,7 @@ class NativeInferenceEngine(InferenceEngine):
         self.cache: Optional[PagePool] = None
         self.runner: Optional[RaggedRunner] = None
         self._ragged = False
+        self._context_limit = self.icfg.context_length
         self._sampled: list = []            # mixer stacks: requests whose sampling parameters the device buffers hold
 
     # ------------------------------------------------------------------ lifecycle
@@ -176,6 +177,8 @@ class NativeInferenceEngine(InferenceEngine):
         # step on that state (``_step_recurrent``).
         self._recompute_decode = bool(getattr(self.model_config, "is_hybrid", False))
         self._ragged = bool(getattr(self.model_config, "is_mixer_stack", False))
+        if getattr(self.model_config, "learned_positions", False):
+            self._context_limit = min(self._context_limit, self.model_config.max_position_embeddings)
         if self._ragged:
             self._init_ragged()
         elif self.device.type == "cuda" and not self._recompute_decode:
@@ -503,6 +506,8 @@ class NativeInferenceEngine(InferenceEngine):
         budget = min(g.max_tokens - len(prompt), g.max_new_tokens)
         if budget <= 0:
             raise ValueError(f"prompt of {len(prompt)} tokens leaves no room under max_tokens={g.max_tokens}")
+        if getattr(self.model_config, "learned_positions", False) and len(prompt) > self._context_limit:
+            raise ValueError(f"prompt of {len(prompt)} tokens is longer than the {self._context_limit} positions of the model")
         out_tok: list[int] = []
         out_lp: list[float] = []
         out_ver: list[int] = []
@@ -697,7 +702,7 @@ class NativeInferenceEngine(InferenceEngine):
                     return "stop"
         if n >= s.max_new:
             return "length"
-        if len(s.tokens) >= self.icfg.context_length:
+        if len(s.tokens) >= self._context_limit:
             return "length"
         return None
 

@@ -13,7 +13,7 @@ import numpy as np
 import torch
 
 from ..ops import lib as oplib
-from ..ops.mixer_ops import ATTN_TILE, SCAN_BLOCK, RaggedBatch
+from ..ops.mixer_ops import ATTN_TILE, SCAN_BLOCK, PageList, RaggedBatch
 from .state_cache import Carried, StateCache
 
 DECODE_BUCKETS = (1, 2, 4, 8, 16, 32, 64, 128, 256, 512)
@@ -31,6 +31,8 @@ class RaggedRunner:
         self.model, self.cache, self.device = model, cache, torch.device(device)
         self.max_batch = max_batch
         self.width = max(1, cache.table_width(context_length))
+        # positions that have a learned vector (None: positions are not limited)
+        self.max_positions = model.cfg.max_position_embeddings if model.cfg.learned_positions else None
         # the routing kernel takes up to 256 experts, 16 per token; beyond that the choice reads back to the host
         moe = [m["mlp"]["router"] for m in model.cfg.mixer_layers if m["mlp"] and m["mlp"]["kind"] == "moe"]
         self.use_graph = use_graph and self.device.type == "cuda" and all(r["experts"] <= 256 and r["top"] <= 16 for r in moe)
@@ -70,23 +72,40 @@ class RaggedRunner:
         slots = pt[row_entry, pos // ps - base[row_entry]].astype(np.int64) * ps + pos % ps if self.cache.has_kv else pos * 0
         n_dec = int((n == 1).sum())
         blocks, tiles = [], []
-        span = getattr(self.cache, "span", 0)
+        sight = getattr(self.cache, "first_visible", lambda p: 0)
         for i in range(n_dec, len(entries)):
             for r in range(0, int(n[i]), SCAN_BLOCK):
                 blocks.append((i, cu[i] + r, min(SCAN_BLOCK, n[i] - r), int(r == 0)))
             tiles += [(i, cu[i] + r) for r in range(0, int(n[i]), ATTN_TILE)]
         # tiles that see the most keys start first: the last ones to run are short
-        tiles.sort(key=lambda t: -(pos[t[1]] % span if span else pos[t[1]]))
+        tiles.sort(key=lambda t: sight(int(pos[t[1]])) - pos[t[1]])
         toks = np.concatenate([np.asarray(e.tokens, np.int64) for e in entries])
         state = np.array([e.carry.slot for e in entries])
         arrs = [toks, pos, slots, row_entry, cu, start, state, pt, base]
         if blocks:
             arrs += [np.array(blocks), np.array(tiles)]
+        windows = sorted(getattr(self.cache, "windows", ())) if blocks else []
+        for w in windows:
+            arrs += self._visible_pages(entries, n_dec, start, n, base, w)
         want = [cu[i] + w for i, e in enumerate(entries) for w in e.want]
         arrs.append(np.array(want, np.int64))
         up = self._upload([a.astype(np.int32) for a in arrs])
-        b = RaggedBatch(*up[:9], blocks=up[9] if blocks else None, tiles=up[10] if blocks else None, n_dec=n_dec, page_size=ps)
+        seen = {w: PageList(*up[11 + 3 * i:14 + 3 * i]) for i, w in enumerate(windows)}
+        b = RaggedBatch(*up[:9], blocks=up[9] if blocks else None, tiles=up[10] if blocks else None, n_dec=n_dec, page_size=ps, seen=seen)
         return b, up[-1]
+
+    def _visible_pages(self, entries: list, n_dec: int, start, n, base, window: int) -> list:
+        """Pages that the portions of a step see through a sliding window, one after the other; and, per entry, the table
+        of their numbers in that list with the page of the sequence that it begins with."""
+        ps = self.cache.page_size
+        first = np.maximum(start - window + 1, 0) // ps if window else start * 0
+        last = (start + n - 1) // ps
+        count = np.where(np.arange(len(entries)) >= n_dec, last - first + 1, 0)
+        table, pages = np.zeros((len(entries), max(1, count.max())), np.int64), []
+        for i in range(n_dec, len(entries)):
+            table[i, :count[i]] = len(pages) + np.arange(count[i])
+            pages += entries[i].carry.pages[first[i] - base[i]:last[i] - base[i] + 1]
+        return [np.array(pages), table, first]
 
     # ------------------------------------------------------------------ the step
     @torch.no_grad()
@@ -97,6 +116,8 @@ class RaggedRunner:
             held = (e.carry.first_page + len(e.carry.pages)) * self.cache.page_size
             if not e.tokens or (self.cache.has_kv and held < e.carry.length + len(e.tokens)):
                 raise ValueError("an entry of a step needs tokens, and pages for all of them")
+            if self.max_positions is not None and e.carry.length + len(e.tokens) > self.max_positions:
+                raise ValueError(f"a sequence of this model has at most {self.max_positions} tokens")
         if self.use_graph and on_layer is None and len(entries) <= self.max_batch and all(
                 len(e.tokens) == 1 and e.want == [0] and len(e.carry.pages) <= self.width for e in entries):
             out = self._decode_graph(entries)

@@ -1,5 +1,5 @@
 """Memory of running requests: the page pool every cache is built on, and the cache of mixer stacks (pages of keys and
-values per attention layer, one state slot per request for the recurrent layers)."""
+values, or of latents, per attention layer, one state slot per request for the recurrent layers)."""
 from __future__ import annotations
 
 from dataclasses import dataclass, field
@@ -63,33 +63,37 @@ class LayerCache:
 
 
 class StateCache(PagePool):
-    """Pages of K and V for the attention layers (``[pages * page_size, heads, dim]`` per layer, each with its own
-    sizes) and fp32 slots for the recurrent ones (convolution tails, recurrence states). A slot is not cleared when it
-    changes hands: kernels take the state of a request that has absorbed nothing as zero."""
+    """Pages for the attention layers (``[pages * page_size, heads, dim]`` of K and V per layer, each with its own sizes; a
+    layer whose keys and values come from one latent has K only) and fp32 slots for the recurrent ones (convolution tails,
+    recurrence states). A slot is not cleared when it changes hands: kernels take the state of a request that has absorbed
+    nothing as zero."""
 
     def __init__(self, mixers: list, num_pages: int, page_size: int, num_slots: int, device, dtype):
         super().__init__(num_pages, page_size)
         self.num_slots = num_slots
         self.layers: list[LayerCache] = []
-        chunks = []
+        self._sight: dict = {}       # attention layers that see the same stretch of positions, once each
+        self.windows: set = set()    # sliding windows of the latent layers
         for mx in mixers:
             lc, shapes = LayerCache(), mx.cache_shapes()
             if "kv" in shapes:
-                lc.k, lc.v = (torch.zeros(num_pages * page_size, *s, device=device, dtype=dtype) for s in shapes["kv"])
-                chunks.append(mx.chunk)
+                lc.k, lc.v = (None if s is None else torch.zeros(num_pages * page_size, *s, device=device, dtype=dtype) for s in shapes["kv"])
+                self._sight[type(mx), mx.span] = mx
+                if lc.v is None:
+                    self.windows.add(mx.span)
             for name in ("tail", "state"):
                 if name in shapes:
                     setattr(lc, name, torch.zeros(num_slots, *shapes[name], device=device, dtype=torch.float32))
             self.layers.append(lc)
-        self.has_kv = bool(chunks)
-        self.chunks = sorted(set(chunks))
+        self.has_kv = bool(self._sight)
+        spans = [mx.span for mx in self._sight.values()]
         # positions the furthest-seeing layer may look at (0: all of them)
-        self.span = 0 if not chunks or min(chunks) == 0 else max(chunks)
+        self.span = 0 if not spans or min(spans) == 0 else max(spans)
         self.free_slots = list(range(num_slots - 1, -1, -1))
 
     @staticmethod
     def bytes_per_page(mixers: list, page_size: int, elem: int) -> int:
-        return sum(h * d for mx in mixers for h, d in mx.cache_shapes().get("kv", ())) * page_size * elem
+        return sum(s[0] * s[1] for mx in mixers for s in mx.cache_shapes().get("kv", ()) if s) * page_size * elem
 
     @staticmethod
     def bytes_per_slot(mixers: list) -> int:
@@ -105,7 +109,7 @@ class StateCache(PagePool):
 
     def first_visible(self, pos: int) -> int:
         """Earliest position that a query at ``pos`` or later can see in any attention layer."""
-        return 0 if self.span == 0 else min(pos // c * c for c in self.chunks)
+        return 0 if self.span == 0 else min(mx.first_visible(pos) for mx in self._sight.values())
 
     def table_width(self, context: int) -> int:
         """Page-table columns a single-token step needs at most."""

@@ -47,7 +47,7 @@ def timed(fn, iters: int = 10, warmup: int = 3, flush=None) -> float:
     return sorted(ts)[len(ts) // 2]
 
 
-def _batch(lens, starts, dev, page_size=64):
+def _batch(lens, starts, dev, page_size=64, windows=()):
     """A ragged batch over consecutive pages; single-token entries first. Returns (batch, cache rows)."""
     from ..engine.ragged_step import Entry, RaggedRunner
     from ..engine.state_cache import Carried
@@ -59,7 +59,7 @@ def _batch(lens, starts, dev, page_size=64):
         at += k
     r = RaggedRunner.__new__(RaggedRunner)
     r.device = torch.device(dev)
-    r.cache = type("C", (), dict(page_size=page_size, has_kv=True))
+    r.cache = type("C", (), dict(page_size=page_size, has_kv=True, windows=windows))
     return RaggedRunner._layout(r, ents)[0], at * page_size
 
 
@@ -175,6 +175,122 @@ def kernel_table(cfg, prefill=(4, 2048), decode=(64, 960), dev="cuda") -> list[d
             add(f"expert_linear down {tag}", lambda: M.expert_linear(hh, wd, rt), (live * If * H + R * k * (H + If)) * 2, 2.0 * R * k * H * If)
             add(f"expert_combine {tag}", lambda: M.expert_combine(ys, rt, rt.topw), R * (k + 1) * H * 2, like=f"gather and sum {tag}")
             add(f"gather and sum {tag}", lambda: (ys.index_select(0, rt.inv).view(R, k, H) * rt.topw.to(ys.dtype).unsqueeze(-1)).sum(1), R * (k + 1) * H * 2)
+    return rows
+
+
+def latent_kernel_table(cfg, prefill=(4, 2048), decode=(64, 960), dev="cuda") -> list[dict]:
+    """As :func:`kernel_table`, for a stack of latent attention (Vogilix)."""
+    bw, fl, _ = peaks()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    bf = dict(device=dev, dtype=torch.bfloat16)
+    f32 = dict(device=dev, dtype=torch.float32)
+    rows = []
+
+    def add(name, fn, nbytes=0.0, flops=0.0, like=None):
+        t = timed(fn, flush=flush)
+        roof = max(nbytes / bw, flops / fl)
+        rows.append(dict(kernel=name, us=round(t * 1e6, 1), roofline_us=round(roof * 1e6, 1), fraction=round(roof / t, 3), like=like))
+
+    Hd, V = cfg.hidden_size, cfg.vocab_size
+    at = cfg.mixer_layers[0]["mixer"]
+    nq, D, Dv, rq, C, scale = at["heads"], at["dim"], at["vdim"], at["q_rank"], at["kv_rank"], at["scale"]
+    windows = sorted({e["mixer"]["mask"]["size"] for e in cfg.mixer_layers})
+    dense = next(e["mlp"] for e in cfg.mixer_layers if e["mlp"] and e["mlp"]["kind"] == "dense")
+    moe = next(e["mlp"] for e in cfg.mixer_layers if e["mlp"] and e["mlp"]["kind"] == "moe")
+    E, k, If, Is = moe["router"]["experts"], moe["router"]["top"], moe["expert"]["ff"], moe["shared"]["ff"]
+    (B, L), (nB, ctx) = prefill, decode
+    pb, prow = _batch([L] * B, [0] * B, dev, windows=windows)
+    db, drow = _batch([1] * nB, [ctx] * nB, dev, windows=windows)
+    w, wrq, wc = torch.zeros(Hd, **f32), torch.ones(rq, **f32), torch.ones(C, **f32)
+    w_kv = torch.randn(nq * (D + Dv), C, **bf) * C ** -0.5
+    w_k, w_v = w_kv[:nq * D].view(nq, D, C), w_kv[nq * D:].view(nq, Dv, C)
+    table, ptab = torch.randn(V, Hd, **bf), torch.randn(cfg.max_position_embeddings, Hd, **bf)
+    side, sd = torch.randn(V, cfg.num_layers * cfg.token_side_dim, **bf), cfg.token_side_dim
+    for tag, b, R, rows_ in (("prefill", pb, B * L, prow), ("decode", db, nB, drow)):
+        # norms, embedding
+        h, res = torch.randn(R, Hd, **bf), torch.randn(R, Hd, **f32)
+        ids = torch.randint(0, V, (R,), device=dev, dtype=torch.int32)
+        add(f"embed_rows {tag}", lambda: M.embed_rows(ids, table, b.pos, ptab), R * Hd * 10, like=f"embedding {tag}")
+        with torch.no_grad():
+            add(f"embedding {tag}", lambda: OF.embedding(ids.long(), table), R * Hd * 4)
+        add(f"post_norm {tag}", lambda: M.post_norm(h, w, res, 1e-6, 0.5, 1.0), R * Hd * 12, like=f"rmsnorm {tag}")
+        r16, w16 = res.bfloat16(), w.bfloat16()
+        with torch.no_grad():
+            add(f"rmsnorm {tag}", lambda: OF.rmsnorm(h, w16, 1e-6, r16), R * Hd * 8)
+        # attention
+        x, cache = torch.randn(R, rq + C, **bf), torch.randn(rows_, 1, C, **bf)
+        add(f"latent_norm_append {tag}", lambda: M.latent_norm_append(x, wrq, wc, 1e-6, b, cache), x.numel() * 4, like=f"qk_norm_append {tag}")
+        kc, vc, wq_ = torch.randn(rows_, 1, 128, **bf), torch.randn(rows_, 1, 128, **bf), torch.ones(rq + C - 256, **f32)
+        add(f"qk_norm_append {tag}", lambda: M.qk_norm_append(x, wq_, wc[:128], 1e-6, b, kc, vc, (rq + C - 256) // 128), x.numel() * 4)
+        q = torch.randn(R, nq, D, **bf)
+        if tag == "prefill":
+            seen = pb.seen[windows[-1]]
+            add("latents gathered prefill", lambda: cache.view(-1, 64 * C).index_select(0, seen.pages), R * C * 4)
+            rows_c = cache.view(-1, C)[:R]
+            add("keys and values prefill (GEMM)", lambda: M.linear(rows_c, w_kv), (R * C + w_kv.numel() + R * nq * (D + Dv)) * 2, 2.0 * R * C * nq * (D + Dv))
+            for win in windows:
+                pairs = B * sum(min(p + 1, win) for p in range(L))
+                flops = 2.0 * nq * (D + Dv) * pairs
+                kv, out = M.linear(rows_c, w_kv), torch.empty(R, nq, Dv, **bf)
+                sn = pb.seen[win]
+
+                def attn():
+                    M._call("ab2_chunk_prefill", q.data_ptr(), pb.cu.data_ptr(), pb.start.data_ptr(), pb.tiles.data_ptr(), pb.tiles.shape[0], out.data_ptr(), R,
+                            kv.shape[0], kv.stride(0), kv.stride(0), kv.data_ptr(), kv[:, nq * D:].data_ptr(), sn.table.data_ptr(), sn.base.data_ptr(),
+                            sn.table.shape[1], 64, nq, nq, D, Dv, scale, 0.0, None, None, 0, win)
+                add(f"window attention {win} prefill", attn, (q.numel() + out.numel() + kv.numel()) * 2, flops, like="attn_fwd prefill")
+                add(f"latent_attention {win} prefill (all of it)", lambda: M.latent_attention(q, cache, w_kv, Dv, pb, scale, win),
+                    (q.numel() * 2 + R * C) * 2, flops + 2.0 * R * C * nq * (D + Dv))
+            if D == Dv and D in (64, 128):
+                k_, v_ = torch.randn(R, nq, D, **bf), torch.randn(R, nq, D, **bf)
+                cu = torch.arange(0, R + 1, L, device=dev, dtype=torch.int32)
+                ti = OF.attn_tile_table(cu, R)
+                add("attn_fwd prefill", lambda: OF.attention_fwd(q, k_, v_, cu, True, D ** -0.5, ti), q.numel() * 8, 4.0 * nq * D * B * L * (L + 1) / 2)
+        else:
+            qc, oc = torch.randn(R, nq, C, **bf), torch.empty(R, nq, C, **bf)
+            add("head_linear of the queries decode", lambda: M.head_linear(q, w_k, w_kn=True), (q.numel() + qc.numel() + w_k.numel()) * 2, 2.0 * R * nq * D * C,
+                like="linear of the same weight bytes decode")
+            add("head_linear of the values decode", lambda: M.head_linear(qc, w_v), (q.numel() + qc.numel() + w_v.numel()) * 2, 2.0 * R * nq * Dv * C,
+                like="linear of the same weight bytes decode")
+            xl, wl = torch.randn(R, C, **bf), torch.randn(nq * D, C, **bf)
+            add("linear of the same weight bytes decode", lambda: M.linear(xl, wl), (xl.numel() + wl.numel() + R * nq * D) * 2, 2.0 * R * nq * D * C)
+            for win in windows:
+                see = min(ctx + 1, win)
+
+                def dec():
+                    M._call("ab2_latent_decode", qc.data_ptr(), b.pos.data_ptr(), b.slots.data_ptr(), b.row_entry.data_ptr(), oc.data_ptr(), R,
+                            cache.data_ptr(), b.pages.data_ptr(), b.page_base.data_ptr(), b.pages.shape[1], 64, nq, C, scale, win)
+                add(f"latent_decode {win} decode", dec, (R * see * C + 2 * qc.numel()) * 2, 4.0 * R * see * nq * C, like="paged_decode decode")
+            nk = max(1, nq // 4)
+            kc, vc = torch.randn(rows_, nk, 128, **bf), torch.randn(rows_, nk, 128, **bf)
+            q2 = torch.randn(R, nq, 128, **bf)
+            lens = torch.full((nB,), ctx + 1, device=dev, dtype=torch.int32)
+            po, ml, o = torch.empty(nB * nq * 4 * 128, **f32), torch.empty(nB * nq * 8, **f32), torch.empty_like(q2)
+
+            def paged():
+                oplib.check(oplib.get_lib().ab2_paged_decode_strided(
+                    q2.data_ptr(), kc.data_ptr(), vc.data_ptr(), b.pages.data_ptr(), lens.data_ptr(), po.data_ptr(), ml.data_ptr(), o.data_ptr(), nB, nq, nk,
+                    128, 64, b.pages.shape[1], 4, 128 ** -0.5, q2.stride(0), oplib.stream_ptr()), "paged_decode")
+            add("paged_decode decode", paged, nB * (ctx + 1) * nk * 256 * 2)
+        # feed-forwards and the token input
+        ff = dense["ff"]
+        z, gu = torch.randn(R, ff, **bf), torch.randn(R, 2 * ff, **bf)
+        add(f"gelu_erf {tag}", lambda: M.gelu_erf(z), R * ff * 4, like=f"swiglu {tag}")
+        with torch.no_grad():
+            add(f"swiglu {tag}", lambda: OF.swiglu(gu), R * ff * 6)
+        rw, x16 = torch.randn(E, Hd, **bf), torch.randn(R, Hd, **bf)
+        add(f"router_logits {tag}", lambda: M.router_logits(x16, rw), (R * Hd + E * Hd) * 2 + R * E * 4, 2.0 * R * E * Hd, like=f"router in the routed decoder {tag}")
+        add(f"router in the routed decoder {tag}", lambda: F.linear(x16.float(), rw.float()), (R * Hd + E * Hd) * 2 + R * E * 4, 2.0 * R * E * Hd)
+        rt = OF.moe_route(torch.randn(R, E, **f32), k, sigmoid=True, norm=False, want_probs=False, want_host=False)
+        eg = torch.randn(R * k, 2 * If, **bf)
+        add(f"glu_clamped experts {tag}", lambda: M.glu_clamped(eg, 6.0, 1.702, rt), R * k * If * 6, like=f"swiglu {tag}")
+        sg = torch.randn(R, 2 * Is, **bf)
+        add(f"glu_clamped shared {tag}", lambda: M.glu_clamped(sg, 7.0, 1.702), R * Is * 6, like=f"swiglu {tag}")
+        y, sh = torch.randn(R * k, Hd, **bf), torch.randn(R, Hd, **bf)
+        add(f"post_norm of experts {tag}", lambda: M.post_norm(M.ExpertSum(y, rt, sh), w, res, 1e-6, 0.5, 1.0), R * Hd * (2 * k + 12), like=f"gather and sum {tag}")
+        add(f"gather and sum {tag}", lambda: (y.index_select(0, rt.inv).view(R, k, Hd) * rt.topw.to(y.dtype).unsqueeze(-1)).sum(1), R * (k + 1) * Hd * 2)
+        g = torch.randn(R, sd, **bf)
+        add(f"side_gate {tag}", lambda: M.side_gate(g, ids, side, 0), R * sd * 6, like=f"swiglu {tag}")
     return rows
 
 
@@ -306,18 +422,45 @@ def like_sized(cfg):
     return hyb, ModelConfig(arch="qwen3", **base), routed
 
 
-def run(steps=True, kernels=True, sizes=("kagolix-8b-layers", "kagolix-2b-layers")) -> dict:
+def latent_like_sized(cfg):
+    """The closest existing models with the same width, heads, feed-forwards, experts and vocabulary as a latent stack: the
+    mixer stack with grouped-query attention in chunks as long as the windows (a key head per four query heads), the dense
+    and the routed decoder."""
+    from ..models.config import ModelConfig
+
+    at = cfg.mixer_layers[0]["mixer"]
+    nk = max(1, at["heads"] // 4)
+    layers = []
+    for e in cfg.mixer_layers:
+        m = dict(heads=at["heads"], kv_heads=nk, dim=at["dim"], vdim=at["vdim"], scale=at["scale"], softcap=30.0, mask=dict(e["mixer"]["mask"]))
+        layers.append(dict(type="attention", mixer=m, mlp=e["mlp"]))
+    stack = ModelConfig.from_hf_dict(dict(architecture="Kagolix", vocab=cfg.vocab_size, width=cfg.hidden_size, norm=dict(eps=1e-6, groups=1),
+                                          logit_softcap=0.0, layers=layers))
+    base = dict(vocab_size=cfg.vocab_size, hidden_size=cfg.hidden_size, num_layers=cfg.num_layers, num_heads=at["heads"], num_kv_heads=nk,
+                head_dim=at["dim"], intermediate_size=cfg.intermediate_size, tie_word_embeddings=False, attention_bias=False, qk_norm=True)
+    routed = ModelConfig(arch="qwen3_moe", **base, num_experts=cfg.num_experts, num_experts_per_tok=cfg.num_experts_per_tok,
+                         moe_intermediate_size=cfg.moe_intermediate_size)
+    return stack, ModelConfig(arch="qwen3", **base), routed
+
+
+def run(steps=True, kernels=True, design="kagolix", sizes=None) -> dict:
     from ..models.config import preset
 
     torch.manual_seed(0)
     bw, fl, src = peaks()
     out = dict(workload="mixer-serve", dtype="bf16", data="synthetic tokens, random weights", roofline=f"{src}: {bw / 1e9:.0f} GB/s, {fl / 1e12:.0f} TFLOP/s",
                sizes={})
-    for name in sizes:
+    for name in sizes or (f"{design}-8b-layers", f"{design}-2b-layers"):
         cfg = preset(name)
         prefill, decode = (4, 2048), (64, 960)
         r = dict(prefill=f"{prefill[0]} x {prefill[1]} tokens", decode=f"{decode[0]} sequences at {decode[1]} tokens")
-        if steps:
+        if steps and design == "vogilix":
+            stack, dense, routed = latent_like_sized(cfg)
+            for key, fn, c in (("vogilix", mixer_steps, cfg), ("mixer_stack_attention", mixer_steps, stack), ("decoder_dense", decoder_steps, dense),
+                               ("decoder_routed", decoder_steps, routed)):
+                r[key] = fn(c, prefill, decode)
+                torch.cuda.empty_cache()
+        elif steps:
             hyb, dense, routed = like_sized(cfg)
             r["mixer_stack"] = mixer_steps(cfg, prefill, decode)
             torch.cuda.empty_cache()
@@ -325,6 +468,6 @@ def run(steps=True, kernels=True, sizes=("kagolix-8b-layers", "kagolix-2b-layers
                 r[key] = fn(c, prefill, decode)
                 torch.cuda.empty_cache()
         if kernels:
-            r["kernels"] = kernel_table(cfg, prefill, decode)
+            r["kernels"] = (latent_kernel_table if design == "vogilix" else kernel_table)(cfg, prefill, decode)
         out["sizes"][name] = r
     return out

@@ -14,7 +14,7 @@ from typing import Optional
 
 @dataclass
 class ModelConfig:
-    arch: str = "qwen2"                 # qwen2 | qwen3 | qwen3_moe | qwen2_moe | qwen3_5 | qwen3_5_moe | kagolix
+    arch: str = "qwen2"                 # qwen2 | qwen3 | qwen3_moe | qwen2_moe | qwen3_5 | qwen3_5_moe | kagolix | vogilix
     vocab_size: int = 151936
     hidden_size: int = 1536
     num_layers: int = 28
@@ -63,11 +63,15 @@ class ModelConfig:
     partial_rotary_factor: float = 1.0
     attn_output_gate: bool = False
     rms_norm_offset: bool = False
-    # mixer stacks (Kagolix): one entry per layer, {"type": mixer kind, "mixer": its sizes, "mlp": feed-forward or
-    # None} as in config.json (see models/mixers.py); grouped RMS norms and a capped output
+    # mixer stacks (Kagolix, Vogilix): one entry per layer, {"type": mixer kind, "mixer": its sizes, "mlp":
+    # feed-forward or None} as in config.json (see models/mixers.py); grouped RMS norms and a capped output
     mixer_layers: list[dict] = field(default_factory=list)
     norm_groups: int = 1
     logit_softcap: float = 0.0
+    norm_placement: str = "sandwich"        # sandwich: before and after every sublayer | post: on its output only
+    residual_mult: float = 1.0              # factor of every sublayer's normed output on its way into the residual sum
+    learned_positions: bool = False         # a vector per position (max_position_embeddings of them) added to the embedding
+    token_side_dim: int = 0                 # > 0: every layer ends with a gated input from its own part of a per-token row
 
     @property
     def is_mixer_stack(self) -> bool:
@@ -238,25 +242,31 @@ class ModelConfig:
     def _from_mixer_stack_dict(cls, d: dict) -> "ModelConfig":
         """config.json of a mixer stack: ``architecture`` names the design, ``layers`` lists every layer's mixer
         and feed-forward with their sizes."""
-        if d["architecture"] != "Kagolix":
-            raise ValueError(f"unsupported architecture '{d['architecture']}'")
-        from .mixers import check_layer_specs
+        from .mixers import DESIGNS, check_layer_specs
 
+        arch = d["architecture"].lower()
+        if arch not in DESIGNS or DESIGNS[arch].name != d["architecture"]:
+            raise ValueError(f"unsupported architecture '{d['architecture']}' (have {sorted(x.name for x in DESIGNS.values())})")
         layers = [dict(type=e["type"], mixer=dict(e["mixer"]), mlp=dict(e["mlp"]) if e.get("mlp") else None) for e in d["layers"]]
-        check_layer_specs(layers, d["width"], d["norm"].get("groups", 1))
-        att = [e["mixer"] for e in layers if e["type"] == "attention"]
+        check_layer_specs(arch, layers, d["width"], d["norm"].get("groups", 1))
+        att = [e["mixer"] for e in layers if "heads" in e["mixer"] and "dim" in e["mixer"]]
         moe = [e["mlp"] for e in layers if e["mlp"] and e["mlp"]["kind"] == "moe"]
-        return cls(arch="kagolix", vocab_size=d["vocab"], hidden_size=d["width"], num_layers=len(layers),
+        own = {}
+        if arch == "vogilix":
+            own = dict(norm_placement="post", rms_norm_offset=True, residual_mult=float(d["residual_mult"]), learned_positions=True,
+                       max_position_embeddings=int(d["max_positions"]), token_side_dim=int((d.get("token_side") or {}).get("dim") or 0))
+        else:
+            own = dict(norm_groups=int(d["norm"].get("groups", 1)), logit_softcap=float(d.get("logit_softcap") or 0.0),
+                       max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)))
+        return cls(arch=arch, vocab_size=d["vocab"], hidden_size=d["width"], num_layers=len(layers),
                    # engine-wide summaries; every layer reads its own sizes from its spec
-                   num_heads=max((m["heads"] for m in att), default=1), num_kv_heads=max((m["kv_heads"] for m in att), default=1),
+                   num_heads=max((m["heads"] for m in att), default=1), num_kv_heads=max((m.get("kv_heads", m["heads"]) for m in att), default=1),
                    head_dim=max((m["dim"] for m in att), default=1),
                    intermediate_size=max((e["mlp"]["ff"] for e in layers if e["mlp"] and e["mlp"]["kind"] == "dense"), default=0),
                    num_experts=max((m["router"]["experts"] for m in moe), default=0),
                    num_experts_per_tok=max((m["router"]["top"] for m in moe), default=0),
                    moe_intermediate_size=max((m["expert"]["ff"] for m in moe), default=0), norm_topk_prob=False,
-                   rms_norm_eps=float(d["norm"]["eps"]), norm_groups=int(d["norm"].get("groups", 1)),
-                   logit_softcap=float(d.get("logit_softcap") or 0.0), tie_word_embeddings=False, attention_bias=False,
-                   mixer_layers=layers, max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)))
+                   rms_norm_eps=float(d["norm"]["eps"]), tie_word_embeddings=False, attention_bias=False, mixer_layers=layers, **own)
 
     @classmethod
     def from_pretrained(cls, path: str) -> "ModelConfig":
@@ -266,9 +276,15 @@ class ModelConfig:
     def to_hf_dict(self) -> dict:
         mt = self.arch
         if self.is_mixer_stack:
-            return dict(architecture="Kagolix", vocab=self.vocab_size, width=self.hidden_size,
-                        norm=dict(eps=self.rms_norm_eps, groups=self.norm_groups), logit_softcap=self.logit_softcap,
-                        layers=[dict(e) for e in self.mixer_layers])
+            from .mixers import DESIGNS
+
+            d = dict(architecture=DESIGNS[mt].name, vocab=self.vocab_size, width=self.hidden_size, layers=[dict(e) for e in self.mixer_layers])
+            if mt == "vogilix":
+                d.update(max_positions=self.max_position_embeddings, norm=dict(eps=self.rms_norm_eps), residual_mult=self.residual_mult,
+                         token_side=dict(dim=self.token_side_dim) if self.token_side_dim else None)
+            else:
+                d.update(norm=dict(eps=self.rms_norm_eps, groups=self.norm_groups), logit_softcap=self.logit_softcap)
+            return d
         d = dict(
             model_type=mt, architectures=[{"qwen2": "Qwen2ForCausalLM", "qwen3": "Qwen3ForCausalLM", "qwen3_5": "Qwen3_5ForCausalLM", "qwen3_5_moe": "Qwen3_5MoeForCausalLM",
                                            "qwen3_moe": "Qwen3MoeForCausalLM", "qwen2_moe": "Qwen2MoeForCausalLM"}[mt]],
@@ -398,6 +414,19 @@ def _mixer_stack_preset(vocab, width, pattern, att, ssm, lru, dense_ff, moe, gro
     return dict(architecture="Kagolix", vocab=vocab, width=width, norm=dict(eps=eps, groups=groups), logit_softcap=softcap, layers=layers)
 
 
+def _latent_stack_preset(vocab, width, pattern, att, windows, dense_ff, moe, shared_ff, side, positions, eps=1e-6, mult=0.5, limits=(6.0, 7.0)):
+    """A Vogilix stack: every layer has the attention ``att`` with the window of its place in ``windows`` (repeated), d in
+    ``pattern`` gives it a dense feed-forward, e experts, - none."""
+    layers = []
+    for i, c in enumerate(pattern):
+        mlp = {"d": dict(kind="dense", ff=dense_ff), "-": None,
+               "e": dict(kind="moe", expert=dict(ff=moe[2], limit=limits[0]), router=dict(experts=moe[0], top=moe[1]),
+                         shared=dict(ff=shared_ff, limit=limits[1]))}[c]
+        layers.append(dict(type="latent_attention", mixer=dict(att, mask=dict(size=windows[i % len(windows)])), mlp=mlp))
+    return dict(architecture="Vogilix", vocab=vocab, width=width, max_positions=positions, norm=dict(eps=eps), residual_mult=mult,
+                token_side=dict(dim=side), layers=layers)
+
+
 MIXER_STACK_PRESETS = {
     "tiny-kagolix": _mixer_stack_preset(
         320, 128, "aMrM", dict(heads=4, kv_heads=2, dim=32, vdim=48, scale=0.2, softcap=25.0, mask=dict(size=40)),
@@ -409,6 +438,14 @@ MIXER_STACK_PRESETS = {
     "kagolix-2b-layers": _mixer_stack_preset(
         32768, 2048, "amRM", dict(heads=16, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, mask=dict(size=1024)),
         dict(heads=64, vdim=64, state=128, groups=4, norm_groups=4, conv=4), dict(width=2560, blocks=10, conv=4), 8192, (64, 8, 768), 8),
+    "tiny-vogilix": _latent_stack_preset(
+        320, 128, "de-", dict(heads=4, dim=32, vdim=48, q_rank=40, kv_rank=56, scale=0.2), (40, 24), 160, (6, 2, 64), 96, 24, 512),
+    # layer sizes of an 8B-class and of a 2B-class model
+    "vogilix-8b-layers": _latent_stack_preset(
+        32768, 4096, "dede", dict(heads=32, dim=128, vdim=128, q_rank=1536, kv_rank=512, scale=128 ** -0.5), (4096, 1024), 12288, (64, 8, 768), 2048,
+        256, 8192),
+    "vogilix-2b-layers": _latent_stack_preset(
+        32768, 2048, "dede", dict(heads=16, dim=128, vdim=128, q_rank=768, kv_rank=512, scale=128 ** -0.5), (1024,), 8192, (64, 8, 768), 1024, 256, 8192),
 }
 
 

@@ -8,6 +8,9 @@
 // indexed by expert, the epilogue masks the rows that spill into the next group. Pipeline (TMA ->
 // 128B-swizzled smem -> tcgen05.mma -> TMEM -> epilogue warps) as in gemm.cu.
 //
+// The same kernel computes every head's own product, C[r, h, :] = op(B[h]) A[r, h, :]: all heads have the same rows, and head
+// h reads and writes its own stretch of columns (ab2_gemm_heads).
+//
 // Takes the place of torch._grouped_mm in the reference's expert layers
 // (areal/experimental/models/archon/moe/grouped_experts.py:100-207) and of the per-expert
 // Python loop of GEMM launches.
@@ -36,16 +39,17 @@ template <int BN, bool B_MN>
 __global__ void __launch_bounds__(192, 1)
 gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
                     __nv_bfloat16* __restrict__ Cptr, const int4* __restrict__ tiles, int num_tiles, int N,
-                    int K, int ldc, int* err, const int* __restrict__ num_rt_dev, int nblk) {
+                    int K, int ldc, int* err, const int* __restrict__ num_rt_dev, int nblk, int head_rows) {
   constexpr bool A_MN = false;
   // Row-tile mode (nblk > 0): `tiles` lists 128-row tiles only, written by the routing kernel together with
   // their number; output tile i covers row tile i / nblk and n-block i % nblk, and the grid was sized for
-  // an upper bound of the row tiles.
-  if (nblk > 0) {
-    const int have = *num_rt_dev * nblk;
-    num_tiles = have < num_tiles ? have : num_tiles;
-  }
+  // an upper bound of the row tiles. Head mode (head_rows > 0): no list; head i / (row tiles * nblk), then row tile, n-block.
+  const int head_rt = (head_rows + BM - 1) / BM;
   auto tile_info = [&](int tile) -> int4 {
+    if (head_rows > 0) {
+      const int rest = tile / nblk, m0 = rest % head_rt * BM;
+      return make_int4(rest / head_rt, m0, min(BM, head_rows - m0), tile % nblk);
+    }
     if (nblk > 0) {
       int4 t = tiles[tile / nblk];
       t.w = tile % nblk;
@@ -91,6 +95,13 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
   tc_fence_after();
   uint32_t tmem_base;
   asm volatile("ld.shared.b32 %0, [%1];" : "=r"(tmem_base) : "r"(tmem_slot));
+  // everything above touches only this kernel's own state
+  pdl_wait();
+  pdl_trigger();
+  if (nblk > 0 && head_rows == 0) {
+    const int have = *num_rt_dev * nblk;
+    num_tiles = have < num_tiles ? have : num_tiles;
+  }
 
   if (warp == 0) {
     // ------------------------------------------------ TMA producer
@@ -102,13 +113,14 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
       for (int tile = blockIdx.x; tile < num_tiles && ok; tile += gridDim.x) {
         const int4 ti = tile_info(tile);
         const int expert = ti.x, m0 = ti.y, n0 = ti.w * BN;
+        const int a0 = head_rows > 0 ? expert * K : 0;      // columns past the head's own meet zero-filled rows of B
         for (int kb = 0; kb < num_kb; ++kb) {
           if (!mbar_wait(empty_bar(stage), phase ^ 1u, err, ERR_WAIT_EMPTY)) { ok = false; break; }
           const uint32_t sA = smem_base + stage * Cfg::STAGE_BYTES;
           const uint32_t sB = sA + Cfg::A_BYTES;
           mbar_expect_tx(full_bar(stage), Cfg::STAGE_BYTES);
           if (!A_MN) {
-            tma_load_2d(sA, &tmA, full_bar(stage), kb * BK, m0);
+            tma_load_2d(sA, &tmA, full_bar(stage), a0 + kb * BK, m0);
           } else {
 #pragma unroll
             for (int c = 0; c < BM / 64; ++c)
@@ -191,7 +203,7 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
         tmem_ld_wait();
         const int col = n0 + c * 32;
         if (row_in_tile < rows_valid && col < N) {       // rows past the expert's group belong to the next one
-          __nv_bfloat16* C = Cptr + (size_t)row * ldc + col;
+          __nv_bfloat16* C = Cptr + (size_t)row * ldc + (head_rows > 0 ? ti.x * N : 0) + col;
           if (col + 32 <= N) {
             uint4* C4 = reinterpret_cast<uint4*>(C);
 #pragma unroll
@@ -222,10 +234,10 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
 
 template <int BN, bool B_MN>
 static int launch_grouped(const void* A, const void* B, void* C, const void* tiles, int num_tiles, int R, int N, int K, int E,
-                          int lda, int ldc, cudaStream_t stream, const int* num_rt_dev = nullptr, int nblk = 0) {
+                          int lda, int ldc, cudaStream_t stream, const int* num_rt_dev = nullptr, int nblk = 0, bool heads = false) {
   using Cfg = GemmCfg<BN>;
   CUtensorMap tmA, tmB;
-  int rc = ab2host::encode_tmap_2d(&tmA, A, 2, (uint64_t)K, (uint64_t)R, (uint64_t)lda * 2, BK, BM, true, 0);
+  int rc = ab2host::encode_tmap_2d(&tmA, A, 2, heads ? (uint64_t)K * E : (uint64_t)K, (uint64_t)R, (uint64_t)lda * 2, BK, BM, true, 0);
   if (rc) return 100 + rc;
   if (!B_MN)  // [E, N, K]
     rc = ab2host::encode_tmap_3d(&tmB, B, 2, (uint64_t)K, (uint64_t)N, (uint64_t)E, (uint64_t)K * 2, (uint64_t)N * K * 2, BK, BN, 1, true, 0);
@@ -240,8 +252,8 @@ static int launch_grouped(const void* A, const void* B, void* C, const void* til
   const int grid = num_tiles < num_sms ? num_tiles : num_sms;
   int* err = ab2host::error_flag();
   if (!err) return 301;
-  kern<<<grid, 192, Cfg::SMEM_BYTES, stream>>>(tmA, tmB, reinterpret_cast<__nv_bfloat16*>(C), reinterpret_cast<const int4*>(tiles),
-                                               num_tiles, N, K, ldc, err, num_rt_dev, nblk);
+  launch_pdl(kern, dim3(grid), dim3(192), (size_t)Cfg::SMEM_BYTES, stream, tmA, tmB, reinterpret_cast<__nv_bfloat16*>(C),
+             reinterpret_cast<const int4*>(tiles), num_tiles, N, K, ldc, err, num_rt_dev, nblk, heads ? R : 0);
   return cudaGetLastError() == cudaSuccess ? 0 : 302;
 }
 
@@ -282,5 +294,21 @@ int ab2_gemm_grouped_rt(const void* A, const void* B, void* C, const void* row_t
                              : launch_grouped<256, false>(A, B, C, row_tiles, (int)max_tiles, R, N, K, E, lda, ldc, s, nrt, nblk);
   return b_mn ? launch_grouped<128, true>(A, B, C, row_tiles, (int)max_tiles, R, N, K, E, lda, ldc, s, nrt, nblk)
               : launch_grouped<128, false>(A, B, C, row_tiles, (int)max_tiles, R, N, K, E, lda, ldc, s, nrt, nblk);
+}
+
+// C[r, h, :] = B[h] A[r, h, :]: A [R, E, K], C [R, E, N], B [E, N, K] (b_mn = 0) or [E, K, N] (b_mn = 1), all bf16 and contiguous.
+int ab2_gemm_heads(const void* A, const void* B, void* C, int R, int E, int N, int K, int b_mn, int bn, void* stream) {
+  using namespace ab2;
+  if (R <= 0 || E <= 0) return 0;
+  if ((K & 7) || (N & 7)) return 10;
+  if (bn != 128 && bn != 256) return 12;
+  const int nblk = (N + bn - 1) / bn;
+  const long long tiles = (long long)E * ((R + BM - 1) / BM) * nblk, cols = (long long)E * (K > N ? K : N);
+  if (tiles > 0x7fffffffLL || cols > 0x7fffffffLL) return 13;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (bn == 256) return b_mn ? launch_grouped<256, true>(A, B, C, nullptr, (int)tiles, R, N, K, E, E * K, E * N, s, nullptr, nblk, true)
+                             : launch_grouped<256, false>(A, B, C, nullptr, (int)tiles, R, N, K, E, E * K, E * N, s, nullptr, nblk, true);
+  return b_mn ? launch_grouped<128, true>(A, B, C, nullptr, (int)tiles, R, N, K, E, E * K, E * N, s, nullptr, nblk, true)
+              : launch_grouped<128, false>(A, B, C, nullptr, (int)tiles, R, N, K, E, E * K, E * N, s, nullptr, nblk, true);
 }
 }

@@ -1,6 +1,7 @@
 // Attention of mixer stacks over the paged cache: scores capped by softcap * tanh(s / softcap), a logarithmic distance
-// bias r1[h] * ln(1 + r2[h] * distance) taken off, and only the earlier keys of the query's own chunk of positions
-// visible (chunks counted from position 0 of the sequence; 0: no limit). Query / key and value sizes may differ.
+// bias r1[h] * ln(1 + r2[h] * distance) taken off (both optional), and only the earlier keys of the query's own chunk of
+// positions visible (chunks counted from position 0 of the sequence), or those of a sliding window (the query's position
+// and the window - 1 before it), or all of them (chunk = window = 0). Query / key and value sizes may differ.
 //
 //   chunk_attn_plain_kernel   any sizes, bf16 or 32-bit: a warp per (row, head)
 //   chunk_decode_kernel       single-token rows, bf16: a cluster of CTAs splits a request's chunk, mma.sync products,
@@ -8,7 +9,7 @@
 //   chunk_prefill_kernel      portions, bf16: tcgen05 products with accumulators in TMEM (second half of this file)
 //
 // Keys and values of the step's own tokens have been appended to the cache before. A query at position i needs rows
-// of pages[entry][j / page_size - page_base[entry]] for the positions j of its chunk.
+// of pages[entry][j / page_size - page_base[entry]] for the positions j that it sees.
 #include <cooperative_groups.h>
 
 #include "mixer_common.cuh"
@@ -21,7 +22,13 @@ struct ChunkArgs {
   int max_pages, page_size, Hq, Hkv, D, Dv;
   float scale, softcap;
   const float *r1, *r2;
-  int chunk;
+  int chunk, window;          // at most one of them set
+
+  // first position that a query at i sees (never decreases with i)
+  __device__ __forceinline__ int first_key(int i) const {
+    if (window > 0) return max(0, i - window + 1);
+    return chunk > 0 ? i / chunk * chunk : 0;
+  }
 };
 
 // Score in base-2 units: log2(e) * (cap(s * scale) - r1 ln(1 + r2 d)). u_scale and s_out are set up by score_consts().
@@ -53,16 +60,18 @@ chunk_attn_plain_kernel(const T* __restrict__ q, const int* __restrict__ pos, co
   const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y * 4 + warp;
   if (h >= p.Hq) return;
-  T* o = out + ((size_t)row * p.Hq + h) * p.Dv;
+  // values wider than one CTA's registers: blockIdx.z takes its stretch of them
+  const int v0 = blockIdx.z * PLAIN_MAX_DV, nv = min(p.Dv - v0, PLAIN_MAX_DV);
+  T* o = out + ((size_t)row * p.Hq + h) * p.Dv + v0;
   if (slots[row] < 0) {
-    for (int d = lane; d < p.Dv; d += 32) stf(o + d, 0.f);
+    for (int d = lane; d < nv; d += 32) stf(o + d, 0.f);
     return;
   }
   float* sq = sq_all + warp * p.D;
   for (int d = lane; d < p.D; d += 32) sq[d] = ldf(q + ((size_t)row * p.Hq + h) * p.D + d) * p.scale;
   __syncwarp();
   const int e = row_entry[row], i = pos[row], kvh = h / (p.Hq / p.Hkv);
-  const int lo = p.chunk > 0 ? i / p.chunk * p.chunk : 0;
+  const int lo = p.first_key(i);
   const int* pt = p.pages + (size_t)e * p.max_pages;
   const int base = p.page_base[e];
   const float r1 = p.r1 ? p.r1[h] : 0.f, r2 = p.r1 ? p.r2[h] : 0.f;
@@ -99,17 +108,17 @@ chunk_attn_plain_kernel(const T* __restrict__ q, const int* __restrict__ pos, co
     const int nj = min(32, i - j0 + 1);
     for (int t = 0; t < nj; ++t) {
       const float wt = __shfl_sync(0xffffffffu, w, t);
-      const T* vr = (const T*)p.vc + __shfl_sync(0xffffffffu, kv, t) * p.Dv;
+      const T* vr = (const T*)p.vc + __shfl_sync(0xffffffffu, kv, t) * p.Dv + v0;
 #pragma unroll
       for (int k = 0; k < PLAIN_MAX_DV / 32; ++k) {
-        if (k * 32 >= p.Dv) break;
-        if (k * 32 + lane < p.Dv) acc[k] += wt * ldf(vr + k * 32 + lane);
+        if (k * 32 >= nv) break;
+        if (k * 32 + lane < nv) acc[k] += wt * ldf(vr + k * 32 + lane);
       }
     }
   }
 #pragma unroll
   for (int k = 0; k < PLAIN_MAX_DV / 32; ++k)
-    if (k * 32 + lane < p.Dv) stf(o + k * 32 + lane, acc[k] / l);
+    if (k * 32 + lane < nv) stf(o + k * 32 + lane, acc[k] / l);
 }
 
 // ------------------------------------------------------------------ single-token rows
@@ -157,7 +166,7 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
   const int G = p.Hq / p.Hkv;
   const int i = pos[b];
   const bool live = slots[b] >= 0;
-  const int lo = p.chunk > 0 ? i / p.chunk * p.chunk : 0;
+  const int lo = p.first_key(i);
   const int len = live ? i + 1 - lo : 0;
   const int per = ((len + SPL - 1) / SPL + CD_KEYS - 1) / CD_KEYS * CD_KEYS;
   const int t0 = lo + spl * per, t1 = min(lo + len, t0 + per);
@@ -375,7 +384,7 @@ struct ChunkPrefillCfg {
   static constexpr int SMEM = BIAS_OFF + 16 * 96 * 4 + 1024;
 };
 
-template <int DK, int DV, bool CAP>
+template <int DK, int DV, bool CAP, bool BIAS>
 __global__ void __launch_bounds__(384, 1)
 chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                      const int* __restrict__ cu, const int* __restrict__ start, const int* __restrict__ tiles, __nv_bfloat16* __restrict__ out,
@@ -386,7 +395,7 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   const int rows = min(2 * CP_Q, cu[e + 1] - row0);
   const int q0 = start[e] + row0 - cu[e];                     // position of the first query row
   const int ntile = rows > CP_Q ? 2 : 1;
-  const int lo0 = p.chunk > 0 ? q0 / p.chunk * p.chunk : 0;
+  const int lo0 = p.first_key(q0);
   const int k0 = lo0 & ~(CP_K - 1);                           // first key block, on a 64-position boundary
   int nb[2];
   nb[0] = (q0 + min(rows, CP_Q) - 1 - k0) / CP_K + 1;
@@ -533,9 +542,9 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     const int nbt = t == 0 ? nb[0] : nb[1];
     const int first = q0 + t * CP_Q;                           // position of the tile's first row
     const int i = first + row;
-    const int lo = p.chunk > 0 ? i / p.chunk * p.chunk : 0;
+    const int lo = p.first_key(i);
     const int last = min(rows - t * CP_Q, CP_Q) - 1;
-    const int lo_last = p.chunk > 0 ? (first + max(last, 0)) / p.chunk * p.chunk : 0;
+    const int lo_last = p.first_key(first + max(last, 0));
     const ScoreConsts sc = score_consts(p.scale, p.softcap);
     const float r1 = p.r1 ? p.r1[head] : 0.f, r2 = p.r1 ? p.r2[head] : 0.f;
     float m_run = -INFINITY, l_run = 0.f;
@@ -544,8 +553,10 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       const int kb = k0 + j * CP_K;
       float* bs = bias + ((warp - 4) * 2 + (j & 1)) * 96;
       // diagonal x of this warp's 32 rows: distance first + 32 qd - kb + x - 63
-      for (int x = lane; x < 95; x += 32) bs[x] = r1 * __log2f(1.f + r2 * (float)max(first + qd * 32 - kb + x - 63, 0));
-      __syncwarp();
+      if constexpr (BIAS) {
+        for (int x = lane; x < 95; x += 32) bs[x] = r1 * __log2f(1.f + r2 * (float)max(first + qd * 32 - kb + x - 63, 0));
+        __syncwarp();
+      }
       ok = __all_sync(0xffffffffu, mbar_wait(s_full(t, j & 1), (uint32_t)(j >> 1) & 1u, err, ERR_WAIT_TMEM_FULL));
       if (!ok) break;                                          // a warp gives up as a whole
       tc_fence_after();
@@ -557,7 +568,8 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       float mx = -INFINITY;
 #pragma unroll
       for (int c = 0; c < 64; ++c) {
-        float v = capped<CAP>(__uint_as_float(u[c]), sc) - bs[lane - c + 63];
+        float v = capped<CAP>(__uint_as_float(u[c]), sc);
+        if constexpr (BIAS) v -= bs[lane - c + 63];
         if (edge && (kb + c > i || kb + c < lo)) v = -INFINITY;
         u[c] = __float_as_uint(v);
         mx = fmaxf(mx, v);
@@ -631,7 +643,7 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   }
 }
 
-template <int DK, int DV, bool CAP>
+template <int DK, int DV, bool CAP, bool>
 static int launch_decode(const void* q, const int* pos, const int* slots, void* out, int R, const ChunkArgs& a, cudaStream_t s) {
   constexpr int SMEM = ChunkDecodeCfg<DK, DV>::SMEM;
   static_assert(2 * ChunkDecodeCfg<DK, DV>::STAGE >= (4 * 16 * DV + 8 * 16) * 4, "the merge buffers alias the stage memory");
@@ -647,16 +659,16 @@ static int launch_decode(const void* q, const int* pos, const int* slots, void* 
   return go(chunk_decode_split_kernel<DK, DV, 8, CAP>, st8);
 }
 
-template <int DK, int DV, bool CAP>
-static int launch_prefill(const void* q, const int* cu, const int* start, const int* tiles, int nt, void* out, int R, int cache_rows,
-                          const ChunkArgs& a, cudaStream_t s) {
+template <int DK, int DV, bool CAP, bool BIAS>
+static int launch_prefill(const void* q, const int* cu, const int* start, const int* tiles, int nt, void* out, int R, int cache_rows, long long ldk,
+                          long long ldv, const ChunkArgs& a, cudaStream_t s) {
   using Cfg = ChunkPrefillCfg<DK, DV>;
   CUtensorMap tq, tk, tv;
   const uint32_t box = a.page_size < CP_K ? a.page_size : CP_K;
   if (ab2host::encode_tmap_3d(&tq, q, 2, a.D, a.Hq, R, (uint64_t)a.D * 2, (uint64_t)a.Hq * a.D * 2, 64, 1, CP_Q, true, 0)) return 100;
-  if (ab2host::encode_tmap_3d(&tk, a.kc, 2, a.D, a.Hkv, cache_rows, (uint64_t)a.D * 2, (uint64_t)a.Hkv * a.D * 2, 64, 1, box, true, 0)) return 101;
-  if (ab2host::encode_tmap_3d(&tv, a.vc, 2, a.Dv, a.Hkv, cache_rows, (uint64_t)a.Dv * 2, (uint64_t)a.Hkv * a.Dv * 2, 64, 1, box, true, 0)) return 102;
-  auto kern = chunk_prefill_kernel<DK, DV, CAP>;
+  if (ab2host::encode_tmap_3d(&tk, a.kc, 2, a.D, a.Hkv, cache_rows, (uint64_t)a.D * 2, (uint64_t)ldk * 2, 64, 1, box, true, 0)) return 101;
+  if (ab2host::encode_tmap_3d(&tv, a.vc, 2, a.Dv, a.Hkv, cache_rows, (uint64_t)a.Dv * 2, (uint64_t)ldv * 2, 64, 1, box, true, 0)) return 102;
+  auto kern = chunk_prefill_kernel<DK, DV, CAP, BIAS>;
   static ab2host::DevState st;
   if (ab2host::prepare_launch(kern, Cfg::SMEM, st, nullptr)) return 300;
   int* err = ab2host::error_flag();
@@ -674,11 +686,11 @@ using namespace ab2;
 // vc [rows, Hkv, Dv]; pages [entries, max_pages] from page number page_base[entry] on. r1 / r2 [Hq] or null. dt 0 bf16, 1 fp32.
 int ab2_chunk_attn_plain(const void* q, const int* pos, const int* slots, const int* row_entry, void* out, int R, const void* kc, const void* vc,
                          const int* pages, const int* page_base, int max_pages, int page_size, int Hq, int Hkv, int D, int Dv, float scale,
-                         float softcap, const float* r1, const float* r2, int chunk, int dt, void* stream) {
+                         float softcap, const float* r1, const float* r2, int chunk, int window, int dt, void* stream) {
   if (R <= 0) return 0;
-  if (Hq % Hkv || Dv > PLAIN_MAX_DV || 16 * D > 48 * 1024) return 10;
-  ChunkArgs a{kc, vc, pages, page_base, max_pages, page_size, Hq, Hkv, D, Dv, scale, softcap, r1, r2, chunk};
-  const dim3 grid(R, (Hq + 3) / 4);
+  if (Hq % Hkv || Dv > 65535 || 16 * D > 48 * 1024) return 10;
+  ChunkArgs a{kc, vc, pages, page_base, max_pages, page_size, Hq, Hkv, D, Dv, scale, softcap, r1, r2, chunk, window};
+  const dim3 grid(R, (Hq + 3) / 4, (Dv + PLAIN_MAX_DV - 1) / PLAIN_MAX_DV);
   if (dt == 0)
     chunk_attn_plain_kernel<__nv_bfloat16><<<grid, 128, 16 * D, (cudaStream_t)stream>>>((const __nv_bfloat16*)q, pos, slots, row_entry,
                                                                                        (__nv_bfloat16*)out, a);
@@ -687,35 +699,35 @@ int ab2_chunk_attn_plain(const void* q, const int* pos, const int* slots, const 
   return cudaGetLastError() == cudaSuccess ? 0 : 1;
 }
 
+#define AB2_BY_SIZE2(FN, CAP, BIAS, ...)                                                                           \
+  if (D <= 64) return Dv <= 64 ? FN<64, 64, CAP, BIAS>(__VA_ARGS__) : FN<64, 128, CAP, BIAS>(__VA_ARGS__);          \
+  return Dv <= 64 ? FN<128, 64, CAP, BIAS>(__VA_ARGS__) : FN<128, 128, CAP, BIAS>(__VA_ARGS__)
 #define AB2_BY_SIZE(FN, ...)                                                                                       \
-  if (a.softcap > 0.f) {                                                                                           \
-    if (D <= 64) return Dv <= 64 ? FN<64, 64, true>(__VA_ARGS__) : FN<64, 128, true>(__VA_ARGS__);                  \
-    return Dv <= 64 ? FN<128, 64, true>(__VA_ARGS__) : FN<128, 128, true>(__VA_ARGS__);                             \
-  }                                                                                                                \
-  if (D <= 64) return Dv <= 64 ? FN<64, 64, false>(__VA_ARGS__) : FN<64, 128, false>(__VA_ARGS__);                  \
-  return Dv <= 64 ? FN<128, 64, false>(__VA_ARGS__) : FN<128, 128, false>(__VA_ARGS__)
+  if (a.softcap > 0.f) { AB2_BY_SIZE2(FN, true, true, __VA_ARGS__); }                                              \
+  if (a.r1 != nullptr) { AB2_BY_SIZE2(FN, false, true, __VA_ARGS__); }                                             \
+  AB2_BY_SIZE2(FN, false, false, __VA_ARGS__)
 
 // Row r is the only row of entry r. bf16; D, Dv multiples of 8 up to 128, at most 16 query heads per key head.
 int ab2_chunk_decode(const void* q, const int* pos, const int* slots, void* out, int R, const void* kc, const void* vc, const int* pages,
                      const int* page_base, int max_pages, int page_size, int Hq, int Hkv, int D, int Dv, float scale, float softcap,
-                     const float* r1, const float* r2, int chunk, void* stream) {
+                     const float* r1, const float* r2, int chunk, int window, void* stream) {
   if (R <= 0) return 0;
   if (Hq % Hkv || Hq / Hkv > 16 || (D & 7) || (Dv & 7) || D > 128 || Dv > 128 || Hkv > 65535) return 10;
   if (!aligned_to(q, 16) || !aligned_to(kc, 16) || !aligned_to(vc, 16)) return 11;
-  ChunkArgs a{kc, vc, pages, page_base, max_pages, page_size, Hq, Hkv, D, Dv, scale, softcap, r1, r2, chunk};
+  ChunkArgs a{kc, vc, pages, page_base, max_pages, page_size, Hq, Hkv, D, Dv, scale, softcap, r1, r2, chunk, window};
   AB2_BY_SIZE(launch_decode, q, pos, slots, out, R, a, (cudaStream_t)stream);
 }
 
 // tiles [nt, 2] = (entry, first row); q / out hold all R rows of the step. bf16; D, Dv multiples of 8 up to 128;
-// page_size 16, 32 or a multiple of 64.
-int ab2_chunk_prefill(const void* q, const int* cu, const int* start, const int* tiles, int nt, void* out, int R, int cache_rows, const void* kc,
-                      const void* vc, const int* pages, const int* page_base, int max_pages, int page_size, int Hq, int Hkv, int D, int Dv,
-                      float scale, float softcap, const float* r1, const float* r2, int chunk, void* stream) {
+// page_size 16, 32 or a multiple of 64. ldk / ldv: elements from one cache row to the next.
+int ab2_chunk_prefill(const void* q, const int* cu, const int* start, const int* tiles, int nt, void* out, int R, int cache_rows, long long ldk,
+                      long long ldv, const void* kc, const void* vc, const int* pages, const int* page_base, int max_pages, int page_size, int Hq, int Hkv, int D, int Dv,
+                      float scale, float softcap, const float* r1, const float* r2, int chunk, int window, void* stream) {
   if (nt <= 0) return 0;
-  if (Hq % Hkv || (D & 7) || (Dv & 7) || D > 128 || Dv > 128 || Hq > 65535) return 10;
+  if (Hq % Hkv || (D & 7) || (Dv & 7) || D > 128 || Dv > 128 || Hq > 65535 || (ldk & 7) || (ldv & 7)) return 10;
   if (!aligned_to(q, 16) || !aligned_to(kc, 16) || !aligned_to(vc, 16) || !aligned_to(out, 16)) return 11;
   if (!(page_size == 16 || page_size == 32 || (page_size > 0 && page_size % 64 == 0))) return 12;
-  ChunkArgs a{kc, vc, pages, page_base, max_pages, page_size, Hq, Hkv, D, Dv, scale, softcap, r1, r2, chunk};
-  AB2_BY_SIZE(launch_prefill, q, cu, start, tiles, nt, out, R, cache_rows, a, (cudaStream_t)stream);
+  ChunkArgs a{kc, vc, pages, page_base, max_pages, page_size, Hq, Hkv, D, Dv, scale, softcap, r1, r2, chunk, window};
+  AB2_BY_SIZE(launch_prefill, q, cu, start, tiles, nt, out, R, cache_rows, ldk, ldv, a, (cudaStream_t)stream);
 }
 }

@@ -1,7 +1,8 @@
 // Elementwise, norm, convolution and small-product kernels of mixer stacks (bf16 or fp32 activations, fp32 residual
-// stream, norm weights and states): grouped sandwich norms, whole-projection q / k norms fused with the cache append,
-// causal convolutions with carried tails, xIELU, SiLU gate, expert combine, capped logits, and a plain grouped product
-// for 32-bit experts and odd sizes.
+// stream, norm weights and states): grouped sandwich norms, norms behind a sublayer (fused with the expert sum), whole-
+// projection q / k norms fused with the cache append, causal convolutions with carried tails, xIELU, GELU, SiLU gate,
+// clamped gated units, token side gate, expert combine, capped logits, and a plain grouped product for 32-bit experts
+// and odd sizes.
 #include "mixer_common.cuh"
 
 namespace ab2 {
@@ -138,6 +139,96 @@ __global__ void gated_norm_kernel(const float* __restrict__ y, const T* __restri
       for (int e = 0; e < V; ++e) a[e] = a[e] * rstd * b[e];
       stv<V>(out + (size_t)row * C + c, a);
     }
+  }
+}
+
+// ------------------------------------------------------------------ norms behind a sublayer
+// h = base row + the sum of the token's k expert rows (either may be missing); resid += mult * norm(h) * (off + w);
+// x = resid, or norm(resid) * (off_next + w_next) when there is a next norm. One CTA per row, the row in shared memory.
+template <typename T, int V>
+__global__ void post_norm_kernel(const T* __restrict__ base, long long ldb, const T* __restrict__ y, const int* __restrict__ inv, int k, int n_rows,
+                                 const float* __restrict__ w, float off, float mult, float* __restrict__ resid, const float* __restrict__ w_next,
+                                 float off_next, T* __restrict__ x, int H, float eps) {
+  extern __shared__ __align__(16) float srow[];       // [H] values, then two rows of partial sums
+  pdl_wait();
+  pdl_trigger();
+  float* sums = srow + ((H + 3) & ~3);
+  const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  auto total = [&](const float* part) {
+    float s = 0.f;
+    for (int i = 0; i < nw; ++i) s += part[i];
+    return s;
+  };
+  float ss = 0.f;
+  for (int c = threadIdx.x * V; c < H; c += blockDim.x * V) {
+    float h[V];
+    if (base != nullptr) ldv<V>(base + (size_t)row * ldb + c, h);
+    else
+      for (int e = 0; e < V; ++e) h[e] = 0.f;
+    for (int s = 0; s < k; ++s) {
+      const int r = inv[(size_t)row * k + s];
+      if (r < 0 || r >= n_rows) continue;
+      float v[V];
+      ldv<V>(y + (size_t)r * H + c, v);
+      for (int e = 0; e < V; ++e) h[e] += v[e];
+    }
+    for (int e = 0; e < V; ++e) ss += h[e] * h[e];
+    stv<V>(srow + c, h);
+  }
+  ss = warp_sum(ss);
+  if (lane == 0) sums[warp] = ss;
+  __syncthreads();
+  const float rstd = mult / sqrtf(total(sums) / H + eps);
+  float* rr = resid + (size_t)row * H;
+  ss = 0.f;
+  for (int c = threadIdx.x * V; c < H; c += blockDim.x * V) {
+    float h[V], r[V], g[V];
+    ldv<V>(srow + c, h);
+    ldv<V>(rr + c, r);
+    ldv<V>(w + c, g);
+    for (int e = 0; e < V; ++e) r[e] += h[e] * rstd * (off + g[e]);
+    stv<V>(rr + c, r);
+    if (w_next == nullptr) {
+      stv<V>(x + (size_t)row * H + c, r);
+    } else {
+      stv<V>(srow + c, r);
+      for (int e = 0; e < V; ++e) ss += r[e] * r[e];
+    }
+  }
+  if (w_next == nullptr) return;
+  ss = warp_sum(ss);
+  if (lane == 0) sums[nw + warp] = ss;
+  __syncthreads();
+  const float rn = 1.f / sqrtf(total(sums + nw) / H + eps);
+  for (int c = threadIdx.x * V; c < H; c += blockDim.x * V) {
+    float r[V], g[V];
+    ldv<V>(srow + c, r);
+    ldv<V>(w_next + c, g);
+    for (int e = 0; e < V; ++e) r[e] = r[e] * rn * (off_next + g[e]);
+    stv<V>(x + (size_t)row * H + c, r);
+  }
+}
+
+// resid = table[ids] (+ pos_table[pos]) in fp32, x the same in T.
+template <typename T, int V>
+__global__ void embed_rows_kernel(const int* __restrict__ ids, const T* __restrict__ table, int vocab, const int* __restrict__ pos,
+                                  const T* __restrict__ pos_table, int n_pos, float* __restrict__ resid, T* __restrict__ x, long long total, int H) {
+  pdl_wait();
+  pdl_trigger();
+  const int hv = H / V;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / hv;
+    const int c = (int)(i - r * hv) * V;
+    const int id = min(max(ids[r], 0), vocab - 1);
+    float v[V];
+    ldv<V>(table + (size_t)id * H + c, v);
+    if (pos_table != nullptr) {
+      float p[V];
+      ldv<V>(pos_table + (size_t)min(max(pos[r], 0), n_pos - 1) * H + c, p);
+      for (int e = 0; e < V; ++e) v[e] += p[e];
+    }
+    stv<V>(resid + r * H + c, v);
+    stv<V>(x + r * H + c, v);
   }
 }
 
@@ -342,6 +433,70 @@ __global__ void glu_silu_kernel(const T* __restrict__ gu, long long ld, T* __res
 }
 
 template <typename T, int V>
+__global__ void gelu_erf_kernel(const T* __restrict__ x, long long ld, T* __restrict__ out, long long total, int C) {
+  pdl_wait();
+  pdl_trigger();
+  const int cv = C / V;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / cv;
+    const int c = (int)(i - r * cv) * V;
+    float v[V];
+    ldv<V>(x + r * ld + c, v);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = 0.5f * v[e] * (1.f + erff(v[e] * 0.7071067811865476f));
+    stv<V>(out + r * C + c, v);
+  }
+}
+
+// Clamped gated units: rows g | u, both first multiplied by the row's weight when there are weights (topw by entry, order:
+// the entry of a row).
+template <typename T, int V>
+__global__ void glu_clamped_kernel(const T* __restrict__ gu, long long ld, const int* __restrict__ order, const float* __restrict__ topw,
+                                   T* __restrict__ out, long long total, int I, float limit, float alpha) {
+  pdl_wait();
+  pdl_trigger();
+  const int cv = I / V;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / cv;
+    const int c = (int)(i - r * cv) * V;
+    float w = 1.f;
+    if (topw != nullptr) {
+      const int n = order[r];
+      w = n >= 0 && n < total / cv ? topw[n] : 0.f;
+    }
+    float g[V], u[V];
+    ldv<V>(gu + r * ld + c, g);
+    ldv<V>(gu + r * ld + I + c, u);
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      const float a = fminf(w * g[e], limit), b = fminf(fmaxf(w * u[e], -limit), limit);
+      g[e] = a * sigmoid_t<sizeof(T) == 2>(alpha * a) * (b + 1.f);
+    }
+    stv<V>(out + r * I + c, g);
+  }
+}
+
+// out = gelu_tanh(g) * table[ids, col:col + D]
+template <typename T, int V>
+__global__ void side_gate_kernel(const T* __restrict__ g, long long ld, const int* __restrict__ ids, const T* __restrict__ table, int vocab,
+                                 long long ldt, int col, T* __restrict__ out, long long total, int D) {
+  pdl_wait();
+  pdl_trigger();
+  const int dv = D / V;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / dv;
+    const int c = (int)(i - r * dv) * V;
+    const int id = min(max(ids[r], 0), vocab - 1);
+    float v[V], t[V];
+    ldv<V>(g + r * ld + c, v);
+    ldv<V>(table + id * ldt + col + c, t);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = gelu_tanh_t<sizeof(T) == 2>(v[e]) * t[e];
+    stv<V>(out + r * D + c, v);
+  }
+}
+
+template <typename T, int V>
 __global__ void expert_combine_kernel(const T* __restrict__ y, const int* __restrict__ inv, const float* __restrict__ topw, T* __restrict__ out,
                                       long long total, int k, int H, int n_rows) {
   pdl_wait();
@@ -464,6 +619,44 @@ int ab2_sandwich_norm(const int* ids, const void* table, int vocab, const void* 
   AB2_DONE;
 }
 
+// x and resid [R, H]; base [R, H] (ldb) and / or y [n_rows, H] with inv [R, k]. w_next may be null.
+int ab2_post_norm(const void* base, long long ldb, const void* y, const int* inv, int k, int n_rows, const float* w, float off, float mult,
+                  float* resid, const float* w_next, float off_next, void* x, int R, int H, float eps, int dt, void* stream) {
+  if (R <= 0) return 0;
+  if (H < 1 || (base == nullptr && y == nullptr)) return 10;
+  const int th = norm_threads(H);
+  const size_t smem = (size_t)(((H + 3) & ~3) + 2 * (th / 32)) * 4;
+  if (smem > 200 * 1024) return 11;
+  const int eb = dt == 0 ? 2 : 4;
+  if (y == nullptr) k = 0;
+  auto fits = [&](int v) {
+    return H % v == 0 && ldb % v == 0 && aligned_to(base, v * eb) && aligned_to(y, v * eb) && aligned_to(x, v * eb) && aligned_to(resid, 16) &&
+           aligned_to(w, 16) && aligned_to(w_next, 16);
+  };
+  AB2_TYPED8(dt, fits(8), fits(4), {
+    auto kern = post_norm_kernel<T, V>;
+    static ab2host::DevState st;
+    if (ab2host::prepare_launch(kern, 200 * 1024, st, nullptr)) return 12;
+    launch_pdl(kern, dim3(R), dim3(th), smem, (cudaStream_t)stream, (const T*)base, ldb, (const T*)y, inv, k, n_rows, w, off, mult, resid, w_next,
+               off_next, (T*)x, H, eps);
+  });
+  AB2_DONE;
+}
+
+int ab2_embed_rows(const int* ids, const void* table, int vocab, const int* pos, const void* pos_table, int n_pos, float* resid, void* x, int R, int H,
+                   int dt, void* stream) {
+  if (R <= 0) return 0;
+  if (vocab < 1 || (pos_table != nullptr && n_pos < 1)) return 10;
+  const int eb = dt == 0 ? 2 : 4;
+  auto fits = [&](int v) { return H % v == 0 && aligned_to(table, v * eb) && aligned_to(pos_table, v * eb) && aligned_to(x, v * eb) && aligned_to(resid, 16); };
+  AB2_TYPED8(dt, fits(8), fits(4), {
+    const long long n = (long long)R * (H / V);
+    launch_pdl(embed_rows_kernel<T, V>, dim3(flat_grid(n)), dim3(256), 0, (cudaStream_t)stream, ids, (const T*)table, vocab, pos, (const T*)pos_table,
+               n_pos, resid, (T*)x, n, H);
+  });
+  AB2_DONE;
+}
+
 int ab2_gated_group_norm(const float* y, const void* z, long long ldz, const float* w, void* out, int R, int C, int groups, float eps, int dt,
                          void* stream) {
   if (R <= 0) return 0;
@@ -552,6 +745,46 @@ int ab2_glu_silu(const void* gu, long long ld, void* out, int R, int I, int dt, 
   AB2_TYPED8(dt, I % 8 == 0 && ld % 8 == 0 && aligned_to(gu, 16), vec, {
     const long long n = (long long)R * (I / V);
     launch_pdl(glu_silu_kernel<T, V>, dim3(flat_grid(n)), dim3(256), 0, (cudaStream_t)stream, (const T*)gu, ld, (T*)out, n, I);
+  });
+  AB2_DONE;
+}
+
+int ab2_gelu_erf(const void* x, long long ld, void* out, int R, int C, int dt, void* stream) {
+  if (R <= 0) return 0;
+  const int eb = dt == 0 ? 2 : 4;
+  auto fits = [&](int v) { return C % v == 0 && ld % v == 0 && aligned_to(x, v * eb) && aligned_to(out, v * eb); };
+  AB2_TYPED8(dt, fits(8), fits(4), {
+    const long long n = (long long)R * (C / V);
+    launch_pdl(gelu_erf_kernel<T, V>, dim3(flat_grid(n)), dim3(256), 0, (cudaStream_t)stream, (const T*)x, ld, (T*)out, n, C);
+  });
+  AB2_DONE;
+}
+
+// order [R] and topw [R] together or not at all
+int ab2_glu_clamped(const void* gu, long long ld, const int* order, const float* topw, void* out, int R, int I, float limit, float alpha, int dt,
+                    void* stream) {
+  if (R <= 0) return 0;
+  if ((order == nullptr) != (topw == nullptr)) return 10;
+  const int eb = dt == 0 ? 2 : 4;
+  auto fits = [&](int v) { return I % v == 0 && ld % v == 0 && aligned_to(gu, v * eb) && aligned_to(out, v * eb); };
+  AB2_TYPED8(dt, fits(8), fits(4), {
+    const long long n = (long long)R * (I / V);
+    launch_pdl(glu_clamped_kernel<T, V>, dim3(flat_grid(n)), dim3(256), 0, (cudaStream_t)stream, (const T*)gu, ld, order, topw, (T*)out, n, I, limit,
+               alpha);
+  });
+  AB2_DONE;
+}
+
+int ab2_side_gate(const void* g, long long ld, const int* ids, const void* table, int vocab, long long ldt, int col, void* out, int R, int D, int dt,
+                  void* stream) {
+  if (R <= 0) return 0;
+  if (vocab < 1 || col < 0 || col + D > ldt) return 10;
+  const int eb = dt == 0 ? 2 : 4;
+  auto fits = [&](int v) { return D % v == 0 && ld % v == 0 && ldt % v == 0 && col % v == 0 && aligned_to(g, v * eb) && aligned_to(table, v * eb); };
+  AB2_TYPED8(dt, fits(8), fits(4), {
+    const long long n = (long long)R * (D / V);
+    launch_pdl(side_gate_kernel<T, V>, dim3(flat_grid(n)), dim3(256), 0, (cudaStream_t)stream, (const T*)g, ld, ids, (const T*)table, vocab, ldt, col,
+               (T*)out, n, D);
   });
   AB2_DONE;
 }

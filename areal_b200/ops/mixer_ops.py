@@ -1,6 +1,7 @@
-"""Ops of mixer stacks: grouped sandwich norms on a 32-bit residual stream, chunked attention with capped scores and
-a logarithmic distance bias over a paged cache, causal convolutions, RG-LRU and Mamba-2 recurrences on slot states,
-xIELU, expert combine and capped logits.
+"""Ops of mixer stacks: norms around (grouped) or behind the sublayers on a 32-bit residual stream, chunked attention
+with capped scores and a logarithmic distance bias over a paged cache, sliding-window attention on cached latents, causal
+convolutions, RG-LRU and Mamba-2 recurrences on slot states, activations, expert combine, per-layer token inputs and
+capped logits.
 
 Every op works on a :class:`RaggedBatch`: the rows of several requests, each bringing any number of its next tokens,
 continuing from the cache pages and state slots that earlier steps left. The first ``n_dec`` entries bring one row
@@ -13,7 +14,7 @@ stream are fp32 everywhere.
 from __future__ import annotations
 
 import math
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import Optional
 
 import torch
@@ -46,6 +47,15 @@ def _call(name: str, *args):
 
 
 @dataclass
+class PageList:
+    """Cache pages that a step's portions see, in one list, and every entry's place in it."""
+
+    pages: torch.Tensor          # [NP] pages of the cache
+    table: torch.Tensor          # [E, P'] numbers in ``pages`` of the entry's pages, from page number ``base`` of its sequence on
+    base: torch.Tensor           # [E]
+
+
+@dataclass
 class RaggedBatch:
     """Rows of one step (all tensors int32 on the model's device)."""
 
@@ -62,6 +72,7 @@ class RaggedBatch:
     tiles: Optional[torch.Tensor]    # [NT, 2] (entry, first row) query tiles of entries >= n_dec
     n_dec: int                   # leading entries with one row
     page_size: int
+    seen: dict = field(default_factory=dict)     # sliding window -> PageList of the entries >= n_dec (latent attention)
 
     @property
     def n_rows(self) -> int:
@@ -95,9 +106,25 @@ def linear(x: torch.Tensor, w: torch.Tensor, fp32_out: bool = False) -> torch.Te
     return F.linear(x, w)
 
 
+def head_linear(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, w_kn: bool = False) -> torch.Tensor:
+    """Every head's own product: ``out[r, h] = w[h] x[r, h]``; x [R, H, K], w [H, N, K] (``w_kn``: [H, K, N]). One tcgen05
+    launch for bf16 with aligned sizes, the library's batched product in 32-bit and for odd sizes."""
+    R, H, K = x.shape
+    N = w.shape[2] if w_kn else w.shape[1]
+    if out is None:
+        out = torch.empty(R, H, N, device=x.device, dtype=x.dtype)
+    if x.is_cuda and x.dtype == torch.bfloat16 and K % 8 == 0 and N % 8 == 0:
+        assert x.is_contiguous() and w.is_contiguous() and out.is_contiguous()
+        bn = 256 if N % 256 == 0 and R > 128 else 128
+        _call("ab2_gemm_heads", _p(x), _p(w), _p(out), R, H, N, K, int(w_kn), bn)
+        return out
+    out.copy_(torch.bmm(x.transpose(0, 1), w if w_kn else w.transpose(1, 2)).transpose(0, 1))
+    return out
+
+
 def router_logits(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
-    """32-bit router logits from (possibly bf16) activations and weights."""
-    return F.linear(x.float(), w.float())
+    """32-bit router logits from (possibly bf16) activations and weights: exact products, 32-bit sums."""
+    return linear(x, w, fp32_out=True)
 
 
 # ----------------------------------------------------------------------------- norms
@@ -129,6 +156,56 @@ def sandwich_norm(h, w_post, resid, w_next, groups: int, eps: float):
     assert h.stride(1) == 1
     x = torch.empty(T, H, device=h.device, dtype=h.dtype)
     _call("ab2_sandwich_norm", None, None, 0, _p(h), h.stride(0), _p(w_post), _p(resid), _p(w_next), _p(x), T, H, groups, eps, _dt(h))
+    return x
+
+
+@dataclass
+class ExpertSum:
+    """A feed-forward output that is still in pieces: the expert-sorted rows ``y``, to be summed per token, and what is
+    added to them. The norm behind the sublayer reads the pieces."""
+
+    y: torch.Tensor                      # [T * k, H]
+    routing: Routing
+    shared: Optional[torch.Tensor]       # [T, H]
+
+    def dense(self) -> torch.Tensor:
+        k = self.routing.k
+        h = self.y.index_select(0, self.routing.inv).view(-1, k, self.y.shape[1]).float().sum(1)
+        return h if self.shared is None else h + self.shared.float()
+
+
+def embed_rows(ids, table, pos, pos_table=None):
+    """``(residual fp32, residual in the table's dtype)``: the embedding rows of ``ids``, plus the rows of ``pos`` in
+    ``pos_table`` when there is one."""
+    if not table.is_cuda:
+        resid = table[ids.long()].float()
+        if pos_table is not None:
+            resid = resid + pos_table[pos.long().clamp(0, pos_table.shape[0] - 1)].float()
+        return resid, resid.to(table.dtype)
+    T, H = ids.shape[0], table.shape[1]
+    resid = torch.empty(T, H, device=table.device, dtype=torch.float32)
+    x = torch.empty(T, H, device=table.device, dtype=table.dtype)
+    _call("ab2_embed_rows", _p(ids), _p(table), table.shape[0], _p(pos), _p(pos_table), 0 if pos_table is None else pos_table.shape[0], _p(resid), _p(x), T, H,
+          _dt(table))
+    return resid, x
+
+
+def post_norm(h, w, resid, eps: float, mult: float = 1.0, offset: float = 0.0, w_next=None, offset_next: float = 0.0):
+    """``resid += mult * rmsnorm(h) * (offset + w)`` (in place, fp32); returns resid in h's dtype, or with ``w_next``
+    ``rmsnorm(resid) * (offset_next + w_next)``. ``h`` is [R, H] or an :class:`ExpertSum`."""
+    parts = isinstance(h, ExpertSum)
+    src = h.y if parts else h
+    if not src.is_cuda:
+        resid += mult * group_norm_ref(h.dense() if parts else h, offset + w, 1, eps)
+        out = resid if w_next is None else group_norm_ref(resid, offset_next + w_next, 1, eps)
+        return out.to(src.dtype)
+    T, H = resid.shape
+    assert src.stride(1) == 1
+    x = torch.empty(T, H, device=src.device, dtype=src.dtype)
+    base = h.shared if parts else h
+    ld = 0 if base is None else base.stride(0)
+    y, inv, k, n = (_p(h.y), _p(h.routing.inv), h.routing.k, h.y.shape[0]) if parts else (None, None, 0, 0)
+    _call("ab2_post_norm", _p(base), ld, y, inv, k, n, _p(w), offset, mult, _p(resid), _p(w_next), offset_next, _p(x), T, H, eps, _dt(src))
     return x
 
 
@@ -187,7 +264,7 @@ def chunk_attention(q, kc, vc, b: RaggedBatch, scale: float, softcap: float = 0.
     R, Hq, D = q.shape
     Hkv, Dv = kc.shape[1], vc.shape[2]
     out = torch.empty(R, Hq, Dv, device=q.device, dtype=q.dtype)
-    common = (_p(kc), _p(vc), _p(b.pages), _p(b.page_base), b.pages.shape[1], b.page_size, Hq, Hkv, D, Dv, scale, softcap, _p(r1), _p(r2), chunk)
+    common = (_p(kc), _p(vc), _p(b.pages), _p(b.page_base), b.pages.shape[1], b.page_size, Hq, Hkv, D, Dv, scale, softcap, _p(r1), _p(r2), chunk, 0)
     fast = q.dtype == torch.bfloat16 and D % 8 == 0 and Dv % 8 == 0 and D <= 128 and Dv <= 128
     nd = b.n_dec
     if nd:
@@ -197,9 +274,81 @@ def chunk_attention(q, kc, vc, b: RaggedBatch, scale: float, softcap: float = 0.
             _call("ab2_chunk_attn_plain", _p(q), _p(b.pos), _p(b.slots), _p(b.row_entry), _p(out), nd, *common, _dt(q))
     if R > nd:
         if fast and b.page_size in (16, 32, 64, 128) and b.tiles is not None:
-            _call("ab2_chunk_prefill", _p(q), _p(b.cu), _p(b.start), _p(b.tiles), b.tiles.shape[0], _p(out), R, kc.shape[0], *common)
+            _call("ab2_chunk_prefill", _p(q), _p(b.cu), _p(b.start), _p(b.tiles), b.tiles.shape[0], _p(out), R, kc.shape[0], Hkv * D, Hkv * Dv, *common)
         else:
             _call("ab2_chunk_attn_plain", _p(q[nd:]), _p(b.pos[nd:]), _p(b.slots[nd:]), _p(b.row_entry[nd:]), _p(out[nd:]), R - nd, *common, _dt(q))
+    return out
+
+
+# ----------------------------------------------------------------------------- attention on cached latents
+def latent_norm_append(x, wq, wc, eps: float, b: RaggedBatch, cache):
+    """RMS norms of the two parts of ``x`` (query latent | cached latent), the second into the cache rows of ``b.slots``;
+    returns the first [R, q_rank]. ``cache`` [S, 1, kv_rank]."""
+    nq, nc = wq.shape[0], wc.shape[0]
+    R = x.shape[0]
+    if not x.is_cuda:
+        ok = b.slots >= 0
+        cache[b.slots[ok].long(), 0] = group_norm_ref(x[:, nq:], wc, 1, eps).to(x.dtype)[ok]
+        return group_norm_ref(x[:, :nq], wq, 1, eps).to(x.dtype)
+    cq = torch.empty(R, nq, device=x.device, dtype=x.dtype)
+    _call("ab2_qk_norm_append", _p(x), x.stride(0), _p(wq), _p(wc), _p(b.slots), _p(cq), _p(cache), None, R, nq, nc, 0, eps, _dt(x))
+    return cq
+
+
+def latent_attention_ref(q, cache, w_kv, Dv, b: RaggedBatch, scale, window):
+    R, H, D = q.shape
+    ps = b.page_size
+    out = torch.zeros(R, H, Dv, dtype=q.dtype)
+    for e, r0, r1, st, _ in _segments(b):
+        i = torch.arange(st, st + r1 - r0)
+        j = torch.arange(max(0, st - window + 1) if window else 0, st + r1 - r0)
+        rows = b.pages[e][(j // ps - b.page_base[e]).long()].long() * ps + j % ps
+        kv = F.linear(cache[rows, 0].float(), w_kv.float())
+        k, v = kv[:, :H * D].view(-1, H, D), kv[:, H * D:].view(-1, H, Dv)
+        s = torch.einsum("ihd,jhd->hij", q[r0:r1].float(), k) * scale
+        dist = i[:, None] - j[None, :]
+        see = (dist >= 0) & (dist < window) if window else dist >= 0
+        w = torch.softmax(s.masked_fill(~see, float("-inf")), -1)
+        out[r0:r1] = torch.einsum("hij,jhd->ihd", w, v).to(q.dtype)
+    return out
+
+
+# portions of up to this many tokens (on average) read the latents as single tokens do: working out keys and values of a
+# whole window would cost more than it saves
+SHORT_PORTION = 16
+
+
+def latent_attention(q, cache, w_kv, Dv: int, b: RaggedBatch, scale: float, window: int = 0):
+    """Attention of the step's queries q [R, H, D] over cached latents (the step's own already appended): head h has keys
+    ``w_kv[h D:(h + 1) D] c`` and values ``w_kv[H D + h Dv:...] c``, softmax of ``scale * q.k`` over the position itself and
+    the ``window - 1`` before it (0: no limit). cache [S, 1, C], w_kv [H (D + Dv), C]. Returns [R, H, Dv]."""
+    R, H, D = q.shape
+    C = w_kv.shape[1]
+    if not q.is_cuda:
+        return latent_attention_ref(q, cache, w_kv, Dv, b, scale, window)
+    w_k, w_v = w_kv[:H * D].view(H, D, C), w_kv[H * D:].view(H, Dv, C)
+    out = torch.empty(R, H, Dv, device=q.device, dtype=q.dtype)
+    nd, bf16 = b.n_dec, q.dtype == torch.bfloat16
+    fast_rows = bf16 and C % 8 == 0 and C <= 512
+    fast_tiles = bf16 and D % 8 == 0 and Dv % 8 == 0 and D <= 128 and Dv <= 128 and C % 8 == 0 and b.page_size in (16, 32, 64, 128)
+    whole = R > nd and fast_tiles and R - nd > SHORT_PORTION * (b.n_entries - nd)
+    n = nd if whole else R
+    if n:
+        # keys applied to the queries: scores against the latents themselves, the values' part after the sum
+        qc = head_linear(q[:n], w_k, w_kn=True)
+        oc = torch.empty_like(qc)
+        args = (_p(qc), _p(b.pos), _p(b.slots), _p(b.row_entry), _p(oc), n)
+        if fast_rows:
+            _call("ab2_latent_decode", *args, _p(cache), _p(b.pages), _p(b.page_base), b.pages.shape[1], b.page_size, H, C, scale, window)
+        else:
+            _call("ab2_chunk_attn_plain", *args, _p(cache), _p(cache), _p(b.pages), _p(b.page_base), b.pages.shape[1], b.page_size, H, 1, C, C, scale, 0.0,
+                  None, None, 0, window, _dt(q))
+        head_linear(oc, w_v, out[:n])
+    if whole:
+        seen, ps = b.seen[window], b.page_size
+        kv = linear(cache.view(-1, ps * C).index_select(0, seen.pages).view(-1, C), w_kv)
+        _call("ab2_chunk_prefill", _p(q), _p(b.cu), _p(b.start), _p(b.tiles), b.tiles.shape[0], _p(out), R, kv.shape[0], kv.stride(0), kv.stride(0),
+              _p(kv), _p(kv[:, H * D:]), _p(seen.table), _p(seen.base), seen.table.shape[1], ps, H, H, D, Dv, scale, 0.0, None, None, 0, window)
     return out
 
 
@@ -328,6 +477,41 @@ def glu_silu(gu):
     return out
 
 
+def gelu_erf(x):
+    """``z (1 + erf(z / sqrt 2)) / 2``."""
+    if not x.is_cuda:
+        return F.gelu(x.float()).to(x.dtype)
+    out = torch.empty(x.shape, device=x.device, dtype=x.dtype)
+    _call("ab2_gelu_erf", _p(x), x.stride(0), _p(out), x.shape[0], x.shape[1], _dt(x))
+    return out
+
+
+def glu_clamped(gu, limit: float, alpha: float, routing: Optional[Routing] = None):
+    """``g sigmoid(alpha g) (u + 1)`` with ``g = min(w g', limit)`` and ``u = clamp(w u', -limit, limit)`` for rows g' | u'.
+    With a routing the rows are its expert-sorted ones and w is each row's gate weight, else 1."""
+    I = gu.shape[1] // 2
+    if not gu.is_cuda:
+        z = gu.float()
+        if routing is not None:
+            z = z * routing.topw.reshape(-1)[routing.order.long()][:, None]
+        g, u = z[:, :I].clamp(max=limit), z[:, I:].clamp(-limit, limit)
+        return (g * torch.sigmoid(alpha * g) * (u + 1)).to(gu.dtype)
+    out = torch.empty(gu.shape[0], I, device=gu.device, dtype=gu.dtype)
+    order, topw = (None, None) if routing is None else (_p(routing.order), _p(routing.topw))
+    _call("ab2_glu_clamped", _p(gu), gu.stride(0), order, topw, _p(out), gu.shape[0], I, limit, alpha, _dt(gu))
+    return out
+
+
+def side_gate(g, ids, table, col: int):
+    """``gelu_tanh(g) * table[ids, col:col + D]`` for g [R, D]."""
+    D = g.shape[1]
+    if not g.is_cuda:
+        return (F.gelu(g.float(), approximate="tanh") * table[ids.long(), col:col + D].float()).to(g.dtype)
+    out = torch.empty(g.shape[0], D, device=g.device, dtype=g.dtype)
+    _call("ab2_side_gate", _p(g), g.stride(0), _p(ids), _p(table), table.shape[0], table.stride(0), col, _p(out), g.shape[0], D, _dt(g))
+    return out
+
+
 def expert_linear(x, w, routing: Routing):
     """Rows of ``x`` sorted by expert times ``w[e]^T``: the grouped tcgen05 GEMM for bf16 with aligned sizes, a plain
     grouped kernel in 32-bit and for odd sizes."""
@@ -364,9 +548,16 @@ def softcap_(logits, cap: float):
 for _n, _a in {
     "ab2_sandwich_norm": [_V, _V, _I, _V, _lib.c_ll, _V, _V, _V, _V, _I, _I, _I, _F, _I],
     "ab2_qk_norm_append": [_V, _lib.c_ll, _V, _V, _V, _V, _V, _V, _I, _I, _I, _I, _F, _I],
-    "ab2_chunk_attn_plain": [_V] * 5 + [_I] + [_V] * 4 + [_I] * 6 + [_F, _F, _V, _V, _I, _I],
-    "ab2_chunk_decode": [_V] * 4 + [_I] + [_V] * 4 + [_I] * 6 + [_F, _F, _V, _V, _I],
-    "ab2_chunk_prefill": [_V] * 4 + [_I, _V, _I, _I] + [_V] * 4 + [_I] * 6 + [_F, _F, _V, _V, _I],
+    "ab2_embed_rows": [_V, _V, _I, _V, _V, _I, _V, _V, _I, _I, _I],
+    "ab2_post_norm": [_V, _lib.c_ll, _V, _V, _I, _I, _V, _F, _F, _V, _V, _F, _V, _I, _I, _F, _I],
+    "ab2_gemm_heads": [_V] * 3 + [_I] * 6,
+    "ab2_chunk_attn_plain": [_V] * 5 + [_I] + [_V] * 4 + [_I] * 6 + [_F, _F, _V, _V, _I, _I, _I],
+    "ab2_chunk_decode": [_V] * 4 + [_I] + [_V] * 4 + [_I] * 6 + [_F, _F, _V, _V, _I, _I],
+    "ab2_chunk_prefill": [_V] * 4 + [_I, _V, _I, _I, _lib.c_ll, _lib.c_ll] + [_V] * 4 + [_I] * 6 + [_F, _F, _V, _V, _I, _I],
+    "ab2_latent_decode": [_V] * 5 + [_I] + [_V] * 3 + [_I] * 4 + [_F, _I],
+    "ab2_gelu_erf": [_V, _lib.c_ll, _V, _I, _I, _I],
+    "ab2_glu_clamped": [_V, _lib.c_ll, _V, _V, _V, _I, _I, _F, _F, _I],
+    "ab2_side_gate": [_V, _lib.c_ll, _V, _V, _I, _lib.c_ll, _I, _V, _I, _I, _I],
     "ab2_causal_conv": [_V, _lib.c_ll, _V, _V, _V, _I] + [_V] * 4 + [_I] * 3 + [_V, _V, _I, _I, _I],
     "ab2_rglru_decode": [_V, _V, _lib.c_ll] + [_V] * 8 + [_I] * 4,
     "ab2_rglru_prefill": [_V, _V, _lib.c_ll] + [_V] * 5 + [_I] * 3 + [_V] * 7 + [_I] * 3,

@@ -55,6 +55,7 @@ def parse_args():
     ap.add_argument("--workload", type=str, default="train", choices=["train", "mixer-serve"],
                     help="train: the headline job; mixer-serve: prefill and decode throughput of the mixer stack beside the closest existing "
                          "models, and its kernels against their rooflines (one GPU, prints its own JSON line)")
+    ap.add_argument("--design", type=str, default="kagolix", choices=["kagolix", "vogilix"], help="mixer-serve: the mixer stack to measure")
     ap.add_argument("--model", type=str, default="qwen3-8b")
     ap.add_argument("--preset", type=str, default="driver", choices=sorted(PRESETS))
     ap.add_argument("--length-scale", type=float, default=None, help="scales prompt / median / cap lengths of the preset")
@@ -182,14 +183,14 @@ def run_reference(args):
     return 0
 
 
-def run_mixer_serve():
+def run_mixer_serve(design):
     os.environ.setdefault("AB2_PDL", "1")
     os.environ.setdefault("AB2_DECODE_SPLITK", "1")
     from areal_b200.infra.bench_mixers import run
 
     clocks = ClockSampler()
     clocks.start()
-    result = run()
+    result = run(design=design)
     result["clocks"] = clocks.stop()
     print(json.dumps(result))
     return 0
@@ -200,7 +201,7 @@ def main():
     if args.impl == "reference":
         return run_reference(args)
     if args.workload == "mixer-serve":
-        return run_mixer_serve()
+        return run_mixer_serve(args.design)
     import faulthandler
 
     # decode-path switches of the kernel library, read once per process at first use: programmatic

@@ -285,8 +285,9 @@ def test_layer_outputs_match(target):
 
 
 # ----------------------------------------------------------------------------- mechanisms
-def ragged(lens, starts, device, page_size=16, seed=0):
-    """A RaggedBatch of entries with scattered pages; single-token entries come first."""
+def ragged(lens, starts, device, page_size=16, seed=0, windows=()):
+    """A RaggedBatch of entries with scattered pages; single-token entries come first. ``windows``: sliding windows of
+    latent layers, whose page lists the batch gets."""
     import numpy as np
 
     from areal_b200.engine.ragged_step import RaggedRunner
@@ -301,7 +302,7 @@ def ragged(lens, starts, device, page_size=16, seed=0):
         entries.append(Entry(Carried(slot=len(lens) - 1 - i, pages=pages, length=s), [0] * n, []))
     runner = RaggedRunner.__new__(RaggedRunner)
     runner.device = torch.device(device)
-    runner.cache = type("C", (), dict(page_size=page_size, has_kv=True))
+    runner.cache = type("C", (), dict(page_size=page_size, has_kv=True, windows=windows))
     b, _ = RaggedRunner._layout(runner, entries)
     assert np.all(np.diff([len(e.tokens) != 1 for e in entries]) >= 0)
     return b, entries, total * page_size
