@@ -259,7 +259,7 @@ def latent_kernel_table(cfg, prefill=(4, 2048), decode=(64, 960), dev="cuda") ->
 
                 def dec():
                     M._call("ab2_latent_decode", qc.data_ptr(), b.pos.data_ptr(), b.slots.data_ptr(), b.row_entry.data_ptr(), oc.data_ptr(), R,
-                            cache.data_ptr(), b.pages.data_ptr(), b.page_base.data_ptr(), b.pages.shape[1], 64, nq, C, scale, win)
+                            cache.data_ptr(), cache.shape[0], b.pages.data_ptr(), b.page_base.data_ptr(), b.pages.shape[1], 64, nq, C, scale, win)
                 add(f"latent_decode {win} decode", dec, (R * see * C + 2 * qc.numel()) * 2, 4.0 * R * see * nq * C, like="paged_decode decode")
             nk = max(1, nq // 4)
             kc, vc = torch.randn(rows_, nk, 128, **bf), torch.randn(rows_, nk, 128, **bf)

@@ -2,50 +2,47 @@
 // own key part has been applied to the queries, their value part is applied to the result). A row sees its own position and
 // the window - 1 before it, or all earlier ones (window = 0).
 //
-// A CTA takes one row and 16 or 32 of its heads; the CTAs of a cluster share the row's keys in consecutive stretches. Pieces
-// of 64 latents are staged by asynchronous copies, once for both products (mma.sync, 32-bit sums):
-//   S = Q C^T     every warp its heads and keys, over the whole latent; to shared memory in 32 bits
-//   softmax       every warp its heads: running maximum and sum in registers, the weights to shared memory
-//   O += P C      every warp its eighth of the latent's columns, for all heads
-// Partial results are merged through distributed shared memory.
+// A CTA takes one row and 16 or 32 of its heads; the CTAs of a cluster share the row's keys in consecutive stretches. One warp
+// brings pieces of 32 latents from the cache pages by TMA (128-byte swizzle, 64 columns a box); each is used twice. Of the
+// eight others every one owns an eighth of the latent's columns, in both products (mma.sync, 32-bit sums):
+//   S = Q C^T     every warp its columns' share of all scores; the shares meet in shared memory in 32 bits
+//   softmax       a few threads per head: sum of the shares, running maximum and sum, the weights to shared memory
+//   O += P C      every warp its columns
+// The shares of piece c + 1 and the output of piece c are computed together. O is rescaled only when a head's maximum has
+// grown by more than 2^8 since its reference was set. Partial results of a cluster are merged through distributed shared memory.
 #include <cooperative_groups.h>
 
 #include "mixer_common.cuh"
 
 namespace ab2 {
 
-constexpr int LD_KEYS = 64, LD_THREADS = 256;
+constexpr int LD_KEYS = 32, LD_WARPS = 8, LD_WORK = 32 * LD_WARPS, LD_THREADS = LD_WORK + 32;
 
 struct LatentArgs {
-  const __nv_bfloat16* cache;
   const int *pages, *page_base;
-  int max_pages, page_size, H, C;
+  int max_pages, page_shift, H, C;
   float scale;
   int window;
+  bool one_box;               // a piece is one box of the tensor map (32 rows, all chunks of 64 columns), else one per chunk (or two)
 };
 
 // DC: latent size rounded up to 128, 256 or 512 (missing columns are zero-filled); MT: 16-head tiles of a CTA
 template <int DC, int MT>
 struct LatentCfg {
-  static constexpr int ROW = DC * 2 + 16;                          // padded rows: matrix loads touch distinct banks
-  static constexpr int STAGE = LD_KEYS * ROW;
-  static constexpr int NS = DC == 128 ? 3 : 2;                     // stages
+  static constexpr int CHUNK = LD_KEYS * 128;                      // 64 columns of a piece
+  static constexpr int STAGE = DC / 64 * CHUNK;
+  static constexpr int NS = DC == 512 ? 5 : 4;                     // stages: two in use, the others on their way
   static constexpr int CTAS = DC == 512 ? 1 : 2;                   // per SM
   static constexpr int HEADS = 16 * MT;
-  static constexpr int SROW = LD_KEYS + 4, PROW = LD_KEYS * 2 + 16;
-  static constexpr int Q_OFF = NS * STAGE;
-  static constexpr int S_OFF = Q_OFF + HEADS * ROW;
-  static constexpr int P_OFF = S_OFF + HEADS * SROW * 4;
+  static constexpr int SROW = LD_KEYS + 8, PROW = LD_KEYS * 2 + 16;
+  static constexpr int S_OFF = NS * STAGE;                         // shares of the scores, [warp][head][key]
+  static constexpr int P_OFF = S_OFF + LD_WARPS * HEADS * SROW * 4;
   static constexpr int A_OFF = P_OFF + HEADS * PROW;               // rescaling factor per head
-  static constexpr int ROWS_OFF = A_OFF + HEADS * 4;               // cache row of every key, two pieces
-  static constexpr int SMEM = ROWS_OFF + 2 * LD_KEYS * 4;
+  static constexpr int BAR_OFF = A_OFF + HEADS * 4;
+  static constexpr int SMEM = BAR_OFF + 2 * NS * 8 + 1024;
   static_assert(NS * STAGE >= HEADS * DC * 4, "the merge buffer aliases the stage memory");
 };
 
-__device__ __forceinline__ void ld_copy16(uint32_t dst, const void* src, bool ok) {
-  const int n = ok ? 16 : 0;
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
-}
 __device__ __forceinline__ void ld_mat(uint32_t a, uint32_t (&r)[4]) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
 }
@@ -56,230 +53,309 @@ __device__ __forceinline__ void ld_mma(float (&c)[4], const uint32_t (&a)[4], ui
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
+__device__ __forceinline__ void ld_sync() { asm volatile("bar.sync 1, %0;" ::"n"(LD_WORK) : "memory"); }     // the working warps
 
 template <int DC, int MT>
 __global__ void __launch_bounds__(LD_THREADS, LatentCfg<DC, MT>::CTAS)
-latent_decode_kernel(const __nv_bfloat16* __restrict__ q, const int* __restrict__ pos, const int* __restrict__ slots,
-                     const int* __restrict__ row_entry, __nv_bfloat16* __restrict__ out, const LatentArgs p) {
+latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat16* __restrict__ q, const int* __restrict__ pos,
+                     const int* __restrict__ slots, const int* __restrict__ row_entry, __nv_bfloat16* __restrict__ out, const LatentArgs p, int* err) {
   namespace cg = cooperative_groups;
   using Cfg = LatentCfg<DC, MT>;
-  constexpr int KS = DC / 16, RW = Cfg::HEADS / 8;                  // k-steps of a score; softmax rows of a warp
-  constexpr int WC = DC / 8, NT = WC / 8;                           // columns of a warp in the second product, in tiles of 8
-  extern __shared__ __align__(128) unsigned char dsm[];
+  constexpr int NS = Cfg::NS, HEADS = Cfg::HEADS;
+  constexpr int WC = DC / LD_WARPS, KS = WC / 16, NT = WC / 8;      // columns of a warp; k-steps and tiles of 8 in them
+  constexpr int TPR = LD_WORK / HEADS, KPT = LD_KEYS / TPR;         // softmax: threads per head, keys per thread
+  extern __shared__ unsigned char dsm_raw[];
   __shared__ float s_ml[2][32];                                     // this CTA's (max, sum) per head
-  pdl_wait();
-  pdl_trigger();
-  const int b = blockIdx.x, h0 = blockIdx.y * Cfg::HEADS, spl = blockIdx.z, nspl = gridDim.z;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, tq = lane & 3;
-  const int mat = lane >> 3, r8 = lane & 7;
-  const int heads = min(Cfg::HEADS, p.H - h0);
-  const int i = pos[b], e = row_entry[b];
-  const int lo = p.window > 0 ? max(0, i - p.window + 1) : 0;
-  const int len = slots[b] >= 0 ? i + 1 - lo : 0;
-  const int per = ((len + nspl - 1) / nspl + LD_KEYS - 1) / LD_KEYS * LD_KEYS;
-  const int t0 = lo + spl * per, t1 = min(lo + len, t0 + per);
-  const int np = t1 > t0 ? (t1 - t0 + LD_KEYS - 1) / LD_KEYS : 0;
-  const int* pt = p.pages + (size_t)e * p.max_pages;
-  const int base = p.page_base[e];
-  const uint32_t sm = smem_u32(dsm);
-  float* s_s = reinterpret_cast<float*>(dsm + Cfg::S_OFF);
-  float* s_alpha = reinterpret_cast<float*>(dsm + Cfg::A_OFF);
-  int* s_row = reinterpret_cast<int*>(dsm + Cfg::ROWS_OFF);
-  auto plan = [&](int c) {
-    if (tid < LD_KEYS && c < np) {
-      const int t = t0 + c * LD_KEYS + tid;
-      s_row[(c & 1) * LD_KEYS + tid] = t < t1 ? pt[t / p.page_size - base] * p.page_size + t % p.page_size : -1;
+  __shared__ float s_wt[8][32];                                     // weights of the cluster's partial results
+  unsigned char* dsm = dsm_raw + ((1024u - (smem_u32(dsm_raw) & 1023u)) & 1023u);
+  const uint32_t sm = smem_u32(dsm), bar = sm + Cfg::BAR_OFF;
+  auto full = [&](int s) { return bar + 8u * s; };
+  auto empty = [&](int s) { return bar + 8u * (NS + s); };
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  if (tid == 0) {
+    prefetch_tmap(&tmC);
+    for (int s = 0; s < NS; ++s) {
+      mbar_init(full(s), 1);
+      mbar_init(empty(s), LD_WARPS);
     }
-  };
-  auto issue = [&](int c) {                                         // past the last piece: an empty group
-    if (c < np) {
-      const uint32_t st = sm + (c % Cfg::NS) * Cfg::STAGE;
-#pragma unroll 4
-      for (int k = 0; k < LD_KEYS * (DC / 8) / LD_THREADS; ++k) {
-        const int idx = tid + k * LD_THREADS, r = idx / (DC / 8), piece = idx % (DC / 8);
-        const int row = s_row[(c & 1) * LD_KEYS + r];
-        const bool ok = row >= 0 && piece * 8 < p.C;
-        ld_copy16(st + r * Cfg::ROW + piece * 16, p.cache + (ok ? (size_t)row * p.C + piece * 8 : 0), ok);
-      }
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-#pragma unroll
-  for (int c = 0; c < Cfg::NS - 1; ++c) {
-    plan(c);
-    __syncthreads();
-    issue(c);
-  }
-  plan(Cfg::NS - 1);
-  for (int k = tid; k < Cfg::HEADS * (DC / 8); k += LD_THREADS) {
-    const int r = k / (DC / 8), piece = k % (DC / 8);
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (r < heads && piece * 8 < p.C) v = *reinterpret_cast<const uint4*>(q + ((size_t)b * p.H + h0 + r) * p.C + piece * 8);
-    *reinterpret_cast<uint4*>(dsm + Cfg::Q_OFF + r * Cfg::ROW + piece * 16) = v;
-  }
-  const float sc = p.scale * 1.4426950408889634f;                   // scores in base-2 units
-  float o[MT][NT][4];
-#pragma unroll
-  for (int m = 0; m < MT; ++m)
-#pragma unroll
-    for (int j = 0; j < NT; ++j) o[m][j][0] = o[m][j][1] = o[m][j][2] = o[m][j][3] = 0.f;
-  float m_run[RW], l_run[RW];                                       // rows warp * RW ...; sums of this lane's keys only
-#pragma unroll
-  for (int r = 0; r < RW; ++r) { m_run[r] = -INFINITY; l_run[r] = 0.f; }
-
-  for (int c = 0; c < np; ++c) {
-    asm volatile("cp.async.wait_group %0;" ::"n"(Cfg::NS - 2) : "memory");
-    __syncthreads();                                                // piece c is here, and nobody reads piece c - 1 any more
-    issue(c + Cfg::NS - 1);
-    const uint32_t st = sm + (c % Cfg::NS) * Cfg::STAGE;
-    // ---- scores
-    if constexpr (MT == 2) {
-      const int mt = warp & 1, kg = warp >> 1;                      // 16 heads x 16 keys
-      const uint32_t qa = sm + Cfg::Q_OFF + (mt * 16 + (mat & 1) * 8 + r8) * Cfg::ROW + (mat >> 1) * 16;
-      const uint32_t ka = st + (kg * 16 + (mat >> 1) * 8 + r8) * Cfg::ROW + (mat & 1) * 16;
-      float s[2][2][4] = {};                                        // [k-step parity][key half]
-#pragma unroll 4
-      for (int ks = 0; ks < KS; ks += 2)
-#pragma unroll
-        for (int x = 0; x < 2; ++x) {
-          uint32_t a[4], k[4];
-          ld_mat(qa + (ks + x) * 32, a);
-          ld_mat(ka + (ks + x) * 32, k);
-          ld_mma(s[x][0], a, k[0], k[1]);
-          ld_mma(s[x][1], a, k[2], k[3]);
-        }
-#pragma unroll
-      for (int n = 0; n < 2; ++n) {
-        float* d = s_s + (mt * 16 + gq) * Cfg::SROW + kg * 16 + n * 8 + 2 * tq;
-        *reinterpret_cast<float2*>(d) = make_float2(s[0][n][0] + s[1][n][0], s[0][n][1] + s[1][n][1]);
-        *reinterpret_cast<float2*>(d + 8 * Cfg::SROW) = make_float2(s[0][n][2] + s[1][n][2], s[0][n][3] + s[1][n][3]);
-      }
-    } else {                                                        // 16 heads x 8 keys
-      const uint32_t qa = sm + Cfg::Q_OFF + ((mat & 1) * 8 + r8) * Cfg::ROW + (mat >> 1) * 16;
-      const uint32_t ka = st + (warp * 8 + r8) * Cfg::ROW + mat * 16;
-      float s[2][4] = {};
-#pragma unroll 4
-      for (int ks = 0; ks < KS; ks += 2) {
-        uint32_t k[4];
-        ld_mat(ka + ks * 32, k);
-#pragma unroll
-        for (int x = 0; x < 2; ++x) {
-          uint32_t a[4];
-          ld_mat(qa + (ks + x) * 32, a);
-          ld_mma(s[x], a, k[2 * x], k[2 * x + 1]);
-        }
-      }
-      float* d = s_s + gq * Cfg::SROW + warp * 8 + 2 * tq;
-      *reinterpret_cast<float2*>(d) = make_float2(s[0][0] + s[1][0], s[0][1] + s[1][1]);
-      *reinterpret_cast<float2*>(d + 8 * Cfg::SROW) = make_float2(s[0][2] + s[1][2], s[0][3] + s[1][3]);
-    }
-    __syncthreads();
-    // ---- softmax: lane has keys 2 lane and 2 lane + 1
-    plan(c + Cfg::NS);
-#pragma unroll
-    for (int r = 0; r < RW; ++r) {
-      const int row = warp * RW + r, t = t0 + c * LD_KEYS + 2 * lane;
-      const float2 v = *reinterpret_cast<const float2*>(s_s + row * Cfg::SROW + 2 * lane);
-      const float a = t < t1 ? v.x * sc : -INFINITY, z = t + 1 < t1 ? v.y * sc : -INFINITY;
-      const float mn = fmaxf(m_run[r], warp_max(fmaxf(a, z)));      // finite: every piece has a visible key
-      const float alpha = fast_exp2(m_run[r] - mn), pa = fast_exp2(a - mn), pz = fast_exp2(z - mn);
-      m_run[r] = mn;
-      l_run[r] = l_run[r] * alpha + pa + pz;
-      *reinterpret_cast<uint32_t*>(dsm + Cfg::P_OFF + row * Cfg::PROW + 4 * lane) = pack_bf16(pa, pz);
-      if (lane == 0) s_alpha[row] = alpha;
-    }
-    __syncthreads();
-    // ---- weighted sum of the latents
-#pragma unroll
-    for (int m = 0; m < MT; ++m) {
-      const float a0 = s_alpha[m * 16 + gq], a1 = s_alpha[m * 16 + gq + 8];
-#pragma unroll
-      for (int j = 0; j < NT; ++j) {
-        o[m][j][0] *= a0; o[m][j][1] *= a0;
-        o[m][j][2] *= a1; o[m][j][3] *= a1;
-      }
-    }
-    const uint32_t pa0 = sm + Cfg::P_OFF + ((mat & 1) * 8 + r8) * Cfg::PROW + (mat >> 1) * 16;
-    const uint32_t va0 = st + ((mat & 1) * 8 + r8) * Cfg::ROW + (warp * WC + (mat >> 1) * 8) * 2;
-#pragma unroll
-    for (int ks = 0; ks < LD_KEYS / 16; ++ks) {
-      uint32_t pf[MT][4];
-#pragma unroll
-      for (int m = 0; m < MT; ++m) ld_mat(pa0 + m * 16 * Cfg::PROW + ks * 32, pf[m]);
-#pragma unroll
-      for (int j = 0; j < NT; j += 2) {
-        uint32_t v[4];
-        ld_mat_t(va0 + ks * 16 * Cfg::ROW + j * 16, v);
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          ld_mma(o[m][j], pf[m], v[0], v[1]);
-          ld_mma(o[m][j + 1], pf[m], v[2], v[3]);
-        }
-      }
-    }
-  }
-  // ---- this CTA's sums
-#pragma unroll
-  for (int r = 0; r < RW; ++r) {
-    const float l = warp_sum(l_run[r]);
-    if (lane == 0) { s_ml[0][warp * RW + r] = m_run[r]; s_ml[1][warp * RW + r] = l; }
+    fence_mbar_init();
   }
   __syncthreads();
-  if (nspl == 1) {
+  pdl_wait();
+  pdl_trigger();
+  const int b = blockIdx.x, h0 = blockIdx.y * HEADS, spl = blockIdx.z, nspl = gridDim.z;
+  const int heads = min(HEADS, p.H - h0);
+  const int i = pos[b];
+  const int lo = p.window > 0 ? max(0, i - p.window + 1) : 0;
+  const int nblk = slots[b] >= 0 ? i / LD_KEYS - lo / LD_KEYS + 1 : 0;      // pieces start at multiples of 32: each lies in one page, or
+  const int per = (nblk + nspl - 1) / nspl;                                 // fills two of 16
+  const int t0 = (lo / LD_KEYS + spl * per) * LD_KEYS;
+  const int np = max(0, min(per, nblk - spl * per));
+  float* s_s = reinterpret_cast<float*>(dsm + Cfg::S_OFF);
+  float* s_alpha = reinterpret_cast<float*>(dsm + Cfg::A_OFF);
+
+  if (warp == LD_WARPS) {
+    if (elect_one() && np > 0) {
+      const int e = row_entry[b];
+      const int* pt = p.pages + (size_t)e * p.max_pages;
+      const int base = p.page_base[e], last = p.max_pages - 1, sh = p.page_shift, two = sh == 4 ? 1 : 0;
+      auto row_at = [&](int t) {                                    // boxes outside the held pages are masked
+        return (pt[min(max((t >> sh) - base, 0), last)] << sh) + (t & ((1 << sh) - 1));
+      };
+      int row0 = row_at(t0), row1 = two ? row_at(t0 + 16) : 0;
+      bool ok = true;
+      for (int c = 0; c < np; ++c) {
+        const int s = c % NS;
+        ok = mbar_wait(empty(s), ((uint32_t)(c / NS) & 1u) ^ 1u, err, ERR_WAIT_EMPTY);
+        if (!ok) break;
+        const uint32_t dst = sm + s * Cfg::STAGE;
+        mbar_expect_tx(full(s), Cfg::STAGE);
+        if (p.one_box) {
+          tma_load_3d(dst, &tmC, full(s), 0, row0, 0);
+        } else {
+#pragma unroll 1
+          for (int k = 0; k < DC / 64; ++k) {
+            tma_load_3d(dst + k * Cfg::CHUNK, &tmC, full(s), k * 64, row0, 0);
+            if (two) tma_load_3d(dst + k * Cfg::CHUNK + 16 * 128, &tmC, full(s), k * 64, row1, 0);
+          }
+        }
+        if (c + 1 < np) {
+          row0 = row_at(t0 + (c + 1) * LD_KEYS);
+          if (two) row1 = row_at(t0 + (c + 1) * LD_KEYS + 16);
+        }
+      }
+      if (!ok) {                                                    // copies in flight get a bounded time to land
+        const long long c0 = clock64();
+        while (clock64() - c0 < 8000000LL) {}
+      }
+    }
+    __syncwarp();
+  } else {
+    const int gq = lane >> 2, tq = lane & 3, mat = lane >> 3, r8 = lane & 7;
+    uint32_t qa[MT][KS][4];
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int hh = 0; hh < 2; ++hh) {
-        const int row = m * 16 + gq + 8 * hh;
-        if (row >= heads) continue;
-        const float l = s_ml[1][row], inv = l > 0.f ? 1.f / l : 0.f;
-        __nv_bfloat16* dst = out + ((size_t)b * p.H + h0 + row) * p.C;
+      for (int ks = 0; ks < KS; ++ks)
 #pragma unroll
-        for (int j = 0; j < NT; ++j) {
-          const int col = warp * WC + j * 8 + 2 * tq;
-          if (col < p.C) *reinterpret_cast<uint32_t*>(dst + col) = pack_bf16(o[m][j][2 * hh] * inv, o[m][j][2 * hh + 1] * inv);
+        for (int x = 0; x < 4; ++x) {
+          const int row = m * 16 + gq + (x & 1) * 8, col = warp * WC + ks * 16 + (x >> 1) * 8 + 2 * tq;
+          qa[m][ks][x] = row < heads && col < p.C ? *reinterpret_cast<const uint32_t*>(q + ((size_t)b * p.H + h0 + row) * p.C + col) : 0u;
+        }
+    const float sc = p.scale * 1.4426950408889634f;                 // scores in base-2 units
+    float o[MT][NT][4];
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int j = 0; j < NT; ++j) o[m][j][0] = o[m][j][1] = o[m][j][2] = o[m][j][3] = 0.f;
+    const int srow = tid / TPR, skey = tid % TPR * KPT;
+    float m_run = -INFINITY, l_run = 0.f;                           // of head srow; the sum over this thread's keys only
+    bool ok = true;                                                 // after a wait that gave up: no more waits, same barriers
+    // this warp's columns inside a stage: chunk and first 16-byte piece of its rows (pieces are swizzled by the row)
+    const uint32_t mine = (warp * WC / 64) * Cfg::CHUNK;
+    constexpr int PIECES = WC / 8;
+    const int c0 = warp * PIECES % 8;
+
+    auto scores = [&](int c) {
+      const uint32_t st = sm + (c % NS) * Cfg::STAGE + mine + ((mat >> 1) * 8 + r8) * 128;
+      float s[MT][LD_KEYS / 8][4] = {};
+#pragma unroll
+      for (int ks = 0; ks < KS; ++ks) {
+        const uint32_t a = st + (((c0 + ks * 2 + (mat & 1)) ^ r8) << 4);
+#pragma unroll
+        for (int n = 0; n < LD_KEYS / 8; n += 2) {
+          uint32_t k[4];
+          ld_mat(a + n * 8 * 128, k);
+#pragma unroll
+          for (int m = 0; m < MT; ++m) {
+            ld_mma(s[m][n], qa[m][ks], k[0], k[1]);
+            ld_mma(s[m][n + 1], qa[m][ks], k[2], k[3]);
+          }
         }
       }
-    return;
-  }
-  // ---- the CTAs of the cluster
-  float* mo = reinterpret_cast<float*>(dsm);                        // [HEADS][DC]
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
+      for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int j = 0; j < NT; ++j) {
-      float* d = mo + (m * 16 + gq) * DC + warp * WC + j * 8 + 2 * tq;
-      *reinterpret_cast<float2*>(d) = make_float2(o[m][j][0], o[m][j][1]);
-      *reinterpret_cast<float2*>(d + 8 * DC) = make_float2(o[m][j][2], o[m][j][3]);
+        for (int n = 0; n < LD_KEYS / 8; ++n) {
+          float* d = s_s + (warp * HEADS + m * 16 + gq) * Cfg::SROW + n * 8 + 2 * tq;
+          *reinterpret_cast<float2*>(d) = make_float2(s[m][n][0], s[m][n][1]);
+          *reinterpret_cast<float2*>(d + 8 * Cfg::SROW) = make_float2(s[m][n][2], s[m][n][3]);
+        }
+    };
+    auto softmax = [&](int c) {
+      float v[KPT] = {};
+#pragma unroll
+      for (int w = 0; w < LD_WARPS; ++w) {
+        const float* d = s_s + (w * HEADS + srow) * Cfg::SROW + skey;
+        if constexpr (KPT == 4) {
+          const float4 x = *reinterpret_cast<const float4*>(d);
+          v[0] += x.x; v[1] += x.y; v[2] += x.z; v[3] += x.w;
+        } else {
+          const float2 x = *reinterpret_cast<const float2*>(d);
+          v[0] += x.x; v[1] += x.y;
+        }
+      }
+      const int t = t0 + c * LD_KEYS + skey;
+      float mx = -INFINITY;
+#pragma unroll
+      for (int k = 0; k < KPT; ++k) {
+        v[k] = t + k >= lo && t + k <= i ? v[k] * sc : -INFINITY;
+        mx = fmaxf(mx, v[k]);
+      }
+#pragma unroll
+      for (int x = TPR / 2; x > 0; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));    // finite: every piece has a visible key
+      float alpha = 1.f;
+      if (mx > m_run + 8.f || m_run == -INFINITY) {
+        alpha = fast_exp2(m_run - mx);
+        m_run = mx;
+      }
+      float sum = 0.f;
+#pragma unroll
+      for (int k = 0; k < KPT; ++k) {
+        v[k] = fast_exp2(v[k] - m_run);
+        sum += v[k];
+      }
+      l_run = l_run * alpha + sum;
+      uint32_t* d = reinterpret_cast<uint32_t*>(dsm + Cfg::P_OFF + srow * Cfg::PROW + skey * 2);
+#pragma unroll
+      for (int k = 0; k < KPT / 2; ++k) d[k] = pack_bf16(v[2 * k], v[2 * k + 1]);
+      if (skey == 0) s_alpha[srow] = alpha;
+    };
+    auto arrived = [&](int c) { ok = ok && mbar_wait(full(c % NS), (uint32_t)(c / NS) & 1u, err, ERR_WAIT_FULL); };
+    const uint32_t pa = sm + Cfg::P_OFF + ((mat & 1) * 8 + r8) * Cfg::PROW + (mat >> 1) * 16;
+    if (np > 0) {
+      arrived(0);
+      __syncwarp();
+      scores(0);
+      ld_sync();
+      softmax(0);
     }
+    for (int c = 0; c < np; ++c) {
+      ld_sync();                                                    // weights of piece c are there, shares of the scores free
+      if (c + 1 < np) {
+        arrived(c + 1);
+        __syncwarp();
+        scores(c + 1);
+      }
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        const float a0 = s_alpha[m * 16 + gq], a1 = s_alpha[m * 16 + gq + 8];
+        if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
+#pragma unroll
+          for (int j = 0; j < NT; ++j) {
+            o[m][j][0] *= a0; o[m][j][1] *= a0;
+            o[m][j][2] *= a1; o[m][j][3] *= a1;
+          }
+        }
+      }
+      const uint32_t st = sm + (c % NS) * Cfg::STAGE + mine + ((mat & 1) * 8 + r8) * 128;
+#pragma unroll
+      for (int ks = 0; ks < LD_KEYS / 16; ++ks) {
+        uint32_t pf[MT][4];
+#pragma unroll
+        for (int m = 0; m < MT; ++m) ld_mat(pa + m * 16 * Cfg::PROW + ks * 32, pf[m]);
+#pragma unroll
+        for (int j = 0; j < NT; j += 2) {
+          uint32_t v[4];
+          ld_mat_t(st + ks * 16 * 128 + (((c0 + j + (mat >> 1)) ^ r8) << 4), v);
+#pragma unroll
+          for (int m = 0; m < MT; ++m) {
+            ld_mma(o[m][j], pf[m], v[0], v[1]);
+            ld_mma(o[m][j + 1], pf[m], v[2], v[3]);
+          }
+        }
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(empty(c % NS));
+      ld_sync();                                                    // shares of piece c + 1 are there, weights of piece c free
+      if (c + 1 < np) softmax(c + 1);
+    }
+    // ---- this CTA's sums
+#pragma unroll
+    for (int x = TPR / 2; x > 0; x >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, x);
+    if (skey == 0) { s_ml[0][srow] = m_run; s_ml[1][srow] = l_run; }
+    ld_sync();
+    if (nspl == 1) {
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int hh = 0; hh < 2; ++hh) {
+          const int row = m * 16 + gq + 8 * hh;
+          if (row >= heads) continue;
+          const float l = s_ml[1][row], inv = l > 0.f ? 1.f / l : 0.f;
+          __nv_bfloat16* dst = out + ((size_t)b * p.H + h0 + row) * p.C;
+#pragma unroll
+          for (int j = 0; j < NT; ++j) {
+            const int col = warp * WC + j * 8 + 2 * tq;
+            if (col < p.C) *reinterpret_cast<uint32_t*>(dst + col) = pack_bf16(o[m][j][2 * hh] * inv, o[m][j][2 * hh + 1] * inv);
+          }
+        }
+    } else {
+      float* mo = reinterpret_cast<float*>(dsm);                    // [HEADS][DC], over the stages: every piece has been used
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+          float* d = mo + (m * 16 + gq) * DC + warp * WC + j * 8 + 2 * tq;
+          *reinterpret_cast<float2*>(d) = make_float2(o[m][j][0], o[m][j][1]);
+          *reinterpret_cast<float2*>(d + 8 * DC) = make_float2(o[m][j][2], o[m][j][3]);
+        }
+    }
+  }
+  if (nspl == 1) return;
+  // ---- the CTAs of the cluster
   cg::cluster_group cl = cg::this_cluster();
   cl.sync();
-  for (int k = spl * LD_THREADS + tid; k < heads * (DC / 2); k += LD_THREADS * nspl) {
-    const int g = k / (DC / 2), col = (k - g * (DC / 2)) * 2;
-    if (col >= p.C) continue;
-    float mx = -INFINITY, ll = 0.f, ox = 0.f, oy = 0.f;
-    for (int c = 0; c < nspl; ++c) mx = fmaxf(mx, cl.map_shared_rank(&s_ml[0][0], c)[g]);
-    for (int c = 0; c < nspl; ++c) {
-      const float* ml = cl.map_shared_rank(&s_ml[0][0], c);
-      const float wt = ml[g] == -INFINITY ? 0.f : fast_exp2(ml[g] - mx);
-      const float2 v = *reinterpret_cast<const float2*>(cl.map_shared_rank(mo, c) + g * DC + col);
-      ll += ml[32 + g] * wt;
-      ox += v.x * wt;
-      oy += v.y * wt;
+  if (tid < heads) {
+    float m[8], l[8], mx = -INFINITY, ll = 0.f;
+#pragma unroll
+    for (int c = 0; c < 8; ++c) {
+      const float* ml = cl.map_shared_rank(&s_ml[0][0], min(c, nspl - 1));
+      m[c] = c < nspl ? ml[tid] : -INFINITY;
+      l[c] = ml[32 + tid];
+      mx = fmaxf(mx, m[c]);
     }
-    const float inv = ll > 0.f ? 1.f / ll : 0.f;
-    *reinterpret_cast<uint32_t*>(out + ((size_t)b * p.H + h0 + g) * p.C + col) = pack_bf16(ox * inv, oy * inv);
+#pragma unroll
+    for (int c = 0; c < 8; ++c) {
+      m[c] = m[c] == -INFINITY ? 0.f : fast_exp2(m[c] - mx);
+      ll += l[c] * m[c];
+    }
+#pragma unroll
+    for (int c = 0; c < 8; ++c) s_wt[c][tid] = ll > 0.f ? m[c] / ll : 0.f;
+  }
+  __syncthreads();
+  const float* mo = reinterpret_cast<const float*>(dsm);
+  for (int k = spl * LD_THREADS + tid; k < heads * (DC / 4); k += LD_THREADS * nspl) {
+    const int g = k / (DC / 4), col = (k - g * (DC / 4)) * 4;
+    if (col >= p.C) continue;
+    float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int c = 0; c < nspl; ++c) {
+      const float w = s_wt[c][g];
+      const float4 v = *reinterpret_cast<const float4*>(cl.map_shared_rank(mo, c) + g * DC + col);
+      s.x += v.x * w; s.y += v.y * w; s.z += v.z * w; s.w += v.w * w;
+    }
+    *reinterpret_cast<uint2*>(out + ((size_t)b * p.H + h0 + g) * p.C + col) = make_uint2(pack_bf16(s.x, s.y), pack_bf16(s.z, s.w));
   }
   cl.sync();                                                        // nobody leaves while its shared memory is being read
 }
 
 template <int DC, int MT>
-static int launch_latent(const void* q, const int* pos, const int* slots, const int* row_entry, void* out, int R, const LatentArgs& a, cudaStream_t s) {
+static int launch_latent(const void* q, const int* pos, const int* slots, const int* row_entry, void* out, int R, const void* cache, int cache_rows,
+                         LatentArgs a, cudaStream_t s) {
   using Cfg = LatentCfg<DC, MT>;
   auto kern = latent_decode_kernel<DC, MT>;
   static ab2host::DevState st;
   int sms = 0;
   if (ab2host::prepare_launch(kern, Cfg::SMEM, st, &sms)) return 300;
+  CUtensorMap tc;
+  a.one_box = a.C % 64 == 0 && a.page_shift > 4;
+  if (a.one_box) {             // (column of the chunk, row, chunk)
+    if (ab2host::encode_tmap_3d(&tc, cache, 2, 64, cache_rows, a.C / 64, (uint64_t)a.C * 2, 128, 64, LD_KEYS, DC / 64, true, 0)) return 100;
+  } else if (ab2host::encode_tmap_3d(&tc, cache, 2, a.C, cache_rows, 1, (uint64_t)a.C * 2, (uint64_t)a.C * 2, 64, a.page_shift > 4 ? LD_KEYS : 16, 1, true, 0)) {
+    return 101;
+  }
+  int* err = ab2host::error_flag();
+  if (!err) return 301;
   const int tiles = (a.H + Cfg::HEADS - 1) / Cfg::HEADS;
   // as many CTAs per row as fit on the GPU at once, and no more than the window has pieces
   const int pieces = a.window > 0 ? (a.window + LD_KEYS - 1) / LD_KEYS : 1 << 20;
@@ -299,7 +375,7 @@ static int launch_latent(const void* q, const int* pos, const int* slots, const 
   attr[1].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr;
   cfg.numAttrs = ab2host::pdl_enabled() ? 2 : 1;
-  return cudaLaunchKernelEx(&cfg, kern, (const __nv_bfloat16*)q, pos, slots, row_entry, (__nv_bfloat16*)out, a) == cudaSuccess ? 0 : 302;
+  return cudaLaunchKernelEx(&cfg, kern, tc, (const __nv_bfloat16*)q, pos, slots, row_entry, (__nv_bfloat16*)out, a, err) == cudaSuccess ? 0 : 302;
 }
 
 }  // namespace ab2
@@ -308,21 +384,23 @@ extern "C" {
 using namespace ab2;
 
 // q, out [R, H, C] bf16; row r reads the pages of entry row_entry[r] up to position pos[r]; slots[r] < 0: padding row (zeros).
-// cache [rows, C] bf16; pages [entries, max_pages] from page number page_base[entry] on. C a multiple of 8 up to 512.
-int ab2_latent_decode(const void* q, const int* pos, const int* slots, const int* row_entry, void* out, int R, const void* cache, const int* pages,
-                      const int* page_base, int max_pages, int page_size, int H, int C, float scale, int window, void* stream) {
+// cache [cache_rows, C] bf16; pages [entries, max_pages] from page number page_base[entry] on. C a multiple of 8 up to 512,
+// page_size a power of two from 16 on.
+int ab2_latent_decode(const void* q, const int* pos, const int* slots, const int* row_entry, void* out, int R, const void* cache, int cache_rows,
+                      const int* pages, const int* page_base, int max_pages, int page_size, int H, int C, float scale, int window, void* stream) {
   if (R <= 0) return 0;
-  if ((C & 7) || C < 8 || C > 512 || H < 1 || H > 32 * 65535 || page_size < 1) return 10;
+  if ((C & 7) || C < 8 || C > 512 || H < 1 || H > 16 * 65535 || page_size < 16 || (page_size & (page_size - 1))) return 10;
   if (!aligned_to(q, 16) || !aligned_to(cache, 16) || !aligned_to(out, 16)) return 11;
-  LatentArgs a{(const __nv_bfloat16*)cache, pages, page_base, max_pages, page_size, H, C, scale, window};
-  cudaStream_t s = (cudaStream_t)stream;
+  LatentArgs a{pages, page_base, max_pages, __builtin_ctz(page_size), H, C, scale, window, false};
+#define AB2_LATENT(DC, MT) return launch_latent<DC, MT>(q, pos, slots, row_entry, out, R, cache, cache_rows, a, (cudaStream_t)stream)
   if (H <= 16) {
-    if (C <= 128) return launch_latent<128, 1>(q, pos, slots, row_entry, out, R, a, s);
-    if (C <= 256) return launch_latent<256, 1>(q, pos, slots, row_entry, out, R, a, s);
-    return launch_latent<512, 1>(q, pos, slots, row_entry, out, R, a, s);
+    if (C <= 128) AB2_LATENT(128, 1);
+    if (C <= 256) AB2_LATENT(256, 1);
+    AB2_LATENT(512, 1);
   }
-  if (C <= 128) return launch_latent<128, 2>(q, pos, slots, row_entry, out, R, a, s);
-  if (C <= 256) return launch_latent<256, 2>(q, pos, slots, row_entry, out, R, a, s);
-  return launch_latent<512, 2>(q, pos, slots, row_entry, out, R, a, s);
+  if (C <= 128) AB2_LATENT(128, 2);
+  if (C <= 256) AB2_LATENT(256, 2);
+  AB2_LATENT(512, 2);
+#undef AB2_LATENT
 }
 }

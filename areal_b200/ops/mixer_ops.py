@@ -329,8 +329,9 @@ def latent_attention(q, cache, w_kv, Dv: int, b: RaggedBatch, scale: float, wind
     w_k, w_v = w_kv[:H * D].view(H, D, C), w_kv[H * D:].view(H, Dv, C)
     out = torch.empty(R, H, Dv, device=q.device, dtype=q.dtype)
     nd, bf16 = b.n_dec, q.dtype == torch.bfloat16
-    fast_rows = bf16 and C % 8 == 0 and C <= 512
-    fast_tiles = bf16 and D % 8 == 0 and Dv % 8 == 0 and D <= 128 and Dv <= 128 and C % 8 == 0 and b.page_size in (16, 32, 64, 128)
+    paged = bf16 and C % 8 == 0 and b.page_size in (16, 32, 64, 128)
+    fast_rows = paged and C <= 512
+    fast_tiles = paged and D % 8 == 0 and Dv % 8 == 0 and D <= 128 and Dv <= 128
     whole = R > nd and fast_tiles and R - nd > SHORT_PORTION * (b.n_entries - nd)
     n = nd if whole else R
     if n:
@@ -339,7 +340,7 @@ def latent_attention(q, cache, w_kv, Dv: int, b: RaggedBatch, scale: float, wind
         oc = torch.empty_like(qc)
         args = (_p(qc), _p(b.pos), _p(b.slots), _p(b.row_entry), _p(oc), n)
         if fast_rows:
-            _call("ab2_latent_decode", *args, _p(cache), _p(b.pages), _p(b.page_base), b.pages.shape[1], b.page_size, H, C, scale, window)
+            _call("ab2_latent_decode", *args, _p(cache), cache.shape[0], _p(b.pages), _p(b.page_base), b.pages.shape[1], b.page_size, H, C, scale, window)
         else:
             _call("ab2_chunk_attn_plain", *args, _p(cache), _p(cache), _p(b.pages), _p(b.page_base), b.pages.shape[1], b.page_size, H, 1, C, C, scale, 0.0,
                   None, None, 0, window, _dt(q))
@@ -554,7 +555,7 @@ for _n, _a in {
     "ab2_chunk_attn_plain": [_V] * 5 + [_I] + [_V] * 4 + [_I] * 6 + [_F, _F, _V, _V, _I, _I, _I],
     "ab2_chunk_decode": [_V] * 4 + [_I] + [_V] * 4 + [_I] * 6 + [_F, _F, _V, _V, _I, _I],
     "ab2_chunk_prefill": [_V] * 4 + [_I, _V, _I, _I, _lib.c_ll, _lib.c_ll] + [_V] * 4 + [_I] * 6 + [_F, _F, _V, _V, _I, _I],
-    "ab2_latent_decode": [_V] * 5 + [_I] + [_V] * 3 + [_I] * 4 + [_F, _I],
+    "ab2_latent_decode": [_V] * 5 + [_I, _V, _I, _V, _V] + [_I] * 4 + [_F, _I],
     "ab2_gelu_erf": [_V, _lib.c_ll, _V, _I, _I, _I],
     "ab2_glu_clamped": [_V, _lib.c_ll, _V, _V, _V, _I, _I, _F, _F, _I],
     "ab2_side_gate": [_V, _lib.c_ll, _V, _V, _I, _lib.c_ll, _I, _V, _I, _I, _I],

@@ -43,13 +43,13 @@ def config(*layers, vocab=104, width=64, mult=0.7, side=24, positions=1024, eps=
 CONFIGS = {
     "mixed": config((mixer(), dense()), (mixer(size=24, vdim=48), moe()), (mixer(heads=3, size=72, kv_rank=64), None), (mixer(size=33), moe(top=3, shared=0))),
     # sizes that no vector width divides
-    "odd": config((mixer(heads=3, dim=20, vdim=12, q_rank=18, kv_rank=30, size=33), moe(experts=5, top=3, ff=20, shared=27)),
-                  (mixer(heads=5, dim=7, vdim=10, q_rank=9, kv_rank=21, size=17), dense(33)), vocab=101, width=60, side=6, mult=1.0, eps=1e-3),
+    "odd": config((mixer(heads=3, dim=20, vdim=12, q_rank=18, kv_rank=30, size=33, peak=1.5), moe(experts=5, top=3, ff=20, shared=27)),
+                  (mixer(heads=5, dim=7, vdim=10, q_rank=9, kv_rank=21, size=17, peak=1.5), dense(33)), vocab=101, width=60, side=6, mult=0.5, eps=1e-2),
     # more than one tile of heads, windows longer than a query tile, every expert chosen
     "wide": config((mixer(heads=20, dim=64, vdim=96, q_rank=72, kv_rank=136, size=320, peak=2.0), dense(96)),
                    (mixer(heads=17, dim=16, vdim=8, q_rank=24, kv_rank=32, size=130), moe(experts=3, top=3)), width=128, vocab=96, mult=0.25),
-    "rank512": config((mixer(heads=2, dim=128, vdim=128, q_rank=160, kv_rank=512, size=200, peak=2.0), moe(experts=9, top=1, limit=0.5)),
-                      (mixer(heads=33, dim=8, vdim=16, q_rank=8, kv_rank=264, size=96, peak=2.0), None), mult=1.5),
+    "rank512": config((mixer(heads=2, dim=128, vdim=128, q_rank=160, kv_rank=512, size=200, peak=1.25), moe(experts=9, top=1, limit=0.5)),
+                      (mixer(heads=33, dim=8, vdim=16, q_rank=8, kv_rank=264, size=96, peak=1.25), None), mult=1.25),
     # a token that sees itself only, windows of a page, no window, no token input
     "edges": config((mixer(heads=2, size=1), dense()), (mixer(size=64), None), (mixer(heads=1, size=65, vdim=112), None), (mixer(size=0, peak=2.0), None), side=0),
 }
@@ -93,18 +93,28 @@ def make_weights(cfg, seed=0):
     return W
 
 
+CLEAR = 0.3              # router logits by which the last chosen expert is ahead of the first one left out
 _ORACLE: dict = {}
 
 
 def oracle(name, n, seed):
-    """Tokens, logits and rows with a clear choice of experts of a random prompt under a named configuration (cached:
-    shared by the targets and the schedules)."""
+    """Tokens, logits and residual streams of a prompt under a named configuration (cached: shared by the targets and the
+    schedules). Tokens whose choice of experts is close are drawn again, until none is: bf16 rounding may turn a close choice,
+    which is another result for this token and for those that look back at it."""
     if (name, n, seed) not in _ORACLE:
-        cfg = CONFIGS[name]
-        t = tokens(n, cfg["vocab"], seed)
-        margins = [torch.ones(n)]
-        logits = plain.forward(make_weights(cfg), cfg, t, margins)[0]
-        _ORACLE[name, n, seed] = (t, logits, torch.stack([m.double() for m in margins]).amin(0) > 0.05)
+        cfg, rnd = CONFIGS[name], random.Random(seed)
+        W, t = make_weights(cfg), tokens(n, cfg["vocab"], seed)
+        for _ in range(40):
+            margins = [torch.full((n,), CLEAR)]
+            logits, states = plain.forward(W, cfg, t, margins)
+            close = torch.where(torch.stack([m.double() for m in margins]).amin(0) < CLEAR - 1e-6)[0].tolist()
+            if not close:
+                break
+            for i in close:
+                t[i] = rnd.randrange(cfg["vocab"])
+        else:
+            raise AssertionError(f"{name}: no prompt of {n} tokens with clear choices")
+        _ORACLE[name, n, seed] = (t, logits, states)
     return _ORACLE[name, n, seed]
 
 
@@ -115,7 +125,7 @@ def test_whole_prompt_portions_and_single_tokens_agree(name, target):
     cfg = CONFIGS[name]
     eng = make_engine(cfg, make_weights(cfg), target)
     n = 150
-    t, want, sure = oracle(name, n, 1)
+    t, want, _ = oracle(name, n, 1)
     cuts = {"whole": [n], "decoded": [90] + [1] * 60, "pairs": [2] * 35 + [80], "ragged": [1, 2, 61, 3, 64, 2, 1, 16]}
     for what, sizes in cuts.items():
         d, at = Driver(eng), 0
@@ -123,7 +133,7 @@ def test_whole_prompt_portions_and_single_tokens_agree(name, target):
         for s in sizes:
             d.step([("a", t[at:at + s])], end=["a"] if at + s == n else [])
             at += s
-        assert_close(d.logits("a"), want, target[1], f"{name} {what}", sure)
+        assert_close(d.logits("a"), want, target[1], f"{name} {what}")
     assert len(eng.cache.free) == eng.cache.num_pages and len(eng.cache.free_slots) == eng.cache.num_slots
 
 
@@ -131,11 +141,11 @@ def test_whole_prompt_portions_and_single_tokens_agree(name, target):
 def test_long_prompt_and_long_decoding_cross_many_windows(target):
     name, n = "wide", 700
     cfg = CONFIGS[name]
-    t, want, sure = oracle(name, n, 2)
+    t, want, _ = oracle(name, n, 2)
     eng = make_engine(cfg, make_weights(cfg), target)
     d = Driver(eng)
     d.step([("a", t)], end=["a"])
-    assert_close(d.logits("a"), want, target[1], "whole", sure)
+    assert_close(d.logits("a"), want, target[1], "whole")
     d = Driver(eng)
     d.step([("a", t[:330])])
     for i in range(330, 450):                      # the window's far end walks over the page borders at 64 and 128
@@ -144,7 +154,7 @@ def test_long_prompt_and_long_decoding_cross_many_windows(target):
     d.step([("a", t[450:637])])
     for i in range(637, n):
         d.step([("a", t[i:i + 1])], end=["a"] if i == n - 1 else [])
-    assert_close(d.logits("a"), want, target[1], "decoded", sure)
+    assert_close(d.logits("a"), want, target[1], "decoded")
 
 
 @pytest.mark.parametrize("target", TARGETS)
@@ -175,7 +185,7 @@ def test_mixed_batches_on_reused_pages_and_slots(target, page_size):
         d.step(portions, end=done)
         live = [r for r in live if r not in done]
     for rid in lens:
-        assert_close(d.logits(rid), ref[rid][1], target[1], rid, ref[rid][2])
+        assert_close(d.logits(rid), ref[rid][1], target[1], rid)
     assert len(eng.cache.free) == eng.cache.num_pages
 
 
@@ -183,10 +193,8 @@ def test_mixed_batches_on_reused_pages_and_slots(target, page_size):
 @pytest.mark.parametrize("name", ["mixed", "odd"])
 def test_layer_outputs_match(name, target):
     cfg = CONFIGS[name]
-    W = make_weights(cfg)
-    t = tokens(70, cfg["vocab"], 5)
-    _, states = plain.forward(W, cfg, t)
-    eng = make_engine(cfg, W, target)
+    t, _, states = oracle(name, 70, 5)
+    eng = make_engine(cfg, make_weights(cfg), target)
     c, seen = eng.cache.open(), []
     eng.cache.grow(c, 70)
     eng.runner.step([Entry(c, t, [69])], on_layer=lambda i, r: seen.append(r.double().cpu().clone()))
@@ -219,7 +227,7 @@ def test_a_wrong_reading_shows_in_the_logits(fault, monkeypatch):
     cfg = CONFIGS["mixed"]
     got = plain.forward(make_weights(cfg), cfg, t)[0]
     err = (got - want).pow(2).mean(-1).sqrt() / want.pow(2).mean().sqrt()
-    assert err.median() > 0.1, float(err.median())
+    assert err.median() > 0.03 and err.max() > 0.18, (float(err.median()), float(err.max()))
 
 
 # ----------------------------------------------------------------------------- mechanisms
@@ -513,7 +521,7 @@ def test_trace_runner_replays_steps(tmp_path, target):
     save_file({n: t.bfloat16().contiguous() for n, t in make_weights(cfg).items()}, str(model / "model.safetensors"))
     eng = trace_engine(str(model), "float32" if target[1] == torch.float32 else "bfloat16", 256, target[0])
     assert eng.cache.num_pages == 4 and eng.cache.num_slots == 4
-    ta, wa, sure = oracle(name, 97, 12)
+    ta, wa, _ = oracle(name, 97, 12)
     tb, wb, _ = oracle(name, 7, 11)
     steps = [dict(step=0, entries=[dict(id="a", tokens=ta[:90], want=[3, 89])], end=[]),
              dict(step=1, entries=[dict(id="a", tokens=ta[90:92], want=[]), dict(id="b", tokens=tb[:1], want=[])], end=[]),
@@ -524,7 +532,7 @@ def test_trace_runner_replays_steps(tmp_path, target):
     assert said == [f"done {i}" for i in range(4)]
     got = {i: torch.from_numpy(np.fromfile(out / f"{i}.f32", dtype="<f4")).view(-1, cfg["vocab"]).double() for i in (0, 2, 3)}
     assert not (out / "1.f32").exists()
-    assert_close(got[0], wa[[3, 89]], target[1], sure=sure[[3, 89]])
-    assert_close(got[2], torch.stack([wa[96], wa[92], wb[1]]), target[1], sure=torch.cat([sure[[96, 92]], sure[:1]]))
+    assert_close(got[0], wa[[3, 89]], target[1])
+    assert_close(got[2], torch.stack([wa[96], wa[92], wb[1]]), target[1])
     assert_close(got[3], wb[[6]], target[1])
     assert len(eng.cache.free) == 4 and len(eng.cache.free_slots) == 4
