@@ -368,8 +368,8 @@ static int launch_gemm(int epi, const void* A, const void* B, void* C, const voi
   return cudaGetLastError() == cudaSuccess ? 0 : 302;
 }
 
-// Sum of the split-K pieces: out[i] = bf16(sum_s ws[s * MN + i] (+ resid[i])). MN is a multiple of 4.
-__global__ void splitk_reduce_kernel(const float* __restrict__ ws, __nv_bfloat16* __restrict__ out,
+// Sum of the split-K pieces: out[i] = bf16(sum_s ws[s * MN + i] (+ resid[i])), or the 32-bit sum into out32. MN is a multiple of 4.
+__global__ void splitk_reduce_kernel(const float* __restrict__ ws, __nv_bfloat16* __restrict__ out, float* __restrict__ out32,
                                      const __nv_bfloat16* __restrict__ resid, int splits, long long MN) {
   pdl_wait();
   pdl_trigger();
@@ -384,15 +384,16 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ ws, __nv_bfloat16
       const float2 a = unpack_bf16(r.x), b = unpack_bf16(r.y);
       acc.x += a.x; acc.y += a.y; acc.z += b.x; acc.w += b.y;
     }
-    *reinterpret_cast<uint2*>(out + i) = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
+    if (out32 != nullptr) *reinterpret_cast<float4*>(out32 + i) = acc;
+    else *reinterpret_cast<uint2*>(out + i) = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
   }
 }
 
-// Y[M, N] (bf16) = A[M, K] B[N, K]^T (+ R) with the K range split over `splits` CTAs per output tile:
+// Y[M, N] (bf16, or 32-bit when f32) = A[M, K] B[N, K]^T (+ R) with the K range split over `splits` CTAs per output tile:
 // pieces go to ws ([splits, M, N] fp32) with plain stores, a second kernel sums them.
 template <int BN>
 static int launch_splitk(const void* A, const void* B, void* Y, const void* R, float* ws, int M, int N, int K, int lda, int ldb,
-                         int splits, cudaStream_t stream) {
+                         int splits, cudaStream_t stream, bool f32 = false) {
   using Cfg = GemmCfg<BN>;
   CUtensorMap tmA, tmB;
   int rc = ab2host::encode_tmap_2d(&tmA, A, 2, (uint64_t)K, (uint64_t)M, (uint64_t)lda * 2, BK, BM, true, 0);
@@ -416,7 +417,8 @@ static int launch_splitk(const void* A, const void* B, void* Y, const void* R, f
   const long long MN = (long long)M * N;
   long long want = (MN / 4 + 255) / 256;
   const int rgrid = (int)(want < 148 * 8 ? want : 148 * 8);
-  if (launch_pdl(splitk_reduce_kernel, dim3(rgrid), dim3(256), 0, stream, (const float*)ws, (__nv_bfloat16*)Y, (const __nv_bfloat16*)R, splits,
+  if (launch_pdl(splitk_reduce_kernel, dim3(rgrid), dim3(256), 0, stream, (const float*)ws, f32 ? nullptr : (__nv_bfloat16*)Y, f32 ? (float*)Y : nullptr,
+                 (const __nv_bfloat16*)R, splits,
                  MN) != cudaSuccess)
     return 303;
   return 0;
@@ -518,6 +520,22 @@ int ab2_gemm_splitk(const void* A, const void* B, void* Y, const void* R, void* 
     case 256: return launch_splitk<256>(A, B, Y, R, w, M, N, K, lda, ldb, splits, s);
     case 128: return launch_splitk<128>(A, B, Y, R, w, M, N, K, lda, ldb, splits, s);
     case 64: return launch_splitk<64>(A, B, Y, R, w, M, N, K, lda, ldb, splits, s);
+  }
+  return 12;
+}
+
+// The same product with a 32-bit result Y [M, N].
+int ab2_gemm_splitk_f32(const void* A, const void* B, void* Y, void* ws, int M, int N, int K, int lda, int ldb, int splits, int bn, void* stream) {
+  using namespace ab2;
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if ((lda & 7) || (ldb & 7) || (N & 3) || splits < 1 || !ws) return 10;
+  if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(B) | reinterpret_cast<uintptr_t>(Y)) & 15) return 11;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  float* w = reinterpret_cast<float*>(ws);
+  switch (bn) {
+    case 256: return launch_splitk<256>(A, B, Y, nullptr, w, M, N, K, lda, ldb, splits, s, true);
+    case 128: return launch_splitk<128>(A, B, Y, nullptr, w, M, N, K, lda, ldb, splits, s, true);
+    case 64: return launch_splitk<64>(A, B, Y, nullptr, w, M, N, K, lda, ldb, splits, s, true);
   }
   return 12;
 }

@@ -40,7 +40,8 @@ struct LatentCfg {
   static constexpr int A_OFF = P_OFF + HEADS * PROW;               // rescaling factor per head
   static constexpr int BAR_OFF = A_OFF + HEADS * 4;
   static constexpr int SMEM = BAR_OFF + 2 * NS * 8 + 1024;
-  static_assert(NS * STAGE >= HEADS * DC * 4, "the merge buffer aliases the stage memory");
+  static constexpr int MROW = DC + 8;                              // floats of a merge row
+  static_assert(NS * STAGE >= HEADS * MROW * 4, "the merge buffer aliases the stage memory");
 };
 
 __device__ __forceinline__ void ld_mat(uint32_t a, uint32_t (&r)[4]) {
@@ -85,7 +86,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
   pdl_trigger();
   const int b = blockIdx.x, h0 = blockIdx.y * HEADS, spl = blockIdx.z, nspl = gridDim.z;
   const int heads = min(HEADS, p.H - h0);
-  const int i = pos[b];
+  const int i = pos[b], e = row_entry[b];
   const int lo = p.window > 0 ? max(0, i - p.window + 1) : 0;
   const int nblk = slots[b] >= 0 ? i / LD_KEYS - lo / LD_KEYS + 1 : 0;      // pieces start at multiples of 32: each lies in one page, or
   const int per = (nblk + nspl - 1) / nspl;                                 // fills two of 16
@@ -96,7 +97,6 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
 
   if (warp == LD_WARPS) {
     if (elect_one() && np > 0) {
-      const int e = row_entry[b];
       const int* pt = p.pages + (size_t)e * p.max_pages;
       const int base = p.page_base[e], last = p.max_pages - 1, sh = p.page_shift, two = sh == 4 ? 1 : 0;
       auto row_at = [&](int t) {                                    // boxes outside the held pages are masked
@@ -104,9 +104,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
       };
       int row0 = row_at(t0), row1 = two ? row_at(t0 + 16) : 0;
       bool ok = true;
+      int s = 0;
+      uint32_t ph = 1u;
       for (int c = 0; c < np; ++c) {
-        const int s = c % NS;
-        ok = mbar_wait(empty(s), ((uint32_t)(c / NS) & 1u) ^ 1u, err, ERR_WAIT_EMPTY);
+        ok = mbar_wait(empty(s), ph, err, ERR_WAIT_EMPTY);
         if (!ok) break;
         const uint32_t dst = sm + s * Cfg::STAGE;
         mbar_expect_tx(full(s), Cfg::STAGE);
@@ -123,6 +124,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
           row0 = row_at(t0 + (c + 1) * LD_KEYS);
           if (two) row1 = row_at(t0 + (c + 1) * LD_KEYS + 16);
         }
+        if (++s == NS) { s = 0; ph ^= 1u; }
       }
       if (!ok) {                                                    // copies in flight get a bounded time to land
         const long long c0 = clock64();
@@ -156,8 +158,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
     constexpr int PIECES = WC / 8;
     const int c0 = warp * PIECES % 8;
 
-    auto scores = [&](int c) {
-      const uint32_t st = sm + (c % NS) * Cfg::STAGE + mine + ((mat >> 1) * 8 + r8) * 128;
+    auto scores = [&](int stage) {
+      const uint32_t st = sm + stage * Cfg::STAGE + mine + ((mat >> 1) * 8 + r8) * 128;
       float s[MT][LD_KEYS / 8][4] = {};
 #pragma unroll
       for (int ks = 0; ks < KS; ++ks) {
@@ -221,21 +223,24 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
       for (int k = 0; k < KPT / 2; ++k) d[k] = pack_bf16(v[2 * k], v[2 * k + 1]);
       if (skey == 0) s_alpha[srow] = alpha;
     };
-    auto arrived = [&](int c) { ok = ok && mbar_wait(full(c % NS), (uint32_t)(c / NS) & 1u, err, ERR_WAIT_FULL); };
+    auto arrived = [&](int stage, uint32_t ph) {
+      ok = ok && mbar_wait(full(stage), ph, err, ERR_WAIT_FULL);
+      __syncwarp();
+    };
     const uint32_t pa = sm + Cfg::P_OFF + ((mat & 1) * 8 + r8) * Cfg::PROW + (mat >> 1) * 16;
     if (np > 0) {
-      arrived(0);
-      __syncwarp();
+      arrived(0, 0u);
       scores(0);
       ld_sync();
       softmax(0);
     }
+    int cur = 0, nxt = 1;                                           // stages of pieces c and c + 1
+    uint32_t ph = 0u;                                               // of piece c + 1
     for (int c = 0; c < np; ++c) {
       ld_sync();                                                    // weights of piece c are there, shares of the scores free
       if (c + 1 < np) {
-        arrived(c + 1);
-        __syncwarp();
-        scores(c + 1);
+        arrived(nxt, ph);
+        scores(nxt);
       }
 #pragma unroll
       for (int m = 0; m < MT; ++m) {
@@ -248,7 +253,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
           }
         }
       }
-      const uint32_t st = sm + (c % NS) * Cfg::STAGE + mine + ((mat & 1) * 8 + r8) * 128;
+      const uint32_t st = sm + cur * Cfg::STAGE + mine + ((mat & 1) * 8 + r8) * 128;
 #pragma unroll
       for (int ks = 0; ks < LD_KEYS / 16; ++ks) {
         uint32_t pf[MT][4];
@@ -266,7 +271,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
         }
       }
       __syncwarp();
-      if (lane == 0) mbar_arrive(empty(c % NS));
+      if (lane == 0) mbar_arrive(empty(cur));
+      cur = nxt;
+      if (++nxt == NS) { nxt = 0; ph ^= 1u; }
       ld_sync();                                                    // shares of piece c + 1 are there, weights of piece c free
       if (c + 1 < np) softmax(c + 1);
     }
@@ -291,14 +298,14 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
           }
         }
     } else {
-      float* mo = reinterpret_cast<float*>(dsm);                    // [HEADS][DC], over the stages: every piece has been used
+      float* mo = reinterpret_cast<float*>(dsm);                    // [HEADS][MROW], over the stages: every piece has been used
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
         for (int j = 0; j < NT; ++j) {
-          float* d = mo + (m * 16 + gq) * DC + warp * WC + j * 8 + 2 * tq;
+          float* d = mo + (m * 16 + gq) * Cfg::MROW + warp * WC + j * 8 + 2 * tq;
           *reinterpret_cast<float2*>(d) = make_float2(o[m][j][0], o[m][j][1]);
-          *reinterpret_cast<float2*>(d + 8 * DC) = make_float2(o[m][j][2], o[m][j][3]);
+          *reinterpret_cast<float2*>(d + 8 * Cfg::MROW) = make_float2(o[m][j][2], o[m][j][3]);
         }
     }
   }
@@ -331,7 +338,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
     float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int c = 0; c < nspl; ++c) {
       const float w = s_wt[c][g];
-      const float4 v = *reinterpret_cast<const float4*>(cl.map_shared_rank(mo, c) + g * DC + col);
+      const float4 v = *reinterpret_cast<const float4*>(cl.map_shared_rank(mo, c) + g * Cfg::MROW + col);
       s.x += v.x * w; s.y += v.y * w; s.z += v.z * w; s.w += v.w * w;
     }
     *reinterpret_cast<uint2*>(out + ((size_t)b * p.H + h0 + g) * p.C + col) = make_uint2(pack_bf16(s.x, s.y), pack_bf16(s.z, s.w));

@@ -165,12 +165,18 @@ __global__ void post_norm_kernel(const T* __restrict__ base, long long ldb, cons
     if (base != nullptr) ldv<V>(base + (size_t)row * ldb + c, h);
     else
       for (int e = 0; e < V; ++e) h[e] = 0.f;
-    for (int s = 0; s < k; ++s) {
-      const int r = inv[(size_t)row * k + s];
-      if (r < 0 || r >= n_rows) continue;
-      float v[V];
-      ldv<V>(y + (size_t)r * H + c, v);
-      for (int e = 0; e < V; ++e) h[e] += v[e];
+    for (int s0 = 0; s0 < k; s0 += 4) {                // four rows on their way at a time
+      float v[4][V];
+#pragma unroll
+      for (int s = 0; s < 4; ++s) {
+        const int r = s0 + s < k ? inv[(size_t)row * k + s0 + s] : -1;
+        if (r >= 0 && r < n_rows) ldv<V>(y + (size_t)r * H + c, v[s]);
+        else
+          for (int e = 0; e < V; ++e) v[s][e] = 0.f;
+      }
+#pragma unroll
+      for (int s = 0; s < 4; ++s)
+        for (int e = 0; e < V; ++e) h[e] += v[s][e];
     }
     for (int e = 0; e < V; ++e) ss += h[e] * h[e];
     stv<V>(srow + c, h);

@@ -333,16 +333,19 @@ def decode_gemm_plan(M: int, N: int, K: int, n_sms: int = 148) -> tuple[int, int
     return best[0], best[1]
 
 
-def gemm_decode(x: torch.Tensor, w: torch.Tensor, resid: Optional[torch.Tensor] = None) -> torch.Tensor:
+def gemm_decode(x: torch.Tensor, w: torch.Tensor, resid: Optional[torch.Tensor] = None, fp32_out: bool = False) -> torch.Tensor:
     """``x @ w^T (+ resid)`` for a handful of rows (decode): output tiles alone cannot fill the
     machine, so K is split over CTAs as well (fp32 pieces in a static workspace, one reduce
-    kernel). Falls back to :func:`gemm` when no split is worth it."""
+    kernel). Falls back to :func:`gemm` when no split is worth it. ``fp32_out``: the 32-bit sums themselves (no ``resid``)."""
     M, K = x.shape
     N = w.shape[0]
     if not x.is_cuda:
         y = x.float() @ w.float().t()
-        return (y + resid.float() if resid is not None else y).to(x.dtype)
+        return y if fp32_out else (y + resid.float() if resid is not None else y).to(x.dtype)
+    assert not (fp32_out and resid is not None)
     bn, splits = decode_gemm_plan(M, N, K)
+    if fp32_out and (splits <= 1 or N % 4 or x.stride(1) != 1 or w.stride(1) != 1):
+        return gemm(x, w, epi=EPI_F32)
     if splits <= 1 or N % 4 or x.stride(1) != 1 or w.stride(1) != 1:
         return gemm(x, w, epi=EPI_BF16_RESID, resid=resid) if resid is not None else gemm(x, w)
     need = splits * M * N
@@ -350,6 +353,11 @@ def gemm_decode(x: torch.Tensor, w: torch.Tensor, resid: Optional[torch.Tensor] 
     ws = _SPLITK_WS.get(key)
     if ws is None or ws.numel() < need:
         ws = _SPLITK_WS[key] = torch.empty(max(need, 4 * DECODE_GEMM_MAX_ROWS * 32768), dtype=torch.float32, device=x.device)
+    if fp32_out:
+        y = torch.empty(M, N, dtype=torch.float32, device=x.device)
+        rc = _L().ab2_gemm_splitk_f32(x.data_ptr(), w.data_ptr(), y.data_ptr(), ws.data_ptr(), M, N, K, x.stride(0), w.stride(0), splits, bn, _s())
+        _lib.check(rc, "ab2_gemm_splitk_f32")
+        return y
     y = torch.empty(M, N, dtype=torch.bfloat16, device=x.device)
     if resid is not None:
         assert resid.shape == y.shape and resid.is_contiguous() and resid.dtype == torch.bfloat16

@@ -95,8 +95,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, fp32_out: bool = False) -> torch.Te
     GEMM, 32-bit ones and odd row lengths the library product."""
     if x.is_cuda and x.dtype == torch.bfloat16 and x.shape[1] % 8 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0:
         N = w.shape[0]
-        if OF.DECODE_SPLITK and not fp32_out and x.shape[0] <= OF.DECODE_GEMM_MAX_ROWS and N % 8 == 0:
-            return OF.gemm_decode(x, w)
+        if OF.DECODE_SPLITK and x.shape[0] <= OF.DECODE_GEMM_MAX_ROWS and N % 8 == 0:
+            return OF.gemm_decode(x, w, fp32_out=fp32_out)
         ld = -(-N // 8) * 8
         out = torch.empty(x.shape[0], ld, device=x.device, dtype=torch.float32 if fp32_out else torch.bfloat16)
         gemm(x, w, out=out[:, :N], epi=EPI_F32 if fp32_out else 0)

@@ -566,6 +566,19 @@ def test_decode_splitk_gemm_matches_fp32(M, N, K, with_resid):
     assert torch.equal(y, y2)
 
 
+@pytest.mark.parametrize("M,N,K", [(64, 64, 4096), (3, 8, 1024), (128, 160, 4096), (64, 32768, 512)])
+def test_decode_splitk_gemm_in_32_bits(M, N, K):
+    """The sums themselves (router logits of a few rows): as exact as the products of the bf16 operands allow."""
+    torch.manual_seed(M + N)
+    x = torch.randn(M, K, device="cuda").bfloat16()
+    w = (torch.randn(N, K, device="cuda") * 0.05).bfloat16()
+    y = OF.gemm_decode(x, w, fp32_out=True)
+    assert y.dtype == torch.float32 and y.shape == (M, N)
+    ref = x.double() @ w.double().t()
+    assert ((y - ref).abs().max() / ref.abs().max()).item() < 1e-5
+    assert oplib.kernel_error() == 0
+
+
 # --------------------------------------------------------------------------- RL losses
 @pytest.mark.parametrize("rs", [None, ("mask", "ratio", None, 5.0), ("clamp", "ratio", 0.5, 2.0), ("mask", "kl_k3", None, 0.05),
                                 ("mask", "binary_kl", None, 0.02), ("mask", "kl_k2", None, 0.02)])
