@@ -8,7 +8,7 @@
 //   S = Q C^T     every warp its columns' share of all scores; the shares meet in shared memory in 32 bits
 //   softmax       a few threads per head: sum of the shares, running maximum and sum, the weights to shared memory
 //   O += P C      every warp its columns
-// The shares of piece c + 1 and the output of piece c are computed together. O is rescaled only when a head's maximum has
+// The output of piece c and the softmax of piece c + 1 run side by side. O is rescaled only when a head's maximum has
 // grown by more than 2^8 since its reference was set. Partial results of a cluster are merged through distributed shared memory.
 #include <cooperative_groups.h>
 
@@ -37,8 +37,8 @@ struct LatentCfg {
   static constexpr int SROW = LD_KEYS + 8, PROW = LD_KEYS * 2 + 16;
   static constexpr int S_OFF = NS * STAGE;                         // shares of the scores, [warp][head][key]
   static constexpr int P_OFF = S_OFF + LD_WARPS * HEADS * SROW * 4;
-  static constexpr int A_OFF = P_OFF + HEADS * PROW;               // rescaling factor per head
-  static constexpr int BAR_OFF = A_OFF + HEADS * 4;
+  static constexpr int A_OFF = P_OFF + 2 * HEADS * PROW;           // rescaling factor per head; these and the weights of two pieces
+  static constexpr int BAR_OFF = A_OFF + 2 * HEADS * 4;
   static constexpr int SMEM = BAR_OFF + 2 * NS * 8 + 1024;
   static constexpr int MROW = DC + 8;                              // floats of a merge row
   static_assert(NS * STAGE >= HEADS * MROW * 4, "the merge buffer aliases the stage memory");
@@ -184,8 +184,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
           *reinterpret_cast<float2*>(d + 8 * Cfg::SROW) = make_float2(s[m][n][2], s[m][n][3]);
         }
     };
-    auto softmax = [&](int c) {
-      float v[KPT] = {};
+    auto sums = [&](float (&v)[KPT]) {
+#pragma unroll
+      for (int k = 0; k < KPT; ++k) v[k] = 0.f;
 #pragma unroll
       for (int w = 0; w < LD_WARPS; ++w) {
         const float* d = s_s + (w * HEADS + srow) * Cfg::SROW + skey;
@@ -197,6 +198,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
           v[0] += x.x; v[1] += x.y;
         }
       }
+    };
+    auto softmax = [&](int c, float (&v)[KPT]) {
       const int t = t0 + c * LD_KEYS + skey;
       float mx = -INFINITY;
 #pragma unroll
@@ -218,10 +221,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
         sum += v[k];
       }
       l_run = l_run * alpha + sum;
-      uint32_t* d = reinterpret_cast<uint32_t*>(dsm + Cfg::P_OFF + srow * Cfg::PROW + skey * 2);
+      uint32_t* d = reinterpret_cast<uint32_t*>(dsm + Cfg::P_OFF + ((c & 1) * HEADS + srow) * Cfg::PROW + skey * 2);
 #pragma unroll
       for (int k = 0; k < KPT / 2; ++k) d[k] = pack_bf16(v[2 * k], v[2 * k + 1]);
-      if (skey == 0) s_alpha[srow] = alpha;
+      if (skey == 0) s_alpha[(c & 1) * HEADS + srow] = alpha;
     };
     auto arrived = [&](int stage, uint32_t ph) {
       ok = ok && mbar_wait(full(stage), ph, err, ERR_WAIT_FULL);
@@ -232,7 +235,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
       arrived(0, 0u);
       scores(0);
       ld_sync();
-      softmax(0);
+      float v[KPT];
+      sums(v);
+      softmax(0, v);
     }
     int cur = 0, nxt = 1;                                           // stages of pieces c and c + 1
     uint32_t ph = 0u;                                               // of piece c + 1
@@ -242,9 +247,13 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
         arrived(nxt, ph);
         scores(nxt);
       }
+      ld_sync();                                                    // shares of piece c + 1 are there
+      float v[KPT];
+      if (c + 1 < np) sums(v);
 #pragma unroll
       for (int m = 0; m < MT; ++m) {
-        const float a0 = s_alpha[m * 16 + gq], a1 = s_alpha[m * 16 + gq + 8];
+        const float* al = s_alpha + (c & 1) * HEADS + m * 16 + gq;
+        const float a0 = al[0], a1 = al[8];
         if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
 #pragma unroll
           for (int j = 0; j < NT; ++j) {
@@ -258,15 +267,15 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
       for (int ks = 0; ks < LD_KEYS / 16; ++ks) {
         uint32_t pf[MT][4];
 #pragma unroll
-        for (int m = 0; m < MT; ++m) ld_mat(pa + m * 16 * Cfg::PROW + ks * 32, pf[m]);
+        for (int m = 0; m < MT; ++m) ld_mat(pa + ((c & 1) * HEADS + m * 16) * Cfg::PROW + ks * 32, pf[m]);
 #pragma unroll
         for (int j = 0; j < NT; j += 2) {
-          uint32_t v[4];
-          ld_mat_t(st + ks * 16 * 128 + (((c0 + j + (mat >> 1)) ^ r8) << 4), v);
+          uint32_t cf[4];
+          ld_mat_t(st + ks * 16 * 128 + (((c0 + j + (mat >> 1)) ^ r8) << 4), cf);
 #pragma unroll
           for (int m = 0; m < MT; ++m) {
-            ld_mma(o[m][j], pf[m], v[0], v[1]);
-            ld_mma(o[m][j + 1], pf[m], v[2], v[3]);
+            ld_mma(o[m][j], pf[m], cf[0], cf[1]);
+            ld_mma(o[m][j + 1], pf[m], cf[2], cf[3]);
           }
         }
       }
@@ -274,8 +283,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
       if (lane == 0) mbar_arrive(empty(cur));
       cur = nxt;
       if (++nxt == NS) { nxt = 0; ph ^= 1u; }
-      ld_sync();                                                    // shares of piece c + 1 are there, weights of piece c free
-      if (c + 1 < np) softmax(c + 1);
+      if (c + 1 < np) softmax(c + 1, v);
     }
     // ---- this CTA's sums
 #pragma unroll

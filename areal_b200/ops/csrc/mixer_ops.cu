@@ -145,7 +145,7 @@ __global__ void gated_norm_kernel(const float* __restrict__ y, const T* __restri
 // ------------------------------------------------------------------ norms behind a sublayer
 // h = base row + the sum of the token's k expert rows (either may be missing); resid += mult * norm(h) * (off + w);
 // x = resid, or norm(resid) * (off_next + w_next) when there is a next norm. One CTA per row, the row in shared memory.
-template <typename T, int V>
+template <typename T, int V, bool EXPERTS>
 __global__ void post_norm_kernel(const T* __restrict__ base, long long ldb, const T* __restrict__ y, const int* __restrict__ inv, int k, int n_rows,
                                  const float* __restrict__ w, float off, float mult, float* __restrict__ resid, const float* __restrict__ w_next,
                                  float off_next, T* __restrict__ x, int H, float eps) {
@@ -165,7 +165,7 @@ __global__ void post_norm_kernel(const T* __restrict__ base, long long ldb, cons
     if (base != nullptr) ldv<V>(base + (size_t)row * ldb + c, h);
     else
       for (int e = 0; e < V; ++e) h[e] = 0.f;
-    for (int s0 = 0; s0 < k; s0 += 4) {                // four rows on their way at a time
+    for (int s0 = 0; EXPERTS && s0 < k; s0 += 4) {     // four rows on their way at a time
       float v[4][V];
 #pragma unroll
       for (int s = 0; s < 4; ++s) {
@@ -640,9 +640,9 @@ int ab2_post_norm(const void* base, long long ldb, const void* y, const int* inv
            aligned_to(w, 16) && aligned_to(w_next, 16);
   };
   AB2_TYPED8(dt, fits(8), fits(4), {
-    auto kern = post_norm_kernel<T, V>;
-    static ab2host::DevState st;
-    if (ab2host::prepare_launch(kern, 200 * 1024, st, nullptr)) return 12;
+    auto kern = k > 0 ? post_norm_kernel<T, V, true> : post_norm_kernel<T, V, false>;
+    static ab2host::DevState st[2];
+    if (ab2host::prepare_launch(kern, 200 * 1024, st[k > 0], nullptr)) return 12;
     launch_pdl(kern, dim3(R), dim3(th), smem, (cudaStream_t)stream, (const T*)base, ldb, (const T*)y, inv, k, n_rows, w, off, mult, resid, w_next,
                off_next, (T*)x, H, eps);
   });
