@@ -261,6 +261,16 @@ def latent_kernel_table(cfg, prefill=(4, 2048), decode=(64, 960), dev="cuda") ->
                     M._call("ab2_latent_decode", qc.data_ptr(), b.pos.data_ptr(), b.slots.data_ptr(), b.row_entry.data_ptr(), oc.data_ptr(), R,
                             cache.data_ptr(), cache.shape[0], b.pages.data_ptr(), b.page_base.data_ptr(), b.pages.shape[1], 64, nq, C, scale, win)
                 add(f"latent_decode {win} decode", dec, (R * see * C + 2 * qc.numel()) * 2, 4.0 * R * see * nq * C, like="paged_decode decode")
+            # as many bytes as the paged kernel below reads: four times the sequences
+            b4, rows4 = _batch([1] * (4 * nB), [ctx] * (4 * nB), dev, windows=windows)
+            cache4, qc4 = torch.randn(rows4, 1, C, **bf), torch.randn(4 * nB, nq, C, **bf)
+            oc4, see = torch.empty_like(qc4), min(ctx + 1, windows[-1])
+
+            def dec4():
+                M._call("ab2_latent_decode", qc4.data_ptr(), b4.pos.data_ptr(), b4.slots.data_ptr(), b4.row_entry.data_ptr(), oc4.data_ptr(), 4 * nB,
+                        cache4.data_ptr(), cache4.shape[0], b4.pages.data_ptr(), b4.page_base.data_ptr(), b4.pages.shape[1], 64, nq, C, scale, windows[-1])
+            add(f"latent_decode {windows[-1]} decode, {4 * nB} sequences", dec4, (4 * nB * see * C + 2 * qc4.numel()) * 2, 16.0 * nB * see * nq * C,
+                like="paged_decode decode")
             nk = max(1, nq // 4)
             kc, vc = torch.randn(rows_, nk, 128, **bf), torch.randn(rows_, nk, 128, **bf)
             q2 = torch.randn(R, nq, 128, **bf)
