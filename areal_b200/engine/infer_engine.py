@@ -297,7 +297,7 @@ class NativeInferenceEngine(InferenceEngine):
         ic, dev = self.icfg, self.device
         if self.tp_size > 1:
             raise NotImplementedError("tensor-parallel rollout of mixer stacks")
-        mixers = [l.mix for l in self.model.layers]
+        mixers = self.model.cache_mixers()
         dtype = self.model.dtype
         self.max_batch = B = max(b for b in DECODE_BUCKETS if b <= max(1, ic.max_running_requests))
         want = ic.max_running_requests * (ic.context_length // ic.page_size + 1)
@@ -327,7 +327,7 @@ class NativeInferenceEngine(InferenceEngine):
     def _make_ragged_runner(self):
         ic = self.icfg
         n_pages, ps, slots = self._ragged_shape
-        self.cache = StateCache([l.mix for l in self.model.layers], n_pages, ps, slots, self.device, self.model.dtype)
+        self.cache = StateCache(self.model.cache_mixers(), n_pages, ps, slots, self.device, self.model.dtype)
         self.runner = RaggedRunner(self.model, self.cache, self.device, slots, ic.context_length, ic.use_cuda_graph)
         if self.device.type == "cuda":
             self.runner.stream = self.stream

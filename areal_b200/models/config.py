@@ -14,7 +14,7 @@ from typing import Optional
 
 @dataclass
 class ModelConfig:
-    arch: str = "qwen2"                 # qwen2 | qwen3 | qwen3_moe | qwen2_moe | qwen3_5 | qwen3_5_moe | kagolix | vogilix
+    arch: str = "qwen2"                 # qwen2 | qwen3 | qwen3_moe | qwen2_moe | qwen3_5 | qwen3_5_moe | kagolix | vogilix | bumotar
     vocab_size: int = 151936
     hidden_size: int = 1536
     num_layers: int = 28
@@ -63,14 +63,16 @@ class ModelConfig:
     partial_rotary_factor: float = 1.0
     attn_output_gate: bool = False
     rms_norm_offset: bool = False
-    # mixer stacks (Kagolix, Vogilix): one entry per layer, {"type": mixer kind, "mixer": its sizes, "mlp":
+    # mixer stacks (Kagolix, Vogilix, Bumotar): one entry per layer, {"type": mixer kind, "mixer": its sizes, "mlp":
     # feed-forward or None} as in config.json (see models/mixers.py); grouped RMS norms and a capped output
     mixer_layers: list[dict] = field(default_factory=list)
     norm_groups: int = 1
     logit_softcap: float = 0.0
-    norm_placement: str = "sandwich"        # sandwich: before and after every sublayer | post: on its output only
+    norm_placement: str = "sandwich"        # sandwich: before and after every sublayer | post: on its output only | pre: on its input only
     residual_mult: float = 1.0              # factor of every sublayer's normed output on its way into the residual sum
     learned_positions: bool = False         # a vector per position (max_position_embeddings of them) added to the embedding
+    logit_scale: float = 1.0                # factor of the logits (part of the final norm)
+    layer_loop: Optional[dict] = None       # {"start", "stop", "times"}: layers start .. stop - 1 run that many times in a row
     token_side_dim: int = 0                 # > 0: every layer ends with a gated input from its own part of a per-token row
 
     @property
@@ -249,12 +251,19 @@ class ModelConfig:
             raise ValueError(f"unsupported architecture '{d['architecture']}' (have {sorted(x.name for x in DESIGNS.values())})")
         layers = [dict(type=e["type"], mixer=dict(e["mixer"]), mlp=dict(e["mlp"]) if e.get("mlp") else None) for e in d["layers"]]
         check_layer_specs(arch, layers, d["width"], d["norm"].get("groups", 1))
-        att = [e["mixer"] for e in layers if "heads" in e["mixer"] and "dim" in e["mixer"]]
+        nested = [e["mixer"]["left"] for e in layers if isinstance(e["mixer"].get("left"), dict)]
+        att = [m for m in [e["mixer"] for e in layers] + nested if "heads" in m and "dim" in m]
         moe = [e["mlp"] for e in layers if e["mlp"] and e["mlp"]["kind"] == "moe"]
         own = {}
         if arch == "vogilix":
             own = dict(norm_placement="post", rms_norm_offset=True, residual_mult=float(d["residual_mult"]), learned_positions=True,
                        max_position_embeddings=int(d["max_positions"]), token_side_dim=int((d.get("token_side") or {}).get("dim") or 0))
+        elif arch == "bumotar":
+            loop = {k: int(d["loop"][k]) for k in ("start", "stop", "times")} if d.get("loop") else None
+            if loop and not (0 <= loop["start"] < loop["stop"] <= len(layers) and loop["times"] >= 1):
+                raise ValueError(f"a loop over layers {loop['start']} to {loop['stop']} of {len(layers)}, {loop['times']} times")
+            own = dict(norm_placement="pre", logit_scale=float(d.get("logit_scale", 1.0)), layer_loop=loop,
+                       max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)))
         else:
             own = dict(norm_groups=int(d["norm"].get("groups", 1)), logit_softcap=float(d.get("logit_softcap") or 0.0),
                        max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)))
@@ -282,6 +291,8 @@ class ModelConfig:
             if mt == "vogilix":
                 d.update(max_positions=self.max_position_embeddings, norm=dict(eps=self.rms_norm_eps), residual_mult=self.residual_mult,
                          token_side=dict(dim=self.token_side_dim) if self.token_side_dim else None)
+            elif mt == "bumotar":
+                d.update(norm=dict(eps=self.rms_norm_eps), logit_scale=self.logit_scale, loop=dict(self.layer_loop) if self.layer_loop else None)
             else:
                 d.update(norm=dict(eps=self.rms_norm_eps, groups=self.norm_groups), logit_softcap=self.logit_softcap)
             return d
@@ -427,6 +438,27 @@ def _latent_stack_preset(vocab, width, pattern, att, windows, dense_ff, moe, sha
                 token_side=dict(dim=side), layers=layers)
 
 
+def _looped_stack_preset(vocab, width, pattern, window, ret, latent, moe, shared_ff, loop, logit_scale, eps=1e-6, scales=(0.7, 0.4)):
+    """A Bumotar stack: p in ``pattern`` is a layer of parallel branches (windowed attention, retention), l latent attention,
+    upper case a layer without feed-forward; ``loop`` = (start, stop, times)."""
+    layers = []
+    for c in pattern:
+        mixer = dict(latent) if c.lower() == "l" else dict(left=dict(window), left_scale=scales[0], right=dict(ret), right_scale=scales[1])
+        mlp = dict(kind="moe", expert=dict(ff=moe[2]), router=dict(experts=moe[0], top=moe[1]), shared=dict(ff=shared_ff)) if c.islower() else None
+        layers.append(dict(type="latent_attention" if c.lower() == "l" else "parallel", mixer=mixer, mlp=mlp))
+    return dict(architecture="Bumotar", vocab=vocab, width=width, norm=dict(eps=eps), logit_scale=logit_scale,
+                loop=dict(start=loop[0], stop=loop[1], times=loop[2]) if loop else None, layers=layers)
+
+
+def _ret(heads, dim, vdim, base=10000.0):
+    """Retention with half-lives from a few tokens to a few thousand, spread over the heads."""
+    return dict(heads=heads, dim=dim, vdim=vdim, rot=dict(base=base, dims=dim), decay=[1.0 - 2.0 ** -(3.0 + 8.0 * h / max(1, heads - 1)) for h in range(heads)])
+
+
+def _yarn(base, dims, factor=4.0, original=4096):
+    return dict(base=base, dims=dims, scaling=dict(factor=factor, original=original, fast=32.0, slow=1.0))
+
+
 MIXER_STACK_PRESETS = {
     "tiny-kagolix": _mixer_stack_preset(
         320, 128, "aMrM", dict(heads=4, kv_heads=2, dim=32, vdim=48, scale=0.2, softcap=25.0, mask=dict(size=40)),
@@ -446,6 +478,19 @@ MIXER_STACK_PRESETS = {
         256, 8192),
     "vogilix-2b-layers": _latent_stack_preset(
         32768, 2048, "dede", dict(heads=16, dim=128, vdim=128, q_rank=768, kv_rank=512, scale=128 ** -0.5), (1024,), 8192, (64, 8, 768), 1024, 256, 8192),
+    "tiny-bumotar": _looped_stack_preset(
+        320, 128, "plPl", dict(heads=4, kv_heads=2, dim=32, vdim=48, scale=0.2, softcap=25.0, mask=dict(size=40),
+                               rot=dict(base=10000.0, dims=16, scaling=dict(factor=3.0))), _ret(2, 48, 32),
+        dict(heads=4, dim=24, rot_dim=16, vdim=40, kv_rank=56, scale=0.15, rot=_yarn(10000.0, 16, original=256)), (6, 2, 64), 96, (1, 3, 2), 0.5),
+    # layer sizes of an 8B-class and of a 2B-class model; two looped layers and two that run once
+    "bumotar-8b-layers": _looped_stack_preset(
+        32768, 4096, "plpl", dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, mask=dict(size=1024),
+                                  rot=dict(base=500000.0, dims=64, scaling=dict(factor=4.0))), _ret(16, 128, 128),
+        dict(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, rot=_yarn(10000.0, 64)), (64, 8, 768), 2048, (0, 2, 2), 0.125),
+    "bumotar-2b-layers": _looped_stack_preset(
+        32768, 2048, "plpl", dict(heads=16, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, mask=dict(size=1024),
+                                  rot=dict(base=500000.0, dims=64, scaling=dict(factor=4.0))), _ret(8, 128, 128),
+        dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, rot=_yarn(10000.0, 64)), (64, 8, 768), 1024, (0, 2, 2), 0.125),
 }
 
 

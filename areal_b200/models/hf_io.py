@@ -20,7 +20,8 @@ from .config import ModelConfig
 
 # --------------------------------------------------------------------------- name mapping
 def hf_to_native_plan(cfg: ModelConfig) -> dict[str, list[tuple[str, Optional[tuple[int, int]], Optional[int]]]]:
-    """native name -> list of (hf name, row range in the native tensor or None, expert idx or None)."""
+    """native name -> list of (hf name, row range in the native tensor or None, expert idx or None). Mixer stacks may give any
+    index of the native tensor in place of the expert's (columns of a fused output projection)."""
     if cfg.is_mixer_stack:
         from .mixers import checkpoint_plan
 

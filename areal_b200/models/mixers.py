@@ -1,22 +1,27 @@
 """Mixer stacks: decoder models whose layers are listed one by one, each with its own token mixer and feed-forward.
 
-Two designs are built from the parts below (:data:`DESIGNS`):
+Three designs are built from the parts below (:data:`DESIGNS`):
 
 * Kagolix normalises twice around every sublayer, in groups: ``x += norm_b(f(norm_a(x)))``; its output is capped;
 * Vogilix normalises the sublayer's output only, ``x += m * norm(f(x))``, adds a learned vector per position to the
-  embedding, and ends every layer with a gated input from the layer's own part of a per-token row.
+  embedding, and ends every layer with a gated input from the layer's own part of a per-token row;
+* Bumotar normalises before every sublayer, ``x += f(norm(x))``, and runs a stretch of its layers several times in a row with
+  the same weights, every pass with caches and states of its own and with the embedding mixed in again before it.
 
-The sum x stays in 32 bits in both. The mixers
+The sum x stays in 32 bits in all of them. The mixers
 
 * ``attention``: grouped-query attention inside chunks of positions, whole-projection RMS norms on q and k, no rotation,
   capped scores and a logarithmic distance bias (two numbers per head);
 * ``rglru``: a gated branch times a real-gated linear recurrence behind a short causal convolution;
 * ``mamba2``: the scalar-decay state-space recurrence, gated and normalised in groups;
 * ``latent_attention``: keys and values of all heads from one normed latent per token (the only thing cached), queries from
-  a latent of their own, no positions, a sliding window;
+  a latent of their own, no positions, a sliding window; or (:class:`RotaryLatentAttention`) queries straight from the layer's
+  input and beside the latent one rotated key part for all heads, sinks and a gate per head;
+* ``parallel``: branches side by side on one input and one output projection: windowed attention with rotated, normed
+  queries and keys, capped scores, a sink and gated channels; retention (linear attention with a fixed decay per head);
 
 and the feed-forwards (dense with xIELU or the exact GELU; experts behind a softmax or a sigmoid router, weighted at their
-output or at their input) are built from the ops of :mod:`..ops.mixer_ops`. A forward pass runs the rows of one step
+output or at their input, with or without a gated shared expert) are built from the ops of :mod:`..ops.mixer_ops`. A forward pass runs the rows of one step
 (:class:`~..ops.mixer_ops.RaggedBatch`) from the pages and state slots of :class:`~..engine.state_cache.StateCache`; whole
 prompts, portions and single tokens are the same call.
 
@@ -25,6 +30,7 @@ parameters) as fp32. Serving only: there is no backward pass.
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 
 import torch
@@ -43,16 +49,9 @@ def check_layer_specs(arch: str, layers: list, width: int, norm_groups: int) -> 
         raise ValueError(f"norm groups {norm_groups} do not divide the width {width}")
     for i, e in enumerate(layers):
         t, m, mlp = e["type"], e["mixer"], e["mlp"]
-        if t not in MIXERS:
-            raise ValueError(f"layer {i}: unknown mixer '{t}' (have {sorted(MIXERS)})")
-        if t == "attention" and m["heads"] % m["kv_heads"]:
-            raise ValueError(f"layer {i}: {m['heads']} query heads over {m['kv_heads']} key/value heads")
-        if t == "rglru" and m["width"] % m["blocks"]:
-            raise ValueError(f"layer {i}: {m['blocks']} blocks do not divide {m['width']}")
-        if t == "mamba2" and (m["heads"] % m["groups"] or (m["heads"] * m["vdim"]) % m["norm_groups"]):
-            raise ValueError(f"layer {i}: groups do not divide the heads or the norm groups the channels")
-        if t == "latent_attention" and min(m[k] for k in ("heads", "dim", "vdim", "q_rank", "kv_rank")) < 1:
-            raise ValueError(f"layer {i}: a latent attention needs positive sizes")
+        if t not in design.mixers:
+            raise ValueError(f"layer {i}: unknown mixer '{t}' (have {sorted(design.mixers)})")
+        design.mixers[t].check(m, f"layer {i}: ")
         if mlp and mlp["kind"] not in design.mlps:
             raise ValueError(f"layer {i}: unknown feed-forward '{mlp['kind']}'")
         if mlp and mlp["kind"] == "moe" and not 1 <= mlp["router"]["top"] <= mlp["router"]["experts"]:
@@ -73,8 +72,53 @@ class _Block(nn.Module):
     def vec(self, *shape):
         return nn.Parameter(torch.empty(*shape, dtype=torch.float32, device=self._device))
 
+    def const(self, values):
+        """Constants of the configuration as an fp32 buffer (no part of a checkpoint)."""
+        return torch.tensor(values, dtype=torch.float32, device=self._device)
+
+    @staticmethod
+    def check(m, where):
+        """Raises ``ValueError`` for sizes that no kernel could run."""
+
+    rotary = None            # (frequencies, factor of cos and sin) when the block rotates; its column in the step's table is ``rot_at``
+
+    def rot(self, b):
+        return b.rot[:, self.rot_at:self.rot_at + len(self.rotary[0])]
+
+
+def _need(ok, where, what):
+    if not ok:
+        raise ValueError(where + what)
+
+
+# ----------------------------------------------------------------------------- rotation frequencies
+def rotary_frequencies(rot: dict):
+    """(frequencies, 1.0) of ``rot.dims / 2`` pairs, all divided by ``rot.scaling.factor`` when there is one."""
+    f = float((rot.get("scaling") or {}).get("factor") or 1.0)
+    return tuple(rot["base"] ** (-2.0 * i / rot["dims"]) / f for i in range(rot["dims"] // 2)), 1.0
+
+
+def yarn_frequencies(rot: dict):
+    """(frequencies, factor of cos and sin) under YaRN: pairs that turn more than ``fast`` times within ``original`` positions
+    keep their frequency, those that turn less than ``slow`` times are stretched by ``factor``, with a ramp between."""
+    s = rot.get("scaling")
+    if not s:
+        return rotary_frequencies(rot)
+    dims, base = rot["dims"], float(rot["base"])
+    at = [dims * math.log(s["original"] / (2.0 * math.pi * turns)) / (2.0 * math.log(base)) for turns in (s["fast"], s["slow"])]
+    lo, hi = max(math.floor(at[0]), 0), min(math.ceil(at[1]), dims - 1)
+    out = []
+    for i in range(dims // 2):
+        f, r = base ** (-2.0 * i / dims), min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+        out.append(f / s["factor"] * r + f * (1.0 - r))
+    return tuple(out), 0.1 * math.log(s["factor"]) + 1.0
+
 
 class ChunkAttention(_Block):
+    @staticmethod
+    def check(m, where):
+        _need(m["heads"] % m["kv_heads"] == 0, where, f"{m['heads']} query heads over {m['kv_heads']} key/value heads")
+
     def __init__(self, cfg, m, dtype, device):
         super().__init__(cfg, dtype, device)
         H, w = cfg.hidden_size, m
@@ -110,6 +154,10 @@ class ChunkAttention(_Block):
 
 
 class RGLRU(_Block):
+    @staticmethod
+    def check(m, where):
+        _need(m["width"] % m["blocks"] == 0, where, f"{m['blocks']} blocks do not divide {m['width']}")
+
     def __init__(self, cfg, m, dtype, device):
         super().__init__(cfg, dtype, device)
         H, W, n = cfg.hidden_size, m["width"], m["blocks"]
@@ -140,6 +188,11 @@ class RGLRU(_Block):
 
 
 class Mamba2(_Block):
+    @staticmethod
+    def check(m, where):
+        _need(m["heads"] % m["groups"] == 0 and (m["heads"] * m["vdim"]) % m["norm_groups"] == 0, where,
+              "groups do not divide the heads or the norm groups the channels")
+
     def __init__(self, cfg, m, dtype, device):
         super().__init__(cfg, dtype, device)
         H = cfg.hidden_size
@@ -174,6 +227,10 @@ class LatentAttention(_Block):
     key part is applied to the queries and the value part to the outputs (all heads then share the latent as key and value),
     for portions the keys and values of the visible tokens are worked out once."""
 
+    @staticmethod
+    def check(m, where):
+        _need(min(m[k] for k in ("heads", "dim", "vdim", "q_rank", "kv_rank")) >= 1, where, "a latent attention needs positive sizes")
+
     def __init__(self, cfg, m, dtype, device):
         super().__init__(cfg, dtype, device)
         H = cfg.hidden_size
@@ -207,6 +264,186 @@ class LatentAttention(_Block):
         return {p + "down_proj": [(h + "dq", (0, rq), None), (h + "dkv", (rq, rq + rc), None)],
                 p + "q_norm": [(h + "dq.norm", None, None)], p + "kv_norm": [(h + "dkv.norm", None, None)], p + "uq_proj": [(h + "uq", None, None)],
                 p + "ukv_proj": [(h + "uk", (0, nk), None), (h + "uv", (nk, nk + nv), None)], p + "o_proj": [(h + "o", None, None)]}
+
+
+class RotaryLatentAttention(_Block):
+    """Latent attention with positions: queries come straight from the layer's input as [unrotated, rotated] heads, and the
+    cache row is the normed latent followed by one rotated key part that all heads share. Rotation of neighbouring pairs,
+    YaRN frequencies; a learned sink and a sigmoid gate per head. Sees everything before it."""
+
+    @staticmethod
+    def check(m, where):
+        _need(min(m[k] for k in ("heads", "dim", "vdim", "kv_rank")) >= 1 and m["rot_dim"] >= 2, where, "a latent attention needs positive sizes")
+        _need(m["rot"]["dims"] == m["rot_dim"] and m["rot_dim"] % 2 == 0, where, "the rotated part turns as a whole, in pairs")
+
+    span = 0
+
+    def __init__(self, cfg, m, dtype, device):
+        super().__init__(cfg, dtype, device)
+        H = cfg.hidden_size
+        self.nq, self.D, self.Dv, self.kv_rank, self.rot_dim = m["heads"], m["dim"], m["vdim"], m["kv_rank"], m["rot_dim"]
+        self.scale, self.rotary = float(m["scale"]), yarn_frequencies(m["rot"])
+        self.q_rows = self.nq * (self.D + self.rot_dim)
+        self.gate_at = self.q_rows + self.kv_rank + self.rot_dim
+        self.in_proj = self.mat(self.gate_at + self.nq, H)                       # queries, latent, shared key part, gate
+        self.kv_norm, self.sink = self.vec(self.kv_rank), self.vec(self.nq)
+        self.ukv_proj = self.mat(self.nq * (self.D + self.Dv), self.kv_rank)
+        self.o_proj = self.mat(H, self.nq * self.Dv)
+
+    def cache_shapes(self):
+        return {"kv": ((1, self.kv_rank + self.rot_dim), None)}
+
+    def first_visible(self, pos: int) -> int:
+        return 0
+
+    def forward(self, x, b, lc):
+        R, z = x.shape[0], M.linear(x, self.in_proj)
+        M.latent_rope_append(z, self.kv_norm, self.eps, self.rot(b), True, b, lc.k, self.nq, self.D)
+        q = z[:, :self.q_rows].unflatten(1, (self.nq, self.D + self.rot_dim))
+        o = M.latent_attention(q, lc.k, self.ukv_proj, self.Dv, b, self.scale, 0, self.rot_dim, self.sink, z[:, self.gate_at:])
+        return M.linear(o.view(R, -1), self.o_proj)
+
+    @staticmethod
+    def checkpoint_names(p, m, h):
+        rq, rd, nk, nv = m["heads"] * (m["dim"] + m["rot_dim"]), m["kv_rank"] + m["rot_dim"], m["heads"] * m["dim"], m["heads"] * m["vdim"]
+        return {p + "in_proj": [(h + "q", (0, rq), None), (h + "dkv", (rq, rq + rd), None), (h + "g", (rq + rd, rq + rd + m["heads"]), None)],
+                p + "kv_norm": [(h + "dkv.norm", None, None)], p + "sink": [(h + "sink", None, None)],
+                p + "ukv_proj": [(h + "uk", (0, nk), None), (h + "uv", (nk, nk + nv), None)], p + "o_proj": [(h + "o", None, None)]}
+
+
+# ----------------------------------------------------------------------------- branches side by side
+class WindowBranch(_Block):
+    """Grouped-query attention in a sliding window: per-head norms and rotation (halves paired) on q and k, capped scores, one
+    added to the softmax's denominator, a gate per output channel. Works on its rows q | k | v | g of a fused projection."""
+
+    parts = ("q", "k", "v", "g")
+    SINK = 0.0               # its exponential is what the denominator gets
+
+    @staticmethod
+    def check(m, where):
+        _need(min(m[k] for k in ("heads", "kv_heads", "dim", "vdim")) >= 1 and m["heads"] % m["kv_heads"] == 0, where,
+              f"{m['heads']} query heads over {m['kv_heads']} key/value heads")
+        _need(m["rot"]["dims"] % 2 == 0 and m["rot"]["dims"] <= m["dim"], where, "rotated numbers come in pairs within a head")
+
+    def __init__(self, cfg, m, dtype, device):
+        super().__init__(cfg, dtype, device)
+        self.nq, self.nkv, self.D, self.Dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        self.scale, self.softcap, self.window = float(m["scale"]), float(m.get("softcap") or 0.0), int((m.get("mask") or {}).get("size") or 0)
+        self.rotary = rotary_frequencies(m["rot"])
+        self.q_norm, self.k_norm = self.vec(self.D), self.vec(self.D)
+
+    @staticmethod
+    def rows(m):
+        return m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"], m["heads"] * m["vdim"]
+
+    def cache_shapes(self):
+        return {"kv": ((self.nkv, self.D), (self.nkv, self.Dv))}
+
+    def forward(self, z, b, lc, factor, out):
+        q = M.qk_head_norm_append(z, self.q_norm, self.k_norm, self.eps, self.rot(b), False, b, lc.k, lc.v, self.nq)
+        gate = z[:, self.nq * self.D + self.nkv * (self.D + self.Dv):][:, :self.nq * self.Dv]
+        M.chunk_attention(q, lc.k, lc.v, b, self.scale, self.softcap, window=self.window, sink=self.SINK, gate=gate, out_scale=factor, out=out)
+
+    @staticmethod
+    def own_names(p, h):
+        return {p + "q_norm": [(h + "q.norm", None, None)], p + "k_norm": [(h + "k.norm", None, None)]}
+
+
+class RetentionBranch(_Block):
+    """Linear attention with a fixed decay per head and no denominator: rotated q and k (halves paired), every head's output
+    over its root mean square, gated. Works on its rows q | k | v | g of a fused projection."""
+
+    parts = ("q", "k", "v", "g")
+
+    @staticmethod
+    def check(m, where):
+        _need(min(m[k] for k in ("heads", "dim", "vdim")) >= 1 and len(m["decay"]) == m["heads"], where, f"{len(m['decay'])} decays for {m['heads']} heads")
+        _need(m["rot"]["dims"] % 2 == 0 and m["rot"]["dims"] <= m["dim"] <= 512, where, "rotated numbers come in pairs within a head of up to 512")
+
+    def __init__(self, cfg, m, dtype, device):
+        super().__init__(cfg, dtype, device)
+        self.heads, self.D, self.Dv = m["heads"], m["dim"], m["vdim"]
+        self.rotary = rotary_frequencies(m["rot"])
+        self.register_buffer("decay", self.const(m["decay"]), persistent=False)
+        self.register_buffer("log2_decay", self.const([max(math.log2(a), -1e4) if a > 0 else -1e4 for a in m["decay"]]), persistent=False)
+
+    @staticmethod
+    def rows(m):
+        return m["heads"] * m["dim"], m["heads"] * m["dim"], m["heads"] * m["vdim"], m["heads"] * m["vdim"]
+
+    def cache_shapes(self):
+        return {"state": (self.heads, self.Dv, self.D)}
+
+    def forward(self, z, b, lc, factor, out):
+        M.retention(z, self.decay, self.log2_decay, self.rot(b), self.eps, factor, out, self.heads, self.D, self.Dv, b, lc.state)
+
+    @staticmethod
+    def own_names(p, h):
+        return {}
+
+
+class Parallel(_Block):
+    """Windowed attention and retention on the same input, their outputs weighted and added: one product makes the rows of
+    both, one takes their outputs, which lie side by side, to the layer's width."""
+
+    BRANCHES = (("left", WindowBranch), ("right", RetentionBranch))
+
+    @classmethod
+    def check(cls, m, where):
+        for n, branch in cls.BRANCHES:
+            branch.check(m[n], f"{where}{n}: ")
+
+    def __init__(self, cfg, m, dtype, device):
+        super().__init__(cfg, dtype, device)
+        H = cfg.hidden_size
+        self.factors = [float(m[n + "_scale"]) for n, _ in self.BRANCHES]
+        self.in_rows, self.out_cols = self._layout(m)
+        self.in_proj, self.o_proj = self.mat(self.in_rows[-1], H), self.mat(H, self.out_cols[-1])
+        self.branches = nn.ModuleList([branch(cfg, m[n], dtype, device) for n, branch in self.BRANCHES])
+        self.window = self.branches[0].window
+
+    @classmethod
+    def _layout(cls, m):
+        """First row of every branch in the input projection and first column in the output projection, and their ends."""
+        rows, cols = [0], [0]
+        for n, branch in cls.BRANCHES:
+            r = branch.rows(m[n])
+            rows.append(rows[-1] + sum(r))
+            cols.append(cols[-1] + r[3])
+        return rows, cols
+
+    def cache_shapes(self):
+        out = {}
+        for br in self.branches:
+            out.update(br.cache_shapes())
+        return out
+
+    def first_visible(self, pos: int) -> int:
+        return max(0, pos - self.window + 1) if self.window else 0
+
+    @property
+    def span(self) -> int:
+        return self.window
+
+    def forward(self, x, b, lc):
+        z = M.linear(x, self.in_proj)
+        o = torch.empty(x.shape[0], self.out_cols[-1], device=x.device, dtype=x.dtype)
+        for i, br in enumerate(self.branches):
+            br(z[:, self.in_rows[i]:self.in_rows[i + 1]], b, lc, self.factors[i], o[:, self.out_cols[i]:self.out_cols[i + 1]])
+        return M.linear(o, self.o_proj)
+
+    @classmethod
+    def checkpoint_names(cls, p, m, h):
+        rows, cols = cls._layout(m)
+        out = {p + "in_proj": [], p + "o_proj": []}
+        for i, (n, branch) in enumerate(cls.BRANCHES):
+            at, hb = rows[i], f"{h}{n}."
+            for part, r in zip(branch.parts, branch.rows(m[n])):
+                out[p + "in_proj"].append((hb + part, (at, at + r), None))
+                at += r
+            out[p + "o_proj"].append((hb + "o", None, (slice(None), slice(cols[i], cols[i + 1]))))
+            out.update(branch.own_names(f"{p}branches.{i}.", hb))
+        return out
 
 
 class XieluMLP(_Block):
@@ -302,7 +539,41 @@ class InputWeightedMLP(_Block):
         return out
 
 
-MIXERS = {"attention": ChunkAttention, "rglru": RGLRU, "mamba2": Mamba2, "latent_attention": LatentAttention}
+class SharedExpertMLP(_Block):
+    """Top-k experts of gated units: softmax scores choose, and the chosen ones, renormalised, weigh the experts' outputs. An
+    expert that every token visits may stand beside them, behind a sigmoid gate of one number per token whose logit is made
+    with the router's."""
+
+    def __init__(self, cfg, m, dtype, device):
+        super().__init__(cfg, dtype, device)
+        E, I, H = m["router"]["experts"], m["expert"]["ff"], cfg.hidden_size
+        self.experts, self.top = E, m["router"]["top"]
+        sh = m.get("shared")
+        self.router = self.mat(-(-(E + 1) // 8) * 8 if sh else E, H)             # experts, the shared one's gate, rows without a use
+        self.w_gate_up, self.w_down = self.mat(E, 2 * I, H), self.mat(E, H, I)
+        self.shared = bool(sh)
+        if sh:
+            self.shared_gate_up, self.shared_down = self.mat(2 * sh["ff"], H), self.mat(H, sh["ff"])
+
+    def forward(self, x):
+        z = M.router_logits(x, self.router)
+        rt = OF.moe_route(z[:, :self.experts], self.top, norm=True, want_probs=False, want_host=False)
+        y = M.expert_linear(M.glu_silu(M.expert_linear(x.index_select(0, rt.token_of), self.w_gate_up, rt)), self.w_down, rt)
+        if not self.shared:
+            return M.ExpertSum(y, rt, None, rt.topw)
+        return M.ExpertSum(y, rt, M.linear(M.glu_silu(M.linear(x, self.shared_gate_up)), self.shared_down), rt.topw, z[:, self.experts])
+
+    @staticmethod
+    def checkpoint_names(p, m, h):
+        E, I = m["router"]["experts"], m["expert"]["ff"]
+        out = {p + "router": [(h + "router", (0, E), None)] + ([(h + "shared.sg", (E, E + 1), None)] if m.get("shared") else []),
+               p + "w_gate_up": [(h + f"e{e}.{n}", r, e) for e in range(E) for n, r in (("gate", (0, I)), ("up", (I, 2 * I)))],
+               p + "w_down": [(h + f"e{e}.down", None, e) for e in range(E)]}
+        if m.get("shared"):
+            I = m["shared"]["ff"]
+            out[p + "shared_gate_up"] = [(h + "shared.gate", (0, I), None), (h + "shared.up", (I, 2 * I), None)]
+            out[p + "shared_down"] = [(h + "shared.down", None, None)]
+        return out
 
 
 @dataclass(frozen=True)
@@ -310,14 +581,17 @@ class Design:
     """What tells one kind of mixer stack from another, apart from the constants of its configuration."""
 
     name: str                    # ``architecture`` in config.json
+    mixers: dict                 # mixer kinds
     mlps: dict                   # feed-forward kinds
     layer_norms: tuple           # norms of a layer with a feed-forward ...
     layer_norms_bare: tuple      # ... and of one without
 
 
 DESIGNS = {
-    "kagolix": Design("Kagolix", {"dense": XieluMLP, "moe": RoutedMLP}, ("norm1", "norm1b", "norm2", "norm2b"), ("norm1", "norm1b")),
-    "vogilix": Design("Vogilix", {"dense": GeluMLP, "moe": InputWeightedMLP}, ("norm1", "norm2"), ("norm1",)),
+    "kagolix": Design("Kagolix", {"attention": ChunkAttention, "rglru": RGLRU, "mamba2": Mamba2}, {"dense": XieluMLP, "moe": RoutedMLP}, ("norm1", "norm1b", "norm2", "norm2b"),
+                      ("norm1", "norm1b")),
+    "vogilix": Design("Vogilix", {"latent_attention": LatentAttention}, {"dense": GeluMLP, "moe": InputWeightedMLP}, ("norm1", "norm2"), ("norm1",)),
+    "bumotar": Design("Bumotar", {"latent_attention": RotaryLatentAttention, "parallel": Parallel}, {"moe": SharedExpertMLP}, ("norm1", "norm2"), ("norm1",)),
 }
 
 
@@ -327,7 +601,7 @@ class MixerLayer(_Block):
         spec, H, design = cfg.mixer_layers[idx], cfg.hidden_size, DESIGNS[cfg.arch]
         for n in design.layer_norms if spec["mlp"] else design.layer_norms_bare:
             setattr(self, n, self.vec(H))
-        self.mix = MIXERS[spec["type"]](cfg, spec["mixer"], dtype, device)
+        self.mix = design.mixers[spec["type"]](cfg, spec["mixer"], dtype, device)
         self.mlp = design.mlps[spec["mlp"]["kind"]](cfg, spec["mlp"], dtype, device) if spec["mlp"] else None
         self.side_dim = cfg.token_side_dim
         if self.side_dim:
@@ -347,11 +621,13 @@ def checkpoint_plan(cfg: ModelConfig) -> dict:
         plan["embed_positions"] = [("pos", None, None)]
     if cfg.token_side_dim:
         plan["embed_side"] = [("side.embed", None, None)]
+    if cfg.layer_loop:
+        plan["loop_in"], plan["loop_step"] = [("loop.in", None, None)], [("loop.step", None, None)]
     for i, e in enumerate(cfg.mixer_layers):
         p, h = f"layers.{i}.", f"l{i}."
         for n in design.layer_norms if e["mlp"] else design.layer_norms_bare:
             plan[p + n] = [(h + n, None, None)]
-        plan.update(MIXERS[e["type"]].checkpoint_names(p + "mix.", e["mixer"], h + "mix."))
+        plan.update(design.mixers[e["type"]].checkpoint_names(p + "mix.", e["mixer"], h + "mix."))
         if e["mlp"]:
             plan.update(design.mlps[e["mlp"]["kind"]].checkpoint_names(p + "mlp.", e["mlp"], h + "mlp."))
         if cfg.token_side_dim:
@@ -377,6 +653,10 @@ class MixerStackLM(CausalLM):
             self.embed_positions = nn.Parameter(torch.empty(cfg.max_position_embeddings, cfg.hidden_size, **like))
         if cfg.token_side_dim:
             self.embed_side = nn.Parameter(torch.empty(cfg.vocab_size, cfg.num_layers * cfg.token_side_dim, **like))
+        if cfg.layer_loop:
+            self.loop_in = nn.Parameter(torch.empty(cfg.hidden_size, 2 * cfg.hidden_size, **like))
+            self.loop_step = nn.Parameter(torch.empty(cfg.layer_loop["times"], cfg.hidden_size, **dict(like, dtype=torch.float32)))
+        self._place_rotations()
         if self.embed_tokens.device.type == "meta":
             return
         super().reset_parameters(std, seed)
@@ -407,10 +687,38 @@ class MixerStackLM(CausalLM):
             elif leaf == "act":
                 p.fill_(0.5)
 
+    def _place_rotations(self):
+        """Every block that rotates gets its columns in the step's table of angles; equal rotations share theirs."""
+        at, freqs, mults = {}, [], []
+        for mod in self.modules():
+            if isinstance(mod, _Block) and mod.rotary is not None:
+                if mod.rotary not in at:
+                    at[mod.rotary] = len(freqs)
+                    freqs += mod.rotary[0]
+                    mults += [mod.rotary[1]] * len(mod.rotary[0])
+                mod.rot_at = at[mod.rotary]
+        if freqs:
+            dev = self.embed_tokens.device
+            self.register_buffer("rot_freq", torch.tensor([f / (2.0 * math.pi) for f in freqs], dtype=torch.float64, device=dev), persistent=False)
+            self.register_buffer("rot_mult", torch.tensor(mults, dtype=torch.float32, device=dev), persistent=False)
+
+    @property
+    def layer_runs(self) -> list[int]:
+        """The layers in the order in which they run; looped ones once per pass."""
+        n, loop = self.cfg.num_layers, self.cfg.layer_loop
+        if not loop:
+            return list(range(n))
+        a, z = loop["start"], loop["stop"]
+        return list(range(a)) + list(range(a, z)) * loop["times"] + list(range(z, n))
+
+    def cache_mixers(self) -> list:
+        """The mixer of every layer run: each has its own pages and states."""
+        return [self.layers[i].mix for i in self.layer_runs]
+
     def forward_step(self, b: M.RaggedBatch, cache, on_layer=None) -> torch.Tensor:
         """Final normed hidden rows [R, H] of one step; reads and advances ``cache``. ``on_layer(i, resid)`` sees the
-        32-bit residual stream after everything a layer adds to it."""
-        return (self._step_post if self.cfg.norm_placement == "post" else self._step_sandwich)(b, cache, on_layer)
+        32-bit residual stream after everything the i-th layer run adds to it."""
+        return {"post": self._step_post, "pre": self._step_pre, "sandwich": self._step_sandwich}[self.cfg.norm_placement](b, cache, on_layer)
 
     def _step_sandwich(self, b, cache, on_layer):
         cfg, layers = self.cfg, self.layers
@@ -444,6 +752,40 @@ class MixerStackLM(CausalLM):
                 x = M.post_norm(sub(), w, resid, eps, mult, o, self.norm if end else None, off)
             if on_layer is not None:
                 on_layer(i, resid)
+        return x
+
+    def _step_pre(self, b, cache, on_layer):
+        cfg, layers, runs, dt = self.cfg, self.layers, self.layer_runs, self.dtype
+        eps, H = cfg.rms_norm_eps, cfg.hidden_size
+        b.rot = M.rotary_table(b.pos, self.rot_freq, self.rot_mult) if hasattr(self, "rot_freq") else None
+        loop = cfg.layer_loop
+        a, size, times = (loop["start"], loop["stop"] - loop["start"], loop["times"]) if loop else (0, 0, 0)
+        enters = {a + t * size: t for t in range(times)}            # layer run -> pass that begins with it
+        if loop:
+            # what enters a pass: the stream beside the embedding
+            both = torch.empty(b.n_rows, 2 * H, device=self.embed_tokens.device, dtype=dt)
+            resid, x = M.embed_rows(b.tokens, self.embed_tokens, b.pos, None, both[:, H:], both[:, :H])
+        else:
+            resid, x = M.embed_rows(b.tokens, self.embed_tokens, b.pos)
+        if 0 not in enters:
+            x = M.residual_norm(None, resid, layers[runs[0]].norm1, eps, dt)
+        for r, i in enumerate(runs):
+            layer = layers[i]
+            if r in enters:
+                resid = M.linear(both, self.loop_in, fp32_out=True).contiguous()
+                x = M.residual_norm(None, resid, layer.norm1, eps, dt, vec=self.loop_step[enters[r]])
+            h = layer.mix(x, b, cache.layers[r])
+            if layer.mlp is not None:
+                h = layer.mlp(M.residual_norm(h, resid, layer.norm2, eps, dt))
+            # the stream and what comes next: a pass's entrance, the next layer's norm, or the final norm (with the logits' factor)
+            if r + 1 in enters:
+                M.residual_norm(h, resid, None, eps, dt, out=both[:, :H])
+            elif r + 1 < len(runs):
+                x = M.residual_norm(h, resid, layers[runs[r + 1]].norm1, eps, dt)
+            else:
+                x = M.residual_norm(h, resid, self.norm, eps, dt, mult=cfg.logit_scale)
+            if on_layer is not None:
+                on_layer(r, resid)
         return x
 
     def logits(self, hidden: torch.Tensor) -> torch.Tensor:

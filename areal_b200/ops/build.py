@@ -24,7 +24,8 @@ BUILD = HERE / "build"
 LIB = HERE / "libab2_kernels.so"
 # the kernels that serve a mixer stack, linked alone: what a fresh checkout compiles before its first trace
 STEP_LIB = HERE / "libab2_step.so"
-STEP_SOURCES = ("runtime", "gemm", "gemm2sm", "gemm_grouped", "router", "infer", "mixer_attention", "mixer_latent", "mixer_ops", "mixer_scan", "mixer_ssd")
+STEP_SOURCES = ("runtime", "gemm", "gemm2sm", "gemm_grouped", "router", "infer", "mixer_attention", "mixer_latent", "mixer_ops",
+                "mixer_retention", "mixer_rotary", "mixer_scan", "mixer_ssd")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",

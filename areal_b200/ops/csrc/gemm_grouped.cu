@@ -39,7 +39,7 @@ template <int BN, bool B_MN>
 __global__ void __launch_bounds__(192, 1)
 gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
                     __nv_bfloat16* __restrict__ Cptr, const int4* __restrict__ tiles, int num_tiles, int N,
-                    int K, int ldc, int* err, const int* __restrict__ num_rt_dev, int nblk, int head_rows) {
+                    int K, int ldc, int* err, const int* __restrict__ num_rt_dev, int nblk, int head_rows, int head_stride) {
   constexpr bool A_MN = false;
   // Row-tile mode (nblk > 0): `tiles` lists 128-row tiles only, written by the routing kernel together with
   // their number; output tile i covers row tile i / nblk and n-block i % nblk, and the grid was sized for
@@ -113,7 +113,7 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
       for (int tile = blockIdx.x; tile < num_tiles && ok; tile += gridDim.x) {
         const int4 ti = tile_info(tile);
         const int expert = ti.x, m0 = ti.y, n0 = ti.w * BN;
-        const int a0 = head_rows > 0 ? expert * K : 0;      // columns past the head's own meet zero-filled rows of B
+        const int a0 = head_rows > 0 ? expert * head_stride : 0;      // columns past the head's own meet zero-filled rows of B
         for (int kb = 0; kb < num_kb; ++kb) {
           if (!mbar_wait(empty_bar(stage), phase ^ 1u, err, ERR_WAIT_EMPTY)) { ok = false; break; }
           const uint32_t sA = smem_base + stage * Cfg::STAGE_BYTES;
@@ -234,10 +234,11 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
 
 template <int BN, bool B_MN>
 static int launch_grouped(const void* A, const void* B, void* C, const void* tiles, int num_tiles, int R, int N, int K, int E,
-                          int lda, int ldc, cudaStream_t stream, const int* num_rt_dev = nullptr, int nblk = 0, bool heads = false) {
+                          int lda, int ldc, cudaStream_t stream, const int* num_rt_dev = nullptr, int nblk = 0, int head_stride = 0) {
+  const bool heads = head_stride > 0;
   using Cfg = GemmCfg<BN>;
   CUtensorMap tmA, tmB;
-  int rc = ab2host::encode_tmap_2d(&tmA, A, 2, heads ? (uint64_t)K * E : (uint64_t)K, (uint64_t)R, (uint64_t)lda * 2, BK, BM, true, 0);
+  int rc = ab2host::encode_tmap_2d(&tmA, A, 2, heads ? (uint64_t)head_stride * (E - 1) + K : (uint64_t)K, (uint64_t)R, (uint64_t)lda * 2, BK, BM, true, 0);
   if (rc) return 100 + rc;
   if (!B_MN)  // [E, N, K]
     rc = ab2host::encode_tmap_3d(&tmB, B, 2, (uint64_t)K, (uint64_t)N, (uint64_t)E, (uint64_t)K * 2, (uint64_t)N * K * 2, BK, BN, 1, true, 0);
@@ -253,7 +254,7 @@ static int launch_grouped(const void* A, const void* B, void* C, const void* til
   int* err = ab2host::error_flag();
   if (!err) return 301;
   launch_pdl(kern, dim3(grid), dim3(192), (size_t)Cfg::SMEM_BYTES, stream, tmA, tmB, reinterpret_cast<__nv_bfloat16*>(C),
-             reinterpret_cast<const int4*>(tiles), num_tiles, N, K, ldc, err, num_rt_dev, nblk, heads ? R : 0);
+             reinterpret_cast<const int4*>(tiles), num_tiles, N, K, ldc, err, num_rt_dev, nblk, heads ? R : 0, head_stride);
   return cudaGetLastError() == cudaSuccess ? 0 : 302;
 }
 
@@ -296,19 +297,20 @@ int ab2_gemm_grouped_rt(const void* A, const void* B, void* C, const void* row_t
               : launch_grouped<128, false>(A, B, C, row_tiles, (int)max_tiles, R, N, K, E, lda, ldc, s, nrt, nblk);
 }
 
-// C[r, h, :] = B[h] A[r, h, :]: A [R, E, K], C [R, E, N], B [E, N, K] (b_mn = 0) or [E, K, N] (b_mn = 1), all bf16 and contiguous.
-int ab2_gemm_heads(const void* A, const void* B, void* C, int R, int E, int N, int K, int b_mn, int bn, void* stream) {
+// C[r, h, :] = B[h] A[r, h, :]: A [R, E, K] with lda elements from row to row and hsa from head to head, C [R, E, N], B [E, N, K]
+// (b_mn = 0) or [E, K, N] (b_mn = 1), all bf16, C and B contiguous.
+int ab2_gemm_heads(const void* A, const void* B, void* C, int R, int E, int N, int K, int lda, int hsa, int b_mn, int bn, void* stream) {
   using namespace ab2;
   if (R <= 0 || E <= 0) return 0;
-  if ((K & 7) || (N & 7)) return 10;
+  if ((K & 7) || (N & 7) || (lda & 7) || (hsa & 7) || hsa < K || (long long)hsa * (E - 1) + K > lda) return 10;
   if (bn != 128 && bn != 256) return 12;
   const int nblk = (N + bn - 1) / bn;
   const long long tiles = (long long)E * ((R + BM - 1) / BM) * nblk, cols = (long long)E * (K > N ? K : N);
   if (tiles > 0x7fffffffLL || cols > 0x7fffffffLL) return 13;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  if (bn == 256) return b_mn ? launch_grouped<256, true>(A, B, C, nullptr, (int)tiles, R, N, K, E, E * K, E * N, s, nullptr, nblk, true)
-                             : launch_grouped<256, false>(A, B, C, nullptr, (int)tiles, R, N, K, E, E * K, E * N, s, nullptr, nblk, true);
-  return b_mn ? launch_grouped<128, true>(A, B, C, nullptr, (int)tiles, R, N, K, E, E * K, E * N, s, nullptr, nblk, true)
-              : launch_grouped<128, false>(A, B, C, nullptr, (int)tiles, R, N, K, E, E * K, E * N, s, nullptr, nblk, true);
+  if (bn == 256) return b_mn ? launch_grouped<256, true>(A, B, C, nullptr, (int)tiles, R, N, K, E, lda, E * N, s, nullptr, nblk, hsa)
+                             : launch_grouped<256, false>(A, B, C, nullptr, (int)tiles, R, N, K, E, lda, E * N, s, nullptr, nblk, hsa);
+  return b_mn ? launch_grouped<128, true>(A, B, C, nullptr, (int)tiles, R, N, K, E, lda, E * N, s, nullptr, nblk, hsa)
+              : launch_grouped<128, false>(A, B, C, nullptr, (int)tiles, R, N, K, E, lda, E * N, s, nullptr, nblk, hsa);
 }
 }

@@ -2,6 +2,9 @@
 // bias r1[h] * ln(1 + r2[h] * distance) taken off (both optional), and only the earlier keys of the query's own chunk of
 // positions visible (chunks counted from position 0 of the sequence), or those of a sliding window (the query's position
 // and the window - 1 before it), or all of them (chunk = window = 0). Query / key and value sizes may differ.
+// Optional, all in AttnExtra: a second part of queries and keys that all heads share a key of (rotated parts beside latents),
+// a sink (a score that only enters the denominator), a sigmoid gate on the output (per head or per channel), a factor of the
+// output, row strides.
 //
 //   chunk_attn_plain_kernel   any sizes, bf16 or 32-bit: a warp per (row, head)
 //   chunk_decode_kernel       single-token rows, bf16: a cluster of CTAs splits a request's chunk, mma.sync products,
@@ -23,6 +26,15 @@ struct ChunkArgs {
   float scale, softcap;
   const float *r1, *r2;
   int chunk, window;          // at most one of them set
+  AttnExtra x;
+
+  __host__ void defaults() {  // strides that were left open: contiguous
+    if (!x.ldq) { x.ldq = (long long)Hq * D; x.hsq = D; }
+    if (!x.ldo) x.ldo = (long long)Hq * Dv;
+    if (!x.ldk) x.ldk = (long long)Hkv * D;
+    if (!x.ldv) x.ldv = (long long)Hkv * Dv;
+    if (!x.q2) x.D2 = 0;
+  }
 
   // first position that a query at i sees (never decreases with i)
   __device__ __forceinline__ int first_key(int i) const {
@@ -62,20 +74,23 @@ chunk_attn_plain_kernel(const T* __restrict__ q, const int* __restrict__ pos, co
   if (h >= p.Hq) return;
   // values wider than one CTA's registers: blockIdx.z takes its stretch of them
   const int v0 = blockIdx.z * PLAIN_MAX_DV, nv = min(p.Dv - v0, PLAIN_MAX_DV);
-  T* o = out + ((size_t)row * p.Hq + h) * p.Dv + v0;
+  T* o = out + row * p.x.ldo + (size_t)h * p.Dv + v0;
   if (slots[row] < 0) {
     for (int d = lane; d < nv; d += 32) stf(o + d, 0.f);
     return;
   }
-  float* sq = sq_all + warp * p.D;
-  for (int d = lane; d < p.D; d += 32) sq[d] = ldf(q + ((size_t)row * p.Hq + h) * p.D + d) * p.scale;
+  float* sq = sq_all + warp * (p.D + p.x.D2);
+  float* sq2 = sq + p.D;
+  for (int d = lane; d < p.D; d += 32) sq[d] = ldf(q + row * p.x.ldq + h * p.x.hsq + d) * p.scale;
+  for (int d = lane; d < p.x.D2; d += 32) sq2[d] = ldf((const T*)p.x.q2 + row * p.x.ldq2 + h * p.x.hsq2 + d) * p.scale;
   __syncwarp();
+  const bool vec = p.D % 4 == 0 && p.x.ldk % 4 == 0;
   const int e = row_entry[row], i = pos[row], kvh = h / (p.Hq / p.Hkv);
   const int lo = p.first_key(i);
   const int* pt = p.pages + (size_t)e * p.max_pages;
   const int base = p.page_base[e];
   const float r1 = p.r1 ? p.r1[h] : 0.f, r2 = p.r1 ? p.r2[h] : 0.f;
-  float m = -INFINITY, l = 0.f, acc[PLAIN_MAX_DV / 32];
+  float m = p.x.sink_of(h), l = m > -INFINITY ? 1.f : 0.f, acc[PLAIN_MAX_DV / 32];
 #pragma unroll
   for (int k = 0; k < PLAIN_MAX_DV / 32; ++k) acc[k] = 0.f;
   for (int j0 = lo; j0 <= i; j0 += 32) {
@@ -83,10 +98,10 @@ chunk_attn_plain_kernel(const T* __restrict__ q, const int* __restrict__ pos, co
     float s = -INFINITY;
     long long kv = 0;
     if (j <= i) {
-      kv = ((long long)pt[j / p.page_size - base] * p.page_size + j % p.page_size) * p.Hkv + kvh;
-      const T* kr = (const T*)p.kc + kv * p.D;
+      kv = (long long)pt[j / p.page_size - base] * p.page_size + j % p.page_size;
+      const T* kr = (const T*)p.kc + kv * p.x.ldk + (size_t)kvh * p.D;
       float dot = 0.f;
-      if (p.D % 4 == 0) {
+      if (vec) {
         for (int d = 0; d < p.D; d += 4) {
           float v[4];
           ldv<4>(kr + d, v);
@@ -95,6 +110,8 @@ chunk_attn_plain_kernel(const T* __restrict__ q, const int* __restrict__ pos, co
       } else {
         for (int d = 0; d < p.D; ++d) dot += ldf(kr + d) * sq[d];
       }
+      const T* k2 = (const T*)p.x.k2 + kv * p.x.ldk2;
+      for (int d = 0; d < p.x.D2; ++d) dot += ldf(k2 + d) * sq2[d];
       s = p.softcap > 0.f ? p.softcap * tanhf(dot / p.softcap) : dot;
       if (p.r1) s -= r1 * log1pf(r2 * (float)(i - j));
     }
@@ -108,7 +125,7 @@ chunk_attn_plain_kernel(const T* __restrict__ q, const int* __restrict__ pos, co
     const int nj = min(32, i - j0 + 1);
     for (int t = 0; t < nj; ++t) {
       const float wt = __shfl_sync(0xffffffffu, w, t);
-      const T* vr = (const T*)p.vc + __shfl_sync(0xffffffffu, kv, t) * p.Dv + v0;
+      const T* vr = (const T*)p.vc + __shfl_sync(0xffffffffu, kv, t) * p.x.ldv + (size_t)kvh * p.Dv + v0;
 #pragma unroll
       for (int k = 0; k < PLAIN_MAX_DV / 32; ++k) {
         if (k * 32 >= nv) break;
@@ -116,9 +133,14 @@ chunk_attn_plain_kernel(const T* __restrict__ q, const int* __restrict__ pos, co
       }
     }
   }
+  const T* gate = (const T*)p.x.gate;
+  const float f = p.x.out_scale * (gate && p.x.gate_per_head ? sigmoid_t<false>(ldf(gate + row * p.x.ldg + h)) : 1.f);
+  const bool each = gate && !p.x.gate_per_head;
 #pragma unroll
-  for (int k = 0; k < PLAIN_MAX_DV / 32; ++k)
-    if (k * 32 + lane < nv) stf(o + k * 32 + lane, acc[k] / l);
+  for (int k = 0; k < PLAIN_MAX_DV / 32; ++k) {
+    const int d = k * 32 + lane;
+    if (d < nv) stf(o + d, acc[k] / l * f * (each ? sigmoid_t<false>(ldf(gate + row * p.x.ldg + (size_t)h * p.Dv + v0 + d)) : 1.f));
+  }
 }
 
 // ------------------------------------------------------------------ single-token rows
@@ -188,14 +210,14 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
       const int idx = tid + k * 128, r = idx / (DK / 8), piece = idx % (DK / 8);
       const int row = s_row[(c & 1) * CD_KEYS + r];
       const bool ok = row >= 0 && piece * 8 < p.D;
-      cd_copy16(st + r * Cfg::KROW + piece * 16, (const __nv_bfloat16*)p.kc + (ok ? ((size_t)row * p.Hkv + h) * p.D + piece * 8 : 0), ok);
+      cd_copy16(st + r * Cfg::KROW + piece * 16, (const __nv_bfloat16*)p.kc + (ok ? row * p.x.ldk + h * p.D + piece * 8 : 0), ok);
     }
 #pragma unroll
     for (int k = 0; k < CD_KEYS * (DV / 8) / 128; ++k) {
       const int idx = tid + k * 128, r = idx / (DV / 8), piece = idx % (DV / 8);
       const int row = s_row[(c & 1) * CD_KEYS + r];
       const bool ok = row >= 0 && piece * 8 < p.Dv;
-      cd_copy16(st + CD_KEYS * Cfg::KROW + r * Cfg::VROW + piece * 16, (const __nv_bfloat16*)p.vc + (ok ? ((size_t)row * p.Hkv + h) * p.Dv + piece * 8 : 0), ok);
+      cd_copy16(st + CD_KEYS * Cfg::KROW + r * Cfg::VROW + piece * 16, (const __nv_bfloat16*)p.vc + (ok ? row * p.x.ldv + h * p.Dv + piece * 8 : 0), ok);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -206,7 +228,7 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
   for (int k = tid; k < 16 * (DK / 8); k += 128) {
     const int r = k / (DK / 8), piece = k % (DK / 8);
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (r < G && piece * 8 < p.D) v = *reinterpret_cast<const uint4*>(q + ((size_t)b * p.Hq + h * G + r) * p.D + piece * 8);
+    if (r < G && piece * 8 < p.D) v = *reinterpret_cast<const uint4*>(q + b * p.x.ldq + (h * G + r) * p.x.hsq + piece * 8);
     *reinterpret_cast<uint4*>(dsm + Cfg::Q_OFF + r * Cfg::KROW + piece * 16) = v;
   }
   __syncthreads();
@@ -309,11 +331,23 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
     ml[warp * 16 + gq] = l_run[0]; ml[warp * 16 + gq + 8] = l_run[1];
   }
   __syncthreads();
+  // the sink joins the denominator where the last sums are made; then gate and factor
+  auto store = [&](int g, int d, float ll, float oo) {
+    if (d >= p.Dv) return;
+    const int head = h * G + g;
+    float f = ll > 0.f ? p.x.out_scale / ll : 0.f;
+    const __nv_bfloat16* gate = (const __nv_bfloat16*)p.x.gate;
+    if (gate) f *= sigmoid_t<true>(__bfloat162float(gate[b * p.x.ldg + (p.x.gate_per_head ? head : head * p.Dv + d)]));
+    out[b * p.x.ldo + (size_t)head * p.Dv + d] = __float2bfloat16(oo * f);
+  };
   for (int k = tid; k < G * DV; k += 128) {
     const int g = k / DV, d = k - g * DV;
     float mx = -INFINITY, ll = 0.f, oo = 0.f;
+    if constexpr (SPL == 1) mx = p.x.sink_of(h * G + g) * 1.4426950408889634f;
+    const float sink = mx;
 #pragma unroll
     for (int w = 0; w < 4; ++w) mx = fmaxf(mx, mm[w * 16 + g]);
+    if (sink > -INFINITY) ll = fast_exp2(sink - mx);
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
       const float mw = mm[w * 16 + g];
@@ -322,7 +356,7 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
       oo += mo[(w * 16 + g) * DV + d] * wt;
     }
     if constexpr (SPL == 1) {
-      if (d < p.Dv) out[((size_t)b * p.Hq + h * G + g) * p.Dv + d] = __float2bfloat16(ll > 0.f ? oo / ll : 0.f);
+      store(g, d, ll, oo);
     } else {
       mo[g * DV + d] = oo;                             // only this thread reads (w, g, d) and writes (0, g, d)
       if (d == 0) { s_ml[0][g] = mx; s_ml[1][g] = ll; }
@@ -333,9 +367,11 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
     cl.sync();
     for (int k = spl * 128 + tid; k < G * DV; k += 128 * SPL) {
       const int g = k / DV, d = k - g * DV;
-      float mx = -INFINITY, ll = 0.f, oo = 0.f;
+      const float sink = p.x.sink_of(h * G + g) * 1.4426950408889634f;
+      float mx = sink, ll = 0.f, oo = 0.f;
 #pragma unroll
       for (int c = 0; c < SPL; ++c) mx = fmaxf(mx, cl.map_shared_rank(&s_ml[0][0], c)[g]);
+      if (sink > -INFINITY) ll = fast_exp2(sink - mx);
 #pragma unroll
       for (int c = 0; c < SPL; ++c) {
         const float mc = cl.map_shared_rank(&s_ml[0][0], c)[g];
@@ -343,7 +379,7 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
         ll += cl.map_shared_rank(&s_ml[0][0], c)[16 + g] * wt;
         oo += cl.map_shared_rank(mo, c)[g * DV + d] * wt;
       }
-      if (d < p.Dv) out[((size_t)b * p.Hq + h * G + g) * p.Dv + d] = __float2bfloat16(ll > 0.f ? oo / ll : 0.f);
+      store(g, d, ll, oo);
     }
     cl.sync();                                         // nobody leaves while its shared memory is being read
   }
@@ -372,11 +408,13 @@ chunk_decode_split_kernel(const __nv_bfloat16* __restrict__ q, const int* __rest
 //   O += P V         tcgen05.mma, P from TMEM, V from shared memory
 // O is rescaled only when a row's maximum has grown by more than 2^8 since its reference was set.
 // 384 threads: warp 0 TMA, warp 1 MMA issue and TMEM, warps 4-7 and 8-11 the softmax of the two tiles.
-constexpr int CP_Q = 128, CP_K = 64, CP_ST = 4;
+constexpr int CP_Q = 128, CP_K = 64;
 
-template <int DK, int DV>
+// DR: 64 when queries and keys have a second part (up to 64 numbers, keys without heads), else 0; it is one more chunk of 64 columns.
+template <int DK, int DV, int DR>
 struct ChunkPrefillCfg {
-  static constexpr int QC = DK / 64, VC = DV / 64;           // 64-column chunks
+  static constexpr int QC = (DK + DR) / 64, VC = DV / 64;    // 64-column chunks
+  static constexpr int CP_ST = DK + DR > 128 ? 3 : 4;        // stages of K and V
   static constexpr int Q_BYTES = QC * CP_Q * 128;            // one tile
   static constexpr int K_BYTES = QC * CP_K * 128, V_BYTES = VC * CP_K * 128;
   static constexpr int BAR_OFF = 2 * Q_BYTES + CP_ST * (K_BYTES + V_BYTES);
@@ -384,12 +422,13 @@ struct ChunkPrefillCfg {
   static constexpr int SMEM = BIAS_OFF + 16 * 96 * 4 + 1024;
 };
 
-template <int DK, int DV, bool CAP, bool BIAS>
+template <int DK, int DV, int DR, bool CAP, bool BIAS>
 __global__ void __launch_bounds__(384, 1)
 chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
-                     const int* __restrict__ cu, const int* __restrict__ start, const int* __restrict__ tiles, __nv_bfloat16* __restrict__ out,
-                     const ChunkArgs p, int* err) {
-  using Cfg = ChunkPrefillCfg<DK, DV>;
+                     const __grid_constant__ CUtensorMap tmQ2, const __grid_constant__ CUtensorMap tmK2, const int* __restrict__ cu,
+                     const int* __restrict__ start, const int* __restrict__ tiles, __nv_bfloat16* __restrict__ out, const ChunkArgs p, int* err) {
+  using Cfg = ChunkPrefillCfg<DK, DV, DR>;
+  constexpr int CP_ST = Cfg::CP_ST, HC = DK / 64;             // chunks of the heads' own part
   const int e = tiles[2 * blockIdx.x], row0 = tiles[2 * blockIdx.x + 1], head = blockIdx.y;
   const int kvh = head / (p.Hq / p.Hkv);
   const int rows = min(2 * CP_Q, cu[e + 1] - row0);
@@ -457,7 +496,7 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       mbar_expect_tx(q_full, ntile * Cfg::Q_BYTES);
       for (int t = 0; t < ntile; ++t)
         for (int c = 0; c < Cfg::QC; ++c)
-          tma_load_3d(sQ + t * Cfg::Q_BYTES + c * CP_Q * 128, &tmQ, q_full, c * 64, head, row0 + t * CP_Q);
+          tma_load_3d(sQ + t * Cfg::Q_BYTES + c * CP_Q * 128, c < HC ? &tmQ : &tmQ2, q_full, c < HC ? c * 64 : 0, head, row0 + t * CP_Q);
       for (int j = 0; j < nmax; ++j) {
         const int s = j % CP_ST;
         const uint32_t ph = (uint32_t)(j / CP_ST) & 1u;
@@ -471,7 +510,8 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         mbar_expect_tx(k_full(s), Cfg::K_BYTES);
         for (int c = 0; c < Cfg::QC; ++c)
           for (int x = 0; x < per; ++x)
-            tma_load_3d(sK + s * Cfg::K_BYTES + c * CP_K * 128 + x * box * 128, &tmK, k_full(s), c * 64, kvh, crow[x]);
+            tma_load_3d(sK + s * Cfg::K_BYTES + c * CP_K * 128 + x * box * 128, c < HC ? &tmK : &tmK2, k_full(s), c < HC ? c * 64 : 0, c < HC ? kvh : 0,
+                        crow[x]);
         if (!mbar_wait(v_empty(s), ph ^ 1u, err, ERR_WAIT_EMPTY)) { ok = false; break; }
         mbar_expect_tx(v_full(s), Cfg::V_BYTES);
         for (int c = 0; c < Cfg::VC; ++c)
@@ -491,7 +531,8 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       auto issue_s = [&](int t, int j) {
         const int s = j % CP_ST;
 #pragma unroll
-        for (int kk = 0; kk < DK / 16; ++kk) {
+        for (int kk = 0; kk < (DK + DR) / 16; ++kk) {
+          if (DR && kk >= DK / 16 && (kk - DK / 16) * 16 >= p.x.D2) break;     // only zeros from here on
           const uint64_t ad = make_smem_desc_sw128(sQ + t * Cfg::Q_BYTES + (kk >> 2) * CP_Q * 128, 16, 1024) + (uint64_t)((kk & 3) * 2);
           const uint64_t bd = make_smem_desc_sw128(sK + s * Cfg::K_BYTES + (kk >> 2) * CP_K * 128, 16, 1024) + (uint64_t)((kk & 3) * 2);
           umma_f16(s_col(t, j & 1), ad, bd, idesc_s, kk != 0 ? 1u : 0u);
@@ -547,7 +588,7 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     const int lo_last = p.first_key(first + max(last, 0));
     const ScoreConsts sc = score_consts(p.scale, p.softcap);
     const float r1 = p.r1 ? p.r1[head] : 0.f, r2 = p.r1 ? p.r2[head] : 0.f;
-    float m_run = -INFINITY, l_run = 0.f;
+    float m_run = p.x.sink_of(head) * 1.4426950408889634f, l_run = m_run > -INFINITY ? 1.f : 0.f;
     bool ok = true;
     for (int j = 0; j < nbt && ok; ++j) {
       const int kb = k0 + j * CP_K;
@@ -615,8 +656,12 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     if (ok && nbt > 0) ok = __all_sync(0xffffffffu, mbar_wait(o_done(t), (uint32_t)(nbt - 1) & 1u, err, ERR_WAIT_MISC));
     if (ok && nbt > 0) {
       tc_fence_after();
-      const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-      __nv_bfloat16* dst = out + ((size_t)(row0 + t * CP_Q + row) * p.Hq + head) * p.Dv;
+      float inv = l_run > 0.f ? p.x.out_scale / l_run : 0.f;
+      const size_t grow_ = row0 + t * CP_Q + min(row, max(last, 0));
+      __nv_bfloat16* dst = out + grow_ * p.x.ldo + (size_t)head * p.Dv;
+      const __nv_bfloat16* gate = (const __nv_bfloat16*)p.x.gate;
+      const __nv_bfloat16* each = gate && !p.x.gate_per_head ? gate + grow_ * p.x.ldg + (size_t)head * p.Dv : nullptr;
+      if (gate && p.x.gate_per_head) inv *= sigmoid_t<true>(__bfloat162float(gate[grow_ * p.x.ldg + head]));
 #pragma unroll 1
       for (int c = 0; c < DV / 32; ++c) {
         uint32_t r[32];
@@ -625,12 +670,17 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         if (row <= last) {
 #pragma unroll
           for (int x = 0; x < 4; ++x)
-            if (c * 32 + x * 8 < p.Dv)
-              *reinterpret_cast<uint4*>(dst + c * 32 + x * 8) =
-                  make_uint4(pack_bf16(__uint_as_float(r[8 * x]) * inv, __uint_as_float(r[8 * x + 1]) * inv),
-                             pack_bf16(__uint_as_float(r[8 * x + 2]) * inv, __uint_as_float(r[8 * x + 3]) * inv),
-                             pack_bf16(__uint_as_float(r[8 * x + 4]) * inv, __uint_as_float(r[8 * x + 5]) * inv),
-                             pack_bf16(__uint_as_float(r[8 * x + 6]) * inv, __uint_as_float(r[8 * x + 7]) * inv));
+            if (c * 32 + x * 8 < p.Dv) {
+              float v[8], g[8];
+#pragma unroll
+              for (int k = 0; k < 8; ++k) v[k] = __uint_as_float(r[8 * x + k]) * inv;
+              if (each) {
+                ldv<8>(each + c * 32 + x * 8, g);
+#pragma unroll
+                for (int k = 0; k < 8; ++k) v[k] *= sigmoid_t<true>(g[k]);
+              }
+              stv<8>(dst + c * 32 + x * 8, v);
+            }
         }
       }
     }
@@ -643,7 +693,7 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   }
 }
 
-template <int DK, int DV, bool CAP, bool>
+template <int DK, int DV, int, bool CAP, bool>
 static int launch_decode(const void* q, const int* pos, const int* slots, void* out, int R, const ChunkArgs& a, cudaStream_t s) {
   constexpr int SMEM = ChunkDecodeCfg<DK, DV>::SMEM;
   static_assert(2 * ChunkDecodeCfg<DK, DV>::STAGE >= (4 * 16 * DV + 8 * 16) * 4, "the merge buffers alias the stage memory");
@@ -659,21 +709,28 @@ static int launch_decode(const void* q, const int* pos, const int* slots, void* 
   return go(chunk_decode_split_kernel<DK, DV, 8, CAP>, st8);
 }
 
-template <int DK, int DV, bool CAP, bool BIAS>
-static int launch_prefill(const void* q, const int* cu, const int* start, const int* tiles, int nt, void* out, int R, int cache_rows, long long ldk,
-                          long long ldv, const ChunkArgs& a, cudaStream_t s) {
-  using Cfg = ChunkPrefillCfg<DK, DV>;
-  CUtensorMap tq, tk, tv;
+template <int DK, int DV, int DR, bool CAP, bool BIAS>
+static int launch_prefill(const void* q, const int* cu, const int* start, const int* tiles, int nt, void* out, int R, int cache_rows, const ChunkArgs& a,
+                          cudaStream_t s) {
+  using Cfg = ChunkPrefillCfg<DK, DV, DR>;
+  CUtensorMap tq, tk, tv, tq2, tk2;
   const uint32_t box = a.page_size < CP_K ? a.page_size : CP_K;
-  if (ab2host::encode_tmap_3d(&tq, q, 2, a.D, a.Hq, R, (uint64_t)a.D * 2, (uint64_t)a.Hq * a.D * 2, 64, 1, CP_Q, true, 0)) return 100;
-  if (ab2host::encode_tmap_3d(&tk, a.kc, 2, a.D, a.Hkv, cache_rows, (uint64_t)a.D * 2, (uint64_t)ldk * 2, 64, 1, box, true, 0)) return 101;
-  if (ab2host::encode_tmap_3d(&tv, a.vc, 2, a.Dv, a.Hkv, cache_rows, (uint64_t)a.Dv * 2, (uint64_t)ldv * 2, 64, 1, box, true, 0)) return 102;
-  auto kern = chunk_prefill_kernel<DK, DV, CAP, BIAS>;
+  auto map = [&](CUtensorMap* m, const void* base, int cols, int heads, int rows, long long head_stride, long long row_stride, uint32_t box_rows) {
+    return ab2host::encode_tmap_3d(m, base, 2, cols, heads, rows, (uint64_t)head_stride * 2, (uint64_t)row_stride * 2, 64, 1, box_rows, true, 0);
+  };
+  if (map(&tq, q, a.D, a.Hq, R, a.x.hsq, a.x.ldq, CP_Q)) return 100;
+  if (map(&tk, a.kc, a.D, a.Hkv, cache_rows, a.D, a.x.ldk, box)) return 101;
+  if (map(&tv, a.vc, a.Dv, a.Hkv, cache_rows, a.Dv, a.x.ldv, box)) return 102;
+  tq2 = tq;
+  tk2 = tk;
+  if (DR && map(&tq2, a.x.q2, a.x.D2, a.Hq, R, a.x.hsq2, a.x.ldq2, CP_Q)) return 103;
+  if (DR && map(&tk2, a.x.k2, a.x.D2, 1, cache_rows, a.x.ldk2, a.x.ldk2, box)) return 104;
+  auto kern = chunk_prefill_kernel<DK, DV, DR, CAP, BIAS>;
   static ab2host::DevState st;
   if (ab2host::prepare_launch(kern, Cfg::SMEM, st, nullptr)) return 300;
   int* err = ab2host::error_flag();
   if (!err) return 301;
-  kern<<<dim3(nt, a.Hq), 384, Cfg::SMEM, s>>>(tq, tk, tv, cu, start, tiles, (__nv_bfloat16*)out, a, err);
+  kern<<<dim3(nt, a.Hq), 384, Cfg::SMEM, s>>>(tq, tk, tv, tq2, tk2, cu, start, tiles, (__nv_bfloat16*)out, a, err);
   return cudaGetLastError() == cudaSuccess ? 0 : 302;
 }
 
@@ -683,51 +740,65 @@ extern "C" {
 using namespace ab2;
 
 // q [R, Hq, D], out [R, Hq, Dv], one row per (pos, slot, entry); slot < 0: padding row (zeros). Cache: kc [rows, Hkv, D],
-// vc [rows, Hkv, Dv]; pages [entries, max_pages] from page number page_base[entry] on. r1 / r2 [Hq] or null. dt 0 bf16, 1 fp32.
+// vc [rows, Hkv, Dv]; pages [entries, max_pages] from page number page_base[entry] on. r1 / r2 [Hq] or null. x: null, or what
+// AttnExtra says. dt 0 bf16, 1 fp32.
 int ab2_chunk_attn_plain(const void* q, const int* pos, const int* slots, const int* row_entry, void* out, int R, const void* kc, const void* vc,
                          const int* pages, const int* page_base, int max_pages, int page_size, int Hq, int Hkv, int D, int Dv, float scale,
-                         float softcap, const float* r1, const float* r2, int chunk, int window, int dt, void* stream) {
+                         float softcap, const float* r1, const float* r2, int chunk, int window, const AttnExtra* x, int dt, void* stream) {
   if (R <= 0) return 0;
-  if (Hq % Hkv || Dv > 65535 || 16 * D > 48 * 1024) return 10;
-  ChunkArgs a{kc, vc, pages, page_base, max_pages, page_size, Hq, Hkv, D, Dv, scale, softcap, r1, r2, chunk, window};
+  ChunkArgs a{kc, vc, pages, page_base, max_pages, page_size, Hq, Hkv, D, Dv, scale, softcap, r1, r2, chunk, window, x ? *x : AttnExtra()};
+  a.defaults();
+  const int smem = 16 * (D + a.x.D2);
+  if (Hq % Hkv || Dv > 65535 || smem > 48 * 1024) return 10;
   const dim3 grid(R, (Hq + 3) / 4, (Dv + PLAIN_MAX_DV - 1) / PLAIN_MAX_DV);
   if (dt == 0)
-    chunk_attn_plain_kernel<__nv_bfloat16><<<grid, 128, 16 * D, (cudaStream_t)stream>>>((const __nv_bfloat16*)q, pos, slots, row_entry,
-                                                                                       (__nv_bfloat16*)out, a);
+    chunk_attn_plain_kernel<__nv_bfloat16><<<grid, 128, smem, (cudaStream_t)stream>>>((const __nv_bfloat16*)q, pos, slots, row_entry,
+                                                                                     (__nv_bfloat16*)out, a);
   else
-    chunk_attn_plain_kernel<float><<<grid, 128, 16 * D, (cudaStream_t)stream>>>((const float*)q, pos, slots, row_entry, (float*)out, a);
+    chunk_attn_plain_kernel<float><<<grid, 128, smem, (cudaStream_t)stream>>>((const float*)q, pos, slots, row_entry, (float*)out, a);
   return cudaGetLastError() == cudaSuccess ? 0 : 1;
 }
 
-#define AB2_BY_SIZE2(FN, CAP, BIAS, ...)                                                                           \
-  if (D <= 64) return Dv <= 64 ? FN<64, 64, CAP, BIAS>(__VA_ARGS__) : FN<64, 128, CAP, BIAS>(__VA_ARGS__);          \
-  return Dv <= 64 ? FN<128, 64, CAP, BIAS>(__VA_ARGS__) : FN<128, 128, CAP, BIAS>(__VA_ARGS__)
-#define AB2_BY_SIZE(FN, ...)                                                                                       \
-  if (a.softcap > 0.f) { AB2_BY_SIZE2(FN, true, true, __VA_ARGS__); }                                              \
-  if (a.r1 != nullptr) { AB2_BY_SIZE2(FN, false, true, __VA_ARGS__); }                                             \
-  AB2_BY_SIZE2(FN, false, false, __VA_ARGS__)
+#define AB2_BY_SIZE2(FN, DR, CAP, BIAS, ...)                                                                               \
+  if (D <= 64) return Dv <= 64 ? FN<64, 64, DR, CAP, BIAS>(__VA_ARGS__) : FN<64, 128, DR, CAP, BIAS>(__VA_ARGS__);          \
+  return Dv <= 64 ? FN<128, 64, DR, CAP, BIAS>(__VA_ARGS__) : FN<128, 128, DR, CAP, BIAS>(__VA_ARGS__)
 
-// Row r is the only row of entry r. bf16; D, Dv multiples of 8 up to 128, at most 16 query heads per key head.
+// Row r is the only row of entry r. bf16; D, Dv multiples of 8 up to 128, at most 16 query heads per key head; no second part.
 int ab2_chunk_decode(const void* q, const int* pos, const int* slots, void* out, int R, const void* kc, const void* vc, const int* pages,
                      const int* page_base, int max_pages, int page_size, int Hq, int Hkv, int D, int Dv, float scale, float softcap,
-                     const float* r1, const float* r2, int chunk, int window, void* stream) {
+                     const float* r1, const float* r2, int chunk, int window, const AttnExtra* x, void* stream) {
   if (R <= 0) return 0;
-  if (Hq % Hkv || Hq / Hkv > 16 || (D & 7) || (Dv & 7) || D > 128 || Dv > 128 || Hkv > 65535) return 10;
-  if (!aligned_to(q, 16) || !aligned_to(kc, 16) || !aligned_to(vc, 16)) return 11;
-  ChunkArgs a{kc, vc, pages, page_base, max_pages, page_size, Hq, Hkv, D, Dv, scale, softcap, r1, r2, chunk, window};
-  AB2_BY_SIZE(launch_decode, q, pos, slots, out, R, a, (cudaStream_t)stream);
+  ChunkArgs a{kc, vc, pages, page_base, max_pages, page_size, Hq, Hkv, D, Dv, scale, softcap, r1, r2, chunk, window, x ? *x : AttnExtra()};
+  a.defaults();
+  if (Hq % Hkv || Hq / Hkv > 16 || (D & 7) || (Dv & 7) || D > 128 || Dv > 128 || Hkv > 65535 || a.x.D2) return 10;
+  if (!aligned_to(q, 16) || !aligned_to(kc, 16) || !aligned_to(vc, 16) || ((a.x.ldq | a.x.hsq | a.x.ldk | a.x.ldv) & 7)) return 11;
+  cudaStream_t s = (cudaStream_t)stream;
+  if (softcap > 0.f) { AB2_BY_SIZE2(launch_decode, 0, true, true, q, pos, slots, out, R, a, s); }
+  AB2_BY_SIZE2(launch_decode, 0, false, true, q, pos, slots, out, R, a, s);
 }
 
-// tiles [nt, 2] = (entry, first row); q / out hold all R rows of the step. bf16; D, Dv multiples of 8 up to 128;
+// tiles [nt, 2] = (entry, first row); q / out hold all R rows of the step. bf16; D, Dv multiples of 8 up to 128; a second part up to 64;
 // page_size 16, 32 or a multiple of 64. ldk / ldv: elements from one cache row to the next.
 int ab2_chunk_prefill(const void* q, const int* cu, const int* start, const int* tiles, int nt, void* out, int R, int cache_rows, long long ldk,
                       long long ldv, const void* kc, const void* vc, const int* pages, const int* page_base, int max_pages, int page_size, int Hq, int Hkv, int D, int Dv,
-                      float scale, float softcap, const float* r1, const float* r2, int chunk, int window, void* stream) {
+                      float scale, float softcap, const float* r1, const float* r2, int chunk, int window, const AttnExtra* x, void* stream) {
   if (nt <= 0) return 0;
-  if (Hq % Hkv || (D & 7) || (Dv & 7) || D > 128 || Dv > 128 || Hq > 65535 || (ldk & 7) || (ldv & 7)) return 10;
+  ChunkArgs a{kc, vc, pages, page_base, max_pages, page_size, Hq, Hkv, D, Dv, scale, softcap, r1, r2, chunk, window, x ? *x : AttnExtra()};
+  a.x.ldk = ldk;
+  a.x.ldv = ldv;
+  a.defaults();
+  const AttnExtra& e = a.x;
+  if (Hq % Hkv || (D & 7) || (Dv & 7) || D > 128 || Dv > 128 || Hq > 65535) return 10;
   if (!aligned_to(q, 16) || !aligned_to(kc, 16) || !aligned_to(vc, 16) || !aligned_to(out, 16)) return 11;
   if (!(page_size == 16 || page_size == 32 || (page_size > 0 && page_size % 64 == 0))) return 12;
-  ChunkArgs a{kc, vc, pages, page_base, max_pages, page_size, Hq, Hkv, D, Dv, scale, softcap, r1, r2, chunk, window};
-  AB2_BY_SIZE(launch_prefill, q, cu, start, tiles, nt, out, R, cache_rows, ldk, ldv, a, (cudaStream_t)stream);
+  if ((e.ldk | e.ldv | e.ldq | e.hsq | e.ldo) & 7) return 13;
+  if (e.gate && !e.gate_per_head && (!aligned_to(e.gate, 16) || (e.ldg & 7))) return 14;
+  if (e.D2 && ((e.D2 & 7) || e.D2 > 64 || ((e.ldq2 | e.hsq2 | e.ldk2) & 7) || !aligned_to(e.q2, 16) || !aligned_to(e.k2, 16) || softcap > 0.f || r1)) return 15;
+  cudaStream_t s = (cudaStream_t)stream;
+  if (e.D2) { AB2_BY_SIZE2(launch_prefill, 64, false, false, q, cu, start, tiles, nt, out, R, cache_rows, a, s); }
+  if (r1 && softcap > 0.f) { AB2_BY_SIZE2(launch_prefill, 0, true, true, q, cu, start, tiles, nt, out, R, cache_rows, a, s); }
+  if (softcap > 0.f) { AB2_BY_SIZE2(launch_prefill, 0, true, false, q, cu, start, tiles, nt, out, R, cache_rows, a, s); }
+  if (r1) { AB2_BY_SIZE2(launch_prefill, 0, false, true, q, cu, start, tiles, nt, out, R, cache_rows, a, s); }
+  AB2_BY_SIZE2(launch_prefill, 0, false, false, q, cu, start, tiles, nt, out, R, cache_rows, a, s);
 }
 }

@@ -91,6 +91,20 @@ __device__ __forceinline__ float gelu_tanh_t(float z) {
 }
 __device__ __forceinline__ float softplusf(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
+// What an attention may have beside queries, keys and values (host side: passed by address, null = none of it).
+struct AttnExtra {
+  const void *q2 = nullptr, *k2 = nullptr;   // second part of queries [R, Hq, D2] and keys [cache rows, D2]: its product is added before the scale
+  const void* gate = nullptr;                // output times sigmoid(gate): [R, Hq] (gate_per_head) or [R, Hq * Dv]
+  const float* sink = nullptr;               // per head: a score (scaled as it stands, never capped) that only enters the denominator
+  // elements between rows (and heads); 0: contiguous
+  long long ldq = 0, hsq = 0, ldq2 = 0, hsq2 = 0, ldk = 0, ldv = 0, ldk2 = 0, ldo = 0, ldg = 0;
+  int D2 = 0, gate_per_head = 0;
+  float sink_const = -INFINITY;              // sink of every head without `sink`; minus infinity: none
+  float out_scale = 1.f;
+
+  __device__ __forceinline__ float sink_of(int h) const { return sink ? sink[h] : sink_const; }
+};
+
 static inline bool aligned_to(const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) % bytes) == 0; }
 
 }  // namespace ab2

@@ -1,11 +1,13 @@
 // Attention of single rows over cached latents: one vector c of C numbers per token is key and value of every head (the heads'
 // own key part has been applied to the queries, their value part is applied to the result). A row sees its own position and
-// the window - 1 before it, or all earlier ones (window = 0).
+// the window - 1 before it, or all earlier ones (window = 0). Keys and queries may have a second, rotated part of up to 64 numbers
+// (stored behind the latent) that adds to the scores; a sink, a gate per head and a factor are those of AttnExtra.
 //
 // A CTA takes one row and 16 or 32 of its heads; the CTAs of a cluster share the row's keys in consecutive stretches. One warp
 // brings pieces of 32 latents from the cache pages by TMA (128-byte swizzle, 64 columns a box); each is used twice. Of the
 // eight others every one owns an eighth of the latent's columns, in both products (mma.sync, 32-bit sums):
-//   S = Q C^T     every warp its columns' share of all scores; the shares meet in shared memory in 32 bits
+//   S = Q C^T     every warp its columns' share of all scores; the shares meet in shared memory in 32 bits (of the second
+//                 part, every warp takes 16 columns of 16 keys)
 //   softmax       a few threads per head: sum of the shares, running maximum and sum, the weights to shared memory
 //   O += P C      every warp its columns
 // The output of piece c and the softmax of piece c + 1 run side by side. O is rescaled only when a head's maximum has
@@ -23,15 +25,17 @@ struct LatentArgs {
   int max_pages, page_shift, H, C;
   float scale;
   int window;
+  AttnExtra x;
   bool one_box;               // a piece is one box of the tensor map (32 rows, all chunks of 64 columns), else one per chunk (or two)
 };
 
-// DC: latent size rounded up to 128, 256 or 512 (missing columns are zero-filled); MT: 16-head tiles of a CTA
-template <int DC, int MT>
+// DC: latent size rounded up to 128, 256 or 512 (missing columns are zero-filled); MT: 16-head tiles of a CTA; DR: 64 with a
+// second part, else 0
+template <int DC, int MT, int DR>
 struct LatentCfg {
   static constexpr int CHUNK = LD_KEYS * 128;                      // 64 columns of a piece
-  static constexpr int STAGE = DC / 64 * CHUNK;
-  static constexpr int NS = DC == 512 ? 5 : 4;                     // stages: two in use, the others on their way
+  static constexpr int STAGE = (DC + DR) / 64 * CHUNK;
+  static constexpr int NS = (DC == 512 ? 5 : 4) - (DR ? 1 : 0);    // stages: two in use, the others on their way
   static constexpr int CTAS = DC == 512 ? 1 : 2;                   // per SM
   static constexpr int HEADS = 16 * MT;
   static constexpr int SROW = LD_KEYS + 8, PROW = LD_KEYS * 2 + 16;
@@ -56,12 +60,13 @@ __device__ __forceinline__ void ld_mma(float (&c)[4], const uint32_t (&a)[4], ui
 }
 __device__ __forceinline__ void ld_sync() { asm volatile("bar.sync 1, %0;" ::"n"(LD_WORK) : "memory"); }     // the working warps
 
-template <int DC, int MT>
-__global__ void __launch_bounds__(LD_THREADS, LatentCfg<DC, MT>::CTAS)
-latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat16* __restrict__ q, const int* __restrict__ pos,
+template <int DC, int MT, int DR>
+__global__ void __launch_bounds__(LD_THREADS, LatentCfg<DC, MT, DR>::CTAS)
+latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant__ CUtensorMap tmR, const __nv_bfloat16* __restrict__ q,
+                     const int* __restrict__ pos,
                      const int* __restrict__ slots, const int* __restrict__ row_entry, __nv_bfloat16* __restrict__ out, const LatentArgs p, int* err) {
   namespace cg = cooperative_groups;
-  using Cfg = LatentCfg<DC, MT>;
+  using Cfg = LatentCfg<DC, MT, DR>;
   constexpr int NS = Cfg::NS, HEADS = Cfg::HEADS;
   constexpr int WC = DC / LD_WARPS, KS = WC / 16, NT = WC / 8;      // columns of a warp; k-steps and tiles of 8 in them
   constexpr int TPR = LD_WORK / HEADS, KPT = LD_KEYS / TPR;         // softmax: threads per head, keys per thread
@@ -94,6 +99,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
   const int np = max(0, min(per, nblk - spl * per));
   float* s_s = reinterpret_cast<float*>(dsm + Cfg::S_OFF);
   float* s_alpha = reinterpret_cast<float*>(dsm + Cfg::A_OFF);
+  auto factor = [&](int row) {                                      // of the output of head h0 + row
+    const __nv_bfloat16* gate = (const __nv_bfloat16*)p.x.gate;
+    return gate ? p.x.out_scale * sigmoid_t<true>(__bfloat162float(gate[b * p.x.ldg + h0 + row])) : p.x.out_scale;
+  };
 
   if (warp == LD_WARPS) {
     if (elect_one() && np > 0) {
@@ -120,6 +129,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
             if (two) tma_load_3d(dst + k * Cfg::CHUNK + 16 * 128, &tmC, full(s), k * 64, row1, 0);
           }
         }
+        if constexpr (DR > 0) {
+          tma_load_3d(dst + DC / 64 * Cfg::CHUNK, &tmR, full(s), 0, row0, 0);
+          if (two) tma_load_3d(dst + DC / 64 * Cfg::CHUNK + 16 * 128, &tmR, full(s), 0, row1, 0);
+        }
         if (c + 1 < np) {
           row0 = row_at(t0 + (c + 1) * LD_KEYS);
           if (two) row1 = row_at(t0 + (c + 1) * LD_KEYS + 16);
@@ -144,6 +157,19 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
           const int row = m * 16 + gq + (x & 1) * 8, col = warp * WC + ks * 16 + (x >> 1) * 8 + 2 * tq;
           qa[m][ks][x] = row < heads && col < p.C ? *reinterpret_cast<const uint32_t*>(q + ((size_t)b * p.H + h0 + row) * p.C + col) : 0u;
         }
+    // of the second part: 16 columns and 16 keys of this warp; these keys come first in its accumulators
+    const int ks2 = warp & 3, keys2 = DR ? warp >> 2 : 0;
+    uint32_t qr[MT][4];
+    if constexpr (DR > 0) {
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+          const int row = m * 16 + gq + (x & 1) * 8, col = ks2 * 16 + (x >> 1) * 8 + 2 * tq;
+          qr[m][x] = row < heads && col < p.x.D2
+                         ? *reinterpret_cast<const uint32_t*>((const __nv_bfloat16*)p.x.q2 + b * p.x.ldq2 + (h0 + row) * p.x.hsq2 + col) : 0u;
+        }
+    }
     const float sc = p.scale * 1.4426950408889634f;                 // scores in base-2 units
     float o[MT][NT][4];
 #pragma unroll
@@ -167,7 +193,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
 #pragma unroll
         for (int n = 0; n < LD_KEYS / 8; n += 2) {
           uint32_t k[4];
-          ld_mat(a + n * 8 * 128, k);
+          ld_mat(a + (n ^ (2 * keys2)) * 8 * 128, k);
 #pragma unroll
           for (int m = 0; m < MT; ++m) {
             ld_mma(s[m][n], qa[m][ks], k[0], k[1]);
@@ -175,11 +201,20 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
           }
         }
       }
+      if constexpr (DR > 0) {
+        uint32_t k[4];
+        ld_mat(sm + stage * Cfg::STAGE + DC / 64 * Cfg::CHUNK + (keys2 * 16 + (mat >> 1) * 8 + r8) * 128 + (((ks2 * 2 + (mat & 1)) ^ r8) << 4), k);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          ld_mma(s[m][0], qr[m], k[0], k[1]);
+          ld_mma(s[m][1], qr[m], k[2], k[3]);
+        }
+      }
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
         for (int n = 0; n < LD_KEYS / 8; ++n) {
-          float* d = s_s + (warp * HEADS + m * 16 + gq) * Cfg::SROW + n * 8 + 2 * tq;
+          float* d = s_s + (warp * HEADS + m * 16 + gq) * Cfg::SROW + (n ^ (2 * keys2)) * 8 + 2 * tq;
           *reinterpret_cast<float2*>(d) = make_float2(s[m][n][0], s[m][n][1]);
           *reinterpret_cast<float2*>(d + 8 * Cfg::SROW) = make_float2(s[m][n][2], s[m][n][3]);
         }
@@ -297,7 +332,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
         for (int hh = 0; hh < 2; ++hh) {
           const int row = m * 16 + gq + 8 * hh;
           if (row >= heads) continue;
-          const float l = s_ml[1][row], inv = l > 0.f ? 1.f / l : 0.f;
+          const float sink = p.x.sink_of(h0 + row) * 1.4426950408889634f, mx = fmaxf(s_ml[0][row], sink);
+          const float w = s_ml[0][row] == -INFINITY ? 0.f : fast_exp2(s_ml[0][row] - mx);
+          const float l = s_ml[1][row] * w + (sink > -INFINITY ? fast_exp2(sink - mx) : 0.f), inv = l > 0.f ? w / l * factor(row) : 0.f;
           __nv_bfloat16* dst = out + ((size_t)b * p.H + h0 + row) * p.C;
 #pragma unroll
           for (int j = 0; j < NT; ++j) {
@@ -322,7 +359,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
   cg::cluster_group cl = cg::this_cluster();
   cl.sync();
   if (tid < heads) {
-    float m[8], l[8], mx = -INFINITY, ll = 0.f;
+    const float sink = p.x.sink_of(h0 + tid) * 1.4426950408889634f, f = factor(tid);
+    float m[8], l[8], mx = sink, ll = 0.f;
 #pragma unroll
     for (int c = 0; c < 8; ++c) {
       const float* ml = cl.map_shared_rank(&s_ml[0][0], min(c, nspl - 1));
@@ -330,13 +368,14 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
       l[c] = ml[32 + tid];
       mx = fmaxf(mx, m[c]);
     }
+    if (sink > -INFINITY) ll = fast_exp2(sink - mx);
 #pragma unroll
     for (int c = 0; c < 8; ++c) {
       m[c] = m[c] == -INFINITY ? 0.f : fast_exp2(m[c] - mx);
       ll += l[c] * m[c];
     }
 #pragma unroll
-    for (int c = 0; c < 8; ++c) s_wt[c][tid] = ll > 0.f ? m[c] / ll : 0.f;
+    for (int c = 0; c < 8; ++c) s_wt[c][tid] = ll > 0.f ? m[c] / ll * f : 0.f;
   }
   __syncthreads();
   const float* mo = reinterpret_cast<const float*>(dsm);
@@ -354,21 +393,25 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __nv_bfloat1
   cl.sync();                                                        // nobody leaves while its shared memory is being read
 }
 
-template <int DC, int MT>
+template <int DC, int MT, int DR>
 static int launch_latent(const void* q, const int* pos, const int* slots, const int* row_entry, void* out, int R, const void* cache, int cache_rows,
                          LatentArgs a, cudaStream_t s) {
-  using Cfg = LatentCfg<DC, MT>;
-  auto kern = latent_decode_kernel<DC, MT>;
+  using Cfg = LatentCfg<DC, MT, DR>;
+  auto kern = latent_decode_kernel<DC, MT, DR>;
   static ab2host::DevState st;
   int sms = 0;
   if (ab2host::prepare_launch(kern, Cfg::SMEM, st, &sms)) return 300;
-  CUtensorMap tc;
+  CUtensorMap tc, tr;
   a.one_box = a.C % 64 == 0 && a.page_shift > 4;
+  const uint64_t ld = (uint64_t)a.x.ldk * 2;
+  const uint32_t box = a.page_shift > 4 ? LD_KEYS : 16;
   if (a.one_box) {             // (column of the chunk, row, chunk)
-    if (ab2host::encode_tmap_3d(&tc, cache, 2, 64, cache_rows, a.C / 64, (uint64_t)a.C * 2, 128, 64, LD_KEYS, DC / 64, true, 0)) return 100;
-  } else if (ab2host::encode_tmap_3d(&tc, cache, 2, a.C, cache_rows, 1, (uint64_t)a.C * 2, (uint64_t)a.C * 2, 64, a.page_shift > 4 ? LD_KEYS : 16, 1, true, 0)) {
+    if (ab2host::encode_tmap_3d(&tc, cache, 2, 64, cache_rows, a.C / 64, ld, 128, 64, LD_KEYS, DC / 64, true, 0)) return 100;
+  } else if (ab2host::encode_tmap_3d(&tc, cache, 2, a.C, cache_rows, 1, ld, ld, 64, box, 1, true, 0)) {
     return 101;
   }
+  tr = tc;
+  if (DR && ab2host::encode_tmap_3d(&tr, a.x.k2, 2, a.x.D2, cache_rows, 1, (uint64_t)a.x.ldk2 * 2, (uint64_t)a.x.ldk2 * 2, 64, box, 1, true, 0)) return 102;
   int* err = ab2host::error_flag();
   if (!err) return 301;
   const int tiles = (a.H + Cfg::HEADS - 1) / Cfg::HEADS;
@@ -390,7 +433,7 @@ static int launch_latent(const void* q, const int* pos, const int* slots, const 
   attr[1].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr;
   cfg.numAttrs = ab2host::pdl_enabled() ? 2 : 1;
-  return cudaLaunchKernelEx(&cfg, kern, tc, (const __nv_bfloat16*)q, pos, slots, row_entry, (__nv_bfloat16*)out, a, err) == cudaSuccess ? 0 : 302;
+  return cudaLaunchKernelEx(&cfg, kern, tc, tr, (const __nv_bfloat16*)q, pos, slots, row_entry, (__nv_bfloat16*)out, a, err) == cudaSuccess ? 0 : 302;
 }
 
 }  // namespace ab2
@@ -399,15 +442,22 @@ extern "C" {
 using namespace ab2;
 
 // q, out [R, H, C] bf16; row r reads the pages of entry row_entry[r] up to position pos[r]; slots[r] < 0: padding row (zeros).
-// cache [cache_rows, C] bf16; pages [entries, max_pages] from page number page_base[entry] on. C a multiple of 8 up to 512,
-// page_size a power of two from 16 on.
+// cache [cache_rows, C] bf16 (x->ldk elements from row to row); pages [entries, max_pages] from page number page_base[entry] on. C a
+// multiple of 8 up to 512, page_size a power of two from 16 on. x: null, or second part (up to 64 numbers), sink, gate per head, factor.
 int ab2_latent_decode(const void* q, const int* pos, const int* slots, const int* row_entry, void* out, int R, const void* cache, int cache_rows,
-                      const int* pages, const int* page_base, int max_pages, int page_size, int H, int C, float scale, int window, void* stream) {
+                      const int* pages, const int* page_base, int max_pages, int page_size, int H, int C, float scale, int window, const AttnExtra* x,
+                      void* stream) {
   if (R <= 0) return 0;
   if ((C & 7) || C < 8 || C > 512 || H < 1 || H > 16 * 65535 || page_size < 16 || (page_size & (page_size - 1))) return 10;
   if (!aligned_to(q, 16) || !aligned_to(cache, 16) || !aligned_to(out, 16)) return 11;
-  LatentArgs a{pages, page_base, max_pages, __builtin_ctz(page_size), H, C, scale, window, false};
-#define AB2_LATENT(DC, MT) return launch_latent<DC, MT>(q, pos, slots, row_entry, out, R, cache, cache_rows, a, (cudaStream_t)stream)
+  LatentArgs a{pages, page_base, max_pages, __builtin_ctz(page_size), H, C, scale, window, x ? *x : AttnExtra(), false};
+  if (!a.x.ldk) a.x.ldk = C;
+  if (!a.x.q2) a.x.D2 = 0;
+  if ((a.x.ldk & 7) || (a.x.gate && !a.x.gate_per_head)) return 12;
+  if (a.x.D2 && ((a.x.D2 & 7) || a.x.D2 > 64 || ((a.x.ldq2 | a.x.hsq2 | a.x.ldk2) & 7) || !aligned_to(a.x.q2, 16) || !aligned_to(a.x.k2, 16))) return 13;
+#define AB2_LATENT(DC, MT)                                                                                                                    \
+  return a.x.D2 ? launch_latent<DC, MT, 64>(q, pos, slots, row_entry, out, R, cache, cache_rows, a, (cudaStream_t)stream)                     \
+                : launch_latent<DC, MT, 0>(q, pos, slots, row_entry, out, R, cache, cache_rows, a, (cudaStream_t)stream)
   if (H <= 16) {
     if (C <= 128) AB2_LATENT(128, 1);
     if (C <= 256) AB2_LATENT(256, 1);

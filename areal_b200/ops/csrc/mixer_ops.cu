@@ -1,5 +1,6 @@
 // Elementwise, norm, convolution and small-product kernels of mixer stacks (bf16 or fp32 activations, fp32 residual
-// stream, norm weights and states): grouped sandwich norms, norms behind a sublayer (fused with the expert sum), whole-
+// stream, norm weights and states): grouped sandwich norms, norms behind a sublayer and residual sums before a norm (both fused
+// with the expert sum), whole-
 // projection q / k norms fused with the cache append, causal convolutions with carried tails, xIELU, GELU, SiLU gate,
 // clamped gated units, token side gate, expert combine, capped logits, and a plain grouped product for 32-bit experts
 // and odd sizes.
@@ -215,10 +216,87 @@ __global__ void post_norm_kernel(const T* __restrict__ base, long long ldb, cons
   }
 }
 
-// resid = table[ids] (+ pos_table[pos]) in fp32, x the same in T.
+// ------------------------------------------------------------------ residual sum, then the next norm
+// h = base row (times sigmoid(logit), if there is one) + the token's k expert rows times their weights + vec, each optional;
+// resid += h; x = norm(resid) * w_next * mult, or resid when there is no norm. One CTA per row, the row in shared memory.
+template <typename T, int V, bool EXPERTS>
+__global__ void residual_norm_kernel(const T* __restrict__ base, long long ldb, const float* __restrict__ logit, long long ldl, const T* __restrict__ y,
+                                     const int* __restrict__ inv, const float* __restrict__ topw, int k, int n_rows, const float* __restrict__ vec,
+                                     float* __restrict__ resid, const float* __restrict__ w_next, float mult, T* __restrict__ x, long long ldx, int H,
+                                     float eps) {
+  extern __shared__ __align__(16) float srow[];       // [H] values, then the partial sums
+  pdl_wait();
+  pdl_trigger();
+  float* sums = srow + ((H + 3) & ~3);
+  const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  const float f = logit != nullptr ? sigmoid_t<false>(logit[row * ldl]) : 1.f;
+  float* rr = resid + (size_t)row * H;
+  T* xr = x + row * ldx;
+  float ss = 0.f;
+  for (int c = threadIdx.x * V; c < H; c += blockDim.x * V) {
+    float r[V];
+    ldv<V>(rr + c, r);
+    if (base != nullptr) {
+      float b[V];
+      ldv<V>(base + row * ldb + c, b);
+#pragma unroll
+      for (int e = 0; e < V; ++e) r[e] += f * b[e];
+    }
+    if (vec != nullptr) {
+      float b[V];
+      ldv<V>(vec + c, b);
+#pragma unroll
+      for (int e = 0; e < V; ++e) r[e] += b[e];
+    }
+    for (int s0 = 0; EXPERTS && s0 < k; s0 += 4) {     // four rows on their way at a time
+      float v[4][V], w[4];
+#pragma unroll
+      for (int s = 0; s < 4; ++s) {
+        const int i = s0 + s < k ? inv[(size_t)row * k + s0 + s] : -1;
+        w[s] = 0.f;
+        if (i >= 0 && i < n_rows) {
+          w[s] = topw[(size_t)row * k + s0 + s];
+          ldv<V>(y + (size_t)i * H + c, v[s]);
+        } else {
+          for (int e = 0; e < V; ++e) v[s][e] = 0.f;
+        }
+      }
+#pragma unroll
+      for (int s = 0; s < 4; ++s)
+#pragma unroll
+        for (int e = 0; e < V; ++e) r[e] += w[s] * v[s][e];
+    }
+    stv<V>(rr + c, r);
+    if (w_next == nullptr) {
+      stv<V>(xr + c, r);
+    } else {
+      stv<V>(srow + c, r);
+#pragma unroll
+      for (int e = 0; e < V; ++e) ss += r[e] * r[e];
+    }
+  }
+  if (w_next == nullptr) return;
+  ss = warp_sum(ss);
+  if (lane == 0) sums[warp] = ss;
+  __syncthreads();
+  ss = 0.f;
+  for (int i = 0; i < nw; ++i) ss += sums[i];
+  const float rstd = mult / sqrtf(ss / H + eps);
+  for (int c = threadIdx.x * V; c < H; c += blockDim.x * V) {
+    float r[V], g[V];
+    ldv<V>(srow + c, r);
+    ldv<V>(w_next + c, g);
+#pragma unroll
+    for (int e = 0; e < V; ++e) r[e] = r[e] * rstd * g[e];
+    stv<V>(xr + c, r);
+  }
+}
+
+// resid = table[ids] (+ pos_table[pos]) in fp32, x the same in T (and once more at x2, if that is given).
 template <typename T, int V>
 __global__ void embed_rows_kernel(const int* __restrict__ ids, const T* __restrict__ table, int vocab, const int* __restrict__ pos,
-                                  const T* __restrict__ pos_table, int n_pos, float* __restrict__ resid, T* __restrict__ x, long long total, int H) {
+                                  const T* __restrict__ pos_table, int n_pos, float* __restrict__ resid, T* __restrict__ x, T* __restrict__ x2,
+                                  long long ldx, long long total, int H) {
   pdl_wait();
   pdl_trigger();
   const int hv = H / V;
@@ -234,7 +312,8 @@ __global__ void embed_rows_kernel(const int* __restrict__ ids, const T* __restri
       for (int e = 0; e < V; ++e) v[e] += p[e];
     }
     stv<V>(resid + r * H + c, v);
-    stv<V>(x + r * H + c, v);
+    stv<V>(x + r * ldx + c, v);
+    if (x2 != nullptr) stv<V>(x2 + r * ldx + c, v);
   }
 }
 
@@ -649,16 +728,45 @@ int ab2_post_norm(const void* base, long long ldb, const void* y, const int* inv
   AB2_DONE;
 }
 
-int ab2_embed_rows(const int* ids, const void* table, int vocab, const int* pos, const void* pos_table, int n_pos, float* resid, void* x, int R, int H,
-                   int dt, void* stream) {
+// resid [R, H], x and x2 (or null) [R, H] with ldx elements from row to row; base [R, H] (ldb) with logit [R] (ldl), y [n_rows, H] with inv
+// and topw [R, k], vec [H]: each may be null, like w_next.
+int ab2_residual_norm(const void* base, long long ldb, const float* logit, long long ldl, const void* y, const int* inv, const float* topw, int k,
+                      int n_rows, const float* vec, float* resid, const float* w_next, float mult, void* x, long long ldx, int R, int H, float eps, int dt,
+                      void* stream) {
+  if (R <= 0) return 0;
+  if (H < 1 || (y != nullptr && (inv == nullptr || topw == nullptr))) return 10;
+  const int th = norm_threads(H);
+  const size_t smem = (size_t)(((H + 3) & ~3) + th / 32) * 4;
+  if (smem > 200 * 1024) return 11;
+  const int eb = dt == 0 ? 2 : 4;
+  if (y == nullptr) k = 0;
+  auto fits = [&](int v) {
+    return H % v == 0 && ldb % v == 0 && ldx % v == 0 && aligned_to(base, v * eb) && aligned_to(y, v * eb) && aligned_to(x, v * eb) &&
+           aligned_to(resid, 16) && aligned_to(vec, 16) && aligned_to(w_next, 16);
+  };
+  AB2_TYPED8(dt, fits(8), fits(4), {
+    auto kern = k > 0 ? residual_norm_kernel<T, V, true> : residual_norm_kernel<T, V, false>;
+    static ab2host::DevState st[2];
+    if (ab2host::prepare_launch(kern, 200 * 1024, st[k > 0], nullptr)) return 12;
+    launch_pdl(kern, dim3(R), dim3(th), smem, (cudaStream_t)stream, (const T*)base, ldb, logit, ldl, (const T*)y, inv, topw, k, n_rows, vec, resid,
+               w_next, mult, (T*)x, ldx, H, eps);
+  });
+  AB2_DONE;
+}
+
+int ab2_embed_rows(const int* ids, const void* table, int vocab, const int* pos, const void* pos_table, int n_pos, float* resid, void* x, void* x2,
+                   long long ldx, int R, int H, int dt, void* stream) {
   if (R <= 0) return 0;
   if (vocab < 1 || (pos_table != nullptr && n_pos < 1)) return 10;
   const int eb = dt == 0 ? 2 : 4;
-  auto fits = [&](int v) { return H % v == 0 && aligned_to(table, v * eb) && aligned_to(pos_table, v * eb) && aligned_to(x, v * eb) && aligned_to(resid, 16); };
+  auto fits = [&](int v) {
+    return H % v == 0 && ldx % v == 0 && aligned_to(table, v * eb) && aligned_to(pos_table, v * eb) && aligned_to(x, v * eb) &&
+           aligned_to(x2, v * eb) && aligned_to(resid, 16);
+  };
   AB2_TYPED8(dt, fits(8), fits(4), {
     const long long n = (long long)R * (H / V);
     launch_pdl(embed_rows_kernel<T, V>, dim3(flat_grid(n)), dim3(256), 0, (cudaStream_t)stream, ids, (const T*)table, vocab, pos, (const T*)pos_table,
-               n_pos, resid, (T*)x, n, H);
+               n_pos, resid, (T*)x, (T*)x2, ldx, n, H);
   });
   AB2_DONE;
 }

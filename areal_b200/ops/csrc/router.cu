@@ -24,7 +24,7 @@ static constexpr int ROUTE_MAX_E = 256;
 static constexpr int ROUTE_MAX_K = 16;
 
 __global__ void __launch_bounds__(256)
-moe_topk_kernel(const float* __restrict__ logits, const float* __restrict__ bias, float* __restrict__ probs,
+moe_topk_kernel(const float* __restrict__ logits, int ldl, const float* __restrict__ bias, float* __restrict__ probs,
                 float* __restrict__ topw, int* __restrict__ tope, int T, int E, int k, int use_sigmoid, int norm,
                 float scale) {
   const int lane = threadIdx.x & 31;
@@ -32,7 +32,7 @@ moe_topk_kernel(const float* __restrict__ logits, const float* __restrict__ bias
   if (t >= T) return;
   constexpr int PER = ROUTE_MAX_E / 32;
   float p[PER], c[PER];
-  const float* row = logits + (size_t)t * E;
+  const float* row = logits + (size_t)t * ldl;
   float m = -INFINITY;
 #pragma unroll
   for (int j = 0; j < PER; ++j) {
@@ -199,11 +199,11 @@ long long ab2_moe_route_workspace(long long n_entries, int E) {
   return (chunks > 0 ? chunks : 1) * E;
 }
 
-// logits [T, E] fp32; bias [E] fp32 or null (added for the choice only). flags: bit 0 sigmoid scores,
+// logits [T, E] fp32 (ldl elements from row to row); bias [E] fp32 or null (added for the choice only). flags: bit 0 sigmoid scores,
 // bit 1 renormalise the chosen weights, bit 2 tope is given (skip the selection; topw / probs untouched).
 // Outputs: probs [T, E] (nullable), topw [T, k] fp32, tope [T, k] int32, counts [E], offs [E + 1],
 // order / token_of [T * k], inv [T * k], row_tiles [max_row_tiles] int4, num_row_tiles [1].
-int ab2_moe_route(const void* logits, const void* bias, int T, int E, int k, int flags, float scale, void* probs, void* topw,
+int ab2_moe_route(const void* logits, int ldl, const void* bias, int T, int E, int k, int flags, float scale, void* probs, void* topw,
                   void* tope, void* counts, void* offs, void* order, void* token_of, void* inv, void* row_tiles,
                   void* num_row_tiles, int max_row_tiles, void* workspace, void* stream) {
   using namespace ab2;
@@ -217,7 +217,7 @@ int ab2_moe_route(const void* logits, const void* bias, int T, int E, int k, int
   if (!(flags & 4)) {
     const int warps = 8;
     moe_topk_kernel<<<(T + warps - 1) / warps, warps * 32, 0, s>>>(
-        reinterpret_cast<const float*>(logits), reinterpret_cast<const float*>(bias), reinterpret_cast<float*>(probs),
+        reinterpret_cast<const float*>(logits), ldl, reinterpret_cast<const float*>(bias), reinterpret_cast<float*>(probs),
         reinterpret_cast<float*>(topw), reinterpret_cast<int*>(tope), T, E, k, flags & 1, (flags >> 1) & 1, scale);
   }
   moe_count_kernel<<<chunks, 256, 0, s>>>(reinterpret_cast<const int*>(tope), n_entries, E, reinterpret_cast<int*>(workspace));

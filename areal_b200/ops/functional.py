@@ -197,7 +197,9 @@ def moe_route(logits: torch.Tensor, k: int, bias: Optional[torch.Tensor] = None,
     if not logits.is_cuda or E > 256 or k > 16:
         return moe_route_ref(logits, k, bias, sigmoid, norm, scale, tope)
     dev = logits.device
-    logits = logits.float().contiguous()
+    logits = logits.float()
+    if logits.stride(1) != 1:
+        logits = logits.contiguous()
     n = T * k
     i32 = dict(dtype=torch.int32, device=dev)
     given = tope is not None
@@ -213,7 +215,7 @@ def moe_route(logits: torch.Tensor, k: int, bias: Optional[torch.Tensor] = None,
     ws = torch.empty(int(L.ab2_moe_route_workspace(n, E)), **i32)
     b = bias.float().contiguous() if bias is not None else None
     flags = (1 if sigmoid else 0) | (2 if norm else 0) | (4 if given else 0)
-    rc = L.ab2_moe_route(logits.data_ptr(), _lib.ptr(b), T, E, k, flags, float(scale), _lib.ptr(probs), _lib.ptr(topw),
+    rc = L.ab2_moe_route(logits.data_ptr(), logits.stride(0), _lib.ptr(b), T, E, k, flags, float(scale), _lib.ptr(probs), _lib.ptr(topw),
                          tope_.data_ptr(), counts.data_ptr(), offs.data_ptr(), order.data_ptr(), token_of.data_ptr(),
                          inv.data_ptr(), row_tiles.data_ptr(), num_rt.data_ptr(), max_rt, ws.data_ptr(), _s())
     _lib.check(rc, "ab2_moe_route")

@@ -1,7 +1,7 @@
-"""Ops of mixer stacks: norms around (grouped) or behind the sublayers on a 32-bit residual stream, chunked attention
-with capped scores and a logarithmic distance bias over a paged cache, sliding-window attention on cached latents, causal
-convolutions, RG-LRU and Mamba-2 recurrences on slot states, activations, expert combine, per-layer token inputs and
-capped logits.
+"""Ops of mixer stacks: norms around (grouped), behind or before the sublayers on a 32-bit residual stream, rotated
+positions, attention over a paged cache (chunks or sliding windows, capped scores, a logarithmic distance bias, sinks, gated
+outputs), attention on cached latents, causal convolutions, RG-LRU, Mamba-2 and retention recurrences on slot states,
+activations, expert combine, per-layer token inputs and capped logits.
 
 Every op works on a :class:`RaggedBatch`: the rows of several requests, each bringing any number of its next tokens,
 continuing from the cache pages and state slots that earlier steps left. The first ``n_dec`` entries bring one row
@@ -13,6 +13,7 @@ stream are fp32 everywhere.
 """
 from __future__ import annotations
 
+import ctypes
 import math
 from dataclasses import dataclass, field
 from typing import Optional
@@ -73,6 +74,7 @@ class RaggedBatch:
     n_dec: int                   # leading entries with one row
     page_size: int
     seen: dict = field(default_factory=dict)     # sliding window -> PageList of the entries >= n_dec (latent attention)
+    rot: Optional[torch.Tensor] = None           # [R, P, 2] (cos, sin) of the step's rows, made by the model (rotary_table)
 
     @property
     def n_rows(self) -> int:
@@ -107,16 +109,17 @@ def linear(x: torch.Tensor, w: torch.Tensor, fp32_out: bool = False) -> torch.Te
 
 
 def head_linear(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, w_kn: bool = False) -> torch.Tensor:
-    """Every head's own product: ``out[r, h] = w[h] x[r, h]``; x [R, H, K], w [H, N, K] (``w_kn``: [H, K, N]). One tcgen05
-    launch for bf16 with aligned sizes, the library's batched product in 32-bit and for odd sizes."""
+    """Every head's own product: ``out[r, h] = w[h] x[r, h]``; x [R, H, K] (rows and heads may be strided), w [H, N, K] (``w_kn``:
+    [H, K, N]). One tcgen05 launch for bf16 with aligned sizes, the library's batched product in 32-bit and for odd sizes."""
     R, H, K = x.shape
     N = w.shape[2] if w_kn else w.shape[1]
     if out is None:
         out = torch.empty(R, H, N, device=x.device, dtype=x.dtype)
-    if x.is_cuda and x.dtype == torch.bfloat16 and K % 8 == 0 and N % 8 == 0:
-        assert x.is_contiguous() and w.is_contiguous() and out.is_contiguous()
+    lda, hsa = x.stride(0), max(x.stride(1), K)          # (a single head has no stride to speak of)
+    if x.is_cuda and x.dtype == torch.bfloat16 and K % 8 == 0 and N % 8 == 0 and lda % 8 == 0 and hsa % 8 == 0 and x.data_ptr() % 16 == 0:
+        assert x.stride(2) == 1 and w.is_contiguous() and out.is_contiguous()
         bn = 256 if N % 256 == 0 and R > 128 else 128
-        _call("ab2_gemm_heads", _p(x), _p(w), _p(out), R, H, N, K, int(w_kn), bn)
+        _call("ab2_gemm_heads", _p(x), _p(w), _p(out), R, H, N, K, max(lda, hsa * (H - 1) + K), hsa, int(w_kn), bn)
         return out
     out.copy_(torch.bmm(x.transpose(0, 1), w if w_kn else w.transpose(1, 2)).transpose(0, 1))
     return out
@@ -161,32 +164,43 @@ def sandwich_norm(h, w_post, resid, w_next, groups: int, eps: float):
 
 @dataclass
 class ExpertSum:
-    """A feed-forward output that is still in pieces: the expert-sorted rows ``y``, to be summed per token, and what is
-    added to them. The norm behind the sublayer reads the pieces."""
+    """A feed-forward output that is still in pieces: the expert-sorted rows ``y``, to be summed per token (weighted when
+    ``weights`` are given), and what is added to them (times ``sigmoid(shared_logit)`` when that is given). The residual sum or
+    the norm behind the sublayer reads the pieces."""
 
     y: torch.Tensor                      # [T * k, H]
     routing: Routing
     shared: Optional[torch.Tensor]       # [T, H]
+    weights: Optional[torch.Tensor] = None        # [T, k]
+    shared_logit: Optional[torch.Tensor] = None   # [T] fp32, may be strided
 
     def dense(self) -> torch.Tensor:
         k = self.routing.k
-        h = self.y.index_select(0, self.routing.inv).view(-1, k, self.y.shape[1]).float().sum(1)
-        return h if self.shared is None else h + self.shared.float()
+        h = self.y.index_select(0, self.routing.inv).view(-1, k, self.y.shape[1]).float()
+        h = (h if self.weights is None else h * self.weights[..., None]).sum(1)
+        if self.shared is None:
+            return h
+        return h + (self.shared.float() if self.shared_logit is None else self.shared.float() * torch.sigmoid(self.shared_logit)[:, None])
 
 
-def embed_rows(ids, table, pos, pos_table=None):
+def embed_rows(ids, table, pos, pos_table=None, out=None, out2=None):
     """``(residual fp32, residual in the table's dtype)``: the embedding rows of ``ids``, plus the rows of ``pos`` in
-    ``pos_table`` when there is one."""
+    ``pos_table`` when there is one. ``out`` / ``out2``: where the second one goes (rows may be strided, both alike)."""
     if not table.is_cuda:
         resid = table[ids.long()].float()
         if pos_table is not None:
             resid = resid + pos_table[pos.long().clamp(0, pos_table.shape[0] - 1)].float()
-        return resid, resid.to(table.dtype)
+        x = resid.to(table.dtype)
+        for o in (out, out2):
+            if o is not None:
+                o.copy_(x)
+        return resid, x if out is None else out
     T, H = ids.shape[0], table.shape[1]
     resid = torch.empty(T, H, device=table.device, dtype=torch.float32)
-    x = torch.empty(T, H, device=table.device, dtype=table.dtype)
-    _call("ab2_embed_rows", _p(ids), _p(table), table.shape[0], _p(pos), _p(pos_table), 0 if pos_table is None else pos_table.shape[0], _p(resid), _p(x), T, H,
-          _dt(table))
+    x = torch.empty(T, H, device=table.device, dtype=table.dtype) if out is None else out
+    assert out2 is None or out2.stride(0) == x.stride(0)
+    _call("ab2_embed_rows", _p(ids), _p(table), table.shape[0], _p(pos), _p(pos_table), 0 if pos_table is None else pos_table.shape[0], _p(resid), _p(x),
+          _p(out2), x.stride(0), T, H, _dt(table))
     return resid, x
 
 
@@ -195,6 +209,7 @@ def post_norm(h, w, resid, eps: float, mult: float = 1.0, offset: float = 0.0, w
     ``rmsnorm(resid) * (offset_next + w_next)``. ``h`` is [R, H] or an :class:`ExpertSum`."""
     parts = isinstance(h, ExpertSum)
     src = h.y if parts else h
+    assert not (parts and (h.weights is not None or h.shared_logit is not None)), "expert rows summed as they are"
     if not src.is_cuda:
         resid += mult * group_norm_ref(h.dense() if parts else h, offset + w, 1, eps)
         out = resid if w_next is None else group_norm_ref(resid, offset_next + w_next, 1, eps)
@@ -209,7 +224,103 @@ def post_norm(h, w, resid, eps: float, mult: float = 1.0, offset: float = 0.0, w
     return x
 
 
+def residual_norm(h, resid, w_next, eps: float, dtype, vec=None, mult: float = 1.0, out=None):
+    """``resid += h + vec`` (in place, fp32; ``h`` is [R, H], an :class:`ExpertSum` or None, ``vec`` [H] or None); returns
+    ``mult * rmsnorm(resid) * w_next`` in ``dtype``, or resid itself without ``w_next``. ``out``: where it goes (rows may be strided)."""
+    parts = isinstance(h, ExpertSum)
+    R, H = resid.shape
+    if not resid.is_cuda:
+        if h is not None:
+            resid += h.dense() if parts else h.float()
+        if vec is not None:
+            resid += vec
+        x = (resid if w_next is None else mult * group_norm_ref(resid, w_next, 1, eps)).to(dtype)
+        return x if out is None else out.copy_(x)
+    x = torch.empty(R, H, device=resid.device, dtype=dtype) if out is None else out
+    base = h.shared if parts else h
+    lg = h.shared_logit if parts else None
+    assert resid.is_contiguous() and x.dtype == dtype and (base is None or (base.stride(1) == 1 and base.dtype == dtype))
+    y, inv, tw, k, n = (_p(h.y), _p(h.routing.inv), _p(h.weights), h.routing.k, h.y.shape[0]) if parts else (None, None, None, 0, 0)
+    _call("ab2_residual_norm", _p(base), 0 if base is None else base.stride(0), _p(lg), 0 if lg is None else lg.stride(0), y, inv, tw, k, n, _p(vec), _p(resid),
+          _p(w_next), mult, _p(x), x.stride(0), R, H, eps, _dt(x))
+    return x
+
+
+# ----------------------------------------------------------------------------- rotated positions
+def rotary_table(pos, freq, mult):
+    """``(cos, sin)`` of the rows' angles times ``mult``: pos [R], freq [P] double in turns per position, mult [P] fp32. Returns
+    [R, P, 2] fp32."""
+    if not pos.is_cuda:
+        turns = pos.double()[:, None] * freq
+        a = ((turns - turns.round()) * (2 * math.pi)).float()
+        return torch.stack([torch.cos(a) * mult, torch.sin(a) * mult], -1)
+    out = torch.empty(pos.shape[0], freq.shape[0], 2, device=pos.device, dtype=torch.float32)
+    _call("ab2_rotary_table", _p(pos), _p(freq), _p(mult), _p(out), pos.shape[0], freq.shape[0])
+    return out
+
+
+def rotate_ref(x, cs, interleaved: bool):
+    """x [R, ..., D] in fp32 with its first pairs turned; cs [R, half, 2]."""
+    half = cs.shape[1]
+    x = x.float().clone()
+    shape = (x.shape[0],) + (1,) * (x.dim() - 2) + (half,)
+    c, s = cs[..., 0].reshape(shape), cs[..., 1].reshape(shape)
+    a, b = (slice(0, 2 * half, 2), slice(1, 2 * half, 2)) if interleaved else (slice(0, half), slice(half, 2 * half))
+    u, v = x[..., a].clone(), x[..., b].clone()
+    x[..., a], x[..., b] = u * c - v * s, v * c + u * s
+    return x
+
+
+def _rot(rot):
+    """Arguments of a stretch [R, half, 2] of a step's table."""
+    return _p(rot), rot.stride(0) // 2, rot.shape[1]
+
+
+def qk_head_norm_append(z, wq, wk, eps: float, rot, interleaved: bool, b: RaggedBatch, kc, vc, Hq: int):
+    """Per-head RMS norms of q and k (weights [D] shared by the heads, None: no norm), rotation of the first ``2 * rot.shape[1]``
+    numbers of every head, then k and v into the cache rows of ``b.slots``; returns q [R, Hq, D]. ``z`` rows begin with q | k | v."""
+    Hkv, D, Dv = kc.shape[1], kc.shape[2], vc.shape[2]
+    R, nq, nk = z.shape[0], Hq * D, Hkv * D
+    if not z.is_cuda:
+        def turn(x, w):
+            x = x.float()
+            return rotate_ref(x if w is None else group_norm_ref(x, w, 1, eps), rot, interleaved).to(z.dtype)
+        ok = b.slots >= 0
+        kc[b.slots[ok].long()] = turn(z[:, nq:nq + nk].reshape(R, Hkv, D), wk)[ok]
+        vc[b.slots[ok].long()] = z[ok, nq + nk:nq + nk + Hkv * Dv].reshape(-1, Hkv, Dv)
+        return turn(z[:, :nq].reshape(R, Hq, D), wq)
+    q = torch.empty(R, Hq, D, device=z.device, dtype=z.dtype)
+    _call("ab2_qk_head_norm_append", _p(z), z.stride(0), _p(wq), _p(wk), *_rot(rot), int(interleaved), _p(b.slots), _p(q), _p(kc), _p(vc), R, Hq, Hkv, D,
+          Hkv * Dv, eps, _dt(z))
+    return q
+
+
 # ----------------------------------------------------------------------------- attention
+class AttnExtra(ctypes.Structure):
+    """Optional inputs of the attention kernels (the struct of the same name in csrc/mixer_common.cuh)."""
+
+    _fields_ = ([(n, ctypes.c_void_p) for n in ("q2", "k2", "gate", "sink")] +
+                [(n, ctypes.c_longlong) for n in ("ldq", "hsq", "ldq2", "hsq2", "ldk", "ldv", "ldk2", "ldo", "ldg")] +
+                [(n, ctypes.c_int) for n in ("D2", "gate_per_head")] + [(n, ctypes.c_float) for n in ("sink_const", "out_scale")])
+
+
+def _extra(sink=None, gate=None, gate_per_head=False, out_scale=1.0, **strides) -> AttnExtra:
+    x = AttnExtra(sink_const=-math.inf if sink is None or torch.is_tensor(sink) else sink, out_scale=out_scale, gate_per_head=int(gate_per_head), **strides)
+    if torch.is_tensor(sink):
+        x.sink = _p(sink)
+    if gate is not None:
+        x.gate, x.ldg = _p(gate), gate.stride(0)
+    return x
+
+
+def softmax_with_sink(s, sink):
+    """Softmax of s [H, i, j] with ``exp(sink)`` added to the denominator (a number or one per head; None: nothing)."""
+    if sink is None:
+        return torch.softmax(s, -1)
+    sink = (sink if torch.is_tensor(sink) else torch.full((s.shape[0],), float(sink))).float()[:, None, None].expand(-1, s.shape[1], 1)
+    return torch.softmax(torch.cat([s, sink], -1), -1)[..., :-1]
+
+
 def qk_norm_append(qkv, wq, wk, eps: float, b: RaggedBatch, kc, vc, Hq: int):
     """Whole-projection RMS norms of q and k, then k and v into the cache rows of ``b.slots``; returns q [R, Hq, D].
     ``qkv`` rows are q | k | v; ``kc`` [S, Hkv, D], ``vc`` [S, Hkv, Dv]."""
@@ -228,14 +339,14 @@ def qk_norm_append(qkv, wq, wk, eps: float, b: RaggedBatch, kc, vc, Hq: int):
     return q
 
 
-def chunk_attention_ref(q, kc, vc, b: RaggedBatch, scale, softcap, r1, r2, chunk):
+def chunk_attention_ref(q, kc, vc, b: RaggedBatch, scale, softcap, r1, r2, chunk, window=0, sink=None):
     R, Hq, D = q.shape
     Hkv, Dv = kc.shape[1], vc.shape[2]
     out = torch.zeros(R, Hq, Dv, dtype=q.dtype)
     rep, ps = Hq // Hkv, b.page_size
     for e, r0, r1_, st, _ in _segments(b):
         end = st + r1_ - r0
-        lo = (st // chunk) * chunk if chunk else 0
+        lo = (st // chunk) * chunk if chunk else (max(0, st - window + 1) if window else 0)
         j = torch.arange(lo, end)
         rows = b.pages[e][(j // ps - b.page_base[e]).long()].long() * ps + j % ps
         k = kc[rows].float().repeat_interleave(rep, 1)
@@ -250,22 +361,34 @@ def chunk_attention_ref(q, kc, vc, b: RaggedBatch, scale, softcap, r1, r2, chunk
         see = dist >= 0
         if chunk:
             see &= (i // chunk)[:, None] == (j // chunk)[None, :]
+        if window:
+            see &= dist < window
         s = s.masked_fill(~see, float("-inf"))
-        out[r0:r1_] = torch.einsum("hij,jhd->ihd", torch.softmax(s, -1), v).to(q.dtype)
+        out[r0:r1_] = torch.einsum("hij,jhd->ihd", softmax_with_sink(s, sink), v).to(q.dtype)
     return out
 
 
-def chunk_attention(q, kc, vc, b: RaggedBatch, scale: float, softcap: float = 0.0, r1=None, r2=None, chunk: int = 0):
+def chunk_attention(q, kc, vc, b: RaggedBatch, scale: float, softcap: float = 0.0, r1=None, r2=None, chunk: int = 0, window: int = 0, sink=None, gate=None,
+                    out_scale: float = 1.0, out=None):
     """Attention of the step's queries over the paged cache (their own keys already appended): ``softcap *
     tanh(q.k * scale / softcap)`` minus ``r1[h] * ln(1 + r2[h] * distance)``, softmax over the earlier positions of
-    the query's own chunk of ``chunk`` positions (0: no limit). Returns [R, Hq, Dv]."""
-    if not q.is_cuda:
-        return chunk_attention_ref(q, kc, vc, b, scale, softcap, r1, r2, chunk)
+    the query's own chunk of ``chunk`` positions, or over itself and the ``window - 1`` before it (0: no limit), with
+    ``exp(sink)`` more in the denominator; then times ``sigmoid(gate)`` (gate [R, Hq * Dv], rows may be strided) and ``out_scale``.
+    Returns [R, Hq, Dv], in ``out`` [R, Hq * Dv] (rows may be strided) when that is given."""
     R, Hq, D = q.shape
     Hkv, Dv = kc.shape[1], vc.shape[2]
-    out = torch.empty(R, Hq, Dv, device=q.device, dtype=q.dtype)
-    common = (_p(kc), _p(vc), _p(b.pages), _p(b.page_base), b.pages.shape[1], b.page_size, Hq, Hkv, D, Dv, scale, softcap, _p(r1), _p(r2), chunk, 0)
+    if not q.is_cuda:
+        o = chunk_attention_ref(q, kc, vc, b, scale, softcap, r1, r2, chunk, window, sink)
+        if gate is not None or out_scale != 1.0:
+            o = (o.float() * (1.0 if gate is None else torch.sigmoid(gate.float()).view(R, Hq, Dv)) * out_scale).to(q.dtype)
+        return o if out is None else out.copy_(o.view(R, -1))
+    if out is None:
+        out = torch.empty(R, Hq, Dv, device=q.device, dtype=q.dtype)
+    x = _extra(sink, gate, out_scale=out_scale, ldo=out.stride(0))
+    common = (_p(kc), _p(vc), _p(b.pages), _p(b.page_base), b.pages.shape[1], b.page_size, Hq, Hkv, D, Dv, scale, softcap, _p(r1), _p(r2), chunk, window,
+              ctypes.byref(x))
     fast = q.dtype == torch.bfloat16 and D % 8 == 0 and Dv % 8 == 0 and D <= 128 and Dv <= 128
+    tiles = fast and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0 and (gate is None or (gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0))
     nd = b.n_dec
     if nd:
         if fast and Hq // Hkv <= 16:
@@ -273,9 +396,11 @@ def chunk_attention(q, kc, vc, b: RaggedBatch, scale: float, softcap: float = 0.
         else:
             _call("ab2_chunk_attn_plain", _p(q), _p(b.pos), _p(b.slots), _p(b.row_entry), _p(out), nd, *common, _dt(q))
     if R > nd:
-        if fast and b.page_size in (16, 32, 64, 128) and b.tiles is not None:
+        if tiles and b.page_size in (16, 32, 64, 128) and b.tiles is not None:
             _call("ab2_chunk_prefill", _p(q), _p(b.cu), _p(b.start), _p(b.tiles), b.tiles.shape[0], _p(out), R, kc.shape[0], Hkv * D, Hkv * Dv, *common)
         else:
+            if gate is not None:
+                x.gate = _p(gate[nd:])
             _call("ab2_chunk_attn_plain", _p(q[nd:]), _p(b.pos[nd:]), _p(b.slots[nd:]), _p(b.row_entry[nd:]), _p(out[nd:]), R - nd, *common, _dt(q))
     return out
 
@@ -295,20 +420,37 @@ def latent_norm_append(x, wq, wc, eps: float, b: RaggedBatch, cache):
     return cq
 
 
-def latent_attention_ref(q, cache, w_kv, Dv, b: RaggedBatch, scale, window):
-    R, H, D = q.shape
-    ps = b.page_size
+def latent_rope_append(z, wc, eps: float, rot, interleaved: bool, b: RaggedBatch, cache, H: int, D: int):
+    """Rows of ``z``: queries [H, D + r] | latent | key part [r]; r = ``2 * rot.shape[1]``. Turns the last r numbers of every query
+    head in place; the RMS-normed latent and the turned key part go into the cache rows of ``b.slots`` (cache [S, 1, C + r])."""
+    r = 2 * rot.shape[1]
+    C, R, nq = cache.shape[2] - r, z.shape[0], H * (D + r)
+    if not z.is_cuda:
+        q = z[:, :nq].view(R, H, D + r)
+        q[..., D:] = rotate_ref(q[..., D:], rot, interleaved).to(z.dtype)
+        ok = b.slots >= 0
+        row = torch.cat([group_norm_ref(z[:, nq:nq + C], wc, 1, eps), rotate_ref(z[:, nq + C:nq + C + r], rot, interleaved)], -1)
+        cache[b.slots[ok].long(), 0] = row.to(z.dtype)[ok]
+        return
+    _call("ab2_latent_rope_append", _p(z), z.stride(0), _p(wc), *_rot(rot), int(interleaved), _p(b.slots), _p(cache), R, H, D, C, eps, _dt(z))
+
+
+def latent_attention_ref(q, cache, w_kv, Dv, b: RaggedBatch, scale, window, rot_dim=0, sink=None):
+    R, H, D = q.shape[0], q.shape[1], q.shape[2] - rot_dim
+    C, ps = w_kv.shape[1], b.page_size
     out = torch.zeros(R, H, Dv, dtype=q.dtype)
     for e, r0, r1, st, _ in _segments(b):
         i = torch.arange(st, st + r1 - r0)
         j = torch.arange(max(0, st - window + 1) if window else 0, st + r1 - r0)
         rows = b.pages[e][(j // ps - b.page_base[e]).long()].long() * ps + j % ps
-        kv = F.linear(cache[rows, 0].float(), w_kv.float())
+        kv = F.linear(cache[rows, 0, :C].float(), w_kv.float())
         k, v = kv[:, :H * D].view(-1, H, D), kv[:, H * D:].view(-1, H, Dv)
-        s = torch.einsum("ihd,jhd->hij", q[r0:r1].float(), k) * scale
+        s = torch.einsum("ihd,jhd->hij", q[r0:r1, :, :D].float(), k)
+        if rot_dim:
+            s = s + torch.einsum("ihd,jd->hij", q[r0:r1, :, D:].float(), cache[rows, 0, C:].float())
         dist = i[:, None] - j[None, :]
         see = (dist >= 0) & (dist < window) if window else dist >= 0
-        w = torch.softmax(s.masked_fill(~see, float("-inf")), -1)
+        w = softmax_with_sink((s * scale).masked_fill(~see, float("-inf")), sink)
         out[r0:r1] = torch.einsum("hij,jhd->ihd", w, v).to(q.dtype)
     return out
 
@@ -318,38 +460,50 @@ def latent_attention_ref(q, cache, w_kv, Dv, b: RaggedBatch, scale, window):
 SHORT_PORTION = 16
 
 
-def latent_attention(q, cache, w_kv, Dv: int, b: RaggedBatch, scale: float, window: int = 0):
-    """Attention of the step's queries q [R, H, D] over cached latents (the step's own already appended): head h has keys
-    ``w_kv[h D:(h + 1) D] c`` and values ``w_kv[H D + h Dv:...] c``, softmax of ``scale * q.k`` over the position itself and
-    the ``window - 1`` before it (0: no limit). cache [S, 1, C], w_kv [H (D + Dv), C]. Returns [R, H, Dv]."""
-    R, H, D = q.shape
-    C = w_kv.shape[1]
+def latent_attention(q, cache, w_kv, Dv: int, b: RaggedBatch, scale: float, window: int = 0, rot_dim: int = 0, sink=None, gate=None):
+    """Attention of the step's queries q [R, H, D + rot_dim] (rows may be strided) over cached latents (the step's own already
+    appended): head h has keys ``w_kv[h D:(h + 1) D] c`` and values ``w_kv[H D + h Dv:...] c``, the last ``rot_dim`` numbers of a
+    query meet the part behind the latent, which is every head's key; softmax of ``scale * q.k`` over the position itself and
+    the ``window - 1`` before it (0: no limit), with ``exp(sink)`` more in the denominator; every head's output times
+    ``sigmoid(gate)`` (gate [R, H], rows may be strided). cache [S, 1, C + rot_dim], w_kv [H (D + Dv), C]. Returns [R, H, Dv]."""
+    R, H, D = q.shape[0], q.shape[1], q.shape[2] - rot_dim
+    C, ld = w_kv.shape[1], cache.shape[2]
     if not q.is_cuda:
-        return latent_attention_ref(q, cache, w_kv, Dv, b, scale, window)
+        o = latent_attention_ref(q, cache, w_kv, Dv, b, scale, window, rot_dim, sink)
+        return o if gate is None else (o.float() * torch.sigmoid(gate.float())[..., None]).to(o.dtype)
     w_k, w_v = w_kv[:H * D].view(H, D, C), w_kv[H * D:].view(H, Dv, C)
     out = torch.empty(R, H, Dv, device=q.device, dtype=q.dtype)
     nd, bf16 = b.n_dec, q.dtype == torch.bfloat16
-    paged = bf16 and C % 8 == 0 and b.page_size in (16, 32, 64, 128)
-    fast_rows = paged and C <= 512
-    fast_tiles = paged and D % 8 == 0 and Dv % 8 == 0 and D <= 128 and Dv <= 128
+    q1, q2, c2 = q[:, :, :D], q[:, :, D:], cache[:, :, C:]
+    hs = max(q.stride(1), D + rot_dim)
+    paged = bf16 and C % 8 == 0 and b.page_size in (16, 32, 64, 128) and rot_dim % 8 == 0 and rot_dim <= 64
+    part2 = not rot_dim or (D % 8 == 0 and q.stride(0) % 8 == 0 and hs % 8 == 0 and q.data_ptr() % 16 == 0)
+    fast_rows = paged and part2 and C <= 512
+    fast_tiles = paged and part2 and D % 8 == 0 and Dv % 8 == 0 and D <= 128 and Dv <= 128 and q.stride(0) % 8 == 0 and hs % 8 == 0 and q.data_ptr() % 16 == 0
     whole = R > nd and fast_tiles and R - nd > SHORT_PORTION * (b.n_entries - nd)
     n = nd if whole else R
+    second = dict(q2=_p(q2), ldq2=q.stride(0), hsq2=hs, D2=rot_dim) if rot_dim else {}
     if n:
         # keys applied to the queries: scores against the latents themselves, the values' part after the sum
-        qc = head_linear(q[:n], w_k, w_kn=True)
+        qc = head_linear(q1[:n], w_k, w_kn=True)
         oc = torch.empty_like(qc)
+        x = _extra(sink, gate, True, ldk=ld, ldv=ld, **second, **(dict(k2=_p(c2), ldk2=ld) if rot_dim else {}))
         args = (_p(qc), _p(b.pos), _p(b.slots), _p(b.row_entry), _p(oc), n)
         if fast_rows:
-            _call("ab2_latent_decode", *args, _p(cache), cache.shape[0], _p(b.pages), _p(b.page_base), b.pages.shape[1], b.page_size, H, C, scale, window)
+            _call("ab2_latent_decode", *args, _p(cache), cache.shape[0], _p(b.pages), _p(b.page_base), b.pages.shape[1], b.page_size, H, C, scale, window,
+                  ctypes.byref(x))
         else:
             _call("ab2_chunk_attn_plain", *args, _p(cache), _p(cache), _p(b.pages), _p(b.page_base), b.pages.shape[1], b.page_size, H, 1, C, C, scale, 0.0,
-                  None, None, 0, window, _dt(q))
+                  None, None, 0, window, ctypes.byref(x), _dt(q))
         head_linear(oc, w_v, out[:n])
     if whole:
         seen, ps = b.seen[window], b.page_size
-        kv = linear(cache.view(-1, ps * C).index_select(0, seen.pages).view(-1, C), w_kv)
+        rows = cache.view(-1, ps * ld).index_select(0, seen.pages).view(-1, ld)
+        kv = linear(rows[:, :C], w_kv)
+        x = _extra(sink, gate, True, ldq=q.stride(0), hsq=hs, **second, **(dict(k2=_p(rows[:, C:]), ldk2=ld) if rot_dim else {}))
         _call("ab2_chunk_prefill", _p(q), _p(b.cu), _p(b.start), _p(b.tiles), b.tiles.shape[0], _p(out), R, kv.shape[0], kv.stride(0), kv.stride(0),
-              _p(kv), _p(kv[:, H * D:]), _p(seen.table), _p(seen.base), seen.table.shape[1], ps, H, H, D, Dv, scale, 0.0, None, None, 0, window)
+              _p(kv), _p(kv[:, H * D:]), _p(seen.table), _p(seen.base), seen.table.shape[1], ps, H, H, D, Dv, scale, 0.0, None, None, 0, window,
+              ctypes.byref(x))
     return out
 
 
@@ -444,6 +598,40 @@ def mamba2_scan(xbc, dt_raw, dt_bias, A_log, D, heads: int, vdim: int, state: in
     if E:
         _call("ab2_mamba2_scan", *args, E, _p(S), _p(y), heads, vdim, state, groups, _dt(xbc))
     return y
+
+
+# ----------------------------------------------------------------------------- retention
+def retention(z, decay, log2_decay, rot, eps: float, scale: float, out, heads: int, dim: int, vdim: int, b: RaggedBatch, S):
+    """Per head ``S_t = decay S_(t-1) + k_t v_t^T`` and ``o_t = S_t^T q_t`` with turned q and k (halves paired) and k times
+    ``dim ** -0.5``; every head's o over its root mean square, times ``silu(gate)`` and ``scale``, goes to ``out`` [R, heads * vdim] (rows
+    may be strided). ``z`` rows begin with q | k | v | gate; S [slots, heads, vdim, dim] is left at every entry's last token."""
+    R, nq, nv = z.shape[0], heads * dim, heads * vdim
+    k_scale = dim ** -0.5
+    if not z.is_cuda:
+        q, k = (rotate_ref(z[:, i * nq:(i + 1) * nq].reshape(R, heads, dim), rot, False) for i in (0, 1))
+        k, v = k * k_scale, z[:, 2 * nq:2 * nq + nv].float().view(R, heads, vdim)
+        o = torch.zeros(R, heads, vdim)
+        for e, r0, r1, st, sl in _segments(b):
+            h = S[sl].clone() if st > 0 else torch.zeros(heads, vdim, dim)
+            for t in range(r0, r1):
+                h = decay[:, None, None] * h + v[t][:, :, None] * k[t][:, None, :]
+                o[t] = (h * q[t][:, None, :]).sum(-1)
+            S[sl] = h
+        o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
+        out.copy_((o.reshape(R, nv) * F.silu(z[:, 2 * nq + nv:2 * nq + 2 * nv].float()) * scale).to(z.dtype))
+        return out
+    nd, E, half = b.n_dec, b.n_entries, rot.shape[1]
+    if nd:
+        _call("ab2_retention_decode", _p(z), z.stride(0), *_rot(rot), _p(decay), k_scale, _p(b.start), _p(b.state), _p(S), _p(out), out.stride(0), nd, heads,
+              dim, vdim, eps, scale, _dt(z))
+    if E > nd:
+        y = torch.empty(R - nd, nv, device=z.device, dtype=torch.float32)
+        blocks = z.dtype == torch.bfloat16 and dim <= 128 and dim % 8 == 0 and vdim % 8 == 0 and half % 4 == 0 and z.stride(0) % 8 == 0 and z.data_ptr() % 16 == 0
+        _call("ab2_retention_portions", _p(z), z.stride(0), *_rot(rot), _p(decay), _p(log2_decay), k_scale, _p(b.cu), _p(b.start), _p(b.state), nd, E, _p(S),
+              _p(y), heads, dim, vdim, int(blocks), _dt(z))
+        gate = z[nd:, 2 * nq + nv:]
+        _call("ab2_head_norm_gate", _p(y), _p(gate), z.stride(0), _p(out[nd:]), out.stride(0), R - nd, heads, vdim, eps, scale, _dt(z))
+    return out
 
 
 def gated_group_norm(y, z, w, groups: int, eps: float):
@@ -549,13 +737,20 @@ def softcap_(logits, cap: float):
 for _n, _a in {
     "ab2_sandwich_norm": [_V, _V, _I, _V, _lib.c_ll, _V, _V, _V, _V, _I, _I, _I, _F, _I],
     "ab2_qk_norm_append": [_V, _lib.c_ll, _V, _V, _V, _V, _V, _V, _I, _I, _I, _I, _F, _I],
-    "ab2_embed_rows": [_V, _V, _I, _V, _V, _I, _V, _V, _I, _I, _I],
+    "ab2_embed_rows": [_V, _V, _I, _V, _V, _I, _V, _V, _V, _lib.c_ll, _I, _I, _I],
+    "ab2_residual_norm": [_V, _lib.c_ll, _V, _lib.c_ll, _V, _V, _V, _I, _I, _V, _V, _V, _F, _V, _lib.c_ll, _I, _I, _F, _I],
+    "ab2_rotary_table": [_V] * 4 + [_I, _I],
+    "ab2_qk_head_norm_append": [_V, _lib.c_ll, _V, _V, _V, _I, _I, _I] + [_V] * 4 + [_I] * 5 + [_F, _I],
+    "ab2_latent_rope_append": [_V, _lib.c_ll, _V, _V, _I, _I, _I, _V, _V] + [_I] * 4 + [_F, _I],
+    "ab2_retention_decode": [_V, _lib.c_ll, _V, _I, _I, _V, _F] + [_V] * 4 + [_lib.c_ll] + [_I] * 4 + [_F, _F, _I],
+    "ab2_retention_portions": [_V, _lib.c_ll, _V, _I, _I, _V, _V, _F] + [_V] * 3 + [_I, _I, _V, _V] + [_I] * 5,
+    "ab2_head_norm_gate": [_V, _V, _lib.c_ll, _V, _lib.c_ll, _I, _I, _I, _F, _F, _I],
     "ab2_post_norm": [_V, _lib.c_ll, _V, _V, _I, _I, _V, _F, _F, _V, _V, _F, _V, _I, _I, _F, _I],
-    "ab2_gemm_heads": [_V] * 3 + [_I] * 6,
-    "ab2_chunk_attn_plain": [_V] * 5 + [_I] + [_V] * 4 + [_I] * 6 + [_F, _F, _V, _V, _I, _I, _I],
-    "ab2_chunk_decode": [_V] * 4 + [_I] + [_V] * 4 + [_I] * 6 + [_F, _F, _V, _V, _I, _I],
-    "ab2_chunk_prefill": [_V] * 4 + [_I, _V, _I, _I, _lib.c_ll, _lib.c_ll] + [_V] * 4 + [_I] * 6 + [_F, _F, _V, _V, _I, _I],
-    "ab2_latent_decode": [_V] * 5 + [_I, _V, _I, _V, _V] + [_I] * 4 + [_F, _I],
+    "ab2_gemm_heads": [_V] * 3 + [_I] * 8,
+    "ab2_chunk_attn_plain": [_V] * 5 + [_I] + [_V] * 4 + [_I] * 6 + [_F, _F, _V, _V, _I, _I, _V, _I],
+    "ab2_chunk_decode": [_V] * 4 + [_I] + [_V] * 4 + [_I] * 6 + [_F, _F, _V, _V, _I, _I, _V],
+    "ab2_chunk_prefill": [_V] * 4 + [_I, _V, _I, _I, _lib.c_ll, _lib.c_ll] + [_V] * 4 + [_I] * 6 + [_F, _F, _V, _V, _I, _I, _V],
+    "ab2_latent_decode": [_V] * 5 + [_I, _V, _I, _V, _V] + [_I] * 4 + [_F, _I, _V],
     "ab2_gelu_erf": [_V, _lib.c_ll, _V, _I, _I, _I],
     "ab2_glu_clamped": [_V, _lib.c_ll, _V, _V, _V, _I, _I, _F, _F, _I],
     "ab2_side_gate": [_V, _lib.c_ll, _V, _V, _I, _lib.c_ll, _I, _V, _I, _I, _I],
