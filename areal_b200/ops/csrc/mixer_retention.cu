@@ -190,8 +190,9 @@ retention_scan_kernel(const T* __restrict__ z, const RetArgs p, int e0, float* _
 // One CTA (four warps) per request, head and 64 channels walks the request's blocks of 64 tokens. With t, s = 0 .. n - 1 in the block:
 //   o_t = sum_{s <= t} a^(t - s) (q_t . k_s) v_s + a^(t + 1) S^T q_t
 //   S  <- a^n S + sum_s a^(n - 1 - s) k_s v_s^T
-// v and the rotated q are bf16; the rotated k, the weights and S are fp32 and enter a product as the sum of two bf16 numbers
-// (rounding and rest); accumulation is fp32.
+// v is bf16; the rotated q and k, the weights and S are fp32 and enter a product as the sum of two bf16 numbers (rounding and rest,
+// without the product of two rests); accumulation is fp32. An output is divided by its own size afterwards, so what a
+// small q . k loses would show.
 constexpr int RB_Q = 64, RB_P = 64;
 
 __device__ __forceinline__ void rb_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
@@ -214,7 +215,7 @@ template <int NP>
 struct RetCfg {
   static constexpr int NROW = NP * 2 + 16, PROW = RB_P * 2 + 16;         // padded rows (bytes)
   static constexpr int MAT = RB_Q * NROW;
-  static constexpr int Q_OFF = 0, KH_OFF = MAT, KL_OFF = 2 * MAT, SH_OFF = 3 * MAT, SL_OFF = 4 * MAT, V_OFF = 5 * MAT;
+  static constexpr int QH_OFF = 0, QL_OFF = MAT, KH_OFF = 2 * MAT, KL_OFF = 3 * MAT, SH_OFF = 4 * MAT, SL_OFF = 5 * MAT, V_OFF = 6 * MAT;
   static constexpr int A_OFF = V_OFF + RB_Q * PROW;                      // a^0 .. a^64
   static constexpr int SMEM = A_OFF + (RB_Q + 4) * 4;
 };
@@ -258,9 +259,12 @@ retention_blocks_kernel(const __nv_bfloat16* __restrict__ z, const RetArgs p, in
     auto put = [&](int r, int c, const float (&q)[4], const float (&k)[4]) {
       const int off = r * Cfg::NROW + c * 2;
       uint2 hi, lo;
+      rb_split(q[0], q[1], hi.x, lo.x);
+      rb_split(q[2], q[3], hi.y, lo.y);
+      *reinterpret_cast<uint2*>(sm + Cfg::QH_OFF + off) = hi;
+      *reinterpret_cast<uint2*>(sm + Cfg::QL_OFF + off) = lo;
       rb_split(k[0], k[1], hi.x, lo.x);
       rb_split(k[2], k[3], hi.y, lo.y);
-      *reinterpret_cast<uint2*>(sm + Cfg::Q_OFF + off) = make_uint2(pack_bf16(q[0], q[1]), pack_bf16(q[2], q[3]));
       *reinterpret_cast<uint2*>(sm + Cfg::KH_OFF + off) = hi;
       *reinterpret_cast<uint2*>(sm + Cfg::KL_OFF + off) = lo;
     };
@@ -324,8 +328,9 @@ retention_blocks_kernel(const __nv_bfloat16* __restrict__ z, const RetArgs p, in
     for (int j = 0; j < 8; ++j) gm[j][0] = gm[j][1] = gm[j][2] = gm[j][3] = o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
 #pragma unroll
     for (int k = 0; k < KN; ++k) {
-      uint32_t qa[4];
-      rb_mat(sb + Cfg::Q_OFF + (t0 + (mat & 1) * 8 + r8) * Cfg::NROW + (k * 16 + (mat >> 1) * 8) * 2, qa);
+      uint32_t qa[4], ql[4];
+      rb_mat(sb + Cfg::QH_OFF + (t0 + (mat & 1) * 8 + r8) * Cfg::NROW + (k * 16 + (mat >> 1) * 8) * 2, qa);
+      rb_mat(sb + Cfg::QL_OFF + (t0 + (mat & 1) * 8 + r8) * Cfg::NROW + (k * 16 + (mat >> 1) * 8) * 2, ql);
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const uint32_t off = (j * 16 + (mat >> 1) * 8 + r8) * Cfg::NROW + (k * 16 + (mat & 1) * 8) * 2;
@@ -334,6 +339,8 @@ retention_blocks_kernel(const __nv_bfloat16* __restrict__ z, const RetArgs p, in
           rb_mat(sb + Cfg::KH_OFF + off, b);
           rb_mma(gm[2 * j], qa, b[0], b[1]);
           rb_mma(gm[2 * j + 1], qa, b[2], b[3]);
+          rb_mma(gm[2 * j], ql, b[0], b[1]);
+          rb_mma(gm[2 * j + 1], ql, b[2], b[3]);
           rb_mat(sb + Cfg::KL_OFF + off, b);
           rb_mma(gm[2 * j], qa, b[0], b[1]);
           rb_mma(gm[2 * j + 1], qa, b[2], b[3]);
@@ -341,6 +348,8 @@ retention_blocks_kernel(const __nv_bfloat16* __restrict__ z, const RetArgs p, in
         rb_mat(sb + Cfg::SH_OFF + off, b);
         rb_mma(o[2 * j], qa, b[0], b[1]);
         rb_mma(o[2 * j + 1], qa, b[2], b[3]);
+        rb_mma(o[2 * j], ql, b[0], b[1]);
+        rb_mma(o[2 * j + 1], ql, b[2], b[3]);
         rb_mat(sb + Cfg::SL_OFF + off, b);
         rb_mma(o[2 * j], qa, b[0], b[1]);
         rb_mma(o[2 * j + 1], qa, b[2], b[3]);

@@ -124,7 +124,7 @@ def latents(W, p, h, m, eps):
     return norm(z[:, :m["kv_rank"]], W[p + "dkv.norm"], eps), z[:, m["kv_rank"]:]
 
 
-def latent_attention(W, p, h, m, eps):
+def latent_attention(W, p, h, m, eps, steady=None):
     L, H, d, r = h.shape[0], m["heads"], m["dim"], m["rot_dim"]
     q = (h @ W[p + "q"].T).view(L, H, d + r)
     c, shared = latents(W, p, h, m, eps)
@@ -149,17 +149,30 @@ def retain(q, k, v, decay):
     return torch.stack(out)
 
 
-def retention(W, p, h, m, eps):
+def steadiness(o, q, k, v, decay):
+    """[L]: size of a head's output beside the terms it is a sum of (per token, of the worst head). What it is divided by is its
+    own size, so an output whose terms cancel carries their rounding, enlarged."""
+    term = torch.zeros(o.shape[1], dtype=o.dtype)
+    a, out = torch.as_tensor(decay, dtype=o.dtype), []
+    for t in range(o.shape[0]):
+        term = a ** 2 * term + (k[t] * k[t]).sum(-1) * (v[t] * v[t]).mean(-1)
+        out.append(((o[t] * o[t]).mean(-1) / (term * (q[t] * q[t]).sum(-1))).sqrt().min())
+    return torch.stack(out)
+
+
+def retention(W, p, h, m, eps, steady=None):
     L, H, d, e = h.shape[0], m["heads"], m["dim"], m["vdim"]
     q, k, v = ((h @ W[p + n].T).view(L, H, x) for n, x in (("q", d), ("k", d), ("v", e)))
     f, pairs = base_frequencies(m["rot"]), halves(m["rot"]["dims"])
     q, k = rotate(q, range(L), f, pairs), rotate(k, range(L), f, pairs) * d ** -0.5
     o = retain(q, k, v, m["decay"])
+    if steady is not None:
+        steady.append(steadiness(o, q, k, v, m["decay"]))
     return ((o / rms(o, eps)).reshape(L, -1) * silu(h @ W[p + "g"].T)) @ W[p + "o"].T
 
 
-def parallel(W, p, h, m, eps):
-    return m["left_scale"] * windowed(W, p + "left.", h, m["left"], eps) + m["right_scale"] * retention(W, p + "right.", h, m["right"], eps)
+def parallel(W, p, h, m, eps, steady=None):
+    return m["left_scale"] * windowed(W, p + "left.", h, m["left"], eps) + m["right_scale"] * retention(W, p + "right.", h, m["right"], eps, steady)
 
 
 # ----------------------------------------------------------------------------- feed-forward
@@ -211,9 +224,10 @@ def enter_pass(W, x, x0, t):
 MIXERS = {"latent_attention": latent_attention, "parallel": parallel}
 
 
-def forward(W, config, tokens, margins=None):
+def forward(W, config, tokens, margins=None, steady=None):
     """Logits [L, vocab] of one sequence, and the residual stream after every layer run. ``margins`` (a list) collects, per
-    routed layer, how far each token's last chosen expert's logit is ahead of the first one left out."""
+    routed layer, how far each token's last chosen expert's logit is ahead of the first one left out, ``steady`` the
+    :func:`steadiness` of every retention."""
     eps = config["norm"]["eps"]
     x0 = x = W["embed"][torch.as_tensor(tokens)]
     states = []
@@ -221,7 +235,7 @@ def forward(W, config, tokens, margins=None):
         layer, p = config["layers"][i], f"l{i}."
         if t is not None and i == config["loop"]["start"]:
             x = enter_pass(W, x, x0, t)
-        x = x + MIXERS[layer["type"]](W, p + "mix.", norm(x, W[p + "norm1"], eps), layer["mixer"], eps)
+        x = x + MIXERS[layer["type"]](W, p + "mix.", norm(x, W[p + "norm1"], eps), layer["mixer"], eps, steady)
         if layer["mlp"] is not None:
             x = x + feed_forward(W, p + "mlp.", norm(x, W[p + "norm2"], eps), layer["mlp"], margins)
         states.append(x)
