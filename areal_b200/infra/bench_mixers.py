@@ -237,7 +237,7 @@ def latent_kernel_table(cfg, prefill=(4, 2048), decode=(64, 960), dev="cuda") ->
                 def attn():
                     M._call("ab2_chunk_prefill", q.data_ptr(), pb.cu.data_ptr(), pb.start.data_ptr(), pb.tiles.data_ptr(), pb.tiles.shape[0], out.data_ptr(), R,
                             kv.shape[0], kv.stride(0), kv.stride(0), kv.data_ptr(), kv[:, nq * D:].data_ptr(), sn.table.data_ptr(), sn.base.data_ptr(),
-                            sn.table.shape[1], 64, nq, nq, D, Dv, scale, 0.0, None, None, 0, win)
+                            sn.table.shape[1], 64, nq, nq, D, Dv, scale, 0.0, None, None, 0, win, None)
                 add(f"window attention {win} prefill", attn, (q.numel() + out.numel() + kv.numel()) * 2, flops, like="attn_fwd prefill")
                 add(f"latent_attention {win} prefill (all of it)", lambda: M.latent_attention(q, cache, w_kv, Dv, pb, scale, win),
                     (q.numel() * 2 + R * C) * 2, flops + 2.0 * R * C * nq * (D + Dv))
@@ -259,7 +259,7 @@ def latent_kernel_table(cfg, prefill=(4, 2048), decode=(64, 960), dev="cuda") ->
 
                 def dec():
                     M._call("ab2_latent_decode", qc.data_ptr(), b.pos.data_ptr(), b.slots.data_ptr(), b.row_entry.data_ptr(), oc.data_ptr(), R,
-                            cache.data_ptr(), cache.shape[0], b.pages.data_ptr(), b.page_base.data_ptr(), b.pages.shape[1], 64, nq, C, scale, win)
+                            cache.data_ptr(), cache.shape[0], b.pages.data_ptr(), b.page_base.data_ptr(), b.pages.shape[1], 64, nq, C, scale, win, None)
                 add(f"latent_decode {win} decode", dec, (R * see * C + 2 * qc.numel()) * 2, 4.0 * R * see * nq * C, like="paged_decode decode")
             # as many bytes as the paged kernel below reads: four times the sequences
             b4, rows4 = _batch([1] * (4 * nB), [ctx] * (4 * nB), dev, windows=windows)
@@ -268,7 +268,8 @@ def latent_kernel_table(cfg, prefill=(4, 2048), decode=(64, 960), dev="cuda") ->
 
             def dec4():
                 M._call("ab2_latent_decode", qc4.data_ptr(), b4.pos.data_ptr(), b4.slots.data_ptr(), b4.row_entry.data_ptr(), oc4.data_ptr(), 4 * nB,
-                        cache4.data_ptr(), cache4.shape[0], b4.pages.data_ptr(), b4.page_base.data_ptr(), b4.pages.shape[1], 64, nq, C, scale, windows[-1])
+                        cache4.data_ptr(), cache4.shape[0], b4.pages.data_ptr(), b4.page_base.data_ptr(), b4.pages.shape[1], 64, nq, C, scale, windows[-1],
+                        None)
             add(f"latent_decode {windows[-1]} decode, {4 * nB} sequences", dec4, (4 * nB * see * C + 2 * qc4.numel()) * 2, 16.0 * nB * see * nq * C,
                 like="paged_decode decode")
             nk = max(1, nq // 4)
@@ -301,6 +302,156 @@ def latent_kernel_table(cfg, prefill=(4, 2048), decode=(64, 960), dev="cuda") ->
         add(f"gather and sum {tag}", lambda: (y.index_select(0, rt.inv).view(R, k, Hd) * rt.topw.to(y.dtype).unsqueeze(-1)).sum(1), R * (k + 1) * Hd * 2)
         g = torch.randn(R, sd, **bf)
         add(f"side_gate {tag}", lambda: M.side_gate(g, ids, side, 0), R * sd * 6, like=f"swiglu {tag}")
+    return rows
+
+
+def looped_kernel_table(cfg, prefill=(4, 2048), decode=(64, 960), dev="cuda") -> list[dict]:
+    """As :func:`kernel_table`, for a stack of parallel branches and latent attention with positions (Bumotar), each kernel beside
+    the like one of the other mixer stacks at the same sizes."""
+    bw, fl, _ = peaks()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    bf = dict(device=dev, dtype=torch.bfloat16)
+    f32 = dict(device=dev, dtype=torch.float32)
+    rows = []
+
+    def add(name, fn, nbytes=0.0, flops=0.0, like=None):
+        t = timed(fn, flush=flush)
+        roof = max(nbytes / bw, flops / fl)
+        rows.append(dict(kernel=name, us=round(t * 1e6, 1), roofline_us=round(roof * 1e6, 1), fraction=round(roof / t, 3), like=like))
+
+    Hd, V = cfg.hidden_size, cfg.vocab_size
+    p = next(e["mixer"] for e in cfg.mixer_layers if e["type"] == "parallel")
+    at = next(e["mixer"] for e in cfg.mixer_layers if e["type"] == "latent_attention")
+    moe = next(e["mlp"] for e in cfg.mixer_layers if e["mlp"])
+    lf, rt_ = p["left"], p["right"]
+    nq, nk, D, Dv, win, cap = lf["heads"], lf["kv_heads"], lf["dim"], lf["vdim"], lf["mask"]["size"], lf["softcap"]
+    Hr, N, P = rt_["heads"], rt_["dim"], rt_["vdim"]
+    nl, Dl, r, Dvl, C, scale = at["heads"], at["dim"], at["rot_dim"], at["vdim"], at["kv_rank"], at["scale"]
+    E, k, If, Is = moe["router"]["experts"], moe["router"]["top"], moe["expert"]["ff"], moe["shared"]["ff"]
+    (B, L), (nB, ctx) = prefill, decode
+    pb, prow = _batch([L] * B, [0] * B, dev, windows=(0,))
+    db, drow = _batch([1] * nB, [ctx] * nB, dev, windows=(0,))
+    w, wc, wh = torch.ones(Hd, **f32), torch.ones(C, **f32), torch.ones(D, **f32)
+    half, hl, hr = lf["rot"]["dims"] // 2, r // 2, rt_["rot"]["dims"] // 2
+    freq, mult = torch.rand(half + hl + hr, device=dev, dtype=torch.float64), torch.ones(half + hl + hr, **f32)
+    w_kv = torch.randn(nl * (Dl + Dvl), C, **bf) * C ** -0.5
+    w_k, w_v = w_kv[:nl * Dl].view(nl, Dl, C), w_kv[nl * Dl:].view(nl, Dvl, C)
+    sink, decay = torch.randn(nl, **f32), torch.tensor(rt_["decay"], **f32)
+    table = torch.randn(V, Hd, **bf)
+    for tag, b, R, rows_, ne in (("prefill", pb, B * L, prow, B), ("decode", db, nB, drow, nB)):
+        ids = torch.randint(0, V, (R,), device=dev, dtype=torch.int32)
+        both = torch.empty(R, 2 * Hd, **bf)
+        add(f"embed_rows into both halves {tag}", lambda: M.embed_rows(ids, table, b.pos, None, both[:, Hd:], both[:, :Hd]), R * Hd * 10, like=f"embed_rows {tag}")
+        add(f"embed_rows {tag}", lambda: M.embed_rows(ids, table, b.pos), R * Hd * 8)
+        add(f"rotary_table {tag}", lambda: M.rotary_table(b.pos, freq, mult), R * (4 + 8 * freq.numel()), like=f"embed_rows {tag}")
+        cs = M.rotary_table(b.pos, freq, mult)
+        # residual sums and norms
+        h, res, res2 = torch.randn(R, Hd, **bf), torch.randn(R, Hd, **f32), torch.randn(R, Hd, **f32)
+        add(f"residual_norm {tag}", lambda: M.residual_norm(h, res, w, 1e-6, torch.bfloat16), R * Hd * 12, like=f"post_norm {tag}")
+        add(f"post_norm {tag}", lambda: M.post_norm(h, w, res2, 1e-6, 0.5, 1.0), R * Hd * 12)
+        rt = OF.moe_route(torch.randn(R, E, **f32), k, want_probs=False, want_host=False)
+        y, sh, lg = torch.randn(R * k, Hd, **bf), torch.randn(R, Hd, **bf), torch.randn(R, E + 8, **f32)
+        add(f"residual_norm of experts {tag}", lambda: M.residual_norm(M.ExpertSum(y, rt, sh, rt.topw, lg[:, E]), res, w, 1e-6, torch.bfloat16),
+            R * Hd * (2 * k + 12), like=f"post_norm of experts {tag}")
+        add(f"post_norm of experts {tag}", lambda: M.post_norm(M.ExpertSum(y, rt, sh), w, res2, 1e-6, 0.5, 1.0), R * Hd * (2 * k + 12))
+        eg = torch.randn(R * k, 2 * If, **bf)
+        add(f"glu_silu experts {tag}", lambda: M.glu_silu(eg), R * k * If * 6, like=f"glu_clamped experts {tag}")
+        add(f"glu_clamped experts {tag}", lambda: M.glu_clamped(eg, 6.0, 1.702, rt), R * k * If * 6)
+        sg = torch.randn(R, 2 * Is, **bf)
+        add(f"glu_silu shared {tag}", lambda: M.glu_silu(sg), R * Is * 6, like=f"glu_clamped shared {tag}")
+        add(f"glu_clamped shared {tag}", lambda: M.glu_clamped(sg, 7.0, 1.702), R * Is * 6)
+        # windowed attention, beside the chunked one that sees the same number of keys, with its distance bias
+        nin = nq * D + nk * (D + Dv) + nq * Dv
+        z = torch.randn(R, nin, **bf)
+        kc, vc = torch.randn(rows_, nk, D, **bf), torch.randn(rows_, nk, Dv, **bf)
+        add(f"qk_head_norm_append {tag}", lambda: M.qk_head_norm_append(z, wh, wh, 1e-6, cs[:, :half], False, b, kc, vc, nq), R * (nin - nq * Dv) * 4 + R * half * 8,
+            like=f"qk_norm_append {tag}")
+        wq, wk = torch.ones(nq * D, **f32), torch.ones(nk * D, **f32)
+        add(f"qk_norm_append {tag}", lambda: M.qk_norm_append(z, wq, wk, 1e-6, b, kc, vc, nq), R * (nin - nq * Dv) * 4)
+        q, o = torch.randn(R, nq, D, **bf), torch.empty(R, nq * Dv + Hr * P, **bf)
+        gate, r1, r2 = z[:, nin - nq * Dv:], torch.rand(nq, **f32), torch.rand(nq, **f32)
+        pairs = B * sum(min(x + 1, win) for x in range(L)) if tag == "prefill" else nB * min(ctx + 1, win)
+        kv_bytes = (nk * (D + Dv)) * 2 * (R if tag == "prefill" else pairs)
+        flops = 2.0 * nq * (D + Dv) * pairs
+        add(f"window attention {tag}", lambda: M.chunk_attention(q, kc, vc, b, D ** -0.5, cap, window=win, sink=0.0, gate=gate, out_scale=0.7, out=o[:, :nq * Dv]),
+            q.numel() * 2 + R * nq * Dv * 4 + kv_bytes, flops, like=f"chunk_attention {tag}")
+        seen = B * sum(x % win + 1 for x in range(L)) if tag == "prefill" else nB * (ctx % win + 1)
+        add(f"chunk_attention {tag}", lambda: M.chunk_attention(q, kc, vc, b, D ** -0.5, cap, r1, r2, win), q.numel() * 2 + R * nq * Dv * 2 +
+            (nk * (D + Dv)) * 2 * (R if tag == "prefill" else seen), 2.0 * nq * (D + Dv) * seen)
+        # retention, beside the Mamba-2 recurrence of the same state, and its norm
+        zr, S = torch.randn(R, Hr * (2 * N + 2 * P), **bf), torch.zeros(ne, Hr, P, N, **f32)
+        ro = o[:, nq * Dv:]
+        log2 = torch.log2(decay)
+        rot_r = cs[:, half + hl:]
+        # (its output is bf16 and gated; 32-bit rows between its two kernels in prompts)
+        add(f"retention {tag}", lambda: M.retention(zr, decay, log2, rot_r, 1e-6, 0.4, ro, Hr, N, P, b, S),
+            zr.numel() * 2 + R * Hr * P * (10 if tag == "prefill" else 2) + R * hr * 8 + 2 * S.numel() * 4, like=f"mamba2_scan and norm {tag}")
+        Cm = Hr * P + 2 * Hr * N
+        xbc, dtr, dd = torch.randn(R, Cm, **bf), torch.randn(R, Hr, **bf), torch.ones(Hr, **f32)
+        zg, nw = torch.randn(R, Hr * P, **bf), torch.ones(Hr * P, **f32)
+        add(f"mamba2_scan and norm {tag}", lambda: M.gated_group_norm(M.mamba2_scan(xbc, dtr, dd, dd, dd, Hr, P, N, Hr, b, S), zg, nw, Hr, 1e-6),
+            (xbc.numel() + dtr.numel()) * 2 + R * Hr * P * 12 + 2 * S.numel() * 4)
+        if tag == "prefill":
+            yr = torch.empty(R, Hr * P, **f32)
+
+            def blocks():
+                M._call("ab2_retention_portions", zr.data_ptr(), zr.stride(0), rot_r.data_ptr(), rot_r.stride(0) // 2, hr, decay.data_ptr(), log2.data_ptr(),
+                        N ** -0.5, b.cu.data_ptr(), b.start.data_ptr(), b.state.data_ptr(), 0, B, S.data_ptr(), yr.data_ptr(), Hr, N, P, 1, 0)
+            add("retention_blocks prefill", blocks, R * Hr * (2 * N + P) * 2 + yr.numel() * 4 + 2 * S.numel() * 4, like="mamba2_scan prefill")
+            add("mamba2_scan prefill", lambda: M.mamba2_scan(xbc, dtr, dd, dd, dd, Hr, P, N, Hr, b, S), (xbc.numel() + dtr.numel()) * 2 + R * Hr * P * 4 + 2 * S.numel() * 4)
+        # latent attention, beside the one without positions
+        ld = nl * (Dl + r) + C + r + nl
+        zl, cache, cache0 = torch.randn(R, ld, **bf), torch.randn(rows_, 1, C + r, **bf), torch.randn(rows_, 1, C, **bf)
+        add(f"latent_rope_append {tag}", lambda: M.latent_rope_append(zl, wc, 1e-6, cs[:, half:half + hl], True, b, cache, nl, Dl),
+            R * (2 * nl * r + 2 * (C + r)) * 2 + R * hl * 8, like=f"latent_norm_append {tag}")
+        wql = torch.ones(1536, **f32)
+        xl = torch.randn(R, 1536 + C, **bf)
+        add(f"latent_norm_append {tag}", lambda: M.latent_norm_append(xl, wql, wc, 1e-6, b, cache0), xl.numel() * 4)
+        ql, q0 = zl[:, :nl * (Dl + r)].unflatten(1, (nl, Dl + r)), torch.randn(R, nl, Dl, **bf)
+        gl = zl[:, ld - nl:]
+        if tag == "prefill":
+            pairs = B * L * (L + 1) // 2
+            out = torch.empty(R, nl, Dvl, **bf)
+            sn = pb.seen[0]
+            rows_c = cache.view(-1, C + r)
+            kv = M.linear(rows_c[:, :C], w_kv)
+            x = M._extra(sink, gl, True, ldq=ld, hsq=Dl + r, q2=ql[:, :, Dl:].data_ptr(), ldq2=ld, hsq2=Dl + r, D2=r, k2=rows_c[:, C:].data_ptr(), ldk2=C + r)
+
+            def tiles(q_, extra):
+                M._call("ab2_chunk_prefill", q_.data_ptr(), pb.cu.data_ptr(), pb.start.data_ptr(), pb.tiles.data_ptr(), pb.tiles.shape[0], out.data_ptr(), R,
+                        kv.shape[0], kv.stride(0), kv.stride(0), kv.data_ptr(), kv[:, nl * Dl:].data_ptr(), sn.table.data_ptr(), sn.base.data_ptr(),
+                        sn.table.shape[1], 64, nl, nl, Dl, Dvl, scale, 0.0, None, None, 0, 0, extra)
+            add("attention with shared key part prefill", lambda: tiles(ql, M.ctypes.byref(x)), 0, 2.0 * nl * (Dl + r + Dvl) * pairs, like="attention prefill")
+            add("attention prefill", lambda: tiles(q0, None), 0, 2.0 * nl * (Dl + Dvl) * pairs)
+            wb = 2.0 * R * C * nl * (Dl + Dvl)
+            add("latent attention with positions prefill (all of it)", lambda: M.latent_attention(ql, cache, w_kv, Dvl, b, scale, 0, r, sink, gl), 0,
+                2.0 * nl * (Dl + r + Dvl) * pairs + wb, like="latent_attention prefill (all of it)")
+            add("latent_attention prefill (all of it)", lambda: M.latent_attention(q0, cache0, w_kv, Dvl, b, scale, 0), 0, 2.0 * nl * (Dl + Dvl) * pairs + wb)
+        else:
+            for n, (bb, rw) in ((nB, (db, drow)), (4 * nB, _batch([1] * (4 * nB), [ctx] * (4 * nB), dev, windows=(0,)))):
+                qc, oc = torch.randn(n, nl, C, **bf), torch.empty(n, nl, C, **bf)
+                zz = torch.randn(n, ld, **bf)
+                qq, ca, ca0 = zz[:, :nl * (Dl + r)].unflatten(1, (nl, Dl + r)), torch.randn(rw, 1, C + r, **bf), torch.randn(rw, 1, C, **bf)
+                xd = M._extra(sink, zz[:, ld - nl:], True, ldk=C + r, q2=qq[:, :, Dl:].data_ptr(), ldq2=ld, hsq2=Dl + r, D2=r, k2=ca[:, :, C:].data_ptr(), ldk2=C + r)
+
+                def dec(c_, extra):
+                    M._call("ab2_latent_decode", qc.data_ptr(), bb.pos.data_ptr(), bb.slots.data_ptr(), bb.row_entry.data_ptr(), oc.data_ptr(), n, c_.data_ptr(),
+                            c_.shape[0], bb.pages.data_ptr(), bb.page_base.data_ptr(), bb.pages.shape[1], 64, nl, C, scale, 0, extra)
+                t = "" if n == nB else f", {n} sequences"
+                add(f"latent_decode with positions{t}", lambda: dec(ca, M.ctypes.byref(xd)), (n * (ctx + 1) * (C + r) + 2 * qc.numel() + n * nl * r) * 2,
+                    2.0 * n * (ctx + 1) * nl * (2 * C + r), like=f"latent_decode{t}")
+                add(f"latent_decode{t}", lambda: dec(ca0, None), (n * (ctx + 1) * C + 2 * qc.numel()) * 2, 4.0 * n * (ctx + 1) * nl * C)
+            add("head_linear of strided queries decode", lambda: M.head_linear(ql[:, :, :Dl], w_k, w_kn=True), (R * nl * (Dl + C) + w_k.numel()) * 2, 2.0 * R * nl * Dl * C,
+                like="head_linear of the queries decode")
+            add("head_linear of the queries decode", lambda: M.head_linear(q0, w_k, w_kn=True), (R * nl * (Dl + C) + w_k.numel()) * 2, 2.0 * R * nl * Dl * C)
+        wl = torch.randn(Hd, 2 * Hd, **bf)
+        add(f"entrance of a pass {tag} (GEMM, 32-bit sums)", lambda: M.linear(both, wl, fp32_out=True), (both.numel() + wl.numel()) * 2 + R * Hd * 4,
+            4.0 * R * Hd * Hd, like=f"the same product, bf16 {tag}")
+        add(f"the same product, bf16 {tag}", lambda: M.linear(both, wl), (both.numel() + wl.numel()) * 2 + R * Hd * 2, 4.0 * R * Hd * Hd)
+        rw_, x16 = torch.randn(-(-(E + 1) // 8) * 8, Hd, **bf), torch.randn(R, Hd, **bf)
+        add(f"router_logits and gate {tag}", lambda: M.router_logits(x16, rw_), (R * Hd + E * Hd) * 2 + R * E * 4, 2.0 * R * E * Hd, like=f"router_logits {tag}")
+        rw0 = rw_[:E]
+        add(f"router_logits {tag}", lambda: M.router_logits(x16, rw0), (R * Hd + E * Hd) * 2 + R * E * 4, 2.0 * R * E * Hd)
     return rows
 
 
@@ -453,6 +604,34 @@ def latent_like_sized(cfg):
     return stack, ModelConfig(arch="qwen3", **base), routed
 
 
+def looped_like_sized(cfg):
+    """The closest existing models with the same width, experts and vocabulary as a looped stack, one layer per layer run:
+    the other latent stack (windows of a whole prompt), the stack with Mamba-2 and chunked attention in place of the parallel
+    branches and of the latents, the routed decoder."""
+    from ..models.config import ModelConfig
+    from ..models.mixers import MixerStackLM
+
+    runs = MixerStackLM.layer_runs.fget(type("S", (), dict(cfg=cfg)))
+    par = next(e["mixer"] for e in cfg.mixer_layers if e["type"] == "parallel")
+    at = next(e["mixer"] for e in cfg.mixer_layers if e["type"] == "latent_attention")
+    moe = next(e["mlp"] for e in cfg.mixer_layers if e["mlp"])
+    lf, rt = par["left"], par["right"]
+    lat = dict(heads=at["heads"], dim=at["dim"], vdim=at["vdim"], q_rank=1536, kv_rank=at["kv_rank"], scale=at["scale"], mask=dict(size=4096))
+    experts = dict(moe, expert=dict(moe["expert"], limit=6.0), shared=dict(moe["shared"], limit=7.0))
+    vog = ModelConfig.from_hf_dict(dict(architecture="Vogilix", vocab=cfg.vocab_size, width=cfg.hidden_size, max_positions=8192, norm=dict(eps=1e-6), residual_mult=0.5,
+                                        token_side=None, layers=[dict(type="latent_attention", mixer=lat, mlp=experts) for _ in runs]))
+    att = dict(heads=lf["heads"], kv_heads=lf["kv_heads"], dim=lf["dim"], vdim=lf["vdim"], scale=lf["scale"], softcap=lf["softcap"], mask=dict(lf["mask"]))
+    ssm = dict(heads=2 * rt["heads"], vdim=rt["vdim"], state=rt["dim"], groups=rt["heads"], norm_groups=rt["heads"], conv=4)
+    stack = ModelConfig.from_hf_dict(dict(
+        architecture="Kagolix", vocab=cfg.vocab_size, width=cfg.hidden_size, norm=dict(eps=1e-6, groups=1), logit_softcap=0.0,
+        layers=[dict(type="attention" if n % 2 else "mamba2", mixer=att if n % 2 else ssm, mlp=dict(moe, shared=None)) for n in range(len(runs))]))
+    base = dict(vocab_size=cfg.vocab_size, hidden_size=cfg.hidden_size, num_layers=len(runs), num_heads=lf["heads"], num_kv_heads=lf["kv_heads"],
+                head_dim=lf["dim"], intermediate_size=0, tie_word_embeddings=False, attention_bias=False, qk_norm=True)
+    routed = ModelConfig(arch="qwen3_moe", **base, num_experts=cfg.num_experts, num_experts_per_tok=cfg.num_experts_per_tok,
+                         moe_intermediate_size=cfg.moe_intermediate_size)
+    return vog, stack, routed
+
+
 def run(steps=True, kernels=True, design="kagolix", sizes=None) -> dict:
     from ..models.config import preset
 
@@ -470,6 +649,11 @@ def run(steps=True, kernels=True, design="kagolix", sizes=None) -> dict:
                                ("decoder_routed", decoder_steps, routed)):
                 r[key] = fn(c, prefill, decode)
                 torch.cuda.empty_cache()
+        elif steps and design == "bumotar":
+            latent, stack, routed = looped_like_sized(cfg)
+            for key, fn, c in (("bumotar", mixer_steps, cfg), ("vogilix", mixer_steps, latent), ("mixer_stack", mixer_steps, stack), ("decoder_routed", decoder_steps, routed)):
+                r[key] = fn(c, prefill, decode)
+                torch.cuda.empty_cache()
         elif steps:
             hyb, dense, routed = like_sized(cfg)
             r["mixer_stack"] = mixer_steps(cfg, prefill, decode)
@@ -478,6 +662,6 @@ def run(steps=True, kernels=True, design="kagolix", sizes=None) -> dict:
                 r[key] = fn(c, prefill, decode)
                 torch.cuda.empty_cache()
         if kernels:
-            r["kernels"] = (latent_kernel_table if design == "vogilix" else kernel_table)(cfg, prefill, decode)
+            r["kernels"] = {"vogilix": latent_kernel_table, "bumotar": looped_kernel_table, "kagolix": kernel_table}[design](cfg, prefill, decode)
         out["sizes"][name] = r
     return out

@@ -187,13 +187,13 @@ retention_scan_kernel(const T* __restrict__ z, const RetArgs p, int e0, float* _
 }
 
 // ------------------------------------------------------------------ portions in blocks
-// One CTA (four warps) per request, head and 64 channels walks the request's blocks of 64 tokens. With t, s = 0 .. n - 1 in the block:
-//   o_t = sum_{s <= t} a^(t - s) (q_t . k_s) v_s + a^(t + 1) S^T q_t
-//   S  <- a^n S + sum_s a^(n - 1 - s) k_s v_s^T
+// One CTA (eight warps) per request, head and 64 channels walks the request's blocks of 64 tokens. With t, s = 0 .. n - 1 in the block:
+//   o_t = sum_{s <= t} a^(t - s) (q_t . k_s) v_s + a^(t + 1) S^T q_t        warps 0 - 3 the first sum, 4 - 7 the second
+//   S  <- a^n S + sum_s a^(n - 1 - s) k_s v_s^T                             all of them, 16 channels and half of the columns each
 // v is bf16; the rotated q and k, the weights and S are fp32 and enter a product as the sum of two bf16 numbers (rounding and rest,
 // without the product of two rests); accumulation is fp32. An output is divided by its own size afterwards, so what a
 // small q . k loses would show.
-constexpr int RB_Q = 64, RB_P = 64;
+constexpr int RB_Q = 64, RB_P = 64, RB_U = 4;
 
 __device__ __forceinline__ void rb_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
@@ -217,15 +217,18 @@ struct RetCfg {
   static constexpr int MAT = RB_Q * NROW;
   static constexpr int QH_OFF = 0, QL_OFF = MAT, KH_OFF = 2 * MAT, KL_OFF = 3 * MAT, SH_OFF = 4 * MAT, SL_OFF = 5 * MAT, V_OFF = 6 * MAT;
   static constexpr int A_OFF = V_OFF + RB_Q * PROW;                      // a^0 .. a^64
-  static constexpr int SMEM = A_OFF + (RB_Q + 4) * 4;
+  static constexpr int ZROW = RB_P + 4;                                  // floats; what the state adds to the outputs, over the state's
+  static constexpr int Z_OFF = NP >= 64 ? SH_OFF : A_OFF + (RB_Q + 4) * 4;     // own matrices where these are large enough
+  static constexpr int SMEM = A_OFF + (RB_Q + 4) * 4 + (NP >= 64 ? 0 : RB_Q * ZROW * 4);
+  static_assert(NP < 64 || 2 * MAT >= RB_Q * ZROW * 4, "the sums fit over the state");
 };
 
 // NP: N rounded up to 32, 64 or 128 (missing columns are zero).
 template <int NP>
-__global__ void __launch_bounds__(128, 2)
-retention_blocks_kernel(const __nv_bfloat16* __restrict__ z, const RetArgs p, int e0, float* __restrict__ y) {
+__global__ void __launch_bounds__(256, NP == 128 ? 1 : 2)
+retention_blocks_kernel(const __nv_bfloat16* __restrict__ z, const float2* __restrict__ rot, const RetArgs p, int e0, float* __restrict__ y) {
   using Cfg = RetCfg<NP>;
-  constexpr int NT = NP / 8, KN = NP / 16;
+  constexpr int NT = NP / 16, KN = NP / 16;                   // tiles of 8 in half of the columns, k-steps of 16 in all
   extern __shared__ __align__(16) unsigned char sm[];
   const uint32_t sb = smem_u32(sm);
   float* pw = reinterpret_cast<float*>(sm + Cfg::A_OFF);
@@ -237,7 +240,8 @@ retention_blocks_kernel(const __nv_bfloat16* __restrict__ z, const RetArgs p, in
   const __nv_bfloat16* qg = z + (size_t)hd * N;
   const __nv_bfloat16* kg = qg + (size_t)p.H * N;
   const __nv_bfloat16* vg = z + (size_t)2 * p.H * N + (size_t)hd * P + p0;
-  // this warp's 16 channels of the state: rows p = 16 warp + gq (+ 8), columns n = 8 j + 2 tq (+ 1)
+  // this warp's part of the state: rows p = 16 (warp % 4) + gq (+ 8), columns n = n0 + 8 j + 2 tq (+ 1)
+  const int wr = warp & 3, n0 = (warp >> 2) * (NP / 2);
   float* Sg = p.S + (((size_t)slot * p.H + hd) * P + p0) * N;
   float st[NT][4];
   const bool fresh = p.start[e] <= 0;
@@ -245,7 +249,7 @@ retention_blocks_kernel(const __nv_bfloat16* __restrict__ z, const RetArgs p, in
   for (int j = 0; j < NT; ++j)
 #pragma unroll
     for (int hh = 0; hh < 2; ++hh) {
-      const int c = warp * 16 + gq + 8 * hh, n = j * 8 + 2 * tq;
+      const int c = wr * 16 + gq + 8 * hh, n = n0 + j * 8 + 2 * tq;
       float2 v = make_float2(0.f, 0.f);
       if (!fresh && c < np && n < N) v = *reinterpret_cast<const float2*>(Sg + (size_t)c * N + n);
       st[j][2 * hh] = v.x;
@@ -268,43 +272,59 @@ retention_blocks_kernel(const __nv_bfloat16* __restrict__ z, const RetArgs p, in
       *reinterpret_cast<uint2*>(sm + Cfg::KH_OFF + off) = hi;
       *reinterpret_cast<uint2*>(sm + Cfg::KL_OFF + off) = lo;
     };
-    for (int i = tid; i < RB_Q * pieces; i += 128) {
-      const int r = i / pieces, x = i - r * pieces;
-      const size_t at = (size_t)(r0 + r) * p.ld;
-      float q[4] = {}, k[4] = {};
-      if (x < pairs) {
-        const int c = x * 4;
-        float q2[4] = {}, k2[4] = {};
-        if (r < nr) {
-          ldv<4>(qg + at + c, q);
-          ldv<4>(qg + at + c + half, q2);
-          ldv<4>(kg + at + c, k);
-          ldv<4>(kg + at + c + half, k2);
-          const float2* cs = p.rot + (size_t)(r0 + r) * p.ldr + c;
+    for (int i0 = tid; i0 < RB_Q * pieces; i0 += 256 * RB_U) {
+      uint2 a[RB_U][4];                                      // q, k; q and k half a turn further on, or nothing
+      float2 t[RB_U][4];
 #pragma unroll
-          for (int u = 0; u < 4; ++u) {
-            const float2 t = cs[u];
-            const float a = q[u], b = q2[u], d = k[u] * p.k_scale, g = k2[u] * p.k_scale;
-            q[u] = a * t.x - b * t.y;
-            q2[u] = b * t.x + a * t.y;
-            k[u] = d * t.x - g * t.y;
-            k2[u] = g * t.x + d * t.y;
+      for (int u = 0; u < RB_U; ++u) {                       // RB_U pieces on their way at a time
+        const int i = i0 + 256 * u, r = i / pieces, x = i - r * pieces, c = x < pairs ? x * 4 : 2 * half + (x - pairs) * 4;
+        const size_t at = (size_t)(r0 + r) * p.ld + c;
+        a[u][0] = a[u][1] = a[u][2] = a[u][3] = make_uint2(0u, 0u);
+        t[u][0] = t[u][1] = t[u][2] = t[u][3] = make_float2(0.f, 0.f);
+        if (r >= nr || c >= N) continue;
+        a[u][0] = *reinterpret_cast<const uint2*>(qg + at);
+        a[u][1] = *reinterpret_cast<const uint2*>(kg + at);
+        if (x < pairs) {
+          a[u][2] = *reinterpret_cast<const uint2*>(qg + at + half);
+          a[u][3] = *reinterpret_cast<const uint2*>(kg + at + half);
+          const float2* cs = rot + (size_t)(r0 + r) * p.ldr + c;
+#pragma unroll
+          for (int w = 0; w < 4; ++w) t[u][w] = cs[w];
+        }
+      }
+#pragma unroll
+      for (int u = 0; u < RB_U; ++u) {
+        const int i = i0 + 256 * u, r = i / pieces, x = i - r * pieces;
+        if (i >= RB_Q * pieces) break;
+        float q[4], k[4], q2[4], k2[4];
+        auto wide = [](const uint2& v, float (&o)[4]) {
+          const float2 lo = unpack_bf16(v.x), hi = unpack_bf16(v.y);
+          o[0] = lo.x; o[1] = lo.y; o[2] = hi.x; o[3] = hi.y;
+        };
+        wide(a[u][0], q);
+        wide(a[u][1], k);
+#pragma unroll
+        for (int w = 0; w < 4; ++w) k[w] *= p.k_scale;
+        if (x < pairs) {
+          wide(a[u][2], q2);
+          wide(a[u][3], k2);
+#pragma unroll
+          for (int w = 0; w < 4; ++w) {
+            const float2 cs = t[u][w];
+            const float b = q[w], d = q2[w], f = k[w], g = k2[w] * p.k_scale;
+            q[w] = b * cs.x - d * cs.y;
+            q2[w] = d * cs.x + b * cs.y;
+            k[w] = f * cs.x - g * cs.y;
+            k2[w] = g * cs.x + f * cs.y;
           }
+          put(r, x * 4, q, k);
+          put(r, x * 4 + half, q2, k2);
+        } else {
+          put(r, 2 * half + (x - pairs) * 4, q, k);
         }
-        put(r, c, q, k);
-        put(r, c + half, q2, k2);
-      } else {
-        const int c = 2 * half + (x - pairs) * 4;
-        if (r < nr && c < N) {
-          ldv<4>(qg + at + c, q);
-          ldv<4>(kg + at + c, k);
-#pragma unroll
-          for (int u = 0; u < 4; ++u) k[u] *= p.k_scale;
-        }
-        put(r, c, q, k);
       }
     }
-    for (int i = tid; i < RB_Q * (RB_P / 8); i += 128) {
+    for (int i = tid; i < RB_Q * (RB_P / 8); i += 256) {
       const int r = i / (RB_P / 8), c = (i % (RB_P / 8)) * 8;
       uint4 v = make_uint4(0u, 0u, 0u, 0u);
       if (r < nr && c < np) v = *reinterpret_cast<const uint4*>(vg + (size_t)(r0 + r) * p.ld + c);
@@ -316,81 +336,112 @@ retention_blocks_kernel(const __nv_bfloat16* __restrict__ z, const RetArgs p, in
       for (int hh = 0; hh < 2; ++hh) {
         uint32_t hi, lo;
         rb_split(st[j][2 * hh], st[j][2 * hh + 1], hi, lo);
-        const int off = (warp * 16 + gq + 8 * hh) * Cfg::NROW + (j * 8 + 2 * tq) * 2;
+        const int off = (wr * 16 + gq + 8 * hh) * Cfg::NROW + (n0 + j * 8 + 2 * tq) * 2;
         *reinterpret_cast<uint32_t*>(sm + Cfg::SH_OFF + off) = hi;
         *reinterpret_cast<uint32_t*>(sm + Cfg::SL_OFF + off) = lo;
       }
     __syncthreads();
-    // ---- this warp's 16 rows t: G = q k^T, o = q S^T
-    const int t0 = warp * 16;
-    float gm[8][4], o[RB_P / 8][4];
+    const int t0 = wr * 16;                                  // this warp's rows t
+    float* zs = reinterpret_cast<float*>(sm + Cfg::Z_OFF);
+    if (warp >= 4) {
+      // ---- a^(t + 1) q S^T
+      float o[RB_P / 8][4];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) gm[j][0] = gm[j][1] = gm[j][2] = gm[j][3] = o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+      for (int j = 0; j < RB_P / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
 #pragma unroll
-    for (int k = 0; k < KN; ++k) {
-      uint32_t qa[4], ql[4];
-      rb_mat(sb + Cfg::QH_OFF + (t0 + (mat & 1) * 8 + r8) * Cfg::NROW + (k * 16 + (mat >> 1) * 8) * 2, qa);
-      rb_mat(sb + Cfg::QL_OFF + (t0 + (mat & 1) * 8 + r8) * Cfg::NROW + (k * 16 + (mat >> 1) * 8) * 2, ql);
+      for (int k = 0; k < KN; ++k) {
+        uint32_t qa[4], ql[4];
+        rb_mat(sb + Cfg::QH_OFF + (t0 + (mat & 1) * 8 + r8) * Cfg::NROW + (k * 16 + (mat >> 1) * 8) * 2, qa);
+        rb_mat(sb + Cfg::QL_OFF + (t0 + (mat & 1) * 8 + r8) * Cfg::NROW + (k * 16 + (mat >> 1) * 8) * 2, ql);
+        uint32_t b[4][4];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const uint32_t off = (j * 16 + (mat >> 1) * 8 + r8) * Cfg::NROW + (k * 16 + (mat & 1) * 8) * 2;
-        uint32_t b[4];
-        if (j <= warp) {                                     // rows s of later 16-row groups are all in the future
+        for (int j = 0; j < 4; ++j) rb_mat(sb + Cfg::SH_OFF + (j * 16 + (mat >> 1) * 8 + r8) * Cfg::NROW + (k * 16 + (mat & 1) * 8) * 2, b[j]);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          rb_mma(o[2 * j], qa, b[j][0], b[j][1]);
+          rb_mma(o[2 * j + 1], qa, b[j][2], b[j][3]);
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          rb_mma(o[2 * j], ql, b[j][0], b[j][1]);
+          rb_mma(o[2 * j + 1], ql, b[j][2], b[j][3]);
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) rb_mat(sb + Cfg::SL_OFF + (j * 16 + (mat >> 1) * 8 + r8) * Cfg::NROW + (k * 16 + (mat & 1) * 8) * 2, b[j]);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          rb_mma(o[2 * j], qa, b[j][0], b[j][1]);
+          rb_mma(o[2 * j + 1], qa, b[j][2], b[j][3]);
+        }
+      }
+      if constexpr (NP >= 64) asm volatile("bar.sync 2, 128;" ::: "memory");       // these four have read the state's matrices
+      const float w0 = pw[t0 + gq + 1], w1 = pw[t0 + gq + 9];
+#pragma unroll
+      for (int j = 0; j < RB_P / 8; ++j) {
+        float* d = zs + (t0 + gq) * Cfg::ZROW + j * 8 + 2 * tq;
+        *reinterpret_cast<float2*>(d) = make_float2(o[j][0] * w0, o[j][1] * w0);
+        *reinterpret_cast<float2*>(d + 8 * Cfg::ZROW) = make_float2(o[j][2] * w1, o[j][3] * w1);
+      }
+      asm volatile("bar.arrive 1, 256;" ::: "memory");
+    } else {
+      // ---- G = q k^T, then (G weighted) v
+      float gm[8][4], o[RB_P / 8][4];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) gm[j][0] = gm[j][1] = gm[j][2] = gm[j][3] = o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+#pragma unroll
+      for (int k = 0; k < KN; ++k) {
+        uint32_t qa[4], ql[4];
+        rb_mat(sb + Cfg::QH_OFF + (t0 + (mat & 1) * 8 + r8) * Cfg::NROW + (k * 16 + (mat >> 1) * 8) * 2, qa);
+        rb_mat(sb + Cfg::QL_OFF + (t0 + (mat & 1) * 8 + r8) * Cfg::NROW + (k * 16 + (mat >> 1) * 8) * 2, ql);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          if (j > warp) break;                               // rows s of later 16-row groups are all in the future
+          const uint32_t off = (j * 16 + (mat >> 1) * 8 + r8) * Cfg::NROW + (k * 16 + (mat & 1) * 8) * 2;
+          uint32_t b[4], c[4];
           rb_mat(sb + Cfg::KH_OFF + off, b);
+          rb_mat(sb + Cfg::KL_OFF + off, c);
           rb_mma(gm[2 * j], qa, b[0], b[1]);
           rb_mma(gm[2 * j + 1], qa, b[2], b[3]);
           rb_mma(gm[2 * j], ql, b[0], b[1]);
           rb_mma(gm[2 * j + 1], ql, b[2], b[3]);
-          rb_mat(sb + Cfg::KL_OFF + off, b);
-          rb_mma(gm[2 * j], qa, b[0], b[1]);
-          rb_mma(gm[2 * j + 1], qa, b[2], b[3]);
+          rb_mma(gm[2 * j], qa, c[0], c[1]);
+          rb_mma(gm[2 * j + 1], qa, c[2], c[3]);
         }
-        rb_mat(sb + Cfg::SH_OFF + off, b);
-        rb_mma(o[2 * j], qa, b[0], b[1]);
-        rb_mma(o[2 * j + 1], qa, b[2], b[3]);
-        rb_mma(o[2 * j], ql, b[0], b[1]);
-        rb_mma(o[2 * j + 1], ql, b[2], b[3]);
-        rb_mat(sb + Cfg::SL_OFF + off, b);
-        rb_mma(o[2 * j], qa, b[0], b[1]);
-        rb_mma(o[2 * j + 1], qa, b[2], b[3]);
       }
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {                          // 16 columns s at a time: accumulators of G become the A operand
+        if (k > warp) break;
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {                        // x: (row half x & 1, column half x >> 1)
+          const int d = t0 + gq + (x & 1) * 8 - (k * 16 + (x >> 1) * 8 + 2 * tq);        // t - s of the first of two columns
+          const float* gv = &gm[2 * k + (x >> 1)][(x & 1) * 2];
+          rb_split(d >= 0 ? gv[0] * pw[max(d, 0)] : 0.f, d >= 1 ? gv[1] * pw[max(d - 1, 0)] : 0.f, hi[x], lo[x]);
+        }
+#pragma unroll
+        for (int j = 0; j < RB_P / 16; ++j) {
+          uint32_t b[4];
+          rb_mat_t(sb + Cfg::V_OFF + (k * 16 + (mat & 1) * 8 + r8) * Cfg::PROW + (j * 16 + (mat >> 1) * 8) * 2, b);
+          rb_mma(o[2 * j], hi, b[0], b[1]);
+          rb_mma(o[2 * j + 1], hi, b[2], b[3]);
+          rb_mma(o[2 * j], lo, b[0], b[1]);
+          rb_mma(o[2 * j + 1], lo, b[2], b[3]);
+        }
+      }
+      asm volatile("bar.sync 1, 256;" ::: "memory");         // the other warps' sums are there
+#pragma unroll
+      for (int j = 0; j < RB_P / 8; ++j)
+#pragma unroll
+        for (int hh = 0; hh < 2; ++hh) {
+          const int t = t0 + gq + 8 * hh, c = j * 8 + 2 * tq;
+          if (t < nr && c < np) {
+            const float2 z2 = *reinterpret_cast<const float2*>(zs + t * Cfg::ZROW + c);
+            *reinterpret_cast<float2*>(y + (size_t)(r0 - first + t) * p.H * P + (size_t)hd * P + p0 + c) =
+                make_float2(o[j][2 * hh] + z2.x, o[j][2 * hh + 1] + z2.y);
+          }
+        }
     }
-    const float w0 = pw[t0 + gq + 1], w1 = pw[t0 + gq + 9];
-#pragma unroll
-    for (int j = 0; j < RB_P / 8; ++j) {
-      o[j][0] *= w0; o[j][1] *= w0;
-      o[j][2] *= w1; o[j][3] *= w1;
-    }
-    // ---- o += (G weighted) v
-#pragma unroll
-    for (int k = 0; k < 4; ++k) {                            // 16 columns s at a time: accumulators of G become the A operand
-      if (k > warp) break;
-      uint32_t hi[4], lo[4];
-#pragma unroll
-      for (int x = 0; x < 4; ++x) {                          // x: (row half x & 1, column half x >> 1)
-        const int d = t0 + gq + (x & 1) * 8 - (k * 16 + (x >> 1) * 8 + 2 * tq);          // t - s of the first of two columns
-        const float* gv = &gm[2 * k + (x >> 1)][(x & 1) * 2];
-        rb_split(d >= 0 ? gv[0] * pw[max(d, 0)] : 0.f, d >= 1 ? gv[1] * pw[max(d - 1, 0)] : 0.f, hi[x], lo[x]);
-      }
-#pragma unroll
-      for (int j = 0; j < RB_P / 16; ++j) {
-        uint32_t b[4];
-        rb_mat_t(sb + Cfg::V_OFF + (k * 16 + (mat & 1) * 8 + r8) * Cfg::PROW + (j * 16 + (mat >> 1) * 8) * 2, b);
-        rb_mma(o[2 * j], hi, b[0], b[1]);
-        rb_mma(o[2 * j + 1], hi, b[2], b[3]);
-        rb_mma(o[2 * j], lo, b[0], b[1]);
-        rb_mma(o[2 * j + 1], lo, b[2], b[3]);
-      }
-    }
-#pragma unroll
-    for (int j = 0; j < RB_P / 8; ++j)
-#pragma unroll
-      for (int hh = 0; hh < 2; ++hh) {
-        const int t = t0 + gq + 8 * hh, c = j * 8 + 2 * tq;
-        if (t < nr && c < np)
-          *reinterpret_cast<float2*>(y + (size_t)(r0 - first + t) * p.H * P + (size_t)hd * P + p0 + c) = make_float2(o[j][2 * hh], o[j][2 * hh + 1]);
-      }
-    // ---- S <- a^n S + (weighted v)^T k over this warp's 16 channels
+    // ---- S <- a^n S + (weighted v)^T k over this warp's part
     const float dec = pw[nr];
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
@@ -400,7 +451,7 @@ retention_blocks_kernel(const __nv_bfloat16* __restrict__ z, const RetArgs p, in
     for (int k = 0; k < 4; ++k) {
       uint32_t va[4], hi[4], lo[4];
       // v^T: rows p, columns s; transposed 8 x 8 pieces (s half of the fragment = mat >> 1, p half = mat & 1)
-      rb_mat_t(sb + Cfg::V_OFF + (k * 16 + (mat >> 1) * 8 + r8) * Cfg::PROW + (warp * 16 + (mat & 1) * 8) * 2, va);
+      rb_mat_t(sb + Cfg::V_OFF + (k * 16 + (mat >> 1) * 8 + r8) * Cfg::PROW + (t0 + (mat & 1) * 8) * 2, va);
 #pragma unroll
       for (int x = 0; x < 4; ++x) {
         const int d = nr - 1 - (k * 16 + (x >> 1) * 8 + 2 * tq);          // rows past the end are zero
@@ -408,8 +459,8 @@ retention_blocks_kernel(const __nv_bfloat16* __restrict__ z, const RetArgs p, in
         rb_split(v.x * pw[max(d, 0)], v.y * pw[max(d - 1, 0)], hi[x], lo[x]);
       }
 #pragma unroll
-      for (int j = 0; j < NP / 16; ++j) {
-        const uint32_t off = (k * 16 + (mat & 1) * 8 + r8) * Cfg::NROW + (j * 16 + (mat >> 1) * 8) * 2;
+      for (int j = 0; j < NT / 2; ++j) {
+        const uint32_t off = (k * 16 + (mat & 1) * 8 + r8) * Cfg::NROW + (n0 + j * 16 + (mat >> 1) * 8) * 2;
         uint32_t b[4];
         rb_mat_t(sb + Cfg::KH_OFF + off, b);
         rb_mma(st[2 * j], hi, b[0], b[1]);
@@ -427,7 +478,7 @@ retention_blocks_kernel(const __nv_bfloat16* __restrict__ z, const RetArgs p, in
   for (int j = 0; j < NT; ++j)
 #pragma unroll
     for (int hh = 0; hh < 2; ++hh) {
-      const int c = warp * 16 + gq + 8 * hh, n = j * 8 + 2 * tq;
+      const int c = wr * 16 + gq + 8 * hh, n = n0 + j * 8 + 2 * tq;
       if (c < np && n < N) *reinterpret_cast<float2*>(Sg + (size_t)c * N + n) = make_float2(st[j][2 * hh], st[j][2 * hh + 1]);
     }
 }
@@ -463,7 +514,7 @@ static int launch_blocks(const __nv_bfloat16* z, const RetArgs& a, int e0, int E
   auto kern = retention_blocks_kernel<NP>;
   static ab2host::DevState st;
   if (ab2host::prepare_launch(kern, RetCfg<NP>::SMEM, st, nullptr)) return 300;
-  kern<<<dim3(E - e0, a.H, (a.P + RB_P - 1) / RB_P), 128, RetCfg<NP>::SMEM, s>>>(z, a, e0, y);
+  kern<<<dim3(E - e0, a.H, (a.P + RB_P - 1) / RB_P), 256, RetCfg<NP>::SMEM, s>>>(z, a.rot, a, e0, y);
   return cudaGetLastError() == cudaSuccess ? 0 : 302;
 }
 

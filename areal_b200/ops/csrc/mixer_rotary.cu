@@ -4,6 +4,8 @@
 //   latent_rope_append    norm of the cached latent and rotation of the key part behind it, both into the cache; rotation of the
 //                         queries' second part in place
 // Pairs are (i, i + half) of the rotated stretch, or (2 i, 2 i + 1) when interleaved.
+#include <type_traits>
+
 #include "mixer_common.cuh"
 
 namespace ab2 {
@@ -25,7 +27,7 @@ rotary_table_kernel(const int* __restrict__ pos, const double* __restrict__ freq
   }
 }
 
-// One CTA per row, a warp per head.
+// One CTA per row, a warp per head, any sizes.
 template <typename T, int V, bool INTERLEAVED>
 __global__ void __launch_bounds__(256)
 qk_head_norm_append_kernel(const T* __restrict__ z, long long ld, const float* __restrict__ wq, const float* __restrict__ wk,
@@ -46,24 +48,43 @@ qk_head_norm_append_kernel(const T* __restrict__ z, long long ld, const float* _
     for (int c = lane * V; c < D; c += 32 * V) {
       float v[V];
       ldv<V>(src + (size_t)u * D + c, v);
+#pragma unroll
       for (int e = 0; e < V; ++e) ss += v[e] * v[e];
       stv<V>(x + c, v);
     }
     const float rstd = w != nullptr ? 1.f / sqrtf(warp_sum(ss) / D + eps) : 1.f;
     __syncwarp();
     T* dst = u < Hq ? q + ((size_t)row * Hq + u) * D : kc + ((size_t)slot * Hkv + u - Hq) * D;
-    auto val = [&](int c) { return x[c] * rstd * (w != nullptr ? w[c] : 1.f); };
-    for (int c = lane * V; c < D; c += 32 * V) {
-      float v[V];
+    auto normed = [&](int c, float (&v)[V]) {
+      ldv<V>(x + c, v);
+      if (w != nullptr) {
+        float g[V];
+        ldv<V>(w + c, g);
 #pragma unroll
-      for (int e = 0; e < V; ++e) {
-        const int d = c + e;
-        v[e] = val(d);
-        if (d < 2 * half) {
-          const bool first = INTERLEAVED ? !(d & 1) : d < half;
-          const float2 r = cs[INTERLEAVED ? d >> 1 : (first ? d : d - half)];
-          const float o = val(INTERLEAVED ? d ^ 1 : (first ? d + half : d - half));
-          v[e] = first ? v[e] * r.x - o * r.y : v[e] * r.x + o * r.y;
+        for (int e = 0; e < V; ++e) v[e] *= rstd * g[e];
+      }
+    };
+    for (int c = lane * V; c < D; c += 32 * V) {              // V numbers turn together or not at all
+      float v[V], o[V];
+      normed(c, v);
+      if (c < 2 * half) {
+        if constexpr (INTERLEAVED && V > 1) {
+#pragma unroll
+          for (int e = 0; e < V; e += 2) {
+            const float2 r = cs[(c + e) >> 1];
+            const float a = v[e], b = v[e + 1];
+            v[e] = a * r.x - b * r.y;
+            v[e + 1] = b * r.x + a * r.y;
+          }
+        } else {
+          const bool first = INTERLEAVED ? !(c & 1) : c < half;
+          normed(INTERLEAVED ? c ^ 1 : (first ? c + half : c - half), o);
+          const float2* r = cs + (INTERLEAVED ? c >> 1 : (first ? c : c - half));
+#pragma unroll
+          for (int e = 0; e < V; ++e) {
+            const float2 t = r[e];
+            v[e] = v[e] * t.x + (first ? -o[e] : o[e]) * t.y;
+          }
         }
       }
       stv<V>(dst + c, v);
@@ -76,6 +97,77 @@ qk_head_norm_append_kernel(const T* __restrict__ z, long long ld, const float* _
       float v[V];
       ldv<V>(sv + c, v);
       stv<V>(vc + (size_t)slot * nv + c, v);
+    }
+  }
+}
+
+// The same for heads of up to 128 numbers, four to a lane: weights and angles of a lane stay in its registers, partners come
+// from another lane, and a warp has several heads on their way.
+constexpr int QK_U = 4;
+
+template <typename T, bool INTERLEAVED>
+__global__ void __launch_bounds__(256)
+qk_head_norm_append_lanes_kernel(const T* __restrict__ z, long long ld, const float* __restrict__ wq, const float* __restrict__ wk,
+                                 const float2* __restrict__ rot, int ldr, int half, const int* __restrict__ slots, T* __restrict__ q, T* __restrict__ kc,
+                                 T* __restrict__ vc, int Hq, int Hkv, int D, int nv, float eps) {
+  pdl_wait();
+  pdl_trigger();
+  const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5, c = lane * 4;
+  const int slot = slots[row], heads = slot >= 0 ? Hq + Hkv : Hq;
+  const T* src = z + (size_t)row * ld;
+  const bool in = c < D, turns = c < 2 * half, first = c < half;
+  const int step = half / 4, partner = turns ? (first ? lane + step : lane - step) : lane;
+  float gq[4], gk[4];
+  float2 cs[4];
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    gq[e] = in && wq != nullptr ? wq[c + e] : 1.f;
+    gk[e] = in && wk != nullptr ? wk[c + e] : 1.f;
+    cs[e] = make_float2(1.f, 0.f);
+    if (turns && (!INTERLEAVED || e < 2)) cs[e] = rot[(size_t)row * ldr + (INTERLEAVED ? (c >> 1) + e : (first ? c : c - half) + e)];
+    if (!INTERLEAVED && first) cs[e].y = -cs[e].y;
+  }
+  for (int u0 = warp; u0 < heads; u0 += QK_U * nw) {
+    float v[QK_U][4];
+#pragma unroll
+    for (int i = 0; i < QK_U; ++i) {
+      const int u = u0 + i * nw;
+      v[i][0] = v[i][1] = v[i][2] = v[i][3] = 0.f;
+      if (u < heads && in) ldv<4>(src + (size_t)u * D + c, v[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < QK_U; ++i) {
+      const int u = u0 + i * nw;
+      if (u >= heads) break;
+      const float ss = warp_sum(v[i][0] * v[i][0] + v[i][1] * v[i][1] + v[i][2] * v[i][2] + v[i][3] * v[i][3]);
+      const bool is_q = u < Hq;
+      const float rstd = (is_q ? wq : wk) != nullptr ? 1.f / sqrtf(ss / D + eps) : 1.f;
+      float x[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) x[e] = v[i][e] * rstd * (is_q ? gq[e] : gk[e]);
+      if constexpr (INTERLEAVED) {
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+          const float a = x[e], b = x[e + 1];
+          x[e] = a * cs[e / 2].x - b * cs[e / 2].y;
+          x[e + 1] = b * cs[e / 2].x + a * cs[e / 2].y;
+        }
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float o = __shfl_sync(0xffffffffu, x[e], partner);
+          x[e] = x[e] * cs[e].x + o * cs[e].y;
+        }
+      }
+      if (in) stv<4>((is_q ? q + ((size_t)row * Hq + u) * D : kc + ((size_t)slot * Hkv + u - Hq) * D) + c, x);
+    }
+  }
+  if (slot >= 0) {
+    const T* sv = src + (size_t)(Hq + Hkv) * D;
+    for (int i = threadIdx.x * 4; i < nv; i += blockDim.x * 4) {
+      float v[4];
+      ldv<4>(sv + i, v);
+      stv<4>(vc + (size_t)slot * nv + i, v);
     }
   }
 }
@@ -98,10 +190,28 @@ latent_rope_append_kernel(T* __restrict__ z, long long ld, const float* __restri
     stf(to + a, u * r.x - v * r.y);
     stf(to + b, v * r.x + u * r.y);
   };
-  for (int k = tid; k < H * half; k += 256) {
-    const int h = k / half;
-    T* p = src + (size_t)h * (D + 2 * half) + D;
-    turn(p, p, k - h * half);
+  if constexpr (V == 8 && INTERLEAVED) {                      // four pairs at a time
+    const int per = half / 4;
+    for (int k = tid; k < H * per; k += 256) {
+      const int h = k / per, c = (k - h * per) * 8;
+      T* p = src + (size_t)h * (D + 2 * half) + D + c;
+      float v[8];
+      ldv<8>(p, v);
+#pragma unroll
+      for (int e = 0; e < 8; e += 2) {
+        const float2 r = cs[(c + e) >> 1];
+        const float a = v[e], b = v[e + 1];
+        v[e] = a * r.x - b * r.y;
+        v[e + 1] = b * r.x + a * r.y;
+      }
+      stv<8>(p, v);
+    }
+  } else {
+    for (int k = tid; k < H * half; k += 256) {
+      const int h = k / half;
+      T* p = src + (size_t)h * (D + 2 * half) + D;
+      turn(p, p, k - h * half);
+    }
   }
   if (slot < 0) return;
   const T* lat = src + (size_t)H * (D + 2 * half);
@@ -167,7 +277,22 @@ int ab2_qk_head_norm_append(const void* z, long long ld, const float* wq, const 
   const size_t smem = (size_t)8 * ((D + 3) & ~3) * 4;
   if (2 * half > D || half < 0 || smem > 48 * 1024) return 10;
   const int eb = dt == 0 ? 2 : 4;
-  auto fits = [&](int v) { return D % v == 0 && nv % v == 0 && ld % v == 0 && aligned_to(z, v * eb) && aligned_to(q, v * eb) && aligned_to(kc, v * eb) && aligned_to(vc, v * eb); };
+  auto fits = [&](int v) {
+    return D % v == 0 && nv % v == 0 && ld % v == 0 && (interleaved ? 2 * half : half) % v == 0 && aligned_to(z, v * eb) && aligned_to(q, v * eb) &&
+           aligned_to(kc, v * eb) && aligned_to(vc, v * eb) && aligned_to(wq, 16) && aligned_to(wk, 16);
+  };
+  if (D <= 128 && fits(4)) {
+    auto go = [&](auto t, auto inter) {
+      using T = decltype(t);
+      launch_pdl(qk_head_norm_append_lanes_kernel<T, decltype(inter)::value>, dim3(R), dim3(256), 0, (cudaStream_t)stream, (const T*)z, ld, wq, wk,
+                 (const float2*)rot, ldr, half, slots, (T*)q, (T*)kc, (T*)vc, Hq, Hkv, D, nv, eps);
+    };
+    if (dt == 0 && interleaved) go(__nv_bfloat16(), std::true_type());
+    else if (dt == 0) go(__nv_bfloat16(), std::false_type());
+    else if (interleaved) go(0.f, std::true_type());
+    else go(0.f, std::false_type());
+    return cudaGetLastError() == cudaSuccess ? 0 : 1;
+  }
   AB2_ROT_TYPED(dt, fits(8), fits(4), interleaved, {
     launch_pdl(qk_head_norm_append_kernel<T, V, INTER>, dim3(R), dim3(256), smem, (cudaStream_t)stream, (const T*)z, ld, wq, wk, (const float2*)rot, ldr,
                half, slots, (T*)q, (T*)kc, (T*)vc, Hq, Hkv, D, nv, eps);
@@ -182,7 +307,7 @@ int ab2_latent_rope_append(void* z, long long ld, const float* wc, const void* r
   if (half < 1 || C < 1) return 10;
   const int eb = dt == 0 ? 2 : 4;
   auto fits = [&](int v) {
-    return C % v == 0 && (2 * half) % v == 0 && ld % v == 0 && (H * (D + 2 * half)) % v == 0 && aligned_to(z, v * eb) && aligned_to(cache, v * eb) && aligned_to(wc, 16);
+    return C % v == 0 && D % v == 0 && (2 * half) % v == 0 && ld % v == 0 && aligned_to(z, v * eb) && aligned_to(cache, v * eb) && aligned_to(wc, 16);
   };
   AB2_ROT_TYPED(dt, fits(8), fits(4), interleaved, {
     launch_pdl(latent_rope_append_kernel<T, V, INTER>, dim3(R), dim3(256), 0, (cudaStream_t)stream, (T*)z, ld, wc, (const float2*)rot, ldr, half, slots,
