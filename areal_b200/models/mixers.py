@@ -585,13 +585,16 @@ class Design:
     mlps: dict                   # feed-forward kinds
     layer_norms: tuple           # norms of a layer with a feed-forward ...
     layer_norms_bare: tuple      # ... and of one without
+    kernels: tuple               # sources of its mixers' kernels (beside those of every stack)
 
 
 DESIGNS = {
     "kagolix": Design("Kagolix", {"attention": ChunkAttention, "rglru": RGLRU, "mamba2": Mamba2}, {"dense": XieluMLP, "moe": RoutedMLP}, ("norm1", "norm1b", "norm2", "norm2b"),
-                      ("norm1", "norm1b")),
-    "vogilix": Design("Vogilix", {"latent_attention": LatentAttention}, {"dense": GeluMLP, "moe": InputWeightedMLP}, ("norm1", "norm2"), ("norm1",)),
-    "bumotar": Design("Bumotar", {"latent_attention": RotaryLatentAttention, "parallel": Parallel}, {"moe": SharedExpertMLP}, ("norm1", "norm2"), ("norm1",)),
+                      ("norm1", "norm1b"), ("mixer_attention", "mixer_scan", "mixer_ssd")),
+    "vogilix": Design("Vogilix", {"latent_attention": LatentAttention}, {"dense": GeluMLP, "moe": InputWeightedMLP}, ("norm1", "norm2"), ("norm1",),
+                      ("mixer_attention", "mixer_latent")),
+    "bumotar": Design("Bumotar", {"latent_attention": RotaryLatentAttention, "parallel": Parallel}, {"moe": SharedExpertMLP}, ("norm1", "norm2"), ("norm1",),
+                      ("mixer_attention", "mixer_latent", "mixer_retention", "mixer_rotary")),
 }
 
 

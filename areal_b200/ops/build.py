@@ -22,10 +22,9 @@ HERE = Path(__file__).resolve().parent
 CSRC = HERE / "csrc"
 BUILD = HERE / "build"
 LIB = HERE / "libab2_kernels.so"
-# the kernels that serve a mixer stack, linked alone: what a fresh checkout compiles before its first trace
-STEP_LIB = HERE / "libab2_step.so"
-STEP_SOURCES = ("runtime", "gemm", "gemm2sm", "gemm_grouped", "router", "infer", "mixer_attention", "mixer_latent", "mixer_ops",
-                "mixer_retention", "mixer_rotary", "mixer_scan", "mixer_ssd")
+# the kernels that serve any mixer stack; with those of a design's own mixers, linked alone, they are what a fresh checkout
+# compiles before its first trace
+STEP_SOURCES = ("runtime", "gemm", "gemm2sm", "gemm_grouped", "router", "infer", "mixer_ops")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -65,9 +64,10 @@ def is_current(lib: Path = LIB, names=None) -> bool:
     return stamp.read_text().strip() == _digest(sources(names) + _headers())
 
 
-def build_step_library() -> Path:
-    """The library a mixer stack is served from: the whole one when it is up to date, else its own subset."""
-    return LIB if is_current() else build(lib=STEP_LIB, names=STEP_SOURCES)
+def build_step_library(design: str, own: tuple) -> Path:
+    """The library a mixer stack is served from: the whole one when it is up to date, else the sources of every stack and the
+    design's ``own``."""
+    return LIB if is_current() else build(lib=HERE / f"libab2_step_{design}.so", names=STEP_SOURCES + own)
 
 
 def build(force: bool = False, verbose: bool = False, lib: Path = LIB, names=None) -> Path:

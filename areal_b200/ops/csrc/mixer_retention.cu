@@ -193,7 +193,7 @@ retention_scan_kernel(const T* __restrict__ z, const RetArgs p, int e0, float* _
 // v is bf16; the rotated q and k, the weights and S are fp32 and enter a product as the sum of two bf16 numbers (rounding and rest,
 // without the product of two rests); accumulation is fp32. An output is divided by its own size afterwards, so what a
 // small q . k loses would show.
-constexpr int RB_Q = 64, RB_P = 64, RB_U = 4;
+constexpr int RB_Q = 64, RB_P = 64;
 
 __device__ __forceinline__ void rb_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
@@ -229,6 +229,7 @@ __global__ void __launch_bounds__(256, NP == 128 ? 1 : 2)
 retention_blocks_kernel(const __nv_bfloat16* __restrict__ z, const float2* __restrict__ rot, const RetArgs p, int e0, float* __restrict__ y) {
   using Cfg = RetCfg<NP>;
   constexpr int NT = NP / 16, KN = NP / 16;                   // tiles of 8 in half of the columns, k-steps of 16 in all
+  constexpr int U = NP / 32;                                  // pieces of q and k of a thread when whole heads turn
   extern __shared__ __align__(16) unsigned char sm[];
   const uint32_t sb = smem_u32(sm);
   float* pw = reinterpret_cast<float*>(sm + Cfg::A_OFF);
@@ -257,78 +258,96 @@ retention_blocks_kernel(const __nv_bfloat16* __restrict__ z, const float2* __res
     }
   if (tid <= RB_Q) pw[tid] = exp2f(p.log2_decay[hd] * (float)tid);
   const int pairs = half / 4, pieces = pairs + (NP - 2 * half) / 4;       // of a row: four pairs, or four numbers that do not turn
+  // A block's rows are on their way while the block before is worked on: U pieces of q and k and two of v per thread.
+  uint2 a[U][4];                                          // q, k; q and k half a turn further on, or nothing
+  float2 t[U][4];
+  uint4 vr[2];
+  auto fetch = [&](int r0, int i0) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + 256 * u, r = i / pieces, x = i - r * pieces, c = x < pairs ? x * 4 : 2 * half + (x - pairs) * 4;
+      const size_t at = (size_t)(r0 + r) * p.ld + c;
+      a[u][0] = a[u][1] = a[u][2] = a[u][3] = make_uint2(0u, 0u);
+      t[u][0] = t[u][1] = t[u][2] = t[u][3] = make_float2(0.f, 0.f);
+      if (r >= RB_Q || r0 + r >= r_end || c >= N) continue;
+      a[u][0] = *reinterpret_cast<const uint2*>(qg + at);
+      a[u][1] = *reinterpret_cast<const uint2*>(kg + at);
+      if (x < pairs) {
+        a[u][2] = *reinterpret_cast<const uint2*>(qg + at + half);
+        a[u][3] = *reinterpret_cast<const uint2*>(kg + at + half);
+        const float2* cs = rot + (size_t)(r0 + r) * p.ldr + c;
+#pragma unroll
+        for (int w = 0; w < 4; ++w) t[u][w] = cs[w];
+      }
+    }
+  };
+  auto fetch_v = [&](int r0) {
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int i = tid + 256 * u, r = i >> 3, c = (i & 7) * 8;
+      vr[u] = make_uint4(0u, 0u, 0u, 0u);
+      if (r0 + r < r_end && c < np) vr[u] = *reinterpret_cast<const uint4*>(vg + (size_t)(r0 + r) * p.ld + c);
+    }
+  };
+  auto put = [&](int r, int c, const float (&q)[4], const float (&k)[4]) {
+    const int off = r * Cfg::NROW + c * 2;
+    uint2 hi, lo;
+    rb_split(q[0], q[1], hi.x, lo.x);
+    rb_split(q[2], q[3], hi.y, lo.y);
+    *reinterpret_cast<uint2*>(sm + Cfg::QH_OFF + off) = hi;
+    *reinterpret_cast<uint2*>(sm + Cfg::QL_OFF + off) = lo;
+    rb_split(k[0], k[1], hi.x, lo.x);
+    rb_split(k[2], k[3], hi.y, lo.y);
+    *reinterpret_cast<uint2*>(sm + Cfg::KH_OFF + off) = hi;
+    *reinterpret_cast<uint2*>(sm + Cfg::KL_OFF + off) = lo;
+  };
+  auto store = [&](int i0) {                                 // turned, as two bf16 matrices each
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + 256 * u, r = i / pieces, x = i - r * pieces;
+      if (r >= RB_Q) break;
+      float q[4], k[4], q2[4], k2[4];
+      auto wide = [](const uint2& v, float (&o)[4]) {
+        const float2 lo = unpack_bf16(v.x), hi = unpack_bf16(v.y);
+        o[0] = lo.x; o[1] = lo.y; o[2] = hi.x; o[3] = hi.y;
+      };
+      wide(a[u][0], q);
+      wide(a[u][1], k);
+#pragma unroll
+      for (int w = 0; w < 4; ++w) k[w] *= p.k_scale;
+      if (x < pairs) {
+        wide(a[u][2], q2);
+        wide(a[u][3], k2);
+#pragma unroll
+        for (int w = 0; w < 4; ++w) {
+          const float2 cs = t[u][w];
+          const float b = q[w], d = q2[w], f = k[w], g = k2[w] * p.k_scale;
+          q[w] = b * cs.x - d * cs.y;
+          q2[w] = d * cs.x + b * cs.y;
+          k[w] = f * cs.x - g * cs.y;
+          k2[w] = g * cs.x + f * cs.y;
+        }
+        put(r, x * 4, q, k);
+        put(r, x * 4 + half, q2, k2);
+      } else {
+        put(r, 2 * half + (x - pairs) * 4, q, k);
+      }
+    }
+  };
+  fetch(p.cu[e], tid);
+  fetch_v(p.cu[e]);
   for (int r0 = p.cu[e]; r0 < r_end; r0 += RB_Q) {
     const int nr = min(RB_Q, r_end - r0);
     // ---- q, k (turned) and v of the block (rows past the end: zero), the state as two bf16 matrices
-    auto put = [&](int r, int c, const float (&q)[4], const float (&k)[4]) {
-      const int off = r * Cfg::NROW + c * 2;
-      uint2 hi, lo;
-      rb_split(q[0], q[1], hi.x, lo.x);
-      rb_split(q[2], q[3], hi.y, lo.y);
-      *reinterpret_cast<uint2*>(sm + Cfg::QH_OFF + off) = hi;
-      *reinterpret_cast<uint2*>(sm + Cfg::QL_OFF + off) = lo;
-      rb_split(k[0], k[1], hi.x, lo.x);
-      rb_split(k[2], k[3], hi.y, lo.y);
-      *reinterpret_cast<uint2*>(sm + Cfg::KH_OFF + off) = hi;
-      *reinterpret_cast<uint2*>(sm + Cfg::KL_OFF + off) = lo;
-    };
-    for (int i0 = tid; i0 < RB_Q * pieces; i0 += 256 * RB_U) {
-      uint2 a[RB_U][4];                                      // q, k; q and k half a turn further on, or nothing
-      float2 t[RB_U][4];
-#pragma unroll
-      for (int u = 0; u < RB_U; ++u) {                       // RB_U pieces on their way at a time
-        const int i = i0 + 256 * u, r = i / pieces, x = i - r * pieces, c = x < pairs ? x * 4 : 2 * half + (x - pairs) * 4;
-        const size_t at = (size_t)(r0 + r) * p.ld + c;
-        a[u][0] = a[u][1] = a[u][2] = a[u][3] = make_uint2(0u, 0u);
-        t[u][0] = t[u][1] = t[u][2] = t[u][3] = make_float2(0.f, 0.f);
-        if (r >= nr || c >= N) continue;
-        a[u][0] = *reinterpret_cast<const uint2*>(qg + at);
-        a[u][1] = *reinterpret_cast<const uint2*>(kg + at);
-        if (x < pairs) {
-          a[u][2] = *reinterpret_cast<const uint2*>(qg + at + half);
-          a[u][3] = *reinterpret_cast<const uint2*>(kg + at + half);
-          const float2* cs = rot + (size_t)(r0 + r) * p.ldr + c;
-#pragma unroll
-          for (int w = 0; w < 4; ++w) t[u][w] = cs[w];
-        }
-      }
-#pragma unroll
-      for (int u = 0; u < RB_U; ++u) {
-        const int i = i0 + 256 * u, r = i / pieces, x = i - r * pieces;
-        if (i >= RB_Q * pieces) break;
-        float q[4], k[4], q2[4], k2[4];
-        auto wide = [](const uint2& v, float (&o)[4]) {
-          const float2 lo = unpack_bf16(v.x), hi = unpack_bf16(v.y);
-          o[0] = lo.x; o[1] = lo.y; o[2] = hi.x; o[3] = hi.y;
-        };
-        wide(a[u][0], q);
-        wide(a[u][1], k);
-#pragma unroll
-        for (int w = 0; w < 4; ++w) k[w] *= p.k_scale;
-        if (x < pairs) {
-          wide(a[u][2], q2);
-          wide(a[u][3], k2);
-#pragma unroll
-          for (int w = 0; w < 4; ++w) {
-            const float2 cs = t[u][w];
-            const float b = q[w], d = q2[w], f = k[w], g = k2[w] * p.k_scale;
-            q[w] = b * cs.x - d * cs.y;
-            q2[w] = d * cs.x + b * cs.y;
-            k[w] = f * cs.x - g * cs.y;
-            k2[w] = g * cs.x + f * cs.y;
-          }
-          put(r, x * 4, q, k);
-          put(r, x * 4 + half, q2, k2);
-        } else {
-          put(r, 2 * half + (x - pairs) * 4, q, k);
-        }
-      }
+    store(tid);
+    for (int i0 = tid + 256 * U; i0 < RB_Q * pieces; i0 += 256 * U) {        // heads that hardly turn have more pieces
+      fetch(r0, i0);
+      store(i0);
     }
-    for (int i = tid; i < RB_Q * (RB_P / 8); i += 256) {
-      const int r = i / (RB_P / 8), c = (i % (RB_P / 8)) * 8;
-      uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (r < nr && c < np) v = *reinterpret_cast<const uint4*>(vg + (size_t)(r0 + r) * p.ld + c);
-      *reinterpret_cast<uint4*>(sm + Cfg::V_OFF + r * Cfg::PROW + c * 2) = v;
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int i = tid + 256 * u;
+      *reinterpret_cast<uint4*>(sm + Cfg::V_OFF + (i >> 3) * Cfg::PROW + (i & 7) * 16) = vr[u];
     }
 #pragma unroll
     for (int j = 0; j < NT; ++j)
@@ -341,6 +360,10 @@ retention_blocks_kernel(const __nv_bfloat16* __restrict__ z, const float2* __res
         *reinterpret_cast<uint32_t*>(sm + Cfg::SL_OFF + off) = lo;
       }
     __syncthreads();
+    if (r0 + RB_Q < r_end) {
+      fetch(r0 + RB_Q, tid);
+      fetch_v(r0 + RB_Q);
+    }
     const int t0 = wr * 16;                                  // this warp's rows t
     float* zs = reinterpret_cast<float*>(sm + Cfg::Z_OFF);
     if (warp >= 4) {

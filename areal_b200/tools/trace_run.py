@@ -86,10 +86,14 @@ def main(argv=None) -> int:
     if not torch.cuda.is_available():
         print("trace_run needs a CUDA device", file=sys.stderr)
         return 1
+    from ..models.config import ModelConfig
+    from ..models.mixers import DESIGNS
     from ..ops import build as kbuild
     from ..ops import lib as oplib
 
-    oplib.use_library(kbuild.build_step_library())
+    cfg = ModelConfig.from_pretrained(a.model)
+    if cfg.is_mixer_stack:
+        oplib.use_library(kbuild.build_step_library(cfg.arch, DESIGNS[cfg.arch].kernels))
     torch.cuda.set_device(0)
     os.makedirs(a.out, exist_ok=True)
     engine = make_engine(a.model, a.dtype, a.max_tokens)

@@ -683,6 +683,14 @@ def test_checkpoint_names_and_shapes_are_the_design_s():
         assert {n: tuple(t.shape) for n, t in back.items()} == {n: tuple(t.shape) for n, t in W.items()}
 
 
+def test_designs_name_their_kernel_sources():
+    from areal_b200.ops import build
+
+    for d in mixers.DESIGNS.values():
+        names = build.STEP_SOURCES + d.kernels
+        assert len(build.sources(names)) == len(set(names)) == len(names)
+
+
 def test_every_pass_has_pages_and_states_of_its_own():
     mc = preset("tiny-bumotar")                        # four layers, the middle two twice
     model = build_model(mc, dtype=torch.float32, seed=1)
