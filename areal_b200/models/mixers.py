@@ -21,9 +21,9 @@ The sum x stays in 32 bits in all of them. The mixers
   queries and keys, capped scores, a sink and gated channels; retention (linear attention with a fixed decay per head);
 
 and the feed-forwards (dense with xIELU or the exact GELU; experts behind a softmax or a sigmoid router, weighted at their
-output or at their input, with or without a gated shared expert) are built from the ops of :mod:`..ops.mixer_ops`. A forward pass runs the rows of one step
-(:class:`~..ops.mixer_ops.RaggedBatch`) from the pages and state slots of :class:`~..engine.state_cache.StateCache`; whole
-prompts, portions and single tokens are the same call.
+output or at their input, with or without a gated shared expert) are built from the ops of :mod:`..ops.mixer_ops`. A forward
+pass runs the rows of one step (:class:`~..ops.mixer_ops.RaggedBatch`) from the pages and state slots of
+:class:`~..engine.state_cache.StateCache`; whole prompts, portions and single tokens are the same call.
 
 Matrices are stored in the model's dtype, everything that is used in 32 bits (norm weights, biases, taps, decay and bias
 parameters) as fp32. Serving only: there is no backward pass.

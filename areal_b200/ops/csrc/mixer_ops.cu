@@ -1,9 +1,8 @@
 // Elementwise, norm, convolution and small-product kernels of mixer stacks (bf16 or fp32 activations, fp32 residual
-// stream, norm weights and states): grouped sandwich norms, norms behind a sublayer and residual sums before a norm (both fused
-// with the expert sum), whole-
-// projection q / k norms fused with the cache append, causal convolutions with carried tails, xIELU, GELU, SiLU gate,
-// clamped gated units, token side gate, expert combine, capped logits, and a plain grouped product for 32-bit experts
-// and odd sizes.
+// stream, norm weights and states): grouped sandwich norms, norms behind a sublayer and residual sums before a norm (both
+// fused with the expert sum), whole-projection q / k norms fused with the cache append, causal convolutions with carried
+// tails, xIELU, GELU, SiLU gate, clamped gated units, token side gate, expert combine, capped logits, and a plain grouped
+// product for 32-bit experts and odd sizes.
 #include "mixer_common.cuh"
 
 namespace ab2 {
