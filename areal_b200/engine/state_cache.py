@@ -2,6 +2,7 @@
 values, or of latents, per attention layer, one state slot per request for the recurrent layers)."""
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
 from typing import Optional
 
@@ -55,17 +56,22 @@ class Carried:
     length: int = 0              # tokens absorbed
 
 
+SLOT_STATES = ("tail", "state", "shift")       # what a layer may keep per request
+
+
 class LayerCache:
-    __slots__ = ("k", "v", "tail", "state")
+    __slots__ = ("k", "v", "key_factor") + SLOT_STATES
 
     def __init__(self):
-        self.k = self.v = self.tail = self.state = None
+        for name in self.__slots__:
+            setattr(self, name, None)
 
 
 class StateCache(PagePool):
     """Pages for the attention layers (``[pages * page_size, heads, dim]`` of K and V per layer, each with its own sizes; a
-    layer whose keys and values come from one latent has K only) and fp32 slots for the recurrent ones (convolution tails,
-    recurrence states). A slot is not cleared when it changes hands: kernels take the state of a request that has absorbed
+    layer whose keys and values come from one latent, or whose keys are its values, has K only, and a number per key beside it
+    when keys are normed as they are read) and fp32 slots for what else a layer carries (convolution tails, recurrence states,
+    the row before for a token shift). A slot is not cleared when it changes hands: kernels take the state of a request that has absorbed
     nothing as zero."""
 
     def __init__(self, mixers: list, num_pages: int, page_size: int, num_slots: int, device, dtype):
@@ -75,13 +81,15 @@ class StateCache(PagePool):
         self._sight: dict = {}       # attention layers that see the same stretch of positions, once each
         self.windows: set = set()    # sliding windows of the latent layers
         for mx in mixers:
-            lc, shapes = LayerCache(), mx.cache_shapes()
+            lc, shapes = LayerCache(), mx.memory()
             if "kv" in shapes:
                 lc.k, lc.v = (None if s is None else torch.zeros(num_pages * page_size, *s, device=device, dtype=dtype) for s in shapes["kv"])
+                if "key_factor" in shapes:
+                    lc.key_factor = torch.zeros(num_pages * page_size, *shapes["key_factor"], device=device, dtype=torch.float32)
                 self._sight[type(mx), mx.span] = mx
-                if lc.v is None:
+                if mx.lists_pages:
                     self.windows.add(mx.span)
-            for name in ("tail", "state"):
+            for name in SLOT_STATES:
                 if name in shapes:
                     setattr(lc, name, torch.zeros(num_slots, *shapes[name], device=device, dtype=torch.float32))
             self.layers.append(lc)
@@ -93,19 +101,15 @@ class StateCache(PagePool):
 
     @staticmethod
     def bytes_per_page(mixers: list, page_size: int, elem: int) -> int:
-        return sum(s[0] * s[1] for mx in mixers for s in mx.cache_shapes().get("kv", ()) if s) * page_size * elem
+        n = 0
+        for mx in mixers:
+            shapes = mx.memory()
+            n += sum(s[0] * s[1] for s in shapes.get("kv", ()) if s) * elem + sum(shapes.get("key_factor", ())) * 4
+        return n * page_size
 
     @staticmethod
     def bytes_per_slot(mixers: list) -> int:
-        n = 0
-        for mx in mixers:
-            for name, s in mx.cache_shapes().items():
-                if name != "kv":
-                    k = 4
-                    for d in s:
-                        k *= d
-                    n += k
-        return n
+        return sum(4 * math.prod(s) for mx in mixers for name, s in mx.memory().items() if name in SLOT_STATES)
 
     def first_visible(self, pos: int) -> int:
         """Earliest position that a query at ``pos`` or later can see in any attention layer."""

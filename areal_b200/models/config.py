@@ -14,7 +14,7 @@ from typing import Optional
 
 @dataclass
 class ModelConfig:
-    arch: str = "qwen2"                 # qwen2 | qwen3 | qwen3_moe | qwen2_moe | qwen3_5 | qwen3_5_moe | kagolix | vogilix | bumotar
+    arch: str = "qwen2"                 # qwen2 | qwen3 | qwen3_moe | qwen2_moe | qwen3_5 | qwen3_5_moe | kagolix | vogilix | bumotar | goganex
     vocab_size: int = 151936
     hidden_size: int = 1536
     num_layers: int = 28
@@ -63,7 +63,7 @@ class ModelConfig:
     partial_rotary_factor: float = 1.0
     attn_output_gate: bool = False
     rms_norm_offset: bool = False
-    # mixer stacks (Kagolix, Vogilix, Bumotar): one entry per layer, {"type": mixer kind, "mixer": its sizes, "mlp":
+    # mixer stacks (Kagolix, Vogilix, Bumotar, Goganex): one entry per layer, {"type": mixer kind, "mixer": its sizes, "mlp":
     # feed-forward or None} as in config.json (see models/mixers.py); grouped RMS norms and a capped output
     mixer_layers: list[dict] = field(default_factory=list)
     norm_groups: int = 1
@@ -73,6 +73,9 @@ class ModelConfig:
     learned_positions: bool = False         # a vector per position (max_position_embeddings of them) added to the embedding
     logit_scale: float = 1.0                # factor of the logits (part of the final norm)
     layer_loop: Optional[dict] = None       # {"start", "stop", "times"}: layers start .. stop - 1 run that many times in a row
+    loop_mixes_embedding: bool = True       # before every pass the stream goes through a product with the embedding (else passes just follow)
+    embedding_scale: float = 1.0            # factor of the embedding rows (in 32 bits)
+    token_shift: bool = False               # what a mixer reads is blended with the same for the token before, number by number
     token_side_dim: int = 0                 # > 0: every layer ends with a gated input from its own part of a per-token row
 
     @property
@@ -258,12 +261,15 @@ class ModelConfig:
         if arch == "vogilix":
             own = dict(norm_placement="post", rms_norm_offset=True, residual_mult=float(d["residual_mult"]), learned_positions=True,
                        max_position_embeddings=int(d["max_positions"]), token_side_dim=int((d.get("token_side") or {}).get("dim") or 0))
-        elif arch == "bumotar":
+        elif arch in ("bumotar", "goganex"):
             loop = {k: int(d["loop"][k]) for k in ("start", "stop", "times")} if d.get("loop") else None
             if loop and not (0 <= loop["start"] < loop["stop"] <= len(layers) and loop["times"] >= 1):
                 raise ValueError(f"a loop over layers {loop['start']} to {loop['stop']} of {len(layers)}, {loop['times']} times")
-            own = dict(norm_placement="pre", logit_scale=float(d.get("logit_scale", 1.0)), layer_loop=loop,
-                       max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)))
+            own = dict(norm_placement="pre", layer_loop=loop, max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)))
+            if arch == "bumotar":
+                own.update(logit_scale=float(d.get("logit_scale", 1.0)))
+            else:
+                own.update(loop_mixes_embedding=False, token_shift=True, embedding_scale=float(d["embedding"]["scale"]))
         else:
             own = dict(norm_groups=int(d["norm"].get("groups", 1)), logit_softcap=float(d.get("logit_softcap") or 0.0),
                        max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)))
@@ -291,8 +297,9 @@ class ModelConfig:
             if mt == "vogilix":
                 d.update(max_positions=self.max_position_embeddings, norm=dict(eps=self.rms_norm_eps), residual_mult=self.residual_mult,
                          token_side=dict(dim=self.token_side_dim) if self.token_side_dim else None)
-            elif mt == "bumotar":
-                d.update(norm=dict(eps=self.rms_norm_eps), logit_scale=self.logit_scale, loop=dict(self.layer_loop) if self.layer_loop else None)
+            elif mt in ("bumotar", "goganex"):
+                d.update(norm=dict(eps=self.rms_norm_eps), loop=dict(self.layer_loop) if self.layer_loop else None)
+                d.update(dict(logit_scale=self.logit_scale) if mt == "bumotar" else dict(embedding=dict(scale=self.embedding_scale)))
             else:
                 d.update(norm=dict(eps=self.rms_norm_eps, groups=self.norm_groups), logit_softcap=self.logit_softcap)
             return d
@@ -450,6 +457,19 @@ def _looped_stack_preset(vocab, width, pattern, window, ret, latent, moe, shared
                 loop=dict(start=loop[0], stop=loop[1], times=loop[2]) if loop else None, layers=layers)
 
 
+def _shifted_stack_preset(vocab, width, pattern, att, left, gru, ff, limit, loop, scale, eps=1e-6):
+    """A Goganex stack: a in ``pattern`` is a layer of rotated attention, p one of parallel branches (attention whose keys are its
+    values, minGRU), upper case a layer without feed-forward; ``loop`` = (start, stop, times)."""
+    layers = [dict(type="attention" if c.lower() == "a" else "parallel", mixer=dict(att) if c.lower() == "a" else dict(left=dict(left), right=dict(width=gru)),
+                   mlp=dict(kind="dense", ff=ff, limit=limit) if c.islower() else None) for c in pattern]
+    return dict(architecture="Goganex", vocab=vocab, width=width, norm=dict(eps=eps), embedding=dict(scale=scale),
+                loop=dict(start=loop[0], stop=loop[1], times=loop[2]) if loop else None, layers=layers)
+
+
+def _llama3(base, dims, factor=8.0, low=1.0, high=4.0, original=8192):
+    return dict(base=base, dims=dims, scaling=dict(factor=factor, low=low, high=high, original=original))
+
+
 def _ret(heads, dim, vdim, base=10000.0):
     """Retention with half-lives from a few tokens to a few thousand, spread over the heads."""
     return dict(heads=heads, dim=dim, vdim=vdim, rot=dict(base=base, dims=dim), decay=[1.0 - 2.0 ** -(3.0 + 8.0 * h / max(1, heads - 1)) for h in range(heads)])
@@ -491,6 +511,16 @@ MIXER_STACK_PRESETS = {
         32768, 2048, "plpl", dict(heads=16, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, mask=dict(size=1024),
                                   rot=dict(base=500000.0, dims=64, scaling=dict(factor=4.0))), _ret(8, 128, 128),
         dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, rot=_yarn(10000.0, 64)), (64, 8, 768), 1024, (0, 2, 2), 0.125),
+    "tiny-goganex": _shifted_stack_preset(
+        320, 128, "apPa", dict(heads=4, kv_heads=2, dim=32, vdim=48, scale=0.2, rot=_llama3(10000.0, 24, original=256)),
+        dict(heads=6, kv_heads=2, dim=40, vdim=40, scale=0.15), 96, 160, 2.0, (1, 3, 2), 0.7),
+    # layer sizes of an 8B-class and of a 2B-class model; two looped layers and two that run once
+    "goganex-8b-layers": _shifted_stack_preset(
+        32768, 4096, "apap", dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, rot=_llama3(500000.0, 128)),
+        dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5), 4096, 12288, 7.0, (0, 2, 2), 4.0),
+    "goganex-2b-layers": _shifted_stack_preset(
+        32768, 2048, "apap", dict(heads=16, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, rot=_llama3(500000.0, 128)),
+        dict(heads=16, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5), 2560, 8192, 7.0, (0, 2, 2), 4.0),
 }
 
 

@@ -1,12 +1,14 @@
 """Mixer stacks: decoder models whose layers are listed one by one, each with its own token mixer and feed-forward.
 
-Three designs are built from the parts below (:data:`DESIGNS`):
+Four designs are built from the parts below (:data:`DESIGNS`):
 
 * Kagolix normalises twice around every sublayer, in groups: ``x += norm_b(f(norm_a(x)))``; its output is capped;
 * Vogilix normalises the sublayer's output only, ``x += m * norm(f(x))``, adds a learned vector per position to the
   embedding, and ends every layer with a gated input from the layer's own part of a per-token row;
 * Bumotar normalises before every sublayer, ``x += f(norm(x))``, and runs a stretch of its layers several times in a row with
-  the same weights, every pass with caches and states of its own and with the embedding mixed in again before it.
+  the same weights, every pass with caches and states of its own and with the embedding mixed in again before it;
+* Goganex does so too, with nothing between the passes, scales the embedding, and blends what a mixer reads with the same row of
+  the token before (token shift).
 
 The sum x stays in 32 bits in all of them. The mixers
 
@@ -18,9 +20,12 @@ The sum x stays in 32 bits in all of them. The mixers
   a latent of their own, no positions, a sliding window; or (:class:`RotaryLatentAttention`) queries straight from the layer's
   input and beside the latent one rotated key part for all heads, sinks and a gate per head;
 * ``parallel``: branches side by side on one input and one output projection: windowed attention with rotated, normed
-  queries and keys, capped scores, a sink and gated channels; retention (linear attention with a fixed decay per head);
+  queries and keys, capped scores, a sink and gated channels; retention (linear attention with a fixed decay per head); or
+  (:class:`NormedParallel`) on output projections of their own whose results are normed before they are added: attention without
+  positions whose keys are its values, and minGRU;
+* ``attention`` as :class:`RotaryAttention`: rotated queries and keys of unit length, a factor per head, a sink;
 
-and the feed-forwards (dense with xIELU or the exact GELU; experts behind a softmax or a sigmoid router, weighted at their
+and the feed-forwards (dense with xIELU, the exact GELU or clamped gated units; experts behind a softmax or a sigmoid router, weighted at their
 output or at their input, with or without a gated shared expert) are built from the ops of :mod:`..ops.mixer_ops`. A forward
 pass runs the rows of one step (:class:`~..ops.mixer_ops.RaggedBatch`) from the pages and state slots of
 :class:`~..engine.state_cache.StateCache`; whole prompts, portions and single tokens are the same call.
@@ -72,6 +77,16 @@ class _Block(nn.Module):
     def vec(self, *shape):
         return nn.Parameter(torch.empty(*shape, dtype=torch.float32, device=self._device))
 
+    carried = {}             # what the layer around the block keeps in a request's slot
+    lists_pages = False      # its portions want the pages that they see in one list
+
+    def cache_shapes(self) -> dict:
+        return {}
+
+    def memory(self) -> dict:
+        """Shapes of what the cache holds for the block, per token and per request."""
+        return {**self.cache_shapes(), **self.carried}
+
     def const(self, values):
         """Constants of the configuration as an fp32 buffer (no part of a checkpoint)."""
         return torch.tensor(values, dtype=torch.float32, device=self._device)
@@ -89,6 +104,11 @@ class _Block(nn.Module):
 def _need(ok, where, what):
     if not ok:
         raise ValueError(where + what)
+
+
+def _check_heads(m, where):
+    _need(min(m[k] for k in ("heads", "kv_heads", "dim", "vdim")) >= 1 and m["heads"] % m["kv_heads"] == 0, where,
+          f"{m['heads']} query heads over {m['kv_heads']} key/value heads")
 
 
 # ----------------------------------------------------------------------------- rotation frequencies
@@ -112,6 +132,20 @@ def yarn_frequencies(rot: dict):
         f, r = base ** (-2.0 * i / dims), min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
         out.append(f / s["factor"] * r + f * (1.0 - r))
     return tuple(out), 0.1 * math.log(s["factor"]) + 1.0
+
+
+def llama3_frequencies(rot: dict):
+    """(frequencies, 1.0) scaled by wavelength: pairs that turn more than ``high`` times within ``original`` positions keep their
+    frequency, those that turn less than ``low`` times are slowed by ``factor``, in between the two are blended."""
+    base, s = rotary_frequencies(dict(rot, scaling=None))[0], rot.get("scaling")
+    if not s:
+        return base, 1.0
+    out = []
+    for f in base:
+        turns = s["original"] * f / (2.0 * math.pi)
+        keep = 1.0 if turns > s["high"] else (0.0 if turns < s["low"] else (turns - s["low"]) / max(s["high"] - s["low"], 1e-30))
+        out.append((1.0 - keep) * f / s["factor"] + keep * f)
+    return tuple(out), 1.0
 
 
 class ChunkAttention(_Block):
@@ -227,6 +261,8 @@ class LatentAttention(_Block):
     key part is applied to the queries and the value part to the outputs (all heads then share the latent as key and value),
     for portions the keys and values of the visible tokens are worked out once."""
 
+    lists_pages = True
+
     @staticmethod
     def check(m, where):
         _need(min(m[k] for k in ("heads", "dim", "vdim", "q_rank", "kv_rank")) >= 1, where, "a latent attention needs positive sizes")
@@ -277,6 +313,7 @@ class RotaryLatentAttention(_Block):
         _need(m["rot"]["dims"] == m["rot_dim"] and m["rot_dim"] % 2 == 0, where, "the rotated part turns as a whole, in pairs")
 
     span = 0
+    lists_pages = True
 
     def __init__(self, cfg, m, dtype, device):
         super().__init__(cfg, dtype, device)
@@ -311,18 +348,58 @@ class RotaryLatentAttention(_Block):
                 p + "ukv_proj": [(h + "uk", (0, nk), None), (h + "uv", (nk, nk + nv), None)], p + "o_proj": [(h + "o", None, None)]}
 
 
+ONE_IN_DENOMINATOR = 0.0       # sink whose exponential is the 1 that a softmax's denominator gets
+
+
+class RotaryAttention(_Block):
+    """Grouped-query attention that sees everything before it. q and k are rotated (neighbouring numbers paired, frequencies
+    scaled by wavelength) and brought to a root mean square of one, scores are multiplied by a learned number per head, the
+    softmax has one more in its denominator."""
+
+    span = 0
+
+    @staticmethod
+    def check(m, where):
+        _check_heads(m, where)
+        _need(2 <= m["rot"]["dims"] <= m["dim"] and m["rot"]["dims"] % 2 == 0, where, "rotated numbers come in pairs within a head")
+
+    def __init__(self, cfg, m, dtype, device):
+        super().__init__(cfg, dtype, device)
+        H = cfg.hidden_size
+        self.nq, self.nkv, self.D, self.Dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        self.scale, self.rotary = float(m["scale"]), llama3_frequencies(m["rot"])
+        self.qkv_proj = self.mat((self.nq + self.nkv) * self.D + self.nkv * self.Dv, H)
+        self.temp = self.vec(self.nq)
+        self.o_proj = self.mat(H, self.nq * self.Dv)
+
+    def cache_shapes(self):
+        return {"kv": ((self.nkv, self.D), (self.nkv, self.Dv))}
+
+    def first_visible(self, pos: int) -> int:
+        return 0
+
+    def forward(self, x, b, lc):
+        q = M.qk_head_norm_append(M.linear(x, self.qkv_proj), None, None, self.eps, self.rot(b), True, b, lc.k, lc.v, self.nq, unit=True, q_factor=self.temp)
+        o = M.chunk_attention(q, lc.k, lc.v, b, self.scale, sink=ONE_IN_DENOMINATOR)
+        return M.linear(o.view(x.shape[0], -1), self.o_proj)
+
+    @staticmethod
+    def checkpoint_names(p, m, h):
+        rq, rk, rv = m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"]
+        return {p + "qkv_proj": [(h + "q", (0, rq), None), (h + "k", (rq, rq + rk), None), (h + "v", (rq + rk, rq + rk + rv), None)],
+                p + "temp": [(h + "temp", None, None)], p + "o_proj": [(h + "o", None, None)]}
+
+
 # ----------------------------------------------------------------------------- branches side by side
 class WindowBranch(_Block):
     """Grouped-query attention in a sliding window: per-head norms and rotation (halves paired) on q and k, capped scores, one
     added to the softmax's denominator, a gate per output channel. Works on its rows q | k | v | g of a fused projection."""
 
     parts = ("q", "k", "v", "g")
-    SINK = 0.0               # its exponential is what the denominator gets
 
     @staticmethod
     def check(m, where):
-        _need(min(m[k] for k in ("heads", "kv_heads", "dim", "vdim")) >= 1 and m["heads"] % m["kv_heads"] == 0, where,
-              f"{m['heads']} query heads over {m['kv_heads']} key/value heads")
+        _check_heads(m, where)
         _need(m["rot"]["dims"] % 2 == 0 and m["rot"]["dims"] <= m["dim"], where, "rotated numbers come in pairs within a head")
 
     def __init__(self, cfg, m, dtype, device):
@@ -336,16 +413,20 @@ class WindowBranch(_Block):
     def rows(m):
         return m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"], m["heads"] * m["vdim"]
 
+    @staticmethod
+    def columns(m):
+        return m["heads"] * m["vdim"]
+
     def cache_shapes(self):
         return {"kv": ((self.nkv, self.D), (self.nkv, self.Dv))}
 
     def forward(self, z, b, lc, factor, out):
         q = M.qk_head_norm_append(z, self.q_norm, self.k_norm, self.eps, self.rot(b), False, b, lc.k, lc.v, self.nq)
         gate = z[:, self.nq * self.D + self.nkv * (self.D + self.Dv):][:, :self.nq * self.Dv]
-        M.chunk_attention(q, lc.k, lc.v, b, self.scale, self.softcap, window=self.window, sink=self.SINK, gate=gate, out_scale=factor, out=out)
+        M.chunk_attention(q, lc.k, lc.v, b, self.scale, self.softcap, window=self.window, sink=ONE_IN_DENOMINATOR, gate=gate, out_scale=factor, out=out)
 
     @staticmethod
-    def own_names(p, h):
+    def own_names(p, m, h):
         return {p + "q_norm": [(h + "q.norm", None, None)], p + "k_norm": [(h + "k.norm", None, None)]}
 
 
@@ -371,6 +452,10 @@ class RetentionBranch(_Block):
     def rows(m):
         return m["heads"] * m["dim"], m["heads"] * m["dim"], m["heads"] * m["vdim"], m["heads"] * m["vdim"]
 
+    @staticmethod
+    def columns(m):
+        return m["heads"] * m["vdim"]
+
     def cache_shapes(self):
         return {"state": (self.heads, self.Dv, self.D)}
 
@@ -378,8 +463,78 @@ class RetentionBranch(_Block):
         M.retention(z, self.decay, self.log2_decay, self.rot(b), self.eps, factor, out, self.heads, self.D, self.Dv, b, lc.state)
 
     @staticmethod
-    def own_names(p, h):
+    def own_names(p, m, h):
         return {}
+
+
+class KeyValueBranch(_Block):
+    """Grouped-query attention without positions that sees everything before it; its keys, as projected, are its values, while q and
+    k meet with a root mean square of one. The cache holds the projected keys once, and the number that norms each of them. Works
+    on its rows q | k of a fused projection."""
+
+    parts = ("q", "k")
+
+    @staticmethod
+    def check(m, where):
+        _check_heads(m, where)
+        _need(m["dim"] == m["vdim"], where, f"keys of {m['dim']} numbers cannot be values of {m['vdim']}")
+
+    def __init__(self, cfg, m, dtype, device):
+        super().__init__(cfg, dtype, device)
+        self.nq, self.nkv, self.D, self.scale = m["heads"], m["kv_heads"], m["dim"], float(m["scale"])
+
+    @staticmethod
+    def rows(m):
+        return m["heads"] * m["dim"], m["kv_heads"] * m["dim"]
+
+    @staticmethod
+    def columns(m):
+        return m["heads"] * m["dim"]
+
+    def cache_shapes(self):
+        return {"kv": ((self.nkv, self.D), None), "key_factor": (self.nkv,)}
+
+    def forward(self, z, b, lc):
+        q = M.qk_head_norm_append(z, None, None, self.eps, None, False, b, lc.k, None, self.nq, unit=True, key_factor=lc.key_factor)
+        return M.chunk_attention(q, lc.k, None, b, self.scale, key_factor=lc.key_factor).view(z.shape[0], -1)
+
+    @staticmethod
+    def own_names(p, m, h):
+        return {}
+
+
+class MinGRUBranch(_Block):
+    """Gated recurrence whose gates read only the current token. Works on its rows z | x | g of a fused projection."""
+
+    parts = ("z", "x", "g")
+
+    @staticmethod
+    def check(m, where):
+        _need(m["width"] >= 1, where, "a recurrence needs a width")
+
+    def __init__(self, cfg, m, dtype, device):
+        super().__init__(cfg, dtype, device)
+        self.W = m["width"]
+        self.zx_bias = self.vec(2 * self.W)
+
+    @staticmethod
+    def rows(m):
+        return (m["width"],) * 3
+
+    @staticmethod
+    def columns(m):
+        return m["width"]
+
+    def cache_shapes(self):
+        return {"state": (self.W,)}
+
+    def forward(self, z, b, lc):
+        return M.min_gru(z, self.zx_bias, b, lc.state)
+
+    @staticmethod
+    def own_names(p, m, h):
+        W = m["width"]
+        return {p + "zx_bias": [(h + "z.b", (0, W), None), (h + "x.b", (W, 2 * W), None)]}
 
 
 class Parallel(_Block):
@@ -407,9 +562,8 @@ class Parallel(_Block):
         """First row of every branch in the input projection and first column in the output projection, and their ends."""
         rows, cols = [0], [0]
         for n, branch in cls.BRANCHES:
-            r = branch.rows(m[n])
-            rows.append(rows[-1] + sum(r))
-            cols.append(cols[-1] + r[3])
+            rows.append(rows[-1] + sum(branch.rows(m[n])))
+            cols.append(cols[-1] + branch.columns(m[n]))
         return rows, cols
 
     def cache_shapes(self):
@@ -442,7 +596,39 @@ class Parallel(_Block):
                 out[p + "in_proj"].append((hb + part, (at, at + r), None))
                 at += r
             out[p + "o_proj"].append((hb + "o", None, (slice(None), slice(cols[i], cols[i + 1]))))
-            out.update(branch.own_names(f"{p}branches.{i}.", hb))
+            out.update(branch.own_names(f"{p}branches.{i}.", m[n], hb))
+        return out
+
+
+class NormedParallel(Parallel):
+    """Attention whose keys are its values beside minGRU: one product makes the rows of both, each has an output projection of its
+    own, and half the sum of the two outputs, each normed over the layer's width, is left to the residual sum behind the mixer."""
+
+    BRANCHES = (("left", KeyValueBranch), ("right", MinGRUBranch))
+    FACTOR = 0.5
+
+    def __init__(self, cfg, m, dtype, device):
+        _Block.__init__(self, cfg, dtype, device)
+        H = cfg.hidden_size
+        self.in_rows, self.out_cols = self._layout(m)
+        self.in_proj = self.mat(self.in_rows[-1], H)
+        self.o_proj = nn.ParameterList([self.mat(H, branch.columns(m[n])) for n, branch in self.BRANCHES])
+        self.left_norm, self.right_norm = self.vec(H), self.vec(H)
+        self.branches = nn.ModuleList([branch(cfg, m[n], dtype, device) for n, branch in self.BRANCHES])
+        self.window = 0
+
+    def forward(self, x, b, lc):
+        z = M.linear(x, self.in_proj)
+        left, right = (M.linear(br(z[:, self.in_rows[i]:self.in_rows[i + 1]], b, lc), self.o_proj[i]) for i, br in enumerate(self.branches))
+        return M.BranchSum(left, right, self.left_norm, self.right_norm, self.FACTOR, self.eps)
+
+    @classmethod
+    def checkpoint_names(cls, p, m, h):
+        out = super().checkpoint_names(p, m, h)
+        del out[p + "o_proj"]
+        for i, (n, _) in enumerate(cls.BRANCHES):
+            out[f"{p}o_proj.{i}"] = [(f"{h}{n}.o", None, None)]
+            out[f"{p}{n}_norm"] = [(f"{h}{n}.out", None, None)]
         return out
 
 
@@ -499,6 +685,23 @@ class GeluMLP(_Block):
 
 
 GLU_ALPHA = 1.702        # slope of the clamped units' gate
+
+
+class ClampedMLP(_Block):
+    """Dense feed-forward of clamped gated units."""
+
+    def __init__(self, cfg, m, dtype, device):
+        super().__init__(cfg, dtype, device)
+        self.limit = float(m["limit"])
+        self.gate_up_proj, self.down_proj = self.mat(2 * m["ff"], cfg.hidden_size), self.mat(cfg.hidden_size, m["ff"])
+
+    def forward(self, x):
+        return M.linear(M.glu_clamped(M.linear(x, self.gate_up_proj), self.limit, GLU_ALPHA), self.down_proj)
+
+    @staticmethod
+    def checkpoint_names(p, m, h):
+        I = m["ff"]
+        return {p + "gate_up_proj": [(h + "gate", (0, I), None), (h + "up", (I, 2 * I), None)], p + "down_proj": [(h + "down", None, None)]}
 
 
 class InputWeightedMLP(_Block):
@@ -595,6 +798,8 @@ DESIGNS = {
                       ("mixer_attention", "mixer_latent")),
     "bumotar": Design("Bumotar", {"latent_attention": RotaryLatentAttention, "parallel": Parallel}, {"moe": SharedExpertMLP}, ("norm1", "norm2"), ("norm1",),
                       ("mixer_attention", "mixer_latent", "mixer_retention", "mixer_rotary")),
+    "goganex": Design("Goganex", {"attention": RotaryAttention, "parallel": NormedParallel}, {"dense": ClampedMLP}, ("norm1", "norm2"), ("norm1",),
+                      ("mixer_attention", "mixer_rotary", "mixer_gru")),
 }
 
 
@@ -606,6 +811,10 @@ class MixerLayer(_Block):
             setattr(self, n, self.vec(H))
         self.mix = design.mixers[spec["type"]](cfg, spec["mixer"], dtype, device)
         self.mlp = design.mlps[spec["mlp"]["kind"]](cfg, spec["mlp"], dtype, device) if spec["mlp"] else None
+        self.shift = None
+        if cfg.token_shift:
+            self.shift = self.vec(H)
+            self.mix.carried = {"shift": (H,)}
         self.side_dim = cfg.token_side_dim
         if self.side_dim:
             self.side_col = idx * self.side_dim
@@ -624,12 +833,14 @@ def checkpoint_plan(cfg: ModelConfig) -> dict:
         plan["embed_positions"] = [("pos", None, None)]
     if cfg.token_side_dim:
         plan["embed_side"] = [("side.embed", None, None)]
-    if cfg.layer_loop:
+    if cfg.layer_loop and cfg.loop_mixes_embedding:
         plan["loop_in"], plan["loop_step"] = [("loop.in", None, None)], [("loop.step", None, None)]
     for i, e in enumerate(cfg.mixer_layers):
         p, h = f"layers.{i}.", f"l{i}."
         for n in design.layer_norms if e["mlp"] else design.layer_norms_bare:
             plan[p + n] = [(h + n, None, None)]
+        if cfg.token_shift:
+            plan[p + "shift"] = [(h + "shift", None, None)]
         plan.update(design.mixers[e["type"]].checkpoint_names(p + "mix.", e["mixer"], h + "mix."))
         if e["mlp"]:
             plan.update(design.mlps[e["mlp"]["kind"]].checkpoint_names(p + "mlp.", e["mlp"], h + "mlp."))
@@ -656,7 +867,7 @@ class MixerStackLM(CausalLM):
             self.embed_positions = nn.Parameter(torch.empty(cfg.max_position_embeddings, cfg.hidden_size, **like))
         if cfg.token_side_dim:
             self.embed_side = nn.Parameter(torch.empty(cfg.vocab_size, cfg.num_layers * cfg.token_side_dim, **like))
-        if cfg.layer_loop:
+        if cfg.layer_loop and cfg.loop_mixes_embedding:
             self.loop_in = nn.Parameter(torch.empty(cfg.hidden_size, 2 * cfg.hidden_size, **like))
             self.loop_step = nn.Parameter(torch.empty(cfg.layer_loop["times"], cfg.hidden_size, **dict(like, dtype=torch.float32)))
         self._place_rotations()
@@ -673,8 +884,10 @@ class MixerStackLM(CausalLM):
             leaf = name.rsplit(".", 1)[-1]
             if leaf in ("norm", "norm1", "norm1b", "norm2", "norm2b") and "mix." not in name:
                 p.fill_(0.0 if cfg.rms_norm_offset else 1.0)
-            elif leaf == "D":
+            elif leaf in ("D", "temp"):
                 p.fill_(1.0)
+            elif leaf == "shift":
+                uniform(p, 0.0, 1.0)
             elif leaf in ("correction", "conv_b", "yx_bias", "gate_b"):
                 p.zero_()
             elif leaf == "conv_w":
@@ -761,22 +974,26 @@ class MixerStackLM(CausalLM):
         cfg, layers, runs, dt = self.cfg, self.layers, self.layer_runs, self.dtype
         eps, H = cfg.rms_norm_eps, cfg.hidden_size
         b.rot = M.rotary_table(b.pos, self.rot_freq, self.rot_mult) if hasattr(self, "rot_freq") else None
-        loop = cfg.layer_loop
+        loop = cfg.layer_loop if cfg.loop_mixes_embedding else None
         a, size, times = (loop["start"], loop["stop"] - loop["start"], loop["times"]) if loop else (0, 0, 0)
         enters = {a + t * size: t for t in range(times)}            # layer run -> pass that begins with it
+
+        def reads(r, src, resid, vec=None):
+            """The stream after ``src`` and ``vec`` were added, and what the mixer of layer run ``r`` reads of it."""
+            layer = layers[runs[r]]
+            return M.stream_norm(src, resid, layer.norm1, eps, dt, vec, layer.shift, b, cache.layers[r].shift)
         if loop:
             # what enters a pass: the stream beside the embedding
             both = torch.empty(b.n_rows, 2 * H, device=self.embed_tokens.device, dtype=dt)
             resid, x = M.embed_rows(b.tokens, self.embed_tokens, b.pos, None, both[:, H:], both[:, :H])
+            if 0 not in enters:
+                resid, x = reads(0, None, resid)
         else:
-            resid, x = M.embed_rows(b.tokens, self.embed_tokens, b.pos)
-        if 0 not in enters:
-            x = M.residual_norm(None, resid, layers[runs[0]].norm1, eps, dt)
+            resid, x = reads(0, M.EmbeddingRows(b.tokens, self.embed_tokens, cfg.embedding_scale), None)
         for r, i in enumerate(runs):
             layer = layers[i]
             if r in enters:
-                resid = M.linear(both, self.loop_in, fp32_out=True).contiguous()
-                x = M.residual_norm(None, resid, layer.norm1, eps, dt, vec=self.loop_step[enters[r]])
+                resid, x = reads(r, None, M.linear(both, self.loop_in, fp32_out=True).contiguous(), self.loop_step[enters[r]])
             h = layer.mix(x, b, cache.layers[r])
             if layer.mlp is not None:
                 h = layer.mlp(M.residual_norm(h, resid, layer.norm2, eps, dt))
@@ -784,7 +1001,7 @@ class MixerStackLM(CausalLM):
             if r + 1 in enters:
                 M.residual_norm(h, resid, None, eps, dt, out=both[:, :H])
             elif r + 1 < len(runs):
-                x = M.residual_norm(h, resid, layers[runs[r + 1]].norm1, eps, dt)
+                resid, x = reads(r + 1, h, resid)
             else:
                 x = M.residual_norm(h, resid, self.norm, eps, dt, mult=cfg.logit_scale)
             if on_layer is not None:

@@ -4,7 +4,7 @@
 // and the window - 1 before it), or all of them (chunk = window = 0). Query / key and value sizes may differ.
 // Optional, all in AttnExtra: a second part of queries and keys that all heads share a key of (rotated parts beside latents),
 // a sink (a score that only enters the denominator), a sigmoid gate on the output (per head or per channel), a factor of the
-// output, row strides.
+// output, a factor per key, row strides. Keys may be the values as well (vc = kc): then single-token rows read them once.
 //
 //   chunk_attn_plain_kernel   any sizes, bf16 or 32-bit: a warp per (row, head)
 //   chunk_decode_kernel       single-token rows, bf16: a cluster of CTAs splits a request's chunk, mma.sync products,
@@ -112,6 +112,7 @@ chunk_attn_plain_kernel(const T* __restrict__ q, const int* __restrict__ pos, co
       }
       const T* k2 = (const T*)p.x.k2 + kv * p.x.ldk2;
       for (int d = 0; d < p.x.D2; ++d) dot += ldf(k2 + d) * sq2[d];
+      if (p.x.kf) dot *= p.x.kf[kv * p.Hkv + kvh];
       s = p.softcap > 0.f ? p.softcap * tanhf(dot / p.softcap) : dot;
       if (p.r1) s -= r1 * log1pf(r2 * (float)(i - j));
     }
@@ -181,6 +182,7 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
   constexpr int KS = DK / 16;
   extern __shared__ __align__(128) unsigned char dsm[];
   __shared__ float s_ml[2][16];                                     // this CTA's merged (max, sum) per head
+  __shared__ float s_kf[2][CD_KEYS];                                // factors of the keys of two pieces
   pdl_wait();
   pdl_trigger();
   const int b = blockIdx.x, h = blockIdx.y, spl = blockIdx.z;
@@ -197,6 +199,7 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
   const int base = p.page_base[b];
   const uint32_t sm = smem_u32(dsm);
   int* s_row = reinterpret_cast<int*>(dsm + Cfg::ROWS_OFF);
+  const bool same = DK == DV && p.vc == p.kc;                       // keys are the values: one copy of a piece serves both products
   auto plan = [&](int c) {
     if (tid < CD_KEYS) {
       const int t = t0 + c * CD_KEYS + tid;
@@ -212,12 +215,19 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
       const bool ok = row >= 0 && piece * 8 < p.D;
       cd_copy16(st + r * Cfg::KROW + piece * 16, (const __nv_bfloat16*)p.kc + (ok ? row * p.x.ldk + h * p.D + piece * 8 : 0), ok);
     }
+    if (!same) {
 #pragma unroll
-    for (int k = 0; k < CD_KEYS * (DV / 8) / 128; ++k) {
-      const int idx = tid + k * 128, r = idx / (DV / 8), piece = idx % (DV / 8);
-      const int row = s_row[(c & 1) * CD_KEYS + r];
-      const bool ok = row >= 0 && piece * 8 < p.Dv;
-      cd_copy16(st + CD_KEYS * Cfg::KROW + r * Cfg::VROW + piece * 16, (const __nv_bfloat16*)p.vc + (ok ? row * p.x.ldv + h * p.Dv + piece * 8 : 0), ok);
+      for (int k = 0; k < CD_KEYS * (DV / 8) / 128; ++k) {
+        const int idx = tid + k * 128, r = idx / (DV / 8), piece = idx % (DV / 8);
+        const int row = s_row[(c & 1) * CD_KEYS + r];
+        const bool ok = row >= 0 && piece * 8 < p.Dv;
+        cd_copy16(st + CD_KEYS * Cfg::KROW + r * Cfg::VROW + piece * 16, (const __nv_bfloat16*)p.vc + (ok ? row * p.x.ldv + h * p.Dv + piece * 8 : 0), ok);
+      }
+    }
+    if (p.x.kf && tid < CD_KEYS) {
+      const int row = s_row[(c & 1) * CD_KEYS + tid];
+      const float* f = p.x.kf + (row >= 0 ? (long long)row * p.Hkv + h : 0);
+      asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_u32(&s_kf[c & 1][tid])), "l"(f), "r"(row >= 0 ? 4 : 0) : "memory");
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -258,7 +268,7 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
     __syncthreads();
     if (c + 2 < np) plan(c + 2);                     // its table half is free: piece c has been issued from it
     const uint32_t ka = sm + (c & 1) * Cfg::STAGE + warp * 16 * Cfg::KROW;
-    const uint32_t va = sm + (c & 1) * Cfg::STAGE + CD_KEYS * Cfg::KROW + warp * 16 * Cfg::VROW;
+    const uint32_t va = same ? ka : sm + (c & 1) * Cfg::STAGE + CD_KEYS * Cfg::KROW + warp * 16 * Cfg::VROW;
     float s[2][4] = {};
 #pragma unroll
     for (int ks = 0; ks < KS; ++ks) {
@@ -268,6 +278,15 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
       cd_mma(s[1], qa[ks], b2, b3);
     }
     const int tok = t0 + c * CD_KEYS + warp * 16 + 2 * tq;
+    if (p.x.kf) {
+      const float* f = &s_kf[c & 1][warp * 16 + 2 * tq];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float v = f[(k >> 1) * 8 + (k & 1)];
+        s[k >> 1][k & 1] *= v;
+        s[k >> 1][2 + (k & 1)] *= v;
+      }
+    }
     uint32_t pa[4];
     float alpha[2];
 #pragma unroll
@@ -422,7 +441,9 @@ struct ChunkPrefillCfg {
   static constexpr int SMEM = BIAS_OFF + 16 * 96 * 4 + 1024;
 };
 
-template <int DK, int DV, int DR, bool CAP, bool BIAS>
+// ADJ: what else a score gets, from shared memory.
+constexpr int ADJ_NONE = 0, ADJ_DISTANCE = 1, ADJ_KEY = 2;
+template <int DK, int DV, int DR, bool CAP, int ADJ>
 __global__ void __launch_bounds__(384, 1)
 chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                      const __grid_constant__ CUtensorMap tmQ2, const __grid_constant__ CUtensorMap tmK2, const int* __restrict__ cu,
@@ -590,11 +611,28 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     const float r1 = p.r1 ? p.r1[head] : 0.f, r2 = p.r1 ? p.r2[head] : 0.f;
     float m_run = p.x.sink_of(head) * 1.4426950408889634f, l_run = m_run > -INFINITY ? 1.f : 0.f;
     bool ok = true;
+    // factors of a block's keys, fetched a block ahead: this lane's are those of its keys lane and lane + 32
+    float kf[2] = {0.f, 0.f};
+    auto fetch_factors = [&](int j) {
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        const int pos = k0 + j * CP_K + lane + 32 * x, pg = min(max(pos / p.page_size - p.page_base[e], 0), p.max_pages - 1);
+        kf[x] = p.x.kf[((long long)p.pages[(size_t)e * p.max_pages + pg] * p.page_size + pos % p.page_size) * p.Hkv + kvh] * sc.u_scale;
+      }
+    };
+    if constexpr (ADJ == ADJ_KEY)
+      if (nbt > 0) fetch_factors(0);
     for (int j = 0; j < nbt && ok; ++j) {
       const int kb = k0 + j * CP_K;
       float* bs = bias + ((warp - 4) * 2 + (j & 1)) * 96;
       // diagonal x of this warp's 32 rows: distance first + 32 qd - kb + x - 63
-      if constexpr (BIAS) {
+      if constexpr (ADJ == ADJ_KEY) {
+        bs[lane] = kf[0];
+        bs[lane + 32] = kf[1];
+        __syncwarp();
+        if (j + 1 < nbt) fetch_factors(j + 1);
+      }
+      if constexpr (ADJ == ADJ_DISTANCE) {
         for (int x = lane; x < 95; x += 32) bs[x] = r1 * __log2f(1.f + r2 * (float)max(first + qd * 32 - kb + x - 63, 0));
         __syncwarp();
       }
@@ -609,8 +647,8 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       float mx = -INFINITY;
 #pragma unroll
       for (int c = 0; c < 64; ++c) {
-        float v = capped<CAP>(__uint_as_float(u[c]), sc);
-        if constexpr (BIAS) v -= bs[lane - c + 63];
+        float v = ADJ == ADJ_KEY ? __uint_as_float(u[c]) * bs[c] : capped<CAP>(__uint_as_float(u[c]), sc);
+        if constexpr (ADJ == ADJ_DISTANCE) v -= bs[lane - c + 63];
         if (edge && (kb + c > i || kb + c < lo)) v = -INFINITY;
         u[c] = __float_as_uint(v);
         mx = fmaxf(mx, v);
@@ -693,7 +731,7 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   }
 }
 
-template <int DK, int DV, int, bool CAP, bool>
+template <int DK, int DV, int, bool CAP, int>
 static int launch_decode(const void* q, const int* pos, const int* slots, void* out, int R, const ChunkArgs& a, cudaStream_t s) {
   constexpr int SMEM = ChunkDecodeCfg<DK, DV>::SMEM;
   static_assert(2 * ChunkDecodeCfg<DK, DV>::STAGE >= (4 * 16 * DV + 8 * 16) * 4, "the merge buffers alias the stage memory");
@@ -709,7 +747,7 @@ static int launch_decode(const void* q, const int* pos, const int* slots, void* 
   return go(chunk_decode_split_kernel<DK, DV, 8, CAP>, st8);
 }
 
-template <int DK, int DV, int DR, bool CAP, bool BIAS>
+template <int DK, int DV, int DR, bool CAP, int ADJ>
 static int launch_prefill(const void* q, const int* cu, const int* start, const int* tiles, int nt, void* out, int R, int cache_rows, const ChunkArgs& a,
                           cudaStream_t s) {
   using Cfg = ChunkPrefillCfg<DK, DV, DR>;
@@ -725,7 +763,7 @@ static int launch_prefill(const void* q, const int* cu, const int* start, const 
   tk2 = tk;
   if (DR && map(&tq2, a.x.q2, a.x.D2, a.Hq, R, a.x.hsq2, a.x.ldq2, CP_Q)) return 103;
   if (DR && map(&tk2, a.x.k2, a.x.D2, 1, cache_rows, a.x.ldk2, a.x.ldk2, box)) return 104;
-  auto kern = chunk_prefill_kernel<DK, DV, DR, CAP, BIAS>;
+  auto kern = chunk_prefill_kernel<DK, DV, DR, CAP, ADJ>;
   static ab2host::DevState st;
   if (ab2host::prepare_launch(kern, Cfg::SMEM, st, nullptr)) return 300;
   int* err = ab2host::error_flag();
@@ -759,9 +797,9 @@ int ab2_chunk_attn_plain(const void* q, const int* pos, const int* slots, const 
   return cudaGetLastError() == cudaSuccess ? 0 : 1;
 }
 
-#define AB2_BY_SIZE2(FN, DR, CAP, BIAS, ...)                                                                               \
-  if (D <= 64) return Dv <= 64 ? FN<64, 64, DR, CAP, BIAS>(__VA_ARGS__) : FN<64, 128, DR, CAP, BIAS>(__VA_ARGS__);          \
-  return Dv <= 64 ? FN<128, 64, DR, CAP, BIAS>(__VA_ARGS__) : FN<128, 128, DR, CAP, BIAS>(__VA_ARGS__)
+#define AB2_BY_SIZE2(FN, DR, CAP, ADJ, ...)                                                                               \
+  if (D <= 64) return Dv <= 64 ? FN<64, 64, DR, CAP, ADJ>(__VA_ARGS__) : FN<64, 128, DR, CAP, ADJ>(__VA_ARGS__);          \
+  return Dv <= 64 ? FN<128, 64, DR, CAP, ADJ>(__VA_ARGS__) : FN<128, 128, DR, CAP, ADJ>(__VA_ARGS__)
 
 // Row r is the only row of entry r. bf16; D, Dv multiples of 8 up to 128, at most 16 query heads per key head; no second part.
 int ab2_chunk_decode(const void* q, const int* pos, const int* slots, void* out, int R, const void* kc, const void* vc, const int* pages,
@@ -773,11 +811,12 @@ int ab2_chunk_decode(const void* q, const int* pos, const int* slots, void* out,
   if (Hq % Hkv || Hq / Hkv > 16 || (D & 7) || (Dv & 7) || D > 128 || Dv > 128 || Hkv > 65535 || a.x.D2) return 10;
   if (!aligned_to(q, 16) || !aligned_to(kc, 16) || !aligned_to(vc, 16) || ((a.x.ldq | a.x.hsq | a.x.ldk | a.x.ldv) & 7)) return 11;
   cudaStream_t s = (cudaStream_t)stream;
-  if (softcap > 0.f) { AB2_BY_SIZE2(launch_decode, 0, true, true, q, pos, slots, out, R, a, s); }
-  AB2_BY_SIZE2(launch_decode, 0, false, true, q, pos, slots, out, R, a, s);
+  if (softcap > 0.f) { AB2_BY_SIZE2(launch_decode, 0, true, 0, q, pos, slots, out, R, a, s); }
+  AB2_BY_SIZE2(launch_decode, 0, false, 0, q, pos, slots, out, R, a, s);
 }
 
 // tiles [nt, 2] = (entry, first row); q / out hold all R rows of the step. bf16; D, Dv multiples of 8 up to 128; a second part up to 64;
+// factors of the keys only without a second part, a cap and a distance bias;
 // page_size 16, 32 or a multiple of 64. ldk / ldv: elements from one cache row to the next.
 int ab2_chunk_prefill(const void* q, const int* cu, const int* start, const int* tiles, int nt, void* out, int R, int cache_rows, long long ldk,
                       long long ldv, const void* kc, const void* vc, const int* pages, const int* page_base, int max_pages, int page_size, int Hq, int Hkv, int D, int Dv,
@@ -795,10 +834,12 @@ int ab2_chunk_prefill(const void* q, const int* cu, const int* start, const int*
   if (e.gate && !e.gate_per_head && (!aligned_to(e.gate, 16) || (e.ldg & 7))) return 14;
   if (e.D2 && ((e.D2 & 7) || e.D2 > 64 || ((e.ldq2 | e.hsq2 | e.ldk2) & 7) || !aligned_to(e.q2, 16) || !aligned_to(e.k2, 16) || softcap > 0.f || r1)) return 15;
   cudaStream_t s = (cudaStream_t)stream;
-  if (e.D2) { AB2_BY_SIZE2(launch_prefill, 64, false, false, q, cu, start, tiles, nt, out, R, cache_rows, a, s); }
-  if (r1 && softcap > 0.f) { AB2_BY_SIZE2(launch_prefill, 0, true, true, q, cu, start, tiles, nt, out, R, cache_rows, a, s); }
-  if (softcap > 0.f) { AB2_BY_SIZE2(launch_prefill, 0, true, false, q, cu, start, tiles, nt, out, R, cache_rows, a, s); }
-  if (r1) { AB2_BY_SIZE2(launch_prefill, 0, false, true, q, cu, start, tiles, nt, out, R, cache_rows, a, s); }
-  AB2_BY_SIZE2(launch_prefill, 0, false, false, q, cu, start, tiles, nt, out, R, cache_rows, a, s);
+  if (e.kf && (e.D2 || r1 || softcap > 0.f)) return 16;
+  if (e.D2) { AB2_BY_SIZE2(launch_prefill, 64, false, ADJ_NONE, q, cu, start, tiles, nt, out, R, cache_rows, a, s); }
+  if (e.kf) { AB2_BY_SIZE2(launch_prefill, 0, false, ADJ_KEY, q, cu, start, tiles, nt, out, R, cache_rows, a, s); }
+  if (r1 && softcap > 0.f) { AB2_BY_SIZE2(launch_prefill, 0, true, ADJ_DISTANCE, q, cu, start, tiles, nt, out, R, cache_rows, a, s); }
+  if (softcap > 0.f) { AB2_BY_SIZE2(launch_prefill, 0, true, ADJ_NONE, q, cu, start, tiles, nt, out, R, cache_rows, a, s); }
+  if (r1) { AB2_BY_SIZE2(launch_prefill, 0, false, ADJ_DISTANCE, q, cu, start, tiles, nt, out, R, cache_rows, a, s); }
+  AB2_BY_SIZE2(launch_prefill, 0, false, ADJ_NONE, q, cu, start, tiles, nt, out, R, cache_rows, a, s);
 }
 }

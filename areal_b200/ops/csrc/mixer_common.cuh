@@ -96,6 +96,7 @@ struct AttnExtra {
   const void *q2 = nullptr, *k2 = nullptr;   // second part of queries [R, Hq, D2] and keys [cache rows, D2]: its product is added before the scale
   const void* gate = nullptr;                // output times sigmoid(gate): [R, Hq] (gate_per_head) or [R, Hq * Dv]
   const float* sink = nullptr;               // per head: a score (scaled as it stands, never capped) that only enters the denominator
+  const float* kf = nullptr;                 // factor of every key's scores (what norms a key that is cached as it is): [cache rows, Hkv]
   // elements between rows (and heads); 0: contiguous
   long long ldq = 0, hsq = 0, ldq2 = 0, hsq2 = 0, ldk = 0, ldv = 0, ldk2 = 0, ldo = 0, ldg = 0;
   int D2 = 0, gate_per_head = 0;

@@ -1,6 +1,8 @@
 // Rotated positions of mixer stacks. A table of (cos, sin) per row of the step and frequency is made once per step; the kernels
 // that rotate read it:
-//   qk_head_norm_append   per-head RMS norms of q and k (optional), rotation, k and v into the paged cache
+//   qk_head_norm_append   per-head RMS norms of q and k (optional; with or without weights), rotation, k and v into the paged cache. A
+//                         turn keeps a head's length, so norms without weights may as well be taken to follow it. Or the keys go into
+//                         the cache as they are (they are the values too) with the number that norms each of them beside them
 //   latent_rope_append    norm of the cached latent and rotation of the key part behind it, both into the cache; rotation of the
 //                         queries' second part in place
 // Pairs are (i, i + half) of the rotated stretch, or (2 i, 2 i + 1) when interleaved.
@@ -27,12 +29,18 @@ rotary_table_kernel(const int* __restrict__ pos, const double* __restrict__ freq
   }
 }
 
+struct QkExtra {
+  const float* qf;            // [Hq] factors of the queries, or null
+  float* kf;                  // [cache rows, Hkv]: keys are stored as they are and their norms' factors here; or null
+  int unit;                   // norms without weights
+};
+
 // One CTA per row, a warp per head, any sizes.
 template <typename T, int V, bool INTERLEAVED>
 __global__ void __launch_bounds__(256)
 qk_head_norm_append_kernel(const T* __restrict__ z, long long ld, const float* __restrict__ wq, const float* __restrict__ wk,
                            const float2* __restrict__ rot, int ldr, int half, const int* __restrict__ slots, T* __restrict__ q, T* __restrict__ kc,
-                           T* __restrict__ vc, int Hq, int Hkv, int D, int nv, float eps) {
+                           T* __restrict__ vc, int Hq, int Hkv, int D, int nv, float eps, const QkExtra x2) {
   extern __shared__ __align__(16) float sm[];
   pdl_wait();
   pdl_trigger();
@@ -52,17 +60,22 @@ qk_head_norm_append_kernel(const T* __restrict__ z, long long ld, const float* _
       for (int e = 0; e < V; ++e) ss += v[e] * v[e];
       stv<V>(x + c, v);
     }
-    const float rstd = w != nullptr ? 1.f / sqrtf(warp_sum(ss) / D + eps) : 1.f;
+    float rstd = w != nullptr || x2.unit ? 1.f / sqrtf(warp_sum(ss) / D + eps) : 1.f;
+    if (u >= Hq && x2.kf != nullptr) {
+      if (lane == 0) x2.kf[(size_t)slot * Hkv + u - Hq] = rstd;
+      rstd = 1.f;
+    }
+    if (u < Hq && x2.qf != nullptr) rstd *= x2.qf[u];
     __syncwarp();
     T* dst = u < Hq ? q + ((size_t)row * Hq + u) * D : kc + ((size_t)slot * Hkv + u - Hq) * D;
     auto normed = [&](int c, float (&v)[V]) {
       ldv<V>(x + c, v);
-      if (w != nullptr) {
-        float g[V];
-        ldv<V>(w + c, g);
+      float g[V];
 #pragma unroll
-        for (int e = 0; e < V; ++e) v[e] *= rstd * g[e];
-      }
+      for (int e = 0; e < V; ++e) g[e] = 1.f;
+      if (w != nullptr) ldv<V>(w + c, g);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] *= rstd * g[e];
     };
     for (int c = lane * V; c < D; c += 32 * V) {              // V numbers turn together or not at all
       float v[V], o[V];
@@ -109,7 +122,7 @@ template <typename T, bool INTERLEAVED>
 __global__ void __launch_bounds__(256)
 qk_head_norm_append_lanes_kernel(const T* __restrict__ z, long long ld, const float* __restrict__ wq, const float* __restrict__ wk,
                                  const float2* __restrict__ rot, int ldr, int half, const int* __restrict__ slots, T* __restrict__ q, T* __restrict__ kc,
-                                 T* __restrict__ vc, int Hq, int Hkv, int D, int nv, float eps) {
+                                 T* __restrict__ vc, int Hq, int Hkv, int D, int nv, float eps, const QkExtra x2) {
   pdl_wait();
   pdl_trigger();
   const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5, c = lane * 4;
@@ -141,7 +154,12 @@ qk_head_norm_append_lanes_kernel(const T* __restrict__ z, long long ld, const fl
       if (u >= heads) break;
       const float ss = warp_sum(v[i][0] * v[i][0] + v[i][1] * v[i][1] + v[i][2] * v[i][2] + v[i][3] * v[i][3]);
       const bool is_q = u < Hq;
-      const float rstd = (is_q ? wq : wk) != nullptr ? 1.f / sqrtf(ss / D + eps) : 1.f;
+      float rstd = (is_q ? wq : wk) != nullptr || x2.unit ? 1.f / sqrtf(ss / D + eps) : 1.f;
+      if (!is_q && x2.kf != nullptr) {
+        if (lane == 0) x2.kf[(size_t)slot * Hkv + u - Hq] = rstd;
+        rstd = 1.f;
+      }
+      if (is_q && x2.qf != nullptr) rstd *= x2.qf[u];
       float x[4];
 #pragma unroll
       for (int e = 0; e < 4; ++e) x[e] = v[i][e] * rstd * (is_q ? gq[e] : gk[e]);
@@ -271,9 +289,14 @@ int ab2_rotary_table(const int* pos, const double* freq, const float* mult, void
 
 // z rows q [Hq, D] | k [Hkv, D] | v [nv]; q [R, Hq, D], kc [S, Hkv, D], vc [S, nv]; wq / wk [D] or null (no norm); rot: the step's
 // table from this mixer's column on, ldr pairs from row to row; the first 2 half numbers of every head turn. slot < 0: nothing cached.
+// unit: norms without weights. qf [Hq] or null: factors of the queries. kf [S, Hkv] or null: keys are stored as they are (then no turn), kf
+// gets what norms them.
 int ab2_qk_head_norm_append(const void* z, long long ld, const float* wq, const float* wk, const void* rot, int ldr, int half, int interleaved,
-                            const int* slots, void* q, void* kc, void* vc, int R, int Hq, int Hkv, int D, int nv, float eps, int dt, void* stream) {
+                            const int* slots, void* q, void* kc, void* vc, int R, int Hq, int Hkv, int D, int nv, float eps, int unit, const float* qf,
+                            float* kf, int dt, void* stream) {
   if (R <= 0) return 0;
+  if ((half > 0 && rot == nullptr) || (kf && (half > 0 || wk || !unit))) return 11;
+  const QkExtra x2{qf, kf, unit};
   const size_t smem = (size_t)8 * ((D + 3) & ~3) * 4;
   if (2 * half > D || half < 0 || smem > 48 * 1024) return 10;
   const int eb = dt == 0 ? 2 : 4;
@@ -285,7 +308,7 @@ int ab2_qk_head_norm_append(const void* z, long long ld, const float* wq, const 
     auto go = [&](auto t, auto inter) {
       using T = decltype(t);
       launch_pdl(qk_head_norm_append_lanes_kernel<T, decltype(inter)::value>, dim3(R), dim3(256), 0, (cudaStream_t)stream, (const T*)z, ld, wq, wk,
-                 (const float2*)rot, ldr, half, slots, (T*)q, (T*)kc, (T*)vc, Hq, Hkv, D, nv, eps);
+                 (const float2*)rot, ldr, half, slots, (T*)q, (T*)kc, (T*)vc, Hq, Hkv, D, nv, eps, x2);
     };
     if (dt == 0 && interleaved) go(__nv_bfloat16(), std::true_type());
     else if (dt == 0) go(__nv_bfloat16(), std::false_type());
@@ -295,7 +318,7 @@ int ab2_qk_head_norm_append(const void* z, long long ld, const float* wq, const 
   }
   AB2_ROT_TYPED(dt, fits(8), fits(4), interleaved, {
     launch_pdl(qk_head_norm_append_kernel<T, V, INTER>, dim3(R), dim3(256), smem, (cudaStream_t)stream, (const T*)z, ld, wq, wk, (const float2*)rot, ldr,
-               half, slots, (T*)q, (T*)kc, (T*)vc, Hq, Hkv, D, nv, eps);
+               half, slots, (T*)q, (T*)kc, (T*)vc, Hq, Hkv, D, nv, eps, x2);
   });
   return cudaGetLastError() == cudaSuccess ? 0 : 1;
 }

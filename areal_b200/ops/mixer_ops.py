@@ -1,7 +1,7 @@
 """Ops of mixer stacks: norms around (grouped), behind or before the sublayers on a 32-bit residual stream, rotated
 positions, attention over a paged cache (chunks or sliding windows, capped scores, a logarithmic distance bias, sinks, gated
-outputs), attention on cached latents, causal convolutions, RG-LRU, Mamba-2 and retention recurrences on slot states,
-activations, expert combine, per-layer token inputs and capped logits.
+outputs, keys that are the values too), attention on cached latents, causal convolutions, token shifts, RG-LRU, minGRU, Mamba-2 and
+retention recurrences on slot states, activations, expert combine, per-layer token inputs and capped logits.
 
 Every op works on a :class:`RaggedBatch`: the rows of several requests, each bringing any number of its next tokens,
 continuing from the cache pages and state slots that earlier steps left. The first ``n_dec`` entries bring one row
@@ -183,6 +183,34 @@ class ExpertSum:
         return h + (self.shared.float() if self.shared_logit is None else self.shared.float() * torch.sigmoid(self.shared_logit)[:, None])
 
 
+@dataclass
+class BranchSum:
+    """A mixer output that is still in two pieces: ``factor`` times the sum of both, each first RMS-normed with its weight. The
+    residual sum behind the mixer reads the pieces."""
+
+    left: torch.Tensor                   # [T, H], rows may be strided
+    right: torch.Tensor
+    w_left: torch.Tensor                 # [H] fp32
+    w_right: torch.Tensor
+    factor: float
+    eps: float
+
+    def dense(self) -> torch.Tensor:
+        return self.factor * (group_norm_ref(self.left, self.w_left, 1, self.eps) + group_norm_ref(self.right, self.w_right, 1, self.eps))
+
+
+@dataclass
+class EmbeddingRows:
+    """What begins a residual stream: ``scale`` times the rows of ``ids``."""
+
+    ids: torch.Tensor
+    table: torch.Tensor
+    scale: float = 1.0
+
+    def dense(self) -> torch.Tensor:
+        return self.table[self.ids.long()].float() * self.scale
+
+
 def embed_rows(ids, table, pos, pos_table=None, out=None, out2=None):
     """``(residual fp32, residual in the table's dtype)``: the embedding rows of ``ids``, plus the rows of ``pos`` in
     ``pos_table`` when there is one. ``out`` / ``out2``: where the second one goes (rows may be strided, both alike)."""
@@ -225,13 +253,17 @@ def post_norm(h, w, resid, eps: float, mult: float = 1.0, offset: float = 0.0, w
 
 
 def residual_norm(h, resid, w_next, eps: float, dtype, vec=None, mult: float = 1.0, out=None):
-    """``resid += h + vec`` (in place, fp32; ``h`` is [R, H], an :class:`ExpertSum` or None, ``vec`` [H] or None); returns
-    ``mult * rmsnorm(resid) * w_next`` in ``dtype``, or resid itself without ``w_next``. ``out``: where it goes (rows may be strided)."""
+    """``resid += h + vec`` (in place, fp32; ``h`` is [R, H], an :class:`ExpertSum`, a :class:`BranchSum` or None, ``vec`` [H] or None);
+    returns ``mult * rmsnorm(resid) * w_next`` in ``dtype``, or resid itself without ``w_next``. ``out``: where it goes (rows may be
+    strided)."""
+    if isinstance(h, BranchSum) and resid.is_cuda:
+        assert w_next is not None, "branches are summed on the way into a norm"
+        return _stream_norm(h, resid, resid, w_next, eps, dtype, vec, mult, out)
     parts = isinstance(h, ExpertSum)
     R, H = resid.shape
     if not resid.is_cuda:
         if h is not None:
-            resid += h.dense() if parts else h.float()
+            resid += h.float() if torch.is_tensor(h) else h.dense()
         if vec is not None:
             resid += vec
         x = (resid if w_next is None else mult * group_norm_ref(resid, w_next, 1, eps)).to(dtype)
@@ -244,6 +276,61 @@ def residual_norm(h, resid, w_next, eps: float, dtype, vec=None, mult: float = 1
     _call("ab2_residual_norm", _p(base), 0 if base is None else base.stride(0), _p(lg), 0 if lg is None else lg.stride(0), y, inv, tw, k, n, _p(vec), _p(resid),
           _p(w_next), mult, _p(x), x.stride(0), R, H, eps, _dt(x))
     return x
+
+
+def _stream_norm(src, resid, new, w, eps, dtype, vec=None, mult=1.0, out=None, shift=None):
+    """The kernel behind :func:`stream_norm`; ``shift`` = (share, batch, slot states)."""
+    R, H = new.shape
+    x = torch.empty(R, H, device=new.device, dtype=dtype) if out is None else out
+    ids = table = a = c = wa = wb = None
+    scale = 1.0
+    if isinstance(src, EmbeddingRows):
+        ids, table, scale = src.ids, src.table, src.scale
+        assert table.is_contiguous() and table.dtype == dtype
+    elif isinstance(src, BranchSum):
+        a, c, wa, wb, scale = src.left, src.right, src.w_left, src.w_right, src.factor
+        assert src.eps == eps
+    else:
+        a = src
+    assert new.is_contiguous() and (resid is None or resid.is_contiguous()) and x.dtype == dtype and x.stride(1) == 1
+    assert all(t is None or (t.dtype == dtype and t.stride(1) == 1 and t.shape == (R, H)) for t in (a, c))
+    share, b, S = shift or (None, None, None)
+    nb = 0 if b is None or b.blocks is None else b.blocks.shape[0]
+    batch = (None,) * 4 + (0, 0) if b is None else (_p(b.cu), _p(b.start), _p(b.state), _p(b.blocks), nb, b.n_dec)
+    # rows that a CTA walks: as many as leave every SM several CTAs
+    stretch = 8 if R >= 4096 else (4 if R >= 512 else 2)
+    _call("ab2_stream_norm", _p(ids), _p(table), 0 if table is None else table.shape[0], _p(a), 0 if a is None else a.stride(0), _p(c),
+          0 if c is None else c.stride(0), _p(wa), _p(wb), scale, _p(vec), _p(resid), _p(new), _p(w), mult, _p(share), _p(x), x.stride(0), *batch, stretch,
+          _p(S), R, H, eps, _dt(x))
+    return x
+
+
+def stream_norm(src, resid, w, eps: float, dtype, vec=None, share=None, b: Optional[RaggedBatch] = None, S=None):
+    """What a mixer reads: ``(stream, x)`` with stream = ``resid`` + ``src`` + ``vec`` in fp32 (``src``: [R, H], an :class:`EmbeddingRows`, which
+    begins the stream, a :class:`BranchSum`, an :class:`ExpertSum` or None) and x = h = ``rmsnorm(stream) * w`` in ``dtype``. With a
+    token shift (``share`` [H]) x = ``h + (h' - h) * share``, h' being the h of the sequence's previous token: the row before, or what
+    the entry's slot in S [slots, H] holds (zeros when the sequence is new); S is left at every entry's last h. ``resid`` may be
+    overwritten."""
+    if isinstance(src, ExpertSum):
+        residual_norm(src, resid, None, eps, dtype)
+        src = None
+    like = src.ids if isinstance(src, EmbeddingRows) else resid
+    if like.is_cuda:
+        R = like.shape[0]
+        new = resid if share is None and resid is not None else torch.empty(R, w.shape[0], device=like.device, dtype=torch.float32)
+        return new, _stream_norm(src, resid, new, w, eps, dtype, vec, shift=None if share is None else (share, b, S))
+    add = 0.0 if src is None else (src.float() if torch.is_tensor(src) else src.dense())
+    stream = (0.0 if resid is None else resid) + add + (0.0 if vec is None else vec)
+    h = group_norm_ref(stream, w, 1, eps)
+    if share is None:
+        return stream, h.to(dtype)
+    x = torch.zeros_like(h)
+    for _, r0, r1, st, sl in _segments(b):
+        old = S[sl] if st > 0 else torch.zeros_like(h[0])
+        before = torch.cat([old[None], h[r0:r1 - 1]])
+        x[r0:r1] = h[r0:r1] + (before - h[r0:r1]) * share
+        S[sl] = h[r1 - 1]
+    return stream, x.to(dtype)
 
 
 # ----------------------------------------------------------------------------- rotated positions
@@ -276,22 +363,37 @@ def _rot(rot):
     return _p(rot), rot.stride(0) // 2, rot.shape[1]
 
 
-def qk_head_norm_append(z, wq, wk, eps: float, rot, interleaved: bool, b: RaggedBatch, kc, vc, Hq: int):
-    """Per-head RMS norms of q and k (weights [D] shared by the heads, None: no norm), rotation of the first ``2 * rot.shape[1]``
-    numbers of every head, then k and v into the cache rows of ``b.slots``; returns q [R, Hq, D]. ``z`` rows begin with q | k | v."""
-    Hkv, D, Dv = kc.shape[1], kc.shape[2], vc.shape[2]
+def qk_head_norm_append(z, wq, wk, eps: float, rot, interleaved: bool, b: RaggedBatch, kc, vc, Hq: int, unit: bool = False, q_factor=None,
+                        key_factor=None):
+    """Per-head RMS norms of q and k (weights [D] shared by the heads; None: no norm, or with ``unit`` one without weights), rotation
+    of the first ``2 * rot.shape[1]`` numbers of every head (rot None: none), q times ``q_factor`` [Hq], then k and v into the cache rows of
+    ``b.slots``; returns q [R, Hq, D]. ``z`` rows begin with q | k | v. A norm without weights may as well follow the rotation, which keeps a
+    head's length. With ``key_factor`` [S, Hkv] (fp32) keys are cached as they are, the numbers that norm them go there, and there is no v."""
+    Hkv, D = kc.shape[1], kc.shape[2]
+    Dv = 0 if vc is None else vc.shape[2]
     R, nq, nk = z.shape[0], Hq * D, Hkv * D
     if not z.is_cuda:
+        ones = torch.ones(D)
+
         def turn(x, w):
-            x = x.float()
-            return rotate_ref(x if w is None else group_norm_ref(x, w, 1, eps), rot, interleaved).to(z.dtype)
+            w = ones if w is None and unit else w
+            x = x.float() if w is None else group_norm_ref(x, w, 1, eps)
+            return x if rot is None else rotate_ref(x, rot, interleaved)
         ok = b.slots >= 0
-        kc[b.slots[ok].long()] = turn(z[:, nq:nq + nk].reshape(R, Hkv, D), wk)[ok]
-        vc[b.slots[ok].long()] = z[ok, nq + nk:nq + nk + Hkv * Dv].reshape(-1, Hkv, Dv)
-        return turn(z[:, :nq].reshape(R, Hq, D), wq)
+        at, k = b.slots[ok].long(), z[:, nq:nq + nk].reshape(R, Hkv, D)
+        if key_factor is None:
+            kc[at] = turn(k, wk).to(z.dtype)[ok]
+        else:
+            kc[at] = k[ok]
+            key_factor[at] = torch.rsqrt(k.float().pow(2).mean(-1) + eps)[ok]
+        if vc is not None:
+            vc[at] = z[ok, nq + nk:nq + nk + Hkv * Dv].reshape(-1, Hkv, Dv)
+        q = turn(z[:, :nq].reshape(R, Hq, D), wq)
+        return (q if q_factor is None else q * q_factor[:, None]).to(z.dtype)
     q = torch.empty(R, Hq, D, device=z.device, dtype=z.dtype)
-    _call("ab2_qk_head_norm_append", _p(z), z.stride(0), _p(wq), _p(wk), *_rot(rot), int(interleaved), _p(b.slots), _p(q), _p(kc), _p(vc), R, Hq, Hkv, D,
-          Hkv * Dv, eps, _dt(z))
+    turned = (None, 0, 0) if rot is None else _rot(rot)
+    _call("ab2_qk_head_norm_append", _p(z), z.stride(0), _p(wq), _p(wk), *turned, int(interleaved), _p(b.slots), _p(q), _p(kc), _p(vc), R, Hq, Hkv, D,
+          Hkv * Dv, eps, int(unit), _p(q_factor), _p(key_factor), _dt(z))
     return q
 
 
@@ -299,7 +401,7 @@ def qk_head_norm_append(z, wq, wk, eps: float, rot, interleaved: bool, b: Ragged
 class AttnExtra(ctypes.Structure):
     """Optional inputs of the attention kernels (the struct of the same name in csrc/mixer_common.cuh)."""
 
-    _fields_ = ([(n, ctypes.c_void_p) for n in ("q2", "k2", "gate", "sink")] +
+    _fields_ = ([(n, ctypes.c_void_p) for n in ("q2", "k2", "gate", "sink", "kf")] +
                 [(n, ctypes.c_longlong) for n in ("ldq", "hsq", "ldq2", "hsq2", "ldk", "ldv", "ldk2", "ldo", "ldg")] +
                 [(n, ctypes.c_int) for n in ("D2", "gate_per_head")] + [(n, ctypes.c_float) for n in ("sink_const", "out_scale")])
 
@@ -339,7 +441,7 @@ def qk_norm_append(qkv, wq, wk, eps: float, b: RaggedBatch, kc, vc, Hq: int):
     return q
 
 
-def chunk_attention_ref(q, kc, vc, b: RaggedBatch, scale, softcap, r1, r2, chunk, window=0, sink=None):
+def chunk_attention_ref(q, kc, vc, b: RaggedBatch, scale, softcap, r1, r2, chunk, window=0, sink=None, key_factor=None):
     R, Hq, D = q.shape
     Hkv, Dv = kc.shape[1], vc.shape[2]
     out = torch.zeros(R, Hq, Dv, dtype=q.dtype)
@@ -349,7 +451,8 @@ def chunk_attention_ref(q, kc, vc, b: RaggedBatch, scale, softcap, r1, r2, chunk
         lo = (st // chunk) * chunk if chunk else (max(0, st - window + 1) if window else 0)
         j = torch.arange(lo, end)
         rows = b.pages[e][(j // ps - b.page_base[e]).long()].long() * ps + j % ps
-        k = kc[rows].float().repeat_interleave(rep, 1)
+        k = kc[rows].float() if key_factor is None else kc[rows].float() * key_factor[rows][..., None]
+        k = k.repeat_interleave(rep, 1)
         v = vc[rows].float().repeat_interleave(rep, 1)
         i = torch.arange(st, end)
         s = torch.einsum("ihd,jhd->hij", q[r0:r1_].float(), k) * scale
@@ -369,26 +472,29 @@ def chunk_attention_ref(q, kc, vc, b: RaggedBatch, scale, softcap, r1, r2, chunk
 
 
 def chunk_attention(q, kc, vc, b: RaggedBatch, scale: float, softcap: float = 0.0, r1=None, r2=None, chunk: int = 0, window: int = 0, sink=None, gate=None,
-                    out_scale: float = 1.0, out=None):
+                    out_scale: float = 1.0, out=None, key_factor=None):
     """Attention of the step's queries over the paged cache (their own keys already appended): ``softcap *
     tanh(q.k * scale / softcap)`` minus ``r1[h] * ln(1 + r2[h] * distance)``, softmax over the earlier positions of
     the query's own chunk of ``chunk`` positions, or over itself and the ``window - 1`` before it (0: no limit), with
     ``exp(sink)`` more in the denominator; then times ``sigmoid(gate)`` (gate [R, Hq * Dv], rows may be strided) and ``out_scale``.
+    Without ``vc`` the keys are the values; ``key_factor`` [S, Hkv] (fp32) multiplies every key's scores, not its value.
     Returns [R, Hq, Dv], in ``out`` [R, Hq * Dv] (rows may be strided) when that is given."""
     R, Hq, D = q.shape
+    vc = kc if vc is None else vc
     Hkv, Dv = kc.shape[1], vc.shape[2]
     if not q.is_cuda:
-        o = chunk_attention_ref(q, kc, vc, b, scale, softcap, r1, r2, chunk, window, sink)
+        o = chunk_attention_ref(q, kc, vc, b, scale, softcap, r1, r2, chunk, window, sink, key_factor)
         if gate is not None or out_scale != 1.0:
             o = (o.float() * (1.0 if gate is None else torch.sigmoid(gate.float()).view(R, Hq, Dv)) * out_scale).to(q.dtype)
         return o if out is None else out.copy_(o.view(R, -1))
     if out is None:
         out = torch.empty(R, Hq, Dv, device=q.device, dtype=q.dtype)
-    x = _extra(sink, gate, out_scale=out_scale, ldo=out.stride(0))
+    x = _extra(sink, gate, out_scale=out_scale, ldo=out.stride(0), kf=_p(key_factor))
     common = (_p(kc), _p(vc), _p(b.pages), _p(b.page_base), b.pages.shape[1], b.page_size, Hq, Hkv, D, Dv, scale, softcap, _p(r1), _p(r2), chunk, window,
               ctypes.byref(x))
     fast = q.dtype == torch.bfloat16 and D % 8 == 0 and Dv % 8 == 0 and D <= 128 and Dv <= 128
     tiles = fast and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0 and (gate is None or (gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0))
+    tiles = tiles and (key_factor is None or (softcap == 0.0 and r1 is None))
     nd = b.n_dec
     if nd:
         if fast and Hq // Hkv <= 16:
@@ -567,6 +673,32 @@ def rglru(u, y, y_bias, gate_w, gate_b, lam, b: RaggedBatch, S):
     return out
 
 
+# ----------------------------------------------------------------------------- minGRU
+def min_gru(zug, bias, b: RaggedBatch, S, out=None):
+    """Element-wise ``S_t = (1 - z) S_(t-1) + z c`` with ``z = sigmoid(zr + bz)``, ``u = ur + bu`` and c = u + 1/2 where u >= 0, else sigmoid(u);
+    returns ``S * silu(g)`` [R, W] in zug's dtype and leaves the last state of every entry in its slot. zug [R, 3 W] rows zr | ur | g (may be
+    strided), bias [2 W] bz | bu, S [slots, W]."""
+    R, W = zug.shape[0], S.shape[1]
+    if not zug.is_cuda:
+        z, u, g = zug.float().view(R, 3, W).unbind(1)
+        z, u = z + bias[:W], u + bias[W:]
+        keep, x = torch.sigmoid(-z), torch.sigmoid(z) * torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
+        y = torch.zeros(R, W)
+        for _, r0, r1, st, sl in _segments(b):
+            h = S[sl].clone() if st > 0 else torch.zeros(W)
+            for t in range(r0, r1):
+                h = keep[t] * h + x[t]
+                y[t] = h
+            S[sl] = h
+        y = (y * F.silu(g)).to(zug.dtype)
+        return y if out is None else out.copy_(y)
+    out = torch.empty(R, W, device=zug.device, dtype=zug.dtype) if out is None else out
+    assert zug.stride(1) == 1 and bias.is_contiguous() and out.stride(1) == 1
+    _call("ab2_min_gru", _p(zug), zug.stride(0), _p(bias), _p(b.cu), _p(b.start), _p(b.state), b.n_dec, b.n_entries, 0 if b.blocks is None else b.blocks.shape[0],
+          _p(S), _p(out), out.stride(0), W, _dt(zug))
+    return out
+
+
 # ----------------------------------------------------------------------------- Mamba-2
 def mamba2_scan(xbc, dt_raw, dt_bias, A_log, D, heads: int, vdim: int, state: int, groups: int, b: RaggedBatch, S):
     """``S_t = exp(-exp(A_log) dt) S_(t-1) + dt B_t x_t^T``, ``y_t = S_t^T C_t + D x_t`` per head, from the convolved
@@ -740,7 +872,9 @@ for _n, _a in {
     "ab2_embed_rows": [_V, _V, _I, _V, _V, _I, _V, _V, _V, _lib.c_ll, _I, _I, _I],
     "ab2_residual_norm": [_V, _lib.c_ll, _V, _lib.c_ll, _V, _V, _V, _I, _I, _V, _V, _V, _F, _V, _lib.c_ll, _I, _I, _F, _I],
     "ab2_rotary_table": [_V] * 4 + [_I, _I],
-    "ab2_qk_head_norm_append": [_V, _lib.c_ll, _V, _V, _V, _I, _I, _I] + [_V] * 4 + [_I] * 5 + [_F, _I],
+    "ab2_qk_head_norm_append": [_V, _lib.c_ll, _V, _V, _V, _I, _I, _I] + [_V] * 4 + [_I] * 5 + [_F, _I, _V, _V, _I],
+    "ab2_stream_norm": [_V, _V, _I, _V, _lib.c_ll, _V, _lib.c_ll, _V, _V, _F] + [_V] * 4 + [_F, _V, _V, _lib.c_ll] + [_V] * 4 + [_I] * 3 + [_V, _I, _I, _F, _I],
+    "ab2_min_gru": [_V, _lib.c_ll] + [_V] * 4 + [_I] * 3 + [_V, _V, _lib.c_ll, _I, _I],
     "ab2_latent_rope_append": [_V, _lib.c_ll, _V, _V, _I, _I, _I, _V, _V] + [_I] * 4 + [_F, _I],
     "ab2_retention_decode": [_V, _lib.c_ll, _V, _I, _I, _V, _F] + [_V] * 4 + [_lib.c_ll] + [_I] * 4 + [_F, _F, _I],
     "ab2_retention_portions": [_V, _lib.c_ll, _V, _I, _I, _V, _V, _F] + [_V] * 3 + [_I, _I, _V, _V] + [_I] * 5,
