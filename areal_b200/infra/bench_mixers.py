@@ -455,6 +455,99 @@ def looped_kernel_table(cfg, prefill=(4, 2048), decode=(64, 960), dev="cuda") ->
     return rows
 
 
+def shifted_kernel_table(cfg, prefill=(4, 2048), decode=(64, 960), dev="cuda") -> list[dict]:
+    """As :func:`kernel_table`, for a stack with a token shift, rotated attention and attention beside minGRU (Goganex), each kernel
+    beside the like one of the other stacks and decoders at the same sizes."""
+    bw, fl, _ = peaks()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    bf = dict(device=dev, dtype=torch.bfloat16)
+    f32 = dict(device=dev, dtype=torch.float32)
+    rows = []
+
+    def add(name, fn, nbytes=0.0, flops=0.0, like=None):
+        t = timed(fn, flush=flush)
+        roof = max(nbytes / bw, flops / fl)
+        rows.append(dict(kernel=name, us=round(t * 1e6, 1), roofline_us=round(roof * 1e6, 1), fraction=round(roof / t, 3), like=like))
+
+    Hd, V, ff = cfg.hidden_size, cfg.vocab_size, cfg.intermediate_size
+    at = next(e["mixer"] for e in cfg.mixer_layers if e["type"] == "attention")
+    p = next(e["mixer"] for e in cfg.mixer_layers if e["type"] == "parallel")
+    nq, nk, D, Dv = at["heads"], at["kv_heads"], at["dim"], at["vdim"]
+    lq, lk, Dl, W = p["left"]["heads"], p["left"]["kv_heads"], p["left"]["dim"], p["right"]["width"]
+    half, blocks = at["rot"]["dims"] // 2, W // 256
+    (B, L), (nB, ctx) = prefill, decode
+    pb, prow = _batch([L] * B, [0] * B, dev)
+    db, drow = _batch([1] * nB, [ctx] * nB, dev)
+    w, share, table, dt = torch.ones(Hd, **f32), torch.rand(Hd, **f32), torch.randn(V, Hd, **bf), torch.bfloat16
+    freq, mult, temp = torch.rand(half, device=dev, dtype=torch.float64), torch.ones(half, **f32), torch.ones(nq, **f32)
+    for tag, b, R, rows_, ne in (("prefill", pb, B * L, prow, B), ("decode", db, nB, drow, nB)):
+        one = tag == "decode"
+        # the stream: sums, norms, shift (a portion's stream goes from one buffer to another)
+        ids = torch.randint(0, V, (R,), device=dev, dtype=torch.int32)
+        h, h2, res, S = torch.randn(R, Hd, **bf), torch.randn(R, Hd, **bf), torch.randn(R, Hd, **f32), torch.zeros(ne, Hd, **f32)
+        slot = 2 * ne * Hd * 4
+        add(f"embedding, norm, shift {tag}", lambda: M.stream_norm(M.EmbeddingRows(ids, table, 4.0), None, w, 1e-6, dt, None, share, b, S), R * Hd * 8 + slot,
+            like=f"embed_rows {tag}")
+        add(f"embed_rows {tag}", lambda: M.embed_rows(ids, table, b.pos), R * Hd * 8)
+        add(f"residual sum, norm, shift {tag}", lambda: M.stream_norm(h, res, w, 1e-6, dt, None, share, b, S), R * Hd * 12 + slot, like=f"residual_norm {tag}")
+        add(f"residual_norm {tag}", lambda: M.residual_norm(h, res, w, 1e-6, dt), R * Hd * 12)
+        pair = M.BranchSum(h, h2, w, w, 0.5, 1e-6)
+        add(f"normed branches, norm, shift {tag}", lambda: M.stream_norm(pair, res, w, 1e-6, dt, None, share, b, S), R * Hd * 14 + slot, like=f"sandwich_norm {tag}")
+        add(f"normed branches, norm {tag}", lambda: M.residual_norm(pair, res, w, 1e-6, dt), R * Hd * 14, like=f"sandwich_norm {tag}")
+        add(f"sandwich_norm {tag}", lambda: M.sandwich_norm(h, w, res, w, 1, 1e-6), R * Hd * 12)
+        # queries and keys
+        cs = M.rotary_table(b.pos, freq, mult)
+        z, wh = torch.randn(R, nq * D + nk * (D + Dv), **bf), torch.ones(D, **f32)
+        kc, vc = torch.randn(rows_, nk, D, **bf), torch.randn(rows_, nk, Dv, **bf)
+        add(f"turn, unit norm, append {tag}", lambda: M.qk_head_norm_append(z, None, None, 1e-6, cs, True, b, kc, vc, nq, unit=True, q_factor=temp),
+            z.numel() * 4 + R * half * 8, like=f"qk_head_norm_append {tag}")
+        add(f"qk_head_norm_append {tag}", lambda: M.qk_head_norm_append(z, wh, wh, 1e-6, cs, False, b, kc, vc, nq), z.numel() * 4 + R * half * 8)
+        zl, kl, kf = torch.randn(R, (lq + lk) * Dl, **bf), torch.randn(rows_, lk, Dl, **bf), torch.rand(rows_, lk, **f32)
+        add(f"unit norm, keys as they are {tag}", lambda: M.qk_head_norm_append(zl, None, None, 1e-6, None, False, b, kl, None, lq, unit=True, key_factor=kf),
+            zl.numel() * 4 + R * lk * 4, like=f"qk_head_norm_append {tag}")
+        # attention over everything before, beside the chunked one (capped, biased) whose chunk is as long, and the decoders'
+        q, ql = torch.randn(R, nq, D, **bf), torch.randn(R, lq, Dl, **bf)
+        pairs = nB * (ctx + 1) if one else B * L * (L + 1) // 2
+        keys = pairs if one else R
+
+        def cost(hq, hk, d, dv, per_key):
+            return R * hq * (d + dv) * 2 + keys * per_key, 2.0 * hq * (d + dv) * pairs
+        add(f"attention with a sink {tag}", lambda: M.chunk_attention(q, kc, vc, b, D ** -0.5, sink=0.0), *cost(nq, nk, D, Dv, nk * (D + Dv) * 2),
+            like=f"chunk_attention {tag}")
+        add(f"attention, keys as values {tag}", lambda: M.chunk_attention(ql, kl, None, b, Dl ** -0.5, key_factor=kf), *cost(lq, lk, Dl, Dl, lk * (Dl * 2 + 4)),
+            like=f"chunk_attention {tag}")
+        r1, r2 = torch.rand(nq, **f32), torch.rand(nq, **f32)
+        add(f"chunk_attention {tag}", lambda: M.chunk_attention(q, kc, vc, b, D ** -0.5, 30.0, r1, r2, 4096), *cost(nq, nk, D, Dv, nk * (D + Dv) * 2))
+        if D == Dv and D in (64, 128):
+            if one:
+                lens = torch.full((nB,), ctx + 1, device=dev, dtype=torch.int32)
+                po, ml, o = torch.empty(nB * nq * 4 * D, **f32), torch.empty(nB * nq * 8, **f32), torch.empty_like(q)
+
+                def paged():
+                    oplib.check(oplib.get_lib().ab2_paged_decode_strided(
+                        q.data_ptr(), kc.data_ptr(), vc.data_ptr(), b.pages.data_ptr(), lens.data_ptr(), po.data_ptr(), ml.data_ptr(), o.data_ptr(), nB, nq, nk, D,
+                        64, b.pages.shape[1], 4, D ** -0.5, q.stride(0), oplib.stream_ptr()), "paged_decode")
+                add("paged_decode decode", paged, *cost(nq, nk, D, Dv, nk * (D + Dv) * 2))
+            else:
+                k, v = torch.randn(R, nk, D, **bf), torch.randn(R, nk, D, **bf)
+                cu = torch.arange(0, R + 1, L, device=dev, dtype=torch.int32)
+                ti = OF.attn_tile_table(cu, R)
+                add("attn_fwd prefill", lambda: OF.attention_fwd(q, k, v, cu, True, D ** -0.5, ti), *cost(nq, nk, D, Dv, nk * (D + Dv) * 2))
+        # recurrence, beside the RG-LRU of the same width (whose gates are products of their own)
+        zug, bias, St = torch.randn(R, 3 * W, **bf), torch.zeros(2 * W, **f32), torch.zeros(ne, W, **f32)
+        add(f"min_gru {tag}", lambda: M.min_gru(zug, bias, b, St), R * W * 8 + 2 * St.numel() * 4, like=f"rglru {tag}")
+        n = W // blocks
+        gw, gb, lam, yb = torch.randn(2, blocks, n, n, **bf) * 0.05, torch.zeros(2, blocks, n, **f32), torch.full((W,), -3.0, **f32), torch.zeros(W, **f32)
+        u, yx = torch.randn(R, W, **bf), torch.randn(R, 2 * W, **bf)
+        add(f"rglru {tag}", lambda: M.rglru(u, yx[:, :W], yb, gw, gb, lam, b, St), R * W * 6 + gw.numel() * 2 + 2 * St.numel() * 4, 4.0 * R * W * n)
+        # feed-forward
+        gu = torch.randn(R, 2 * ff, **bf)
+        add(f"glu_clamped {tag}", lambda: M.glu_clamped(gu, 7.0, 1.702), R * ff * 6, like=f"swiglu {tag}")
+        with torch.no_grad():
+            add(f"swiglu {tag}", lambda: OF.swiglu(gu), R * ff * 6)
+    return rows
+
+
 # ----------------------------------------------------------------------------- whole steps
 def _engine(cfg, seqs, total, prefill_tokens):
     from ..api.cli_args import InferenceEngineConfig, NativeInferConfig
@@ -632,6 +725,26 @@ def looped_like_sized(cfg):
     return vog, stack, routed
 
 
+def shifted_like_sized(cfg):
+    """The closest existing models with the same width, heads and vocabulary as a shifted stack, one layer per layer run: the stack
+    that alternates chunked attention (chunks longer than the prompts) and RG-LRU, its dense feed-forwards (two matrices) one and a
+    half times as wide for the same weights; the dense decoder."""
+    from ..models.config import ModelConfig
+    from ..models.mixers import MixerStackLM
+
+    runs = MixerStackLM.layer_runs.fget(type("S", (), dict(cfg=cfg)))
+    at = next(e["mixer"] for e in cfg.mixer_layers if e["type"] == "attention")
+    W, ff = next(e["mixer"] for e in cfg.mixer_layers if e["type"] == "parallel")["right"]["width"], cfg.intermediate_size
+    att = dict(heads=at["heads"], kv_heads=at["kv_heads"], dim=at["dim"], vdim=at["vdim"], scale=at["scale"], softcap=30.0, mask=dict(size=4096))
+    lru = dict(width=W, blocks=W // 256, conv=4)
+    stack = ModelConfig.from_hf_dict(dict(
+        architecture="Kagolix", vocab=cfg.vocab_size, width=cfg.hidden_size, norm=dict(eps=1e-6, groups=1), logit_softcap=0.0,
+        layers=[dict(type="rglru" if n % 2 else "attention", mixer=lru if n % 2 else att, mlp=dict(kind="dense", ff=3 * ff // 2)) for n in range(len(runs))]))
+    dense = ModelConfig(arch="qwen3", vocab_size=cfg.vocab_size, hidden_size=cfg.hidden_size, num_layers=len(runs), num_heads=at["heads"],
+                        num_kv_heads=at["kv_heads"], head_dim=at["dim"], intermediate_size=ff, tie_word_embeddings=False, attention_bias=False, qk_norm=True)
+    return stack, dense
+
+
 def run(steps=True, kernels=True, design="kagolix", sizes=None) -> dict:
     from ..models.config import preset
 
@@ -654,6 +767,11 @@ def run(steps=True, kernels=True, design="kagolix", sizes=None) -> dict:
             for key, fn, c in (("bumotar", mixer_steps, cfg), ("vogilix", mixer_steps, latent), ("mixer_stack", mixer_steps, stack), ("decoder_routed", decoder_steps, routed)):
                 r[key] = fn(c, prefill, decode)
                 torch.cuda.empty_cache()
+        elif steps and design == "goganex":
+            stack, dense = shifted_like_sized(cfg)
+            for key, fn, c in (("goganex", mixer_steps, cfg), ("mixer_stack", mixer_steps, stack), ("decoder_dense", decoder_steps, dense)):
+                r[key] = fn(c, prefill, decode)
+                torch.cuda.empty_cache()
         elif steps:
             hyb, dense, routed = like_sized(cfg)
             r["mixer_stack"] = mixer_steps(cfg, prefill, decode)
@@ -662,6 +780,7 @@ def run(steps=True, kernels=True, design="kagolix", sizes=None) -> dict:
                 r[key] = fn(c, prefill, decode)
                 torch.cuda.empty_cache()
         if kernels:
-            r["kernels"] = {"vogilix": latent_kernel_table, "bumotar": looped_kernel_table, "kagolix": kernel_table}[design](cfg, prefill, decode)
+            r["kernels"] = {"vogilix": latent_kernel_table, "bumotar": looped_kernel_table, "goganex": shifted_kernel_table,
+                            "kagolix": kernel_table}[design](cfg, prefill, decode)
         out["sizes"][name] = r
     return out

@@ -55,7 +55,7 @@ def parse_args():
     ap.add_argument("--workload", type=str, default="train", choices=["train", "mixer-serve"],
                     help="train: the headline job; mixer-serve: prefill and decode throughput of the mixer stack beside the closest existing "
                          "models, and its kernels against their rooflines (one GPU, prints its own JSON line)")
-    ap.add_argument("--design", type=str, default="kagolix", choices=["kagolix", "vogilix", "bumotar"], help="mixer-serve: the mixer stack to measure")
+    ap.add_argument("--design", type=str, default="kagolix", choices=["kagolix", "vogilix", "bumotar", "goganex"], help="mixer-serve: the mixer stack to measure")
     ap.add_argument("--model", type=str, default="qwen3-8b")
     ap.add_argument("--preset", type=str, default="driver", choices=sorted(PRESETS))
     ap.add_argument("--length-scale", type=float, default=None, help="scales prompt / median / cap lengths of the preset")

@@ -60,8 +60,8 @@ CONFIGS = {
     "wide": config((att(heads=17, kv=1, dim=64, vdim=96, turn=llama3(64)), dense(96)), (par(heads=20, kv=4, dim=96, width=200), dense(40)),
                    width=128, vocab=96, loop=(1, 2, 1), scale=1.0),
     "dim128": config((par(heads=2, kv=1, dim=128, width=8), dense(64)), (att(heads=2, kv=2, dim=128, vdim=128, turn=llama3(128)), dense(64)), loop=(1, 2, 2), scale=2.5),
-    # no loop, parallel branches first and last, a key head per query head, small and very large heads, one channel
-    "edges": config((par(heads=3, kv=3, dim=8, width=1), dense(16)), (att(heads=2, kv=1, dim=136, vdim=24, turn=rot(100)), None),
+    # no loop, parallel branches first and last, a key head per query head, small and very large heads, few channels
+    "edges": config((par(heads=3, kv=3, dim=8, width=10), dense(16)), (att(heads=2, kv=1, dim=136, vdim=24, turn=rot(100)), None),
                     (att(heads=2, kv=2, dim=8, vdim=40, turn=llama3(2)), dense()), (par(heads=2, kv=1, dim=136, width=130), dense(24)), width=40, loop=None),
 }
 
