@@ -170,8 +170,8 @@ struct ChunkDecodeCfg {
   static constexpr int KROW = DK * 2 + 16, VROW = DV * 2 + 16;     // padded rows: matrix loads touch distinct banks
   static constexpr int STAGE = CD_KEYS * (KROW + VROW);
   static constexpr int Q_OFF = 2 * STAGE;
-  static constexpr int ROWS_OFF = Q_OFF + 16 * KROW;               // cache row of every key, two pieces
-  static constexpr int SMEM = ROWS_OFF + 2 * CD_KEYS * 4;
+  static constexpr int ROWS_OFF = Q_OFF + 16 * KROW;               // cache row of every key, four pieces
+  static constexpr int SMEM = ROWS_OFF + 4 * CD_KEYS * 4;
 };
 
 template <int DK, int DV, int SPL, bool CAP>
@@ -182,7 +182,7 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
   constexpr int KS = DK / 16;
   extern __shared__ __align__(128) unsigned char dsm[];
   __shared__ float s_ml[2][16];                                     // this CTA's merged (max, sum) per head
-  __shared__ float s_kf[2][CD_KEYS];                                // factors of the keys of two pieces
+  __shared__ float s_kf[4][CD_KEYS];                                // factors of the keys of four pieces
   pdl_wait();
   pdl_trigger();
   const int b = blockIdx.x, h = blockIdx.y, spl = blockIdx.z;
@@ -199,19 +199,22 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
   const int base = p.page_base[b];
   const uint32_t sm = smem_u32(dsm);
   int* s_row = reinterpret_cast<int*>(dsm + Cfg::ROWS_OFF);
-  const bool same = DK == DV && p.vc == p.kc;                       // keys are the values: one copy of a piece serves both products
-  auto plan = [&](int c) {
-    if (tid < CD_KEYS) {
-      const int t = t0 + c * CD_KEYS + tid;
-      s_row[(c & 1) * CD_KEYS + tid] = t < t1 ? pt[t / p.page_size - base] * p.page_size + t % p.page_size : -1;
-    }
+  // keys that are the values: one copy of a piece serves both products, and twice as many pieces are on their way
+  const bool same = DK == DV && p.vc == p.kc;
+  const int ahead = same ? 3 : 1, stage = same ? CD_KEYS * Cfg::KROW : Cfg::STAGE;
+  auto row_of = [&](int c) {                                        // cache row of this thread's key of piece c
+    const int t = t0 + c * CD_KEYS + tid;
+    return tid < CD_KEYS && t < t1 ? pt[t / p.page_size - base] * p.page_size + t % p.page_size : -1;
+  };
+  auto plan = [&](int c, int row) {
+    if (tid < CD_KEYS) s_row[(c & 3) * CD_KEYS + tid] = row;
   };
   auto issue = [&](int c) {
-    const uint32_t st = sm + (c & 1) * Cfg::STAGE;
+    const uint32_t st = sm + (c & ahead) * stage;
 #pragma unroll
     for (int k = 0; k < CD_KEYS * (DK / 8) / 128; ++k) {
       const int idx = tid + k * 128, r = idx / (DK / 8), piece = idx % (DK / 8);
-      const int row = s_row[(c & 1) * CD_KEYS + r];
+      const int row = s_row[(c & 3) * CD_KEYS + r];
       const bool ok = row >= 0 && piece * 8 < p.D;
       cd_copy16(st + r * Cfg::KROW + piece * 16, (const __nv_bfloat16*)p.kc + (ok ? row * p.x.ldk + h * p.D + piece * 8 : 0), ok);
     }
@@ -219,22 +222,23 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
 #pragma unroll
       for (int k = 0; k < CD_KEYS * (DV / 8) / 128; ++k) {
         const int idx = tid + k * 128, r = idx / (DV / 8), piece = idx % (DV / 8);
-        const int row = s_row[(c & 1) * CD_KEYS + r];
+        const int row = s_row[(c & 3) * CD_KEYS + r];
         const bool ok = row >= 0 && piece * 8 < p.Dv;
         cd_copy16(st + CD_KEYS * Cfg::KROW + r * Cfg::VROW + piece * 16, (const __nv_bfloat16*)p.vc + (ok ? row * p.x.ldv + h * p.Dv + piece * 8 : 0), ok);
       }
     }
     if (p.x.kf && tid < CD_KEYS) {
-      const int row = s_row[(c & 1) * CD_KEYS + tid];
+      const int row = s_row[(c & 3) * CD_KEYS + tid];
       const float* f = p.x.kf + (row >= 0 ? (long long)row * p.Hkv + h : 0);
-      asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_u32(&s_kf[c & 1][tid])), "l"(f), "r"(row >= 0 ? 4 : 0) : "memory");
+      asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_u32(&s_kf[c & 3][tid])), "l"(f), "r"(row >= 0 ? 4 : 0) : "memory");
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  if (np > 0) plan(0);
-  if (np > 1) plan(1);
+#pragma unroll
+  for (int c = 0; c < 4; ++c)
+    if (c < np && c <= ahead) plan(c, row_of(c));
   __syncthreads();
-  if (np > 0) issue(0);
+  for (int c = 0; c < min(np, ahead); ++c) issue(c);
   for (int k = tid; k < 16 * (DK / 8); k += 128) {
     const int r = k / (DK / 8), piece = k % (DK / 8);
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
@@ -259,15 +263,15 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
   for (int j = 0; j < DV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   for (int c = 0; c < np; ++c) {
-    if (c + 1 < np) {
-      issue(c + 1);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
-    } else {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
-    }
+    if (c + ahead < np) issue(c + ahead);
+    const int later = min(np - 1 - c, ahead);         // pieces that need not be there yet
+    if (later == 0) asm volatile("cp.async.wait_group 0;" ::: "memory");
+    else if (later == 1) asm volatile("cp.async.wait_group 1;" ::: "memory");
+    else if (later == 2) asm volatile("cp.async.wait_group 2;" ::: "memory");
+    else asm volatile("cp.async.wait_group 3;" ::: "memory");
     __syncthreads();
-    if (c + 2 < np) plan(c + 2);                     // its table half is free: piece c has been issued from it
-    const uint32_t ka = sm + (c & 1) * Cfg::STAGE + warp * 16 * Cfg::KROW;
+    const int next = c + ahead + 1 < np ? row_of(c + ahead + 1) : -1;      // looked up while this piece is worked on
+    const uint32_t ka = sm + (c & ahead) * stage + warp * 16 * Cfg::KROW;
     const uint32_t va = same ? ka : sm + (c & 1) * Cfg::STAGE + CD_KEYS * Cfg::KROW + warp * 16 * Cfg::VROW;
     float s[2][4] = {};
 #pragma unroll
@@ -279,7 +283,7 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
     }
     const int tok = t0 + c * CD_KEYS + warp * 16 + 2 * tq;
     if (p.x.kf) {
-      const float* f = &s_kf[c & 1][warp * 16 + 2 * tq];
+      const float* f = &s_kf[c & 3][warp * 16 + 2 * tq];
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
         const float v = f[(k >> 1) * 8 + (k & 1)];
@@ -328,6 +332,7 @@ __device__ __forceinline__ void chunk_decode_body(const __nv_bfloat16* __restric
       cd_mma(o[2 * jj], pa, b0, b1);
       cd_mma(o[2 * jj + 1], pa, b2, b3);
     }
+    if (c + ahead + 1 < np) plan(c + ahead + 1, next);                     // that part of the table is free: its piece has been issued
     __syncthreads();
   }
   // ---- the four warps, then the CTAs of the cluster
@@ -645,9 +650,19 @@ chunk_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       tmem_ld_wait();
       const bool edge = kb < lo_last || kb + CP_K - 1 > first;
       float mx = -INFINITY;
+      if constexpr (ADJ == ADJ_KEY) {
+#pragma unroll
+        for (int c = 0; c < 64; c += 4) {
+          const float4 f = *reinterpret_cast<const float4*>(bs + c);
+          u[c] = __float_as_uint(__uint_as_float(u[c]) * f.x);
+          u[c + 1] = __float_as_uint(__uint_as_float(u[c + 1]) * f.y);
+          u[c + 2] = __float_as_uint(__uint_as_float(u[c + 2]) * f.z);
+          u[c + 3] = __float_as_uint(__uint_as_float(u[c + 3]) * f.w);
+        }
+      }
 #pragma unroll
       for (int c = 0; c < 64; ++c) {
-        float v = ADJ == ADJ_KEY ? __uint_as_float(u[c]) * bs[c] : capped<CAP>(__uint_as_float(u[c]), sc);
+        float v = ADJ == ADJ_KEY ? __uint_as_float(u[c]) : capped<CAP>(__uint_as_float(u[c]), sc);
         if constexpr (ADJ == ADJ_DISTANCE) v -= bs[lane - c + 63];
         if (edge && (kb + c > i || kb + c < lo)) v = -INFINITY;
         u[c] = __float_as_uint(v);
@@ -735,14 +750,17 @@ template <int DK, int DV, int, bool CAP, int>
 static int launch_decode(const void* q, const int* pos, const int* slots, void* out, int R, const ChunkArgs& a, cudaStream_t s) {
   constexpr int SMEM = ChunkDecodeCfg<DK, DV>::SMEM;
   static_assert(2 * ChunkDecodeCfg<DK, DV>::STAGE >= (4 * 16 * DV + 8 * 16) * 4, "the merge buffers alias the stage memory");
-  const int spl = R * a.Hkv >= 1776 ? 1 : (R * a.Hkv >= 111 ? 4 : 8);      // several waves of three CTAs per SM, or all there is
+  // as many pieces of a request as still run at once (three CTAs per SM); halves where whole requests leave a short second wave
+  const long long pairs = (long long)R * a.Hkv, room = 3 * 148;
+  const int spl = pairs * 8 <= room ? 8 : (pairs * 4 <= room ? 4 : (pairs * 2 <= room || (pairs > room && pairs < 2 * room) ? 2 : 1));
   auto go = [&](auto kern, ab2host::DevState& st) -> int {
     if (ab2host::prepare_launch(kern, SMEM, st, nullptr)) return 300;
     launch_pdl(kern, dim3(R, a.Hkv, spl), dim3(128), (size_t)SMEM, s, (const __nv_bfloat16*)q, pos, slots, (__nv_bfloat16*)out, a);
     return cudaGetLastError() == cudaSuccess ? 0 : 302;
   };
-  static ab2host::DevState st1, st4, st8;
+  static ab2host::DevState st1, st2, st4, st8;
   if (spl == 1) return go(chunk_decode_kernel<DK, DV, CAP>, st1);
+  if (spl == 2) return go(chunk_decode_split_kernel<DK, DV, 2, CAP>, st2);
   if (spl == 4) return go(chunk_decode_split_kernel<DK, DV, 4, CAP>, st4);
   return go(chunk_decode_split_kernel<DK, DV, 8, CAP>, st8);
 }

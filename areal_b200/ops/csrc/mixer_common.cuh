@@ -9,7 +9,7 @@ __device__ __forceinline__ float ldf(const __nv_bfloat16* p) { return __bfloat16
 __device__ __forceinline__ void stf(float* p, float v) { *p = v; }
 __device__ __forceinline__ void stf(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 
-// V consecutive elements (V = 1, 4 or 8; the address is aligned to V elements)
+// V consecutive elements (V = 1, 2, 4 or 8; the address is aligned to V elements)
 template <int V>
 __device__ __forceinline__ void ldv(const float* p, float (&v)[V]) {
   if constexpr (V == 8) {
@@ -18,6 +18,9 @@ __device__ __forceinline__ void ldv(const float* p, float (&v)[V]) {
   } else if constexpr (V == 4) {
     const float4 a = *reinterpret_cast<const float4*>(p);
     v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+  } else if constexpr (V == 2) {
+    const float2 a = *reinterpret_cast<const float2*>(p);
+    v[0] = a.x; v[1] = a.y;
   } else {
     v[0] = *p;
   }
@@ -37,6 +40,9 @@ __device__ __forceinline__ void ldv(const __nv_bfloat16* p, float (&v)[V]) {
     const uint2 a = *reinterpret_cast<const uint2*>(p);
     const float2 x = unpack_bf16(a.x), y = unpack_bf16(a.y);
     v[0] = x.x; v[1] = x.y; v[2] = y.x; v[3] = y.y;
+  } else if constexpr (V == 2) {
+    const float2 x = unpack_bf16(*reinterpret_cast<const uint32_t*>(p));
+    v[0] = x.x; v[1] = x.y;
   } else {
     v[0] = __bfloat162float(*p);
   }
@@ -47,6 +53,7 @@ __device__ __forceinline__ void stv(float* p, const float (&v)[V]) {
     reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
     reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
   } else if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  else if constexpr (V == 2) *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
   else *p = v[0];
 }
 template <int V>
@@ -54,7 +61,16 @@ __device__ __forceinline__ void stv(__nv_bfloat16* p, const float (&v)[V]) {
   if constexpr (V == 8) {
     *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
   } else if constexpr (V == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
+  else if constexpr (V == 2) *reinterpret_cast<uint32_t*>(p) = pack_bf16(v[0], v[1]);
   else *p = __float2bfloat16(v[0]);
+}
+
+// Copy of N bytes from global into shared memory that the copying thread alone will read, after its own wait (cp.async.wait_group).
+template <int N>
+__device__ __forceinline__ void copy_own(void* dst, const void* src) {
+  if constexpr (N == 2) *reinterpret_cast<uint16_t*>(dst) = *reinterpret_cast<const uint16_t*>(src);
+  else if constexpr (N == 16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+  else asm volatile("cp.async.ca.shared.global [%0], [%1], %2;" ::"r"(smem_u32(dst)), "l"(src), "n"(N) : "memory");
 }
 
 // Scalar functions. FAST (beside bf16 activations) takes the hardware exponential, logarithm and division, about 1e-6

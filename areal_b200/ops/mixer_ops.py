@@ -278,6 +278,14 @@ def residual_norm(h, resid, w_next, eps: float, dtype, vec=None, mult: float = 1
     return x
 
 
+def _stretch(rows: int, blocks: Optional[int]) -> int:
+    """Rows that a CTA of the stream kernel walks: few of them make more CTAs, many read less twice (``blocks``: 64-row blocks of the
+    portions when rows are shifted, else None)."""
+    if blocks is None:
+        return 4 if rows >= 2048 else 1
+    return 7 if blocks >= 16 else 3
+
+
 def _stream_norm(src, resid, new, w, eps, dtype, vec=None, mult=1.0, out=None, shift=None):
     """The kernel behind :func:`stream_norm`; ``shift`` = (share, batch, slot states)."""
     R, H = new.shape
@@ -297,10 +305,9 @@ def _stream_norm(src, resid, new, w, eps, dtype, vec=None, mult=1.0, out=None, s
     share, b, S = shift or (None, None, None)
     nb = 0 if b is None or b.blocks is None else b.blocks.shape[0]
     batch = (None,) * 4 + (0, 0) if b is None else (_p(b.cu), _p(b.start), _p(b.state), _p(b.blocks), nb, b.n_dec)
-    # rows that a CTA walks: as many as leave every SM several CTAs
-    stretch = 8 if R >= 4096 else (4 if R >= 512 else 2)
     _call("ab2_stream_norm", _p(ids), _p(table), 0 if table is None else table.shape[0], _p(a), 0 if a is None else a.stride(0), _p(c),
-          0 if c is None else c.stride(0), _p(wa), _p(wb), scale, _p(vec), _p(resid), _p(new), _p(w), mult, _p(share), _p(x), x.stride(0), *batch, stretch,
+          0 if c is None else c.stride(0), _p(wa), _p(wb), scale, _p(vec), _p(resid), _p(new), _p(w), mult, _p(share), _p(x), x.stride(0), *batch,
+          _stretch(R, None if b is None else nb),
           _p(S), R, H, eps, _dt(x))
     return x
 
@@ -674,10 +681,10 @@ def rglru(u, y, y_bias, gate_w, gate_b, lam, b: RaggedBatch, S):
 
 
 # ----------------------------------------------------------------------------- minGRU
-def min_gru(zug, bias, b: RaggedBatch, S, out=None):
+def min_gru(zug, bias, b: RaggedBatch, S, out=None, cluster: int = 0):
     """Element-wise ``S_t = (1 - z) S_(t-1) + z c`` with ``z = sigmoid(zr + bz)``, ``u = ur + bu`` and c = u + 1/2 where u >= 0, else sigmoid(u);
     returns ``S * silu(g)`` [R, W] in zug's dtype and leaves the last state of every entry in its slot. zug [R, 3 W] rows zr | ur | g (may be
-    strided), bias [2 W] bz | bu, S [slots, W]."""
+    strided), bias [2 W] bz | bu, S [slots, W]. ``cluster``: CTAs that share a portion (0: by size)."""
     R, W = zug.shape[0], S.shape[1]
     if not zug.is_cuda:
         z, u, g = zug.float().view(R, 3, W).unbind(1)
@@ -695,7 +702,7 @@ def min_gru(zug, bias, b: RaggedBatch, S, out=None):
     out = torch.empty(R, W, device=zug.device, dtype=zug.dtype) if out is None else out
     assert zug.stride(1) == 1 and bias.is_contiguous() and out.stride(1) == 1
     _call("ab2_min_gru", _p(zug), zug.stride(0), _p(bias), _p(b.cu), _p(b.start), _p(b.state), b.n_dec, b.n_entries, 0 if b.blocks is None else b.blocks.shape[0],
-          _p(S), _p(out), out.stride(0), W, _dt(zug))
+          cluster, _p(S), _p(out), out.stride(0), W, _dt(zug))
     return out
 
 
@@ -874,7 +881,7 @@ for _n, _a in {
     "ab2_rotary_table": [_V] * 4 + [_I, _I],
     "ab2_qk_head_norm_append": [_V, _lib.c_ll, _V, _V, _V, _I, _I, _I] + [_V] * 4 + [_I] * 5 + [_F, _I, _V, _V, _I],
     "ab2_stream_norm": [_V, _V, _I, _V, _lib.c_ll, _V, _lib.c_ll, _V, _V, _F] + [_V] * 4 + [_F, _V, _V, _lib.c_ll] + [_V] * 4 + [_I] * 3 + [_V, _I, _I, _F, _I],
-    "ab2_min_gru": [_V, _lib.c_ll] + [_V] * 4 + [_I] * 3 + [_V, _V, _lib.c_ll, _I, _I],
+    "ab2_min_gru": [_V, _lib.c_ll] + [_V] * 4 + [_I] * 4 + [_V, _V, _lib.c_ll, _I, _I],
     "ab2_latent_rope_append": [_V, _lib.c_ll, _V, _V, _I, _I, _I, _V, _V] + [_I] * 4 + [_F, _I],
     "ab2_retention_decode": [_V, _lib.c_ll, _V, _I, _I, _V, _F] + [_V] * 4 + [_lib.c_ll] + [_I] * 4 + [_F, _F, _I],
     "ab2_retention_portions": [_V, _lib.c_ll, _V, _I, _I, _V, _V, _F] + [_V] * 3 + [_I, _I, _V, _V] + [_I] * 5,

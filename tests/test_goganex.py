@@ -390,7 +390,7 @@ def test_factors_of_keys_go_with_caps_and_distance_biases(target):
 @pytest.mark.parametrize("lens,starts", [([1, 1, 1, 130, 64, 2, 200], [0, 47, 5, 0, 63, 118, 3]), ([1, 700, 513, 2], [9, 0, 20, 0]), ([3, 2, 64], [0, 1, 30])])
 def test_min_gru(lens, starts, width, target):
     """Portions and single tokens from carried states, in slots that hold what an earlier request left; gates from nearly shut to
-    nearly open. Portions of one block, of several, and of several rounds of a cluster's blocks."""
+    nearly open. Portions of one block, of several, and of several rounds of blocks, by one CTA and by clusters."""
     g = torch.Generator().manual_seed(width)
     b, entries, _ = ragged(lens, starts, target[0])
     R, bias = sum(lens), bf16_values((2 * width,), g, 1.0)
@@ -406,9 +406,9 @@ def test_min_gru(lens, starts, width, target):
         rows.append(x[s:]), ends.append(states[-1]), wants.append((states * plain.silu(x[:, 2 * width:]))[s:])
     wide = torch.zeros(R, 3 * width + 9, dtype=target[1], device=target[0])                  # rows of a wider product, not aligned
     wide[:, 1:3 * width + 1] = dev(torch.cat(rows), target)
-    for zug in (wide[:, 1:3 * width + 1], wide[:, 1:3 * width + 1].contiguous()):
+    for zug, cluster in [(wide[:, 1:3 * width + 1], 0), *((wide[:, 1:3 * width + 1].contiguous(), c) for c in (0, 1, 2, 4, 8))]:
         S2 = S.clone()
-        got, at = M.min_gru(zug, f32(bias, target), b, S2).double().cpu(), 0
+        got, at = M.min_gru(zug, f32(bias, target), b, S2, cluster=cluster).double().cpu(), 0
         for e, n in enumerate(lens):
             err = (got[at:at + n] - wants[e]).abs().max() / wants[e].abs().max()
             assert err < (1e-5 if target[1] == torch.float32 else 0.01), (e, float(err))
