@@ -504,7 +504,7 @@ class KeyValueBranch(_Block):
 
 
 class MinGRUBranch(_Block):
-    """Gated recurrence whose gates read only the current token. Works on its rows z | x | g of a fused projection."""
+    """Element-wise recurrence with gates made from the token alone, not from the state. Works on its rows z | x | g of a fused projection."""
 
     parts = ("z", "x", "g")
 
@@ -788,18 +788,20 @@ class Design:
     mlps: dict                   # feed-forward kinds
     layer_norms: tuple           # norms of a layer with a feed-forward ...
     layer_norms_bare: tuple      # ... and of one without
-    kernels: tuple               # sources of its mixers' kernels (beside those of every stack)
+    kernels: tuple               # sources of its own kernels (beside those of every stack)
 
+
+EXPERTS = ("gemm_grouped", "router")         # kernel sources of routed feed-forwards (and of products per head)
 
 DESIGNS = {
     "kagolix": Design("Kagolix", {"attention": ChunkAttention, "rglru": RGLRU, "mamba2": Mamba2}, {"dense": XieluMLP, "moe": RoutedMLP}, ("norm1", "norm1b", "norm2", "norm2b"),
-                      ("norm1", "norm1b"), ("mixer_attention", "mixer_scan", "mixer_ssd")),
+                      ("norm1", "norm1b"), ("mixer_attention", "mixer_scan", "mixer_ssd", *EXPERTS)),
     "vogilix": Design("Vogilix", {"latent_attention": LatentAttention}, {"dense": GeluMLP, "moe": InputWeightedMLP}, ("norm1", "norm2"), ("norm1",),
-                      ("mixer_attention", "mixer_latent")),
+                      ("mixer_attention", "mixer_latent", *EXPERTS)),
     "bumotar": Design("Bumotar", {"latent_attention": RotaryLatentAttention, "parallel": Parallel}, {"moe": SharedExpertMLP}, ("norm1", "norm2"), ("norm1",),
-                      ("mixer_attention", "mixer_latent", "mixer_retention", "mixer_rotary")),
+                      ("mixer_attention", "mixer_latent", "mixer_retention", "mixer_rotary", "mixer_stream", *EXPERTS)),
     "goganex": Design("Goganex", {"attention": RotaryAttention, "parallel": NormedParallel}, {"dense": ClampedMLP}, ("norm1", "norm2"), ("norm1",),
-                      ("mixer_attention", "mixer_rotary", "mixer_gru")),
+                      ("mixer_attention", "mixer_rotary", "mixer_stream", "mixer_gru")),
 }
 
 

@@ -24,7 +24,7 @@ BUILD = HERE / "build"
 LIB = HERE / "libab2_kernels.so"
 # the kernels that serve any mixer stack; with those of a design's own mixers, linked alone, they are what a fresh checkout
 # compiles before its first trace
-STEP_SOURCES = ("runtime", "gemm", "gemm2sm", "gemm_grouped", "router", "infer", "mixer_ops", "mixer_stream")
+STEP_SOURCES = ("runtime", "gemm", "gemm2sm", "infer", "mixer_ops")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",

@@ -1,4 +1,4 @@
-// Element-wise gated recurrence whose gates read only the current token (minGRU), on per-request state slots:
+// minGRU: an element-wise recurrence with gates made from the token alone, not from the state; on per-request state slots:
 //   z = sigmoid(zr + bz);  c = u + 1/2 for u = ur + bu >= 0, else sigmoid(u);  S = (1 - z) S + z c;  out = S * silu(g)
 // Gates, candidates and states are fp32; rows of the projections z | u | g and the output are bf16 or fp32.
 //
