@@ -92,10 +92,10 @@ class AgentGateway:
             base = f"http://{self.inference}/v1" if self.inference else ""
             res = call(f"http://{s['worker']}/turn", dict(session_key=s["key"], message=run["message"], base_url=base, api_key=s["api_key"],
                                                           history=s["history"]), timeout=self.turn_timeout)
-            run["result"], run["status"] = res, "ok"
+            run["result"], status = res, "ok"
             s["history"] += [{"role": "user", "content": run["message"]}, {"role": "assistant", "content": res.get("text", "")}]
         except Exception as e:  # the run fails, the session stays usable
-            run["error"], run["status"] = repr(e), "error"
+            run["error"], status = repr(e), "error"
         nxt = None
         with self._lock:
             s["active"] = None
@@ -109,6 +109,7 @@ class AgentGateway:
                     nxt = s["queue"].pop(0)
                 follow = self._start_run(s, nxt[0], nxt[1])
                 run["followup_run_id"] = follow["run_id"]
+            run["status"] = status          # last: whoever waits for the run sees its follow-up and the session's history
 
     # ---- routes
     def _install(self):
